@@ -5,6 +5,7 @@ from .gotulorn import GotulornConfig
 from .konovik import KonovikConfig
 from .lefulorn import LefulornConfig
 from .llama import LlamaConfig, RopeScaling
+from .tedisun import TedisunConfig
 
-__all__ = ["ConfigError", "ModelConfig", "DizepelConfig", "GotulornConfig", "KonovikConfig", "LefulornConfig", "LlamaConfig", "RopeScaling", "architecture_of", "architectures",
+__all__ = ["ConfigError", "ModelConfig", "DizepelConfig", "GotulornConfig", "KonovikConfig", "LefulornConfig", "LlamaConfig", "RopeScaling", "TedisunConfig", "architecture_of", "architectures",
            "config_from_dict", "load_config", "lookup_architecture", "register_architecture"]

@@ -51,6 +51,8 @@ LIBRARIES: Dict[str, tuple] = {
     "token_mix": ("token_mix.cu", []),
     "norm_conv": ("norm_conv.cu", []),
     "ssd": ("ssd.cu", []),
+    "matrix_memory": ("matrix_memory.cu", []),
+    "streams": ("streams.cu", []),
 }
 
 _HEADERS = ["common.cuh", "page_map.cuh"]

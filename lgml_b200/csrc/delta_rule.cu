@@ -1,4 +1,4 @@
-// The gated delta rule with a decay per key channel, and what surrounds it in a mixer: short
+// The gated delta rule with a decay per key channel or one per head, and what surrounds it in a mixer: short
 // causal convolutions with SiLU on q, k and v, unit-length q and k, the write strength beta, the
 // decay, the recurrence itself, and the gated per-head RMS norm of what it reads out.
 //
@@ -11,6 +11,10 @@
 // (S of every head, then the last taps - 1 inputs of the convolutions) lives in one float32
 // vector per request slot.
 //
+// With one decay per head the convolutions are a kernel of their own (short_conv, norm_conv.cu), and
+// delta_head_prepare makes the unit vectors in place and the per-head decay and beta; delta_scan then
+// reads a row of four floats (decay, beta, two zeros) per head.
+//
 // Four kernels a step:
 //   delta_prepare      one block per token, all tokens at once: convolution (the inputs before a
 //                      portion's first token come from the slot), SiLU, norms, beta, decay (beta
@@ -21,7 +25,7 @@
 //                      column of S in registers; the R threads of a column add up S^T k and S^T q
 //                      by shuffles in a fixed order.  Columns never talk to each other, so the
 //                      result does not depend on how a prompt was cut or what else is in the batch.
-//   delta_output       per (token, head): o / rms(o) * weight * sigmoid(gate)
+//   delta_output       per (token, head): o / rms(o) * weight * sigmoid(gate) (or silu(gate))
 #include <math.h>
 
 #include "common.cuh"
@@ -110,6 +114,55 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_conv_state_kernel(
         }
 }
 
+// One decay per head.  qkv [n, C] (q (G D) | k (G D) | v ...) after convolution and SiLU: q and k become unit vectors per
+// head in place, q also times D^-1/2.  gb [n, H, 4] = (decay, beta, 0, 0) from the projections a and b.  A warp takes a head.
+__global__ void __launch_bounds__(PREP_THREADS) delta_head_prepare_kernel(float *__restrict__ qkv, int C, const float *__restrict__ a_pre, int lda,
+                                                                          const float *__restrict__ b_pre, int ldb, const float *__restrict__ a_log,
+                                                                          const float *__restrict__ dt_bias, float *__restrict__ gb, int n_tokens, int H,
+                                                                          int G, int D, int vec) {
+    pdl_trigger();
+    pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const int hpt = 2 * G + 1;                  // q heads, k heads, and one unit for the token's decays and betas
+    const long long total = (long long)n_tokens * hpt;
+    for (long long u = (long long)blockIdx.x * (PREP_THREADS / 32) + (threadIdx.x >> 5); u < total; u += (long long)gridDim.x * (PREP_THREADS / 32)) {
+        const int t = (int)(u / hpt), hd = (int)(u - (long long)t * hpt);
+        if (hd == 2 * G) {
+            for (int h = lane; h < H; h += 32) {
+                const float g = expf(-expf(a_log[h]) * softplus_f(act_load(a_pre + (size_t)t * lda + h) + dt_bias[h]));
+                const float beta = sigmoid_f(act_load(b_pre + (size_t)t * ldb + h));
+                *reinterpret_cast<float4 *>(gb + ((size_t)t * H + h) * 4) = make_float4(g, beta, 0.f, 0.f);
+            }
+            continue;
+        }
+        float *row = qkv + (size_t)t * C + (size_t)hd * D;
+        const float scale = hd < G ? 1.0f / sqrtf((float)D) : 1.f;
+        float ss = 0.f;
+        if (vec && D <= 512) {
+            float4 v[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int d = (i * 32 + lane) * 4;
+                v[i] = d < D ? act_load(reinterpret_cast<const float4 *>(row + d)) : make_float4(0.f, 0.f, 0.f, 0.f);
+                ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
+            }
+            const float inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f) * scale;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int d = (i * 32 + lane) * 4;
+                if (d < D) *reinterpret_cast<float4 *>(row + d) = make_float4(v[i].x * inv, v[i].y * inv, v[i].z * inv, v[i].w * inv);
+            }
+            continue;
+        }
+        for (int d = lane; d < D; d += 32) {
+            const float v = act_load(row + d);
+            ss = fmaf(v, v, ss);
+        }
+        const float inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f) * scale;
+        for (int d = lane; d < D; d += 32) row[d] = act_load(row + d) * inv;
+    }
+}
+
 __device__ __forceinline__ void cp_async_16(void *dst, const void *src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
@@ -124,7 +177,8 @@ template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile(
 // with cp.async (through L2) while this one is computed; else one buffer filled with plain loads.
 // NC columns a thread (column c of a thread lies SCAN_THREADS / R columns after its column c - 1):
 // two independent chains per thread fill the waits of each other, and k, q and the decays are read once for both.
-template <int NPT, bool ASYNC, int NC>
+// HEAD: one decay per head; gb rows are (decay, beta, 0, 0) and a token's row of the decay buffer is those four floats.
+template <int NPT, bool ASYNC, int NC, bool HEAD>
 __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
     const float *__restrict__ qkv_c, const float *__restrict__ gb, float *__restrict__ state, long long state_stride,
     const int *__restrict__ seq_start, const int *__restrict__ slots, float *__restrict__ o_out, int H, int G, int D, int Dv, int R) {
@@ -133,7 +187,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
     extern __shared__ __align__(16) float sm[];
     constexpr int RUN = NPT + 4;                          // floats from one thread's run to the next
     const int DP = RUN * R;
-    const int DB = D + 4, GP = DP + 4;
+    const int DB = HEAD ? 4 : D + 4, GP = HEAD ? 4 : DP + 4;
     const int tcols = SCAN_THREADS / R;                   // columns side by side in a block; a thread's columns lie tcols apart
     const int cols = NC * tcols;
     const int buf_floats = TCH * (2 * DP + GP + cols);
@@ -160,7 +214,8 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
         for (int b = 0; b < nb; ++b) {
             float *k_s = sm + b * buf_floats, *q_s = k_s + TCH * DP, *g_s = q_s + TCH * DP, *v_s = g_s + TCH * GP;
             for (int e = tid; e < rows * DP; e += SCAN_THREADS) k_s[e] = q_s[e] = 0.f;
-            for (int e = tid; e < rows * GP; e += SCAN_THREADS) g_s[e] = (e % GP) < DP ? 1.f : 0.f;
+            if (!HEAD)
+                for (int e = tid; e < rows * GP; e += SCAN_THREADS) g_s[e] = (e % GP) < DP ? 1.f : 0.f;
             for (int e = tid; e < rows * cols; e += SCAN_THREADS) v_s[e] = 0.f;
         }
     }
@@ -181,7 +236,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
             for (int e = tid; e < nt * b4; e += SCAN_THREADS) {
                 const int i = e / b4, d = (e - i * b4) * 4;
                 // the decays go to their places, beta (the row's last four floats) behind the padded row
-                cp_async_16(g_s + i * GP + (d < D ? (d / NPT) * RUN + d % NPT : DP), gb + ((size_t)(t0 + c0 + i) * H + h) * DB + d);
+                cp_async_16(g_s + i * GP + (HEAD ? 0 : (d < D ? (d / NPT) * RUN + d % NPT : DP)), gb + ((size_t)(t0 + c0 + i) * H + h) * DB + d);
             }
             for (int e = tid; e < nt * c4; e += SCAN_THREADS) {
                 const int i = e / c4, cl = (e - i * c4) * 4;
@@ -195,9 +250,10 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
                 q_s[i * DP + at] = act_load(row);
                 k_s[i * DP + at] = act_load(row + G * D);
             }
-            for (int e = tid; e < nt * (D + 1); e += SCAN_THREADS) {
-                const int i = e / (D + 1), d = e - i * (D + 1);
-                g_s[i * GP + (d < D ? (d / NPT) * RUN + d % NPT : DP)] = act_load(gb + ((size_t)(t0 + c0 + i) * H + h) * DB + d);
+            const int gn = HEAD ? 2 : D + 1;
+            for (int e = tid; e < nt * gn; e += SCAN_THREADS) {
+                const int i = e / gn, d = e - i * gn;
+                g_s[i * GP + (HEAD ? d : (d < D ? (d / NPT) * RUN + d % NPT : DP))] = act_load(gb + ((size_t)(t0 + c0 + i) * H + h) * DB + d);
             }
             for (int e = tid; e < nt * cols; e += SCAN_THREADS) {
                 const int i = e / cols, cl = e - i * cols;
@@ -229,18 +285,19 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
 #pragma unroll
             for (int j = 0; j < NPT; j += 4) {
                 *reinterpret_cast<float4 *>(kk + j) = *reinterpret_cast<const float4 *>(k_s + i * DP + r * RUN + j);
-                *reinterpret_cast<float4 *>(gg + j) = *reinterpret_cast<const float4 *>(g_s + i * GP + r * RUN + j);
+                if (!HEAD) *reinterpret_cast<float4 *>(gg + j) = *reinterpret_cast<const float4 *>(g_s + i * GP + r * RUN + j);
                 *reinterpret_cast<float4 *>(qq + j) = *reinterpret_cast<const float4 *>(q_s + i * DP + r * RUN + j);
             }
             // four partial sums each (NPT is a multiple of 4), added in a fixed order: the chain of
             // dependent operations per token is a quarter as long, and the next token waits on it
             float ks[NC], oq[NC];
+            const float g_head = HEAD ? g_s[i * GP] : 1.f;
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
                 float ka[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                 for (int j = 0; j < NPT; ++j) {
-                    S[c][j] *= gg[j];
+                    S[c][j] *= HEAD ? g_head : gg[j];
                     ka[j & 3] = fmaf(kk[j], S[c][j], ka[j & 3]);
                 }
                 ks[c] = (ka[0] + ka[1]) + (ka[2] + ka[3]);
@@ -248,7 +305,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
             for (int o = 1; o < R; o <<= 1)
 #pragma unroll
                 for (int c = 0; c < NC; ++c) ks[c] += __shfl_xor_sync(0xffffffffu, ks[c], o);
-            const float beta = g_s[i * GP + DP];
+            const float beta = g_s[i * GP + (HEAD ? 1 : DP)];
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
                 const float u = beta * (v_s[i * cols + col_local + c * tcols] - ks[c]);
@@ -286,7 +343,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
 template <typename T>
 __global__ void __launch_bounds__(128) delta_output_kernel(const float *__restrict__ o, const float *__restrict__ weight,
                                                            const float *__restrict__ gate, int ldg, T *__restrict__ out, int ldo, int H,
-                                                           int Dv, float eps) {
+                                                           int Dv, float eps, int act) {
     pdl_trigger();
     pdl_wait();
     __shared__ float red[32];
@@ -300,19 +357,20 @@ __global__ void __launch_bounds__(128) delta_output_kernel(const float *__restri
     ss = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)Dv + eps);
     for (int d = threadIdx.x; d < Dv; d += blockDim.x) {
-        const float v = act_load(row + d) * inv * weight[d] * sigmoid_f(act_load(gate + (size_t)t * ldg + (size_t)h * Dv + d));
+        const float z = act_load(gate + (size_t)t * ldg + (size_t)h * Dv + d);
+        const float v = act_load(row + d) * inv * weight[d] * (act ? z * sigmoid_f(z) : sigmoid_f(z));
         out[(size_t)t * ldo + (size_t)h * Dv + d] = from_f32<T>(v);
     }
 }
 
-template <int NPT, bool ASYNC, int NC>
+template <int NPT, bool ASYNC, int NC, bool HEAD>
 int launch_scan(dim3 grid, size_t smem, cudaStream_t stream, const float *qkv_c, const float *gb, float *state, long long state_stride,
                 const int *seq_start, const int *slots, float *o_out, int H, int G, int D, int Dv, int R) {
     if (smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NPT, ASYNC, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NPT, ASYNC, NC, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) LGML_FAIL("delta_scan: cannot have %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
     }
-    lgml_launch(delta_scan_kernel<NPT, ASYNC, NC>, grid, SCAN_THREADS, smem, stream, qkv_c, gb, state, state_stride, seq_start, slots, o_out, H, G, D,
+    lgml_launch(delta_scan_kernel<NPT, ASYNC, NC, HEAD>, grid, SCAN_THREADS, smem, stream, qkv_c, gb, state, state_stride, seq_start, slots, o_out, H, G, D,
                 Dv, R);
     return lgml_launch_status("delta_scan");
 }
@@ -338,9 +396,23 @@ LGML_API int lgml_delta_prepare(const float *proj, int ldp, const float *a_pre, 
     return lgml_launch_status("delta_conv_state");
 }
 
-// gb: float32 [tokens, H, D + 4] as delta_prepare writes it (decays, beta, zeros).
-LGML_API int lgml_delta_scan(const float *qkv_c, const float *gb, float *state, long long state_stride, const int *seq_start,
-                             const int *slots, float *o_out, int n_seqs, int H, int G, int D, int Dv, cudaStream_t stream) {
+// qkv float32 [n, C], C >= 2 G D; a_pre / b_pre: rows of H floats, lda / ldb apart; gb float32 [n, H, 4], 16-byte aligned.
+LGML_API int lgml_delta_head_prepare(float *qkv, int C, const float *a_pre, int lda, const float *b_pre, int ldb, const float *a_log,
+                                     const float *dt_bias, float *gb, int n_tokens, int H, int G, int D, cudaStream_t stream) {
+    LGML_REQUIRE(n_tokens >= 0 && H > 0 && G > 0 && D > 0 && H % G == 0, "delta_head_prepare: bad sizes");
+    LGML_REQUIRE(C >= 2 * G * D && lda >= H && ldb >= H, "delta_head_prepare: rows too short");
+    LGML_REQUIRE(((uintptr_t)gb & 15) == 0, "delta_head_prepare: the decays must be 16-byte aligned");
+    if (n_tokens == 0) return 0;
+    const int vec = C % 4 == 0 && D % 4 == 0 && ((uintptr_t)qkv & 15) == 0;
+    const long long blocks = ((long long)n_tokens * (2 * G + 1) + PREP_THREADS / 32 - 1) / (PREP_THREADS / 32);
+    lgml_launch(delta_head_prepare_kernel, (int)(blocks < 148 * 16 ? blocks : 148 * 16), PREP_THREADS, 0, stream, qkv, C, a_pre, lda, b_pre, ldb, a_log,
+                dt_bias, gb, n_tokens, H, G, D, vec);
+    return lgml_launch_status("delta_head_prepare");
+}
+
+// gb: float32 [tokens, H, D + 4] as delta_prepare writes it (decays, beta, zeros); head_decay: [tokens, H, 4] (decay, beta, zeros).
+LGML_API int lgml_delta_scan_form(const float *qkv_c, const float *gb, float *state, long long state_stride, const int *seq_start,
+                                  const int *slots, float *o_out, int n_seqs, int H, int G, int D, int Dv, int head_decay, cudaStream_t stream) {
     LGML_REQUIRE(n_seqs >= 0 && H > 0 && G > 0 && D > 0 && Dv > 0 && H % G == 0, "delta_scan: bad sizes");
     LGML_REQUIRE(D <= 1024, "delta_scan: key size %d is over 1024", D);
     LGML_REQUIRE(H <= 65535, "delta_scan: too many heads");
@@ -363,12 +435,15 @@ LGML_API int lgml_delta_scan(const float *qkv_c, const float *gb, float *state, 
     const int nc = wide ? 2 : 1;
     const int cols = nc * (SCAN_THREADS / R);
     const bool async = D % 4 == 0 && Dv % 4 == 0 && (((uintptr_t)qkv_c | (uintptr_t)gb) & 15) == 0;
-    const size_t smem = sizeof(float) * (size_t)(async ? 2 : 1) * TCH * (3 * (size_t)(npt + 4) * R + 4 + cols);
+    const size_t smem = sizeof(float) * (size_t)(async ? 2 : 1) * TCH * ((head_decay ? 2 : 3) * (size_t)(npt + 4) * R + 4 + cols);
     dim3 grid(n_seqs, H, (Dv + cols - 1) / cols);
 #define LGML_SCAN_ARGS grid, smem, stream, qkv_c, gb, state, state_stride, seq_start, slots, o_out, H, G, D, Dv, R
-#define LGML_SCAN_CASE(N)                                                                                          \
-    if (nc == 2) return async ? launch_scan<N, true, 2>(LGML_SCAN_ARGS) : launch_scan<N, false, 2>(LGML_SCAN_ARGS); \
-    return async ? launch_scan<N, true, 1>(LGML_SCAN_ARGS) : launch_scan<N, false, 1>(LGML_SCAN_ARGS);
+#define LGML_SCAN_FORM(N, NC) \
+    (head_decay ? (async ? launch_scan<N, true, NC, true>(LGML_SCAN_ARGS) : launch_scan<N, false, NC, true>(LGML_SCAN_ARGS)) \
+                : (async ? launch_scan<N, true, NC, false>(LGML_SCAN_ARGS) : launch_scan<N, false, NC, false>(LGML_SCAN_ARGS)))
+#define LGML_SCAN_CASE(N)                    \
+    if (nc == 2) return LGML_SCAN_FORM(N, 2); \
+    return LGML_SCAN_FORM(N, 1);
     switch (npt) {
         case 4: LGML_SCAN_CASE(4)
         case 8: LGML_SCAN_CASE(8)
@@ -376,20 +451,32 @@ LGML_API int lgml_delta_scan(const float *qkv_c, const float *gb, float *state, 
         default: LGML_SCAN_CASE(32)
     }
 #undef LGML_SCAN_CASE
+#undef LGML_SCAN_FORM
 #undef LGML_SCAN_ARGS
 }
 
-LGML_API int lgml_delta_output(const float *o, const float *weight, const float *gate, int ldg, void *out, int dtype, int ldo,
-                               int n_tokens, int H, int Dv, float eps, cudaStream_t stream) {
+LGML_API int lgml_delta_scan(const float *qkv_c, const float *gb, float *state, long long state_stride, const int *seq_start,
+                             const int *slots, float *o_out, int n_seqs, int H, int G, int D, int Dv, cudaStream_t stream) {
+    return lgml_delta_scan_form(qkv_c, gb, state, state_stride, seq_start, slots, o_out, n_seqs, H, G, D, Dv, 0, stream);
+}
+
+// act 0: the gate is sigmoid(gate); 1: silu(gate)
+LGML_API int lgml_delta_output_act(const float *o, const float *weight, const float *gate, int ldg, void *out, int dtype, int ldo,
+                               int n_tokens, int H, int Dv, float eps, int act, cudaStream_t stream) {
     LGML_REQUIRE(n_tokens >= 0 && H > 0 && Dv > 0 && H <= 65535, "delta_output: bad sizes");
     LGML_REQUIRE(ldg >= H * Dv && ldo >= H * Dv, "delta_output: a row stride is below H Dv");
     if (n_tokens == 0) return 0;
     dim3 grid(n_tokens, H);
     if (dtype == LGML_F32)
-        lgml_launch(delta_output_kernel<float>, grid, 128, 0, stream, o, weight, gate, ldg, (float *)out, ldo, H, Dv, eps);
+        lgml_launch(delta_output_kernel<float>, grid, 128, 0, stream, o, weight, gate, ldg, (float *)out, ldo, H, Dv, eps, act);
     else if (dtype == LGML_BF16)
-        lgml_launch(delta_output_kernel<__nv_bfloat16>, grid, 128, 0, stream, o, weight, gate, ldg, (__nv_bfloat16 *)out, ldo, H, Dv, eps);
+        lgml_launch(delta_output_kernel<__nv_bfloat16>, grid, 128, 0, stream, o, weight, gate, ldg, (__nv_bfloat16 *)out, ldo, H, Dv, eps, act);
     else
         LGML_FAIL("delta_output: unknown type %d", dtype);
     return lgml_launch_status("delta_output");
+}
+
+LGML_API int lgml_delta_output(const float *o, const float *weight, const float *gate, int ldg, void *out, int dtype, int ldo,
+                               int n_tokens, int H, int Dv, float eps, cudaStream_t stream) {
+    return lgml_delta_output_act(o, weight, gate, ldg, out, dtype, ldo, n_tokens, H, Dv, eps, 0, stream);
 }

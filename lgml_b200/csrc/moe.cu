@@ -5,6 +5,11 @@
 //   chosen = the `top` largest z (ties: the lower index), w = softmax over the chosen z alone
 //   y      = sum_e w_e W_down[e] (silu(W_gate[e] h) * (W_up[e] h))
 //
+// Mode 2 of the router: the scores are the softmax over ALL experts, the chosen are those with the largest score + b_r, and
+// the weights are their scores as they are.  The last n_identity of the router's rows may be experts that return their
+// input: a slot that chose one holds -1 (no expert's matrices), and the sum of their weights is the token's weight on
+// its own row (`also`).
+//
 // moe_router writes the chosen experts and their weights, [tokens, top] each.  The experts'
 // matrices lie stacked: gate and up as [X, 2 F, E] with the gate row of a feature followed by its up row (the layout
 // whose product has both in one thread's hands), down as [X, E, F].
@@ -24,7 +29,8 @@ namespace {
 template <typename T>
 __global__ void __launch_bounds__(128) moe_router_kernel(const T *__restrict__ h, int ldh, const float *__restrict__ wr, const float *__restrict__ br,
                                                          int *__restrict__ ids, float *__restrict__ wts, int E, int X, int top, int mode,
-                                                         float route_scale, int n_extra, float *__restrict__ extra) {
+                                                         float route_scale, int n_extra, float *__restrict__ extra, int n_identity,
+                                                         float *__restrict__ identity_w) {
     pdl_trigger();
     pdl_wait();
     // X choice values (+ n_extra logits of rows that are no experts), X scores (mode 1), then the token's row (E floats, from a 16-byte boundary)
@@ -61,13 +67,29 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const T *__restrict__ h
                 sc[e] = sg;
                 z[e] = sg + (br ? br[e] : 0.f);
             } else {
-                z[e] = dot + (br ? br[e] : 0.f);
+                z[e] = dot + (br && mode == 0 ? br[e] : 0.f);
             }
         }
     }
     __syncthreads();
     if (warp != 0) return;
-    float zmax = 0.f, sum = 0.f;
+    float zmax = 0.f, sum = 0.f, own = 0.f;
+    if (mode == 2) {
+        // scores over all logits (z holds them without the bias)
+        float mx = -INFINITY, all = 0.f;
+        for (int e = lane; e < X; e += 32) mx = fmaxf(mx, z[e]);
+        mx = warp_max(mx);
+        for (int e = lane; e < X; e += 32) {
+            sc[e] = expf(z[e] - mx);
+            all += sc[e];
+        }
+        all = 1.0f / warp_sum(all);
+        for (int e = lane; e < X; e += 32) {
+            sc[e] *= all;
+            z[e] = sc[e] + (br ? br[e] : 0.f);
+        }
+        __syncwarp();
+    }
     for (int s = 0; s < top; ++s) {
         float best = -INFINITY;
         int at = 0x7fffffff;
@@ -83,17 +105,22 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const T *__restrict__ h
         }
         if (at == 0x7fffffff) at = 0;               // every logit was -inf or NaN
         if (s == 0) zmax = best;
-        const float p = mode == 1 ? sc[at] : expf(best - zmax);
+        const float p = mode != 0 ? sc[at] : expf(best - zmax);
         sum += p;
+        const bool identity = at >= X - n_identity;
+        if (identity) own += p;
         if (lane == 0) {
-            ids[(size_t)t * top + s] = at;
+            ids[(size_t)t * top + s] = identity ? -1 : at;
             wts[(size_t)t * top + s] = p;
             z[at] = -INFINITY;
         }
         __syncwarp();
     }
     // mode 0: softmax over the chosen logits; mode 1: the chosen scores over their sum (+ 1e-20), times a constant
-    const float inv = mode == 1 ? route_scale / (sum + 1e-20f) : 1.0f / sum;
+    // mode 2: the chosen scores as they are
+    const float inv = mode == 2 ? 1.f : (mode == 1 ? route_scale / (sum + 1e-20f) : 1.0f / sum);
+    if (identity_w != nullptr && lane == 0) identity_w[t] = own * inv;
+    __syncwarp();
     for (int s = lane; s < top; s += 32) wts[(size_t)t * top + s] *= inv;
 }
 
@@ -132,7 +159,8 @@ __global__ void __launch_bounds__(GU_WARPS * 32) moe_gate_up_kernel(const T *__r
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     for (int k = threadIdx.x; k < E; k += blockDim.x) hs[k] = to_f32(act_load(h + (size_t)t * ldh + k));
     int e = act_load(ids + row);
-    e = e < 0 ? 0 : (e >= X ? X - 1 : e);
+    if (e < 0) return;                          // a slot without an expert
+    e = e >= X ? X - 1 : e;
     __syncthreads();
     const int f0 = (blockIdx.y * GU_WARPS + warp) * GU_PER_WARP;
     if (f0 >= F) return;
@@ -198,16 +226,17 @@ __global__ void __launch_bounds__(GU_WARPS * 32) moe_gate_up_kernel(const T *__r
 // out[t, j] = sum_s wts[t, s] (Wd[ids[t, s]] act[t top + s])[j], float32; the chosen experts in their order.  A warp takes
 // DN_PER_WARP outputs at once.
 constexpr int DN_WARPS = 4, DN_PER_WARP = 4;
-template <typename T>
+template <typename T, typename TA>
 __global__ void __launch_bounds__(DN_WARPS * 32) moe_down_kernel(const T *__restrict__ act, const int *__restrict__ ids, const float *__restrict__ wts,
                                                                  const T *__restrict__ wd, float *__restrict__ out, int E, int F, int X, int top,
-                                                                 const float *__restrict__ also, const float *__restrict__ also_w) {
+                                                                 const TA *__restrict__ also, int lda, const float *__restrict__ also_w) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float as[];       // top rows of F
     const int t = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int k = threadIdx.x; k < top * F; k += blockDim.x) as[k] = to_f32(act_load(act + (size_t)t * top * F + k));
+    for (int k = threadIdx.x; k < top * F; k += blockDim.x)
+        as[k] = act_load(ids + (size_t)t * top + k / F) >= 0 ? to_f32(act_load(act + (size_t)t * top * F + k)) : 0.f;
     __syncthreads();
     const int j0 = (blockIdx.y * DN_WARPS + warp) * DN_PER_WARP;
     if (j0 >= E) return;
@@ -217,7 +246,8 @@ __global__ void __launch_bounds__(DN_WARPS * 32) moe_down_kernel(const T *__rest
     for (int i = 0; i < DN_PER_WARP; ++i) total[i] = 0.f;
     for (int s = 0; s < top; ++s) {
         int e = act_load(ids + (size_t)t * top + s);
-        e = e < 0 ? 0 : (e >= X ? X - 1 : e);
+        if (e < 0) continue;                    // a slot without an expert
+        e = e >= X ? X - 1 : e;
         const float w = act_load(wts + (size_t)t * top + s);
         float r[DN_PER_WARP];
         if (vec) {
@@ -243,7 +273,7 @@ __global__ void __launch_bounds__(DN_WARPS * 32) moe_down_kernel(const T *__rest
         for (int i = 0; i < DN_PER_WARP; ++i)
             if (j0 + i < E) {
                 float v = total[i];
-                if (also) v = fmaf(act_load(also_w + t), act_load(also + (size_t)t * E + j0 + i), v);
+                if (also) v = fmaf(act_load(also_w + t), to_f32(act_load(also + (size_t)t * lda + j0 + i)), v);
                 out[(size_t)t * E + j0 + i] = v;
             }
 }
@@ -262,24 +292,34 @@ static int need_smem(K kernel, size_t smem, const char *who) {
 //   mode 0: the chosen by the largest logits + br, weights = softmax over the chosen logits
 //   mode 1: scores = sigmoid(logits), the chosen by the largest score + br, weights = score / (sum of the chosen scores + 1e-20) * route_scale
 //   wr holds n_extra more rows behind the experts': extra[n, n_extra] = sigmoid of their logits
-LGML_API int lgml_moe_router_mode(const void *h, int dtype, int ldh, const float *wr, const float *br, int *ids, float *wts, int n_tokens, int E, int X,
-                                  int top, int mode, float route_scale, int n_extra, float *extra, cudaStream_t stream) {
+//   mode 2: scores = softmax over all X logits, the chosen by the largest score + br, weights = their scores
+//   n_identity: the last n_identity of the X rows are experts without matrices: a slot that chose one holds -1, and identity_w[n]
+//   (or null) gets the sum of their weights
+LGML_API int lgml_moe_router_form(const void *h, int dtype, int ldh, const float *wr, const float *br, int *ids, float *wts, int n_tokens, int E, int X,
+                                  int top, int mode, float route_scale, int n_extra, float *extra, int n_identity, float *identity_w, cudaStream_t stream) {
     LGML_REQUIRE(n_tokens >= 0 && E > 0 && X > 0 && top > 0 && top <= X, "moe_router: bad sizes (%d experts, %d chosen)", X, top);
     LGML_REQUIRE(X <= 8192, "moe_router: at most 8192 experts");
-    LGML_REQUIRE(mode == 0 || mode == 1, "moe_router: unknown mode %d", mode);
+    LGML_REQUIRE(mode >= 0 && mode <= 2, "moe_router: unknown mode %d", mode);
     LGML_REQUIRE(n_extra >= 0 && n_extra <= 64 && (n_extra == 0 || extra != nullptr), "moe_router: bad extra rows");
+    LGML_REQUIRE(n_identity >= 0 && n_identity <= X, "moe_router: bad identity experts");
     if (n_tokens == 0) return 0;
     const size_t smem = sizeof(float) * (2 * (size_t)((X + n_extra + 3) & ~3) + (size_t)E);
     LGML_REQUIRE(smem <= 200 * 1024, "moe_router: %d experts and rows of %d do not fit shared memory", X, E);
     if (need_smem(moe_router_kernel<float>, smem, "moe_router") || need_smem(moe_router_kernel<__nv_bfloat16>, smem, "moe_router")) return -1;
     if (dtype == LGML_F32)
-        lgml_launch(moe_router_kernel<float>, n_tokens, 128, smem, stream, (const float *)h, ldh, wr, br, ids, wts, E, X, top, mode, route_scale, n_extra, extra);
+        lgml_launch(moe_router_kernel<float>, n_tokens, 128, smem, stream, (const float *)h, ldh, wr, br, ids, wts, E, X, top, mode, route_scale, n_extra, extra,
+                    n_identity, identity_w);
     else if (dtype == LGML_BF16)
         lgml_launch(moe_router_kernel<__nv_bfloat16>, n_tokens, 128, smem, stream, (const __nv_bfloat16 *)h, ldh, wr, br, ids, wts, E, X, top, mode,
-                    route_scale, n_extra, extra);
+                    route_scale, n_extra, extra, n_identity, identity_w);
     else
         LGML_FAIL("moe_router: unknown type %d", dtype);
     return lgml_launch_status("moe_router");
+}
+
+LGML_API int lgml_moe_router_mode(const void *h, int dtype, int ldh, const float *wr, const float *br, int *ids, float *wts, int n_tokens, int E, int X,
+                                  int top, int mode, float route_scale, int n_extra, float *extra, cudaStream_t stream) {
+    return lgml_moe_router_form(h, dtype, ldh, wr, br, ids, wts, n_tokens, E, X, top, mode, route_scale, n_extra, extra, 0, nullptr, stream);
 }
 
 LGML_API int lgml_moe_router(const void *h, int dtype, int ldh, const float *wr, const float *br, int *ids, float *wts, int n_tokens, int E, int X,
@@ -288,10 +328,11 @@ LGML_API int lgml_moe_router(const void *h, int dtype, int ldh, const float *wr,
 }
 
 // The row form: act [n top, F] in the compute type (scratch of the caller), out float32 [n, E].
-// plain = 1: experts without a gate (wgu is [X, F, E], act = relu(W_up h)^2).  also / also_w: float32 [n, E] and [n], out += also_w[t] also[t] (or null).
+// plain = 1: experts without a gate (wgu is [X, F, E], act = relu(W_up h)^2).  also / also_w: rows of E entries, lda apart, float32 or (also_own = 1) in the
+// compute type, and float32 [n]: out += also_w[t] also[t] (or null).
 LGML_API int lgml_moe_experts_rows_form(const void *h, int dtype, int ldh, const int *ids, const float *wts, const void *wgu, const void *wd,
-                                        void *act, float *out, int n_tokens, int E, int F, int X, int top, int plain, const float *also,
-                                        const float *also_w, cudaStream_t stream) {
+                                        void *act, float *out, int n_tokens, int E, int F, int X, int top, int plain, const void *also,
+                                        int also_own, int lda, const float *also_w, cudaStream_t stream) {
     LGML_REQUIRE(n_tokens >= 0 && E > 0 && F > 0 && X > 0 && top > 0, "moe_experts_rows: bad sizes");
     if (n_tokens == 0) return 0;
     const size_t smem_gu = sizeof(float) * (size_t)E, smem_dn = sizeof(float) * (size_t)top * F;
@@ -299,19 +340,24 @@ LGML_API int lgml_moe_experts_rows_form(const void *h, int dtype, int ldh, const
     dim3 grid_gu(n_tokens * top, (F + GU_WARPS * GU_PER_WARP - 1) / (GU_WARPS * GU_PER_WARP));
     dim3 grid_dn(n_tokens, (E + DN_WARPS * DN_PER_WARP - 1) / (DN_WARPS * DN_PER_WARP));
     if (dtype == LGML_F32) {
-        if (need_smem(moe_gate_up_kernel<float>, smem_gu, "moe_experts_rows") || need_smem(moe_down_kernel<float>, smem_dn, "moe_experts_rows")) return -1;
+        if (need_smem(moe_gate_up_kernel<float>, smem_gu, "moe_experts_rows") || need_smem(moe_down_kernel<float, float>, smem_dn, "moe_experts_rows")) return -1;
         lgml_launch(moe_gate_up_kernel<float>, grid_gu, GU_WARPS * 32, smem_gu, stream, (const float *)h, ldh, ids, (const float *)wgu, (float *)act, E, F, X,
                     top, plain);
-        lgml_launch(moe_down_kernel<float>, grid_dn, DN_WARPS * 32, smem_dn, stream, (const float *)act, ids, wts, (const float *)wd, out, E, F, X, top,
-                    also, also_w);
+        lgml_launch(moe_down_kernel<float, float>, grid_dn, DN_WARPS * 32, smem_dn, stream, (const float *)act, ids, wts, (const float *)wd, out, E, F, X, top,
+                    (const float *)also, lda, also_w);
     } else if (dtype == LGML_BF16) {
         if (need_smem(moe_gate_up_kernel<__nv_bfloat16>, smem_gu, "moe_experts_rows") ||
-            need_smem(moe_down_kernel<__nv_bfloat16>, smem_dn, "moe_experts_rows"))
+            need_smem(moe_down_kernel<__nv_bfloat16, float>, smem_dn, "moe_experts_rows") ||
+            need_smem(moe_down_kernel<__nv_bfloat16, __nv_bfloat16>, smem_dn, "moe_experts_rows"))
             return -1;
         lgml_launch(moe_gate_up_kernel<__nv_bfloat16>, grid_gu, GU_WARPS * 32, smem_gu, stream, (const __nv_bfloat16 *)h, ldh, ids,
                     (const __nv_bfloat16 *)wgu, (__nv_bfloat16 *)act, E, F, X, top, plain);
-        lgml_launch(moe_down_kernel<__nv_bfloat16>, grid_dn, DN_WARPS * 32, smem_dn, stream, (const __nv_bfloat16 *)act, ids, wts,
-                    (const __nv_bfloat16 *)wd, out, E, F, X, top, also, also_w);
+        if (also_own)
+            lgml_launch(moe_down_kernel<__nv_bfloat16, __nv_bfloat16>, grid_dn, DN_WARPS * 32, smem_dn, stream, (const __nv_bfloat16 *)act, ids, wts,
+                        (const __nv_bfloat16 *)wd, out, E, F, X, top, (const __nv_bfloat16 *)also, lda, also_w);
+        else
+            lgml_launch(moe_down_kernel<__nv_bfloat16, float>, grid_dn, DN_WARPS * 32, smem_dn, stream, (const __nv_bfloat16 *)act, ids, wts,
+                        (const __nv_bfloat16 *)wd, out, E, F, X, top, (const float *)also, lda, also_w);
     } else {
         LGML_FAIL("moe_experts_rows: unknown type %d", dtype);
     }
@@ -320,7 +366,7 @@ LGML_API int lgml_moe_experts_rows_form(const void *h, int dtype, int ldh, const
 
 LGML_API int lgml_moe_experts_rows(const void *h, int dtype, int ldh, const int *ids, const float *wts, const void *wgu, const void *wd,
                                    void *act, float *out, int n_tokens, int E, int F, int X, int top, cudaStream_t stream) {
-    return lgml_moe_experts_rows_form(h, dtype, ldh, ids, wts, wgu, wd, act, out, n_tokens, E, F, X, top, 0, nullptr, nullptr, stream);
+    return lgml_moe_experts_rows_form(h, dtype, ldh, ids, wts, wgu, wd, act, out, n_tokens, E, F, X, top, 0, nullptr, 0, E, nullptr, stream);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -351,7 +397,8 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int *__restrict__
     __syncthreads();
     for (int r = threadIdx.x; r < n_rows; r += blockDim.x) {
         int e = act_load(ids + r);
-        e = e < 0 ? 0 : (e >= X ? X - 1 : e);
+        if (e < 0) continue;                    // a slot without an expert is in no tile
+        e = e >= X ? X - 1 : e;
         atomicAdd(&counts[e], 1);
     }
     __syncthreads();
@@ -367,7 +414,8 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int *__restrict__
     __syncthreads();
     for (int r = threadIdx.x; r < n_rows; r += blockDim.x) {
         int e = act_load(ids + r);
-        e = e < 0 ? 0 : (e >= X ? X - 1 : e);
+        if (e < 0) continue;
+        e = e >= X ? X - 1 : e;
         rows[first[e] + atomicAdd(&cursor[e], 1)] = r;
     }
     for (int e = threadIdx.x; e < X; e += blockDim.x) {
@@ -584,25 +632,36 @@ __global__ void __launch_bounds__(128) moe_gather_rows_kernel(const __nv_bfloat1
     for (int c = threadIdx.x; c < E / 8; c += blockDim.x) dst[c] = act_load(src + c);
 }
 
-__global__ void __launch_bounds__(256) moe_weighted_sum_kernel(const float *__restrict__ y, const int *__restrict__ pos, const float *__restrict__ wts,
-                                                               float *__restrict__ out, int n_tokens, int E, int top,
-                                                               const float *__restrict__ also, const float *__restrict__ also_w) {
+__device__ __forceinline__ float4 quad_of(const float *p) { return act_load(reinterpret_cast<const float4 *>(p)); }
+__device__ __forceinline__ float4 quad_of(const __nv_bfloat16 *p) {
+    const float2 raw = act_load(reinterpret_cast<const float2 *>(p));
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
+// A slot whose id is negative holds no expert and adds nothing.
+template <typename TA>
+__global__ void __launch_bounds__(256) moe_weighted_sum_kernel(const float *__restrict__ y, const int *__restrict__ pos, const int *__restrict__ ids,
+                                                               const float *__restrict__ wts, float *__restrict__ out, int n_tokens, int E, int top,
+                                                               const TA *__restrict__ also, int lda, const float *__restrict__ also_w) {
     pdl_trigger();
     pdl_wait();
-    if (E % 4 == 0 && ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(also)) & 15) == 0) {
+    if (E % 4 == 0 && lda % 4 == 0 &&
+        ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(also)) & 15) == 0) {
         const int quads = E / 4;
         const size_t total = (size_t)n_tokens * quads;
         for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
             const size_t t = i / quads, j = (i - t * quads) * 4;
             float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
             for (int k = 0; k < top; ++k) {
+                if (ids != nullptr && act_load(ids + t * top + k) < 0) continue;
                 const float w = act_load(wts + t * top + k);
                 const float4 v = act_load(reinterpret_cast<const float4 *>(y + (size_t)act_load(pos + t * top + k) * E + j));
                 s.x = fmaf(w, v.x, s.x), s.y = fmaf(w, v.y, s.y), s.z = fmaf(w, v.z, s.z), s.w = fmaf(w, v.w, s.w);
             }
             if (also) {
                 const float w = act_load(also_w + t);
-                const float4 v = act_load(reinterpret_cast<const float4 *>(also + t * E + j));
+                const float4 v = quad_of(also + t * lda + j);
                 s.x = fmaf(w, v.x, s.x), s.y = fmaf(w, v.y, s.y), s.z = fmaf(w, v.z, s.z), s.w = fmaf(w, v.w, s.w);
             }
             *reinterpret_cast<float4 *>(out + t * E + j) = s;
@@ -613,8 +672,9 @@ __global__ void __launch_bounds__(256) moe_weighted_sum_kernel(const float *__re
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
         const size_t t = i / E, j = i - t * E;
         float s = 0.f;
-        for (int k = 0; k < top; ++k) s = fmaf(act_load(wts + t * top + k), act_load(y + (size_t)act_load(pos + t * top + k) * E + j), s);
-        if (also) s = fmaf(act_load(also_w + t), act_load(also + i), s);
+        for (int k = 0; k < top; ++k)
+            if (ids == nullptr || act_load(ids + t * top + k) >= 0) s = fmaf(act_load(wts + t * top + k), act_load(y + (size_t)act_load(pos + t * top + k) * E + j), s);
+        if (also) s = fmaf(act_load(also_w + t), to_f32(act_load(also + t * lda + j)), s);
         out[i] = s;
     }
 }
@@ -642,16 +702,20 @@ LGML_API int lgml_moe_gather_rows(const void *h, int ldh, const int *rows, const
     return lgml_launch_status("moe_gather_rows");
 }
 
-LGML_API int lgml_moe_weighted_sum_also(const float *y, const int *pos, const float *wts, float *out, int n_tokens, int E, int top, const float *also,
-                                        const float *also_w, cudaStream_t stream) {
-    LGML_REQUIRE(n_tokens >= 0 && E > 0 && top > 0, "moe_weighted_sum: bad sizes");
+// ids int32 [n top] or null (every slot holds an expert); also: rows of E entries, lda apart, float32 or (also_bf16 = 1) bfloat16, or null
+LGML_API int lgml_moe_weighted_sum_form(const float *y, const int *pos, const int *ids, const float *wts, float *out, int n_tokens, int E, int top,
+                                        const void *also, int also_bf16, int lda, const float *also_w, cudaStream_t stream) {
+    LGML_REQUIRE(n_tokens >= 0 && E > 0 && top > 0 && (also == nullptr || (also_w != nullptr && lda >= E)), "moe_weighted_sum: bad sizes");
     if (n_tokens == 0) return 0;
     const size_t total = (size_t)n_tokens * E;
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
-    lgml_launch(moe_weighted_sum_kernel, blocks, 256, 0, stream, y, pos, wts, out, n_tokens, E, top, also, also_w);
+    if (also_bf16)
+        lgml_launch(moe_weighted_sum_kernel<__nv_bfloat16>, blocks, 256, 0, stream, y, pos, ids, wts, out, n_tokens, E, top, (const __nv_bfloat16 *)also, lda, also_w);
+    else
+        lgml_launch(moe_weighted_sum_kernel<float>, blocks, 256, 0, stream, y, pos, ids, wts, out, n_tokens, E, top, (const float *)also, lda, also_w);
     return lgml_launch_status("moe_weighted_sum");
 }
 
 LGML_API int lgml_moe_weighted_sum(const float *y, const int *pos, const float *wts, float *out, int n_tokens, int E, int top, cudaStream_t stream) {
-    return lgml_moe_weighted_sum_also(y, pos, wts, out, n_tokens, E, top, nullptr, nullptr, stream);
+    return lgml_moe_weighted_sum_form(y, pos, nullptr, wts, out, n_tokens, E, top, nullptr, 0, E, nullptr, stream);
 }

@@ -464,6 +464,96 @@ __global__ void __launch_bounds__(ITEMS) conv_rope_store_kernel(
     }
     }
 }
+// ---------------------------------------------------------------------------------------------
+// norm_rope_store: q and k are normed head by head (over the root mean square of the head's D entries, times a weight of
+// size D shared by the heads; weight null: no norm), then turn by their positions (pairs (i, i + n_rot / 2) of the first
+// n_rot entries); k and v (times v_scale) go to their cells, q to its buffer.
+//   proj float32 [n, ldp]: q at column 0 (H D), k behind it (G D), v behind that (G Dv).
+// Block: a token and a share of its heads; a warp takes one head at a time through a row of shared memory.  The cosines
+// and sines of the token's position are computed once per block.
+constexpr int NRS_WARPS = 4;
+
+template <typename T, int V>
+__global__ void __launch_bounds__(NRS_WARPS * 32) norm_rope_store_kernel(
+    const float *__restrict__ proj, int ldp, const float *__restrict__ q_w, const float *__restrict__ k_w, float eps, T *__restrict__ q_out, int ldq,
+    const int *__restrict__ positions, const int *__restrict__ seq_of_token, const int *__restrict__ block_table, int max_blocks,
+    const float *__restrict__ inv_freq, const float *__restrict__ inv_freq_lo, int n_rot, T *__restrict__ k_pages, T *__restrict__ v_pages, int n_pages,
+    int page_size, int H, int G, int D, int Dv, float v_scale, int write_kv, int *__restrict__ status) {
+    pdl_trigger();
+    pdl_wait();
+    using X = CrsVec<V>;
+    extern __shared__ __align__(16) float nrs[];
+    const int half = n_rot / 2, DS = (max(D, Dv) + 3) & ~3;
+    float *cosv = nrs, *sinv = nrs + half, *rows = nrs + ((n_rot + 3) & ~3);
+    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int pos = positions[t];
+    for (int i = threadIdx.x; i < half; i += NRS_WARPS * 32) rope_sincos(pos, inv_freq[i], inv_freq_lo ? inv_freq_lo[i] : 0.f, sinv + i, cosv + i);
+    int page = -1;
+    if (write_kv) {
+        const int blk = pos / page_size;
+        if (pos >= 0 && blk < max_blocks) page = block_table[(size_t)seq_of_token[t] * max_blocks + blk];
+        if (page < 0 || page >= n_pages) {       // the host reserves pages first; never write outside the pool
+            if (threadIdx.x == 0 && blockIdx.y == 0) atomicExch(status, 2);
+            page = -1;
+        }
+    }
+    __syncthreads();
+    float *buf = rows + (size_t)warp * DS;
+    const float *row = proj + (size_t)t * ldp;
+    const int n_heads = write_kv ? H + 2 * G : H;
+    for (int head = blockIdx.y * NRS_WARPS + warp; head < n_heads; head += gridDim.y * NRS_WARPS) {
+        const size_t cell_row = (size_t)(pos % page_size);
+        if (head >= H + G) {
+            if (page < 0) continue;
+            const int g = head - H - G;
+            const float *src = row + (size_t)(H + G) * D + (size_t)g * Dv;
+            T *dst = v_pages + (((size_t)page * G + g) * page_size + cell_row) * Dv;
+            for (int d = lane * V; d < Dv; d += 32 * V) {
+                float v[V];
+                X::load(src + d, v);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] *= v_scale;
+                X::store(dst + d, v);
+            }
+            continue;
+        }
+        const bool is_q = head < H;
+        const float *w = is_q ? q_w : k_w, *src = row + (size_t)head * D;
+        float ss = 0.f;
+        for (int d = lane * V; d < D; d += 32 * V) {
+            float v[V];
+            X::load(src + d, v);
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss = fmaf(v[e], v[e], ss), buf[d + e] = v[e];
+        }
+        float inv = 1.f;
+        if (w != nullptr) {
+            inv = 1.0f / sqrtf(warp_sum(ss) / (float)D + eps);
+            for (int d = lane * V; d < D; d += 32 * V) {
+                float g[V];
+                X::load_w(w + d, g);
+#pragma unroll
+                for (int e = 0; e < V; ++e) buf[d + e] = buf[d + e] * inv * g[e];
+            }
+        }
+        __syncwarp();
+        T *dst = is_q ? q_out + (size_t)t * ldq + (size_t)head * D
+                      : (page >= 0 ? k_pages + (((size_t)page * G + (head - H)) * page_size + cell_row) * D : nullptr);
+        if (dst != nullptr)
+            for (int d = lane * V; d < D; d += 32 * V) {
+                float y[V];
+#pragma unroll
+                for (int e = 0; e < V; ++e) {
+                    const int i = d + e;
+                    y[e] = buf[i];
+                    if (i < half) y[e] = buf[i] * cosv[i] - buf[i + half] * sinv[i];
+                    else if (i < n_rot) y[e] = buf[i] * cosv[i - half] + buf[i - half] * sinv[i - half];
+                }
+                X::store(dst + d, y);
+            }
+        __syncwarp();
+    }
+}
 }  // namespace
 
 // src: [n_parts][n_tokens][(H + 2 Hkv) D] of src_dtype (row stride lds, part_stride elements between
@@ -531,4 +621,33 @@ LGML_API int lgml_conv_rope_store(const float *proj, int ldp, const float *wT, f
 #undef LGML_CRS
 #undef LGML_CRS_T
     return lgml_launch_status("conv_rope_store");
+}
+
+// The norm per head, the turn and the cache write; see the kernel.  q_w / k_w: float32 [D] or null.
+LGML_API int lgml_norm_rope_store(const float *proj, int ldp, const float *q_w, const float *k_w, float eps, void *q_out, int dtype, int ldq,
+                                  const int *positions, const int *seq_of_token, const int *block_table, int max_blocks, const float *inv_freq,
+                                  const float *inv_freq_lo, int n_rot, void *k_pages, void *v_pages, int n_pages, int page_size, int n_tokens, int H, int G,
+                                  int D, int Dv, float v_scale, int write_kv, int *status, cudaStream_t stream) {
+    LGML_REQUIRE(n_tokens >= 0 && H > 0 && G > 0 && D > 0 && Dv > 0 && page_size > 0 && max_blocks > 0, "norm_rope_store: bad sizes");
+    LGML_REQUIRE(n_rot >= 0 && n_rot <= D && n_rot % 2 == 0, "norm_rope_store: n_rot %d must be even and at most the head size %d", n_rot, D);
+    LGML_REQUIRE(ldp >= (H + G) * D + G * Dv && ldq >= H * D, "norm_rope_store: rows too short");
+    if (n_tokens == 0) return 0;
+    const int DS = ((D > Dv ? D : Dv) + 3) & ~3;
+    const size_t smem = sizeof(float) * (size_t)(((n_rot + 3) & ~3) + NRS_WARPS * DS);
+    LGML_REQUIRE(smem <= 48 * 1024, "norm_rope_store: heads of %d and %d do not fit shared memory", D, Dv);
+    const bool vec = D % 4 == 0 && Dv % 4 == 0 && ldp % 4 == 0 && ldq % 4 == 0 &&
+                     ((((uintptr_t)proj | (uintptr_t)q_w | (uintptr_t)k_w | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages) & 15) == 0);
+    // a token's heads go over several blocks while tokens alone do not fill the SMs
+    const int n_heads = write_kv ? H + 2 * G : H;
+    int splits = (n_heads + NRS_WARPS - 1) / NRS_WARPS;
+    while (splits > 1 && (long long)n_tokens * splits > 148 * 16) splits = (splits + 1) / 2;
+    dim3 grid(n_tokens, splits);
+#define LGML_NRS(T, V) lgml_launch(norm_rope_store_kernel<T, V>, grid, NRS_WARPS * 32, smem, stream, proj, ldp, q_w, k_w, eps, (T *)q_out, ldq, positions, \
+                                   seq_of_token, block_table, max_blocks, inv_freq, inv_freq_lo, n_rot, (T *)k_pages, (T *)v_pages, n_pages, page_size, H, G, \
+                                   D, Dv, v_scale, write_kv, status)
+    if (dtype == LGML_F32) { if (vec) LGML_NRS(float, 4); else LGML_NRS(float, 1); }
+    else if (dtype == LGML_BF16) { if (vec) LGML_NRS(__nv_bfloat16, 4); else LGML_NRS(__nv_bfloat16, 1); }
+    else LGML_FAIL("norm_rope_store: unknown type %d", dtype);
+#undef LGML_NRS
+    return lgml_launch_status("norm_rope_store");
 }

@@ -4,7 +4,9 @@
 //   S_t  = exp(-exp(A_log_h) dt_t) S_(t-1) + dt_t B_t x_t^T      S is [N, P] per head; B, C are shared by the heads of a group
 //   y_t  = S_t^T C_t + D_h x_t
 //
-//   ssd_scan       the recurrence over a step's tokens, request by request, S in the request's state slot
+//   ssd_scan       the recurrence over a step's tokens, request by request, S in the request's state slot; the same kernel
+//                  runs S_t = a_t S_(t-1) + b_t B_t x_t^T with decays a and write weights b given per (token, head), with
+//                  one column more than x has whose x is 1 (the sum of the written B, a normaliser) if asked for
 //   ssd_gate_norm  (y silu(z)) over the root mean square of each of `groups` equal parts, times a weight
 //
 // Everything is float32 arithmetic in both compute types.  The state of a head is stored column by
@@ -30,13 +32,16 @@ __device__ __forceinline__ float silu_(float v) { return v / (1.0f + expf(-v)); 
 // read neighbouring 16-byte pieces of B and C from shared memory (no bank is asked twice) and of the state from memory.
 // The step's tokens come through shared memory in groups of TT: B, C (rows of NS = LN RN floats, zeros behind N),
 // the tile's x, dt and the decay.
-template <int RN, int CQ>
+// GIVEN: dt_raw holds the write weights themselves and a_given the decays (row stride ldd too); no skip term.  x has Px
+// columns per head; columns Px .. P - 1 of the state are written with x = 1.
+template <int RN, int CQ, bool GIVEN>
 __global__ void __launch_bounds__(SCAN_THREADS) ssd_scan_kernel(const float *__restrict__ xbc, int ldx, const float *__restrict__ dt_raw, int ldd,
                                                                 const float *__restrict__ dt_bias, const float *__restrict__ a_log,
                                                                 const float *__restrict__ d_skip, float *__restrict__ state, long long state_ld,
                                                                 const int *__restrict__ seq_start, const int *__restrict__ slots,
                                                                 float *__restrict__ y, int ldy, int Hs, int G, int P, int N, int LN, int TT,
-                                                                int pieces, int zero_start, float *__restrict__ decay_out, int vec) {
+                                                                int pieces, int zero_start, float *__restrict__ decay_out, int vec,
+                                                                const float *__restrict__ a_given, int Px) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float sm[];
@@ -49,8 +54,8 @@ __global__ void __launch_bounds__(SCAN_THREADS) ssd_scan_kernel(const float *__r
     auto n_of = [&](int i) { return ((i >> 2) * LN + ln) * 4 + (i & 3); };      // the state entry behind this lane's i-th register
     // pieces: the step's tokens in pieces of consecutive tokens, rows (first, past the last) of an [n, 2] table
     const int t0 = pieces ? seq_start[2 * s] : seq_start[s], t1 = pieces ? seq_start[2 * s + 1] : seq_start[s + 1];
-    const int x_cols = Hs * P;
-    const float a = expf(__ldg(a_log + h)), bias = __ldg(dt_bias + h), dsk = __ldg(d_skip + h);
+    const int x_cols = Hs * Px;
+    const float a = GIVEN ? 0.f : expf(__ldg(a_log + h)), bias = GIVEN ? 0.f : __ldg(dt_bias + h), dsk = GIVEN ? 0.f : __ldg(d_skip + h);
     float *st = state + (size_t)(slots ? slots[s] : s) * state_ld + (size_t)h * P * N;
     float S[CQ][RN];
 #pragma unroll
@@ -97,12 +102,13 @@ __global__ void __launch_bounds__(SCAN_THREADS) ssd_scan_kernel(const float *__r
         for (int i = tid; i < nt * CPB; i += SCAN_THREADS) {
             const int k = i / CPB, c = i - k * CPB;
             const int pc = blockIdx.x * CPB + c;
-            xs[k * CPB + c] = pc < P ? act_load(xbc + (size_t)(tb + k) * ldx + (size_t)h * P + pc) : 0.f;
+            xs[k * CPB + c] = pc < Px ? act_load(xbc + (size_t)(tb + k) * ldx + (size_t)h * Px + pc) : (GIVEN && pc < P ? 1.f : 0.f);
         }
         for (int k = tid; k < nt; k += SCAN_THREADS) {
-            const float dt = softplus_(act_load(dt_raw + (size_t)(tb + k) * ldd + h) + bias);
+            const float raw = act_load(dt_raw + (size_t)(tb + k) * ldd + h);
+            const float dt = GIVEN ? raw : softplus_(raw + bias);
             dts[k] = dt;
-            dAs[k] = expf(-a * dt);
+            dAs[k] = GIVEN ? act_load(a_given + (size_t)(tb + k) * ldd + h) : expf(-a * dt);
         }
         __syncthreads();
         for (int k = 0; k < nt; ++k) {
@@ -208,14 +214,15 @@ __global__ void __launch_bounds__(NT) ssd_gate_norm_kernel(const float *__restri
 
 }  // namespace
 
-LGML_API int lgml_ssd_scan(const float *xbc, int ldx, const float *dt_raw, int ldd, const float *dt_bias, const float *a_log, const float *d_skip,
+namespace {
+int scan_any(const float *xbc, int ldx, const float *dt_raw, int ldd, const float *dt_bias, const float *a_log, const float *d_skip,
                            float *state, long long state_ld, const int *seq_start, const int *slots, float *y, int ldy, int n_seqs, int Hs, int G,
-                           int P, int N, int pieces, int zero_start, float *decay_out, cudaStream_t stream) {
-    LGML_REQUIRE(n_seqs >= 0 && Hs > 0 && G > 0 && P > 0 && N > 0, "ssd_scan: bad sizes");
+                           int P, int N, int pieces, int zero_start, float *decay_out, const float *a_given, int Px, cudaStream_t stream) {
+    LGML_REQUIRE(n_seqs >= 0 && Hs > 0 && G > 0 && P > 0 && N > 0 && Px > 0 && Px <= P, "ssd_scan: bad sizes");
     LGML_REQUIRE(Hs % G == 0, "ssd_scan: %d heads are no multiple of %d groups", Hs, G);
     LGML_REQUIRE(N <= 1024, "ssd_scan: a state of %d numbers per column is more than 1024", N);
     LGML_REQUIRE(state_ld >= (long long)Hs * P * N, "ssd_scan: the state's rows do not hold %d x %d x %d floats", Hs, P, N);
-    LGML_REQUIRE(ldx >= Hs * P + 2 * G * N && ldd >= Hs && ldy >= Hs * P, "ssd_scan: rows too short");
+    LGML_REQUIRE(ldx >= Hs * Px + 2 * G * N && ldd >= Hs && ldy >= Hs * P, "ssd_scan: rows too short");
     LGML_REQUIRE(n_seqs <= 65535 && Hs <= 65535, "ssd_scan: too many requests, pieces or heads");
     LGML_REQUIRE(slots != nullptr || pieces, "ssd_scan: requests come with their slots");
     if (n_seqs == 0) return 0;
@@ -238,9 +245,10 @@ LGML_API int lgml_ssd_scan(const float *xbc, int ldx, const float *dt_raw, int l
     while (TT > 1 && (size_t)TT * (2 * NS + CPB + 2) * sizeof(float) > 46 * 1024) TT /= 2;
     const size_t smem = (size_t)TT * (2 * NS + CPB + 2) * sizeof(float);
     dim3 grid((P + CPB - 1) / CPB, Hs, n_seqs);
-    const int vec = N % 4 == 0 && ldx % 4 == 0 && (Hs * P) % 4 == 0 && ((uintptr_t)xbc & 15) == 0;
-#define LGML_SCAN(RN, CQ) lgml_launch(ssd_scan_kernel<RN, CQ>, grid, SCAN_THREADS, smem, stream, xbc, ldx, dt_raw, ldd, dt_bias, a_log, d_skip, state, \
-                                      state_ld, seq_start, slots, y, ldy, Hs, G, P, N, LN, TT, pieces, zero_start, decay_out, vec)
+    const int vec = N % 4 == 0 && ldx % 4 == 0 && (Hs * Px) % 4 == 0 && ((uintptr_t)xbc & 15) == 0;
+#define LGML_SCAN_K(RN, CQ, GIVEN) lgml_launch(ssd_scan_kernel<RN, CQ, GIVEN>, grid, SCAN_THREADS, smem, stream, xbc, ldx, dt_raw, ldd, dt_bias, a_log, d_skip, \
+                                               state, state_ld, seq_start, slots, y, ldy, Hs, G, P, N, LN, TT, pieces, zero_start, decay_out, vec, a_given, Px)
+#define LGML_SCAN(RN, CQ) do { if (a_given != nullptr) LGML_SCAN_K(RN, CQ, true); else LGML_SCAN_K(RN, CQ, false); } while (0)
     if (quad) {
         switch (best_rn) {
             case 4: LGML_SCAN(4, 4); break;
@@ -258,7 +266,26 @@ LGML_API int lgml_ssd_scan(const float *xbc, int ldx, const float *dt_raw, int l
         }
     }
 #undef LGML_SCAN
+#undef LGML_SCAN_K
     return lgml_launch_status("ssd_scan");
+}
+}  // namespace
+
+LGML_API int lgml_ssd_scan(const float *xbc, int ldx, const float *dt_raw, int ldd, const float *dt_bias, const float *a_log, const float *d_skip,
+                           float *state, long long state_ld, const int *seq_start, const int *slots, float *y, int ldy, int n_seqs, int Hs, int G,
+                           int P, int N, int pieces, int zero_start, float *decay_out, cudaStream_t stream) {
+    return scan_any(xbc, ldx, dt_raw, ldd, dt_bias, a_log, d_skip, state, state_ld, seq_start, slots, y, ldy, n_seqs, Hs, G, P, N, pieces, zero_start,
+                    decay_out, nullptr, P, stream);
+}
+
+// The recurrence with decays and write weights given: decay / weight float32 rows of Hs entries, ldd apart.  x has Px columns per head,
+// the state and y have P >= Px; columns from Px on are written with x = 1.
+LGML_API int lgml_ssd_scan_given(const float *xbc, int ldx, const float *weight, const float *decay, int ldd, float *state, long long state_ld,
+                                 const int *seq_start, const int *slots, float *y, int ldy, int n_seqs, int Hs, int G, int Px, int P, int N, int pieces,
+                                 int zero_start, float *decay_out, cudaStream_t stream) {
+    LGML_REQUIRE(decay != nullptr && weight != nullptr, "ssd_scan: decays and write weights are missing");
+    return scan_any(xbc, ldx, weight, ldd, nullptr, nullptr, nullptr, state, state_ld, seq_start, slots, y, ldy, n_seqs, Hs, G, P, N, pieces, zero_start,
+                    decay_out, decay, Px, stream);
 }
 
 LGML_API int lgml_ssd_gate_norm(const float *y, int ldy, const float *z, int ldz, const float *w, void *out, int out_dtype, int ldo, int n_tokens,

@@ -6,6 +6,7 @@ from . import lefulorn  # noqa: F401  (registers Lefulorn)
 from . import gotulorn  # noqa: F401  (registers Gotulorn)
 from . import konovik  # noqa: F401  (registers Konovik)
 from . import dizepel  # noqa: F401  (registers Dizepel)
+from . import tedisun  # noqa: F401  (registers Tedisun)
 
 
 def build_model(config):

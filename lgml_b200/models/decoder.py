@@ -21,6 +21,7 @@ import torch
 
 from .. import ops
 from ..parts.norm import PendingDelta, UnitMix
+from ..parts.streams import PendingStreams
 from ..weights import VECTOR, TensorSpec
 
 
@@ -37,8 +38,10 @@ class DecoderModel:
                  block_prefix: str = "model.layers.{}", final_norm_prefix: str = "model.norm",
                  embed_scale: Optional[float] = None, logit_scale: Optional[float] = None, logit_softcap: Optional[float] = None,
                  ignored_tensors: Sequence[str] = (), embed_norm=None, embed_norm_prefix: str = "model.embed_norm",
-                 delta_dtype: Optional[torch.dtype] = None, pass_rows: Optional[str] = None):
+                 delta_dtype: Optional[torch.dtype] = None, pass_rows: Optional[str] = None, streams: int = 0):
         self.config = config
+        # the residual in this many streams (``parts/streams.py``; the blocks and the final norm are made for them); 0: one x
+        self.streams = int(streams)
         # the type in which mixers and feed-forwards hand their results to the residual stream (None: the compute type)
         self.delta_dtype = delta_dtype
         # the name of a tensor [rows, width] whose rows schedule entries add to x (``LayerCall.add_row``)
@@ -68,6 +71,8 @@ class DecoderModel:
                     raise ValueError(f"schedule entry {ci} reads the cache of entry {call.cache}, which has none of its own")
             if call.add_row is not None and pass_rows is None:
                 raise ValueError(f"schedule entry {ci} adds a pass vector, but the model names no table of them")
+            if self.streams and (call.add_row is not None or call.add_input):
+                raise ValueError(f"schedule entry {ci} adds a row to x, which is {self.streams} streams")
         self.n_pass_rows = 1 + max((call.add_row for call in self.schedule if call.add_row is not None), default=-1)
         self.vocab_size = head.vocab
         parts = [embedding, final_norm, head] + self.blocks + ([embed_norm] if embed_norm is not None else [])
@@ -139,13 +144,16 @@ class DecoderModel:
     def forward(self, rt, batch) -> torch.Tensor:
         """float32 logits [len(batch.logit_rows), vocab] for the tokens of ``batch``."""
         x = self.embedding.forward(rt, batch.token_ids)
-        if self.embed_scale is not None:
+        if self.embed_scale is not None and not (self.streams and self.embed_norm is None):
             ops.scale_cap(x, self.embed_scale)
         if self.embed_norm is not None:
             x = self.embed_norm.forward(rt, x, torch.float32)
         rt.delta_dtype = self.delta_dtype
         x_in = x.clone() if any(call.add_input for call in self.schedule) else None
         pending = None
+        if self.streams:        # the first norm's kernel makes the streams from the (scaled) rows
+            pending = PendingStreams(start=x, start_scale=self.embed_scale if self.embed_scale is not None and self.embed_norm is None else 1.0)
+            x = torch.empty((x.shape[0], self.streams, x.shape[1]), dtype=torch.float32, device=x.device)
         for ci, call in enumerate(self.schedule):
             if call.add_input:
                 if pending is not None:

@@ -828,24 +828,27 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_head_stri
 # mixture of experts
 # ----------------------------------------------------------------------------------------
 
-ROUTER_MODES = {"softmax": 0, "sigmoid": 1}
+ROUTER_MODES = {"softmax": 0, "sigmoid": 1, "softmax_all": 2}
 
 
 def moe_router(h: torch.Tensor, w_router: torch.Tensor, b_router: Optional[torch.Tensor], top: int, mode: str = "softmax",
-               route_scale: float = 1.0, n_extra: int = 0):
+               route_scale: float = 1.0, n_extra: int = 0, n_identity: int = 0):
     """The ``top`` experts with the largest float32 logits W_r h + b_r per token (ties: the lower index)
     and the softmax over those logits alone: (ids int32 [tokens, top], weights float32 [tokens, top]).
     ``mode`` "sigmoid": the scores are sigmoid(W_r h); the experts with the largest score + b_r are chosen, and
     the weights are the chosen scores over their sum (+ 1e-20), times ``route_scale``.  ``n_extra``: the last
     rows of ``w_router`` are no experts; the sigmoids of their logits come back as a third result
-    float32 [tokens, n_extra]."""
+    float32 [tokens, n_extra].  ``mode`` "softmax_all": the scores are the softmax over all logits; the experts with the
+    largest score + b_r are chosen, and the weights are their scores as they are.  ``n_identity``: the last of the experts
+    return their input; a slot that chose one holds the id -1, and the sum of their weights per token comes back as a
+    third result float32 [tokens]."""
     _need(h, "router input", ndim=2)
     _need(w_router, "router weight", torch.float32, 2)
     ldh = _rows_contiguous(h, "router input")
     n, E = h.shape
     X = w_router.shape[0] - int(n_extra)
-    if mode not in ROUTER_MODES or n_extra < 0 or X <= 0:
-        raise KernelError(f"moe_router: mode '{mode}' with {n_extra} extra rows of {w_router.shape[0]}")
+    if mode not in ROUTER_MODES or n_extra < 0 or X <= 0 or not 0 <= n_identity <= X or (n_extra and n_identity):
+        raise KernelError(f"moe_router: mode '{mode}' with {n_extra} extra rows and {n_identity} identity experts of {w_router.shape[0]}")
     if w_router.shape[1] != E or not w_router.is_contiguous() or not 0 < top <= X:
         raise KernelError(f"moe_router: weight {tuple(w_router.shape)} does not fit rows of {E}, or {top} of {X} experts")
     if b_router is not None:
@@ -855,21 +858,26 @@ def moe_router(h: torch.Tensor, w_router: torch.Tensor, b_router: Optional[torch
     ids = torch.empty((n, top), dtype=torch.int32, device=h.device)
     wts = torch.empty((n, top), dtype=torch.float32, device=h.device)
     extra = torch.empty((n, n_extra), dtype=torch.float32, device=h.device) if n_extra else None
-    fn = _fn("moe", "lgml_moe_router_mode", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
-                                             c_int, c_void_p, c_void_p], label="moe_router")
+    own = torch.empty(n, dtype=torch.float32, device=h.device) if n_identity else None
+    fn = _fn("moe", "lgml_moe_router_form", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
+                                             c_int, c_void_p, c_int, c_void_p, c_void_p], label="moe_router")
     _check("moe", fn(_ptr(h), dtype_code(h.dtype), ldh, _ptr(w_router), _ptr(b_router), _ptr(ids), _ptr(wts), n, E, X, int(top), ROUTER_MODES[mode],
-                     float(route_scale), int(n_extra), _ptr(extra), _stream()), "moe_router")
+                     float(route_scale), int(n_extra), _ptr(extra), int(n_identity), _ptr(own), _stream()), "moe_router")
+    if n_identity:
+        return ids, wts, own
     return (ids, wts, extra) if n_extra else (ids, wts)
 
 
-def _also(also, also_w, n: int, E: int, who: str):
-    """A term every token gets beside its experts' (float32 [tokens, E]) and the token's weight on it (float32 [tokens])."""
+def _also(also, also_w, n: int, E: int, dtype: torch.dtype, who: str):
+    """A term every token gets beside its experts' (float32 or the compute type, [tokens, E]) and the token's weight on it
+    (float32 [tokens]).  Returns (1 if the term is bfloat16, its row stride)."""
     if also is None:
-        return
-    _need(also, "shared term", torch.float32, 2)
+        return 0, E
+    _need(also, "shared term", ndim=2)
     _need(also_w, "shared term's weights", torch.float32)
-    if tuple(also.shape) != (n, E) or also_w.numel() != n or not also.is_contiguous() or not also_w.is_contiguous():
-        raise KernelError(f"{who}: shared term {tuple(also.shape)} with weights {tuple(also_w.shape)} does not fit [{n}, {E}]")
+    if tuple(also.shape) != (n, E) or also.dtype not in (torch.float32, dtype) or also_w.numel() != n or not also_w.is_contiguous():
+        raise KernelError(f"{who}: shared term {tuple(also.shape)} {also.dtype} with weights {tuple(also_w.shape)} does not fit [{n}, {E}]")
+    return 1 if also.dtype == torch.bfloat16 else 0, _rows_contiguous(also, "shared term")
 
 
 def _moe_shapes(h, ids, wts, w_gu, w_down, who: str, gated: bool = True):
@@ -894,17 +902,18 @@ def moe_experts_rows(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gu
     [tokens, E].  The experts' matrices stacked: ``w_gu`` [X, 2 F, E] with the gate row of a feature followed
     by its up row, ``w_down`` [X, E, F].  A block per (token, chosen expert): the form for few tokens and for
     the 32-bit path.  ``gated`` False: experts without a gate, ``w_gu`` [X, F, E] and the activation relu squared.
-    ``also`` / ``also_w``: out += also_w[t] * also[t] (a shared expert's output and the token's gate on it)."""
+    ``also`` / ``also_w``: out += also_w[t] * also[t] (a shared expert's output and the token's gate on it; the token's own row
+    and the weight of its identity experts).  A slot whose id is -1 holds no expert."""
     _need(h, "experts' input", ndim=2)
     ldh = _rows_contiguous(h, "experts' input")
     n, E, F, X, top = _moe_shapes(h, ids, wts, w_gu, w_down, "moe_experts_rows", gated)
-    _also(also, also_w, n, E, "moe_experts_rows")
+    also_own, lda = _also(also, also_w, n, E, h.dtype, "moe_experts_rows")
     act = torch.empty((n * top, F), dtype=h.dtype, device=h.device)
     out = torch.empty((n, E), dtype=torch.float32, device=h.device)
     fn = _fn("moe", "lgml_moe_experts_rows_form", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                                   c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p])
+                                                   c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p])
     _check("moe", fn(_ptr(h), dtype_code(h.dtype), ldh, _ptr(ids), _ptr(wts), _ptr(w_gu), _ptr(w_down), _ptr(act), _ptr(out), n, E, F, X,
-                     top, 0 if gated else 1, _ptr(also), _ptr(also_w), _stream()), "moe_experts_rows")
+                     top, 0 if gated else 1, _ptr(also), also_own, lda, _ptr(also_w), _stream()), "moe_experts_rows")
     return out
 
 
@@ -957,7 +966,7 @@ def moe_experts_tcgen05(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w
     _need(h, "experts' input", torch.bfloat16, 2)
     ldh = _rows_contiguous(h, "experts' input")
     n, E, F, X, top = _moe_shapes(h, ids, wts, w_gu, w_down, "moe_experts_tcgen05", gated)
-    _also(also, also_w, n, E, "moe_experts_tcgen05")
+    also_bf16, lda = _also(also, also_w, n, E, h.dtype, "moe_experts_tcgen05")
     if not moe_grouped_supports(h, w_gu, gated):
         raise KernelError("moe_experts_tcgen05: widths and row strides must be multiples of 8 and the input 16-byte aligned")
     n_rows = n * top
@@ -981,8 +990,9 @@ def moe_experts_tcgen05(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w
                               _ptr(status), stream), "gemm_tcgen05_grouped")
     _check("gemm_tcgen05", fn(_ptr(act), _ptr(w_down), _ptr(y), 1, max_tiles, E, F, X, E, _ptr(tiles), 0, _ptr(status), stream),
            "gemm_tcgen05_grouped")
-    fn = _fn("moe", "lgml_moe_weighted_sum_also", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p], label="moe_weighted_sum")
-    _check("moe", fn(_ptr(y), _ptr(pos), _ptr(wts), _ptr(out), n, E, top, _ptr(also), _ptr(also_w), stream), "moe_weighted_sum")
+    fn = _fn("moe", "lgml_moe_weighted_sum_form", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p,
+                                                   c_void_p], label="moe_weighted_sum")
+    _check("moe", fn(_ptr(y), _ptr(pos), _ptr(ids), _ptr(wts), _ptr(out), n, E, top, _ptr(also), also_bf16, lda, _ptr(also_w), stream), "moe_weighted_sum")
     return out
 
 
@@ -1352,20 +1362,26 @@ def ssd_scan(xbc: torch.Tensor, dt_raw: torch.Tensor, dt_bias: torch.Tensor, a_l
     if pieces is None:
         scan(state, ld_state, seq_start, slots, y, n_seqs, False, False, None)
         return y
+    _scan_in_pieces(scan, pieces, n_seqs, n_heads, head_dim, n_state, state, ld_state, slots, y)
+    return y
+
+
+def _scan_in_pieces(scan, pieces, n_seqs: int, n_heads: int, head_dim: int, n_state: int, state: torch.Tensor, ld_state: int, slots: torch.Tensor,
+                    y: torch.Tensor) -> None:
+    """The three launches of a recurrence whose pieces run side by side: from zero, the chain, from the true starts."""
     rows, first = pieces
     _need(rows, "pieces", torch.int32, 2)
     _need(first, "first pieces", torch.int32, 1)
     if rows.shape[1] != 2 or not rows.is_contiguous() or first.numel() != n_seqs + 1:
         raise KernelError("ssd_scan: pieces are a contiguous [n, 2] and one first piece per request and one behind")
-    n_pieces = rows.shape[0]
-    scratch = torch.empty((n_pieces, inner * n_state), dtype=torch.float32, device=xbc.device)
-    decay = torch.empty((n_pieces, n_heads), dtype=torch.float32, device=xbc.device)
-    scan(scratch, inner * n_state, rows, None, None, n_pieces, True, True, decay)
+    n_pieces, floats = rows.shape[0], n_heads * head_dim * n_state
+    scratch = torch.empty((n_pieces, floats), dtype=torch.float32, device=y.device)
+    decay = torch.empty((n_pieces, n_heads), dtype=torch.float32, device=y.device)
+    scan(scratch, floats, rows, None, None, n_pieces, True, True, decay)
     chain = _fn("ssd", "lgml_ssd_chain", [c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-    _check("ssd", chain(_ptr(scratch), inner * n_state, _ptr(decay), _ptr(state), ld_state, _ptr(first), _ptr(slots), n_seqs, n_heads, head_dim, n_state,
+    _check("ssd", chain(_ptr(scratch), floats, _ptr(decay), _ptr(state), ld_state, _ptr(first), _ptr(slots), n_seqs, n_heads, head_dim, n_state,
                         _stream()), "ssd_chain")
-    scan(scratch, inner * n_state, rows, None, y, n_pieces, True, False, None)
-    return y
+    scan(scratch, floats, rows, None, y, n_pieces, True, False, None)
 
 
 def ssd_gate_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
@@ -1385,7 +1401,213 @@ def ssd_gate_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups
     return out
 
 
+MAX_STREAMS = 8
+
+
+def stream_norm(x: torch.Tensor, eps: float, out: Optional[torch.Tensor], weight: Optional[torch.Tensor], w_in: Optional[torch.Tensor] = None,
+                start: Optional[torch.Tensor] = None, start_scale: float = 1.0, delta=None, gate: Optional[torch.Tensor] = None,
+                w_out: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None):
+    """One kernel over the rows of the float32 residual streams x [tokens, R, E]:
+
+        z   = delta [* sigmoid(gate)]                      (``delta``: float32 [tokens, E] or ``Partials``; ``gate`` before its sigmoid)
+        x_t = sum_s mix[s, t] x_s + w_out[t] z             (without ``delta`` the streams stay as they are)
+        u   = sum_s w_in[s] x_s                            (``w_in`` None: the plain sum)
+        out = u / sqrt(mean(u^2) + eps) * weight           (``weight`` None: no output)
+
+    ``start`` (float32 [tokens, E]): the streams do not exist yet, each becomes the token's row times ``start_scale``.
+    With ``rows`` (int32 on the device) only those tokens are normed and x is not written."""
+    _need(x, "residual streams", torch.float32, 3)
+    n, R, E = x.shape
+    if not x.is_contiguous() or not 1 <= R <= MAX_STREAMS:
+        raise KernelError(f"stream_norm: streams {tuple(x.shape)} must be contiguous, 1 to {MAX_STREAMS} of them")
+    for t, what, size in ((w_in, "in weights", R), (w_out, "out weights", R), (mix, "mix matrix", R * R), (weight, "norm weight", E)):
+        if t is not None:
+            _need(t, what, torch.float32)
+            if t.numel() != size or not t.is_contiguous():
+                raise KernelError(f"stream_norm: the {what} must hold {size} floats")
+    if start is not None:
+        _need(start, "first rows", torch.float32, 2)
+        if tuple(start.shape) != (n, E) or not start.is_contiguous() or delta is not None or rows is not None:
+            raise KernelError("stream_norm: the streams start from contiguous rows, for all tokens, with nothing pending")
+    d = dbias = None
+    n_parts, stride = 1, 0
+    if isinstance(delta, Partials):
+        d, dbias = delta.data, delta.bias
+        _need(d, "delta parts", torch.float32, 3)
+        n_parts, stride = d.shape[0], n * E
+        if tuple(d.shape[1:]) != (n, E) or not d.is_contiguous():
+            raise KernelError(f"stream_norm: delta parts must be contiguous [parts, {n}, {E}]")
+    elif delta is not None:
+        d = delta
+        _need(d, "delta", torch.float32, 2)
+        if tuple(d.shape) != (n, E) or not d.is_contiguous():
+            raise KernelError(f"stream_norm: the delta must be a contiguous float32 [{n}, {E}]")
+    if d is not None and (w_out is None or mix is None):
+        raise KernelError("stream_norm: a delta comes with its out weights and mix matrix")
+    ldg = 0
+    if gate is not None:
+        _need(gate, "gate", torch.float32, 2)
+        ldg = _rows_contiguous(gate, "gate")
+        if tuple(gate.shape) != (n, E):
+            raise KernelError(f"stream_norm: gate {tuple(gate.shape)} is not [{n}, {E}]")
+    n_out = n
+    if rows is not None:
+        _need(rows, "rows", torch.int32, 1)
+        n_out = rows.numel()
+    if weight is not None:
+        _need(out, "norm output", ndim=2)
+        if tuple(out.shape) != (n_out, E) or not out.is_contiguous():
+            raise KernelError(f"stream_norm: output {tuple(out.shape)} is not a contiguous [{n_out}, {E}]")
+    else:
+        out = None
+    if n_out == 0:
+        return out
+    fn = _fn("streams", "lgml_stream_norm", [c_void_p, c_void_p, c_float, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                                             c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p])
+    _check("streams", fn(_ptr(x), _ptr(start), float(start_scale), _ptr(d), n_parts, stride, _ptr(dbias), _ptr(gate), ldg, _ptr(w_out), _ptr(mix),
+                         _ptr(w_in), _ptr(weight), _ptr(rows), _ptr(out), dtype_code(out.dtype) if out is not None else F32, n_out, E, R, float(eps),
+                         _stream()), "stream_norm")
+    return out
+
+
+def norm_rope_store(proj: torch.Tensor, q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor], eps: float, positions: torch.Tensor,
+                    seq_of_token: torch.Tensor, block_table: torch.Tensor, inv_freq: torch.Tensor, n_rot: int, k_pages: torch.Tensor,
+                    v_pages: torch.Tensor, n_heads: int, status: torch.Tensor, v_scale: float = 1.0, write_kv: bool = True) -> torch.Tensor:
+    """From the float32 projection ``proj`` [tokens, q (H D) | k (G D) | v (G Dv)] (may be a column slice): q and k over the
+    root mean square of each head times ``q_w`` / ``k_w`` (float32 [D]; None: no norm), then the turn of their first ``n_rot``
+    entries (pairs (i, i + n_rot / 2), ``inv_freq`` float32 [2, n_rot / 2] as rotary parts hold it); k and v times ``v_scale``
+    go to their cells, q comes back in the cache's type [tokens, H D]."""
+    _need(proj, "projection output", torch.float32, 2)
+    ldp = _rows_contiguous(proj, "projection output")
+    _need(k_pages, "key pages", ndim=4)
+    _need(v_pages, "value pages", k_pages.dtype, 4)
+    n = proj.shape[0]
+    n_pages, G, page, D = k_pages.shape
+    Dv = v_pages.shape[3]
+    if tuple(v_pages.shape[:3]) != (n_pages, G, page) or not k_pages.is_contiguous() or not v_pages.is_contiguous():
+        raise KernelError(f"norm_rope_store: key pages {tuple(k_pages.shape)} and value pages {tuple(v_pages.shape)} do not go together")
+    if proj.shape[1] != (n_heads + G) * D + G * Dv:
+        raise KernelError(f"norm_rope_store: {proj.shape[1]} columns are not q, k and v of {n_heads} and {G} heads of {D} and {Dv}")
+    for t, what in ((positions, "positions"), (seq_of_token, "request index of tokens")):
+        _need(t, what, torch.int32, 1)
+        if t.numel() != n:
+            raise KernelError(f"norm_rope_store: one of the {what} per token")
+    _need(block_table, "block table", torch.int32, 2)
+    _need(inv_freq, "frequencies", torch.float32, 2)
+    if not block_table.is_contiguous() or inv_freq.shape[0] != 2 or inv_freq.shape[1] < n_rot // 2 or not inv_freq.is_contiguous():
+        raise KernelError("norm_rope_store: a contiguous block table and [2, n_rot / 2] frequencies")
+    for t, what in ((q_w, "query norm weight"), (k_w, "key norm weight")):
+        if t is not None:
+            _need(t, what, torch.float32, 1)
+            if t.numel() != D:
+                raise KernelError(f"norm_rope_store: the {what} must hold {D} floats")
+    q = torch.empty((n, n_heads * D), dtype=k_pages.dtype, device=proj.device)
+    fn = _fn("rope_cache", "lgml_norm_rope_store", [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
+                                                    c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                                                    c_float, c_int, c_void_p, c_void_p])
+    _check("rope_cache", fn(_ptr(proj), ldp, _ptr(q_w), _ptr(k_w), float(eps), _ptr(q), dtype_code(q.dtype), n_heads * D, _ptr(positions), _ptr(seq_of_token),
+                            _ptr(block_table), block_table.shape[1], _ptr(inv_freq[0]), _ptr(inv_freq[1]), int(n_rot), _ptr(k_pages), _ptr(v_pages), n_pages,
+                            page, n, n_heads, G, D, Dv, float(v_scale), 1 if write_kv else 0, _ptr(status), _stream()), "norm_rope_store")
+    return q
+
+
 # ----------------------------------------------------------------------------------------
+# matrix memory with exponential gates
+# ----------------------------------------------------------------------------------------
+
+def memory_gates(zi: torch.Tensor, zf: torch.Tensor, cap: float, m_state: torch.Tensor, seq_start: torch.Tensor, slots: torch.Tensor) -> torch.Tensor:
+    """From the gates' logits zi, zf float32 [tokens, H] (column slices of one projection): i = cap tanh(zi / cap), f =
+    logsigmoid(cap tanh(zf / cap)) and, request by request, m <- max(f + m, i) (``m_state`` float32 [slots, H], a column slice of
+    the state rows, holds m between steps).  Returns float32 [tokens, 3 H]: exp(f + m_before - m) | exp(i - m) | exp(-m)."""
+    _need(zi, "input gate logits", torch.float32, 2)
+    _need(zf, "forget gate logits", torch.float32, 2)
+    _need(m_state, "running maxima", torch.float32, 2)
+    n, H = zi.shape
+    ldz = _rows_contiguous(zi, "input gate logits") if n else H
+    if tuple(zf.shape) != (n, H) or (n and zf.stride(0) != ldz) or zf.stride(1) != 1 or m_state.shape[1] != H or m_state.stride(1) != 1:
+        raise KernelError(f"memory_gates: gates {tuple(zi.shape)} / {tuple(zf.shape)} and maxima {tuple(m_state.shape)} do not fit")
+    gates = torch.empty((n, 3 * H), dtype=torch.float32, device=zi.device)
+    fn = _fn("matrix_memory", "lgml_memory_gates", [c_void_p, c_void_p, c_int, c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
+    _check("matrix_memory", fn(_ptr(zi), _ptr(zf), ldz, float(cap), _ptr(m_state), m_state.stride(0), _ptr(seq_start), _ptr(slots), _ptr(gates),
+                               slots.numel(), H, _stream()), "memory_gates")
+    return gates
+
+
+def memory_output(y: torch.Tensor, gates: torch.Tensor, q_scale: float, weight: torch.Tensor, gate: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
+    """y float32 [tokens, H (P + 1)] (per head S^T q, then n . q, q not yet scaled): o = s S^T q / (max(s |n . q|, exp(-m)) + 1e-6),
+    then per head over its root mean square, times ``weight`` [H P], times sigmoid(gate); into ``out`` [tokens, H P] (dense rows)."""
+    _need(y, "read-out", torch.float32, 2)
+    _need(gates, "gates", torch.float32, 2)
+    _need(weight, "norm weight", torch.float32, 1)
+    _need(gate, "output gate", torch.float32, 2)
+    _need(out, "output", ndim=2)
+    n, H = y.shape[0], gates.shape[1] // 3
+    P = y.shape[1] // H - 1
+    ldg, ldo = _rows_contiguous(gate, "output gate"), _rows_contiguous(out, "output")
+    if y.shape[1] != H * (P + 1) or tuple(gates.shape) != (n, 3 * H) or weight.numel() != H * P or tuple(gate.shape) != (n, H * P) \
+            or tuple(out.shape) != (n, H * P) or not (y.is_contiguous() and gates.is_contiguous() and weight.is_contiguous()):
+        raise KernelError(f"memory_output: y {tuple(y.shape)}, gates {tuple(gates.shape)}, weight {tuple(weight.shape)}, out {tuple(out.shape)} do not fit")
+    fn = _fn("matrix_memory", "lgml_memory_output", [c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
+                                                     c_void_p])
+    _check("matrix_memory", fn(_ptr(y), _ptr(gates), float(q_scale), _ptr(weight), _ptr(gate), ldg, _ptr(out), dtype_code(out.dtype), ldo, n, H, P,
+                               float(eps), _stream()), "memory_output")
+    return out
+
+
+def memory_scan(vkq: torch.Tensor, gates: torch.Tensor, state: torch.Tensor, seq_start: torch.Tensor, slots: torch.Tensor, n_heads: int, head_dim: int,
+                v_head_dim: int, pieces=None) -> torch.Tensor:
+    """S <- a S + b k v^T, n <- a n + b k; y = (S^T q, n . q) per head, over each request's tokens in order.  ``vkq`` float32
+    [tokens, v (H P) | k (H N) | q (H N)] (may be a column slice); ``gates`` as ``memory_gates`` returns them; S and n ([P + 1][N] per
+    head, n the last row) live in ``state[slot]``.  Returns y float32 [tokens, H (P + 1)].  ``pieces`` as for ``ssd_scan``."""
+    _need(vkq, "values, keys and queries", torch.float32, 2)
+    _need(gates, "gates", torch.float32, 2)
+    H, N, P1 = n_heads, head_dim, v_head_dim + 1
+    n = vkq.shape[0]
+    ldx = _rows_contiguous(vkq, "values, keys and queries")
+    if vkq.shape[1] != H * (v_head_dim + 2 * N) or tuple(gates.shape) != (n, 3 * H) or not gates.is_contiguous():
+        raise KernelError(f"memory_scan: {tuple(vkq.shape)} and gates {tuple(gates.shape)} do not fit {H} heads of {N} and {v_head_dim}")
+    ld_state = _state_rows(state, H * P1 * N, "memory_scan")
+    y = torch.empty((n, H * P1), dtype=torch.float32, device=vkq.device)
+    fn = _fn("ssd", "lgml_ssd_scan_given", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                                            c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p], label="memory_scan")
+
+    def scan(st, ld, starts, slot_ids, out, count, in_pieces, from_zero, decay):
+        _check("ssd", fn(_ptr(vkq), ldx, _ptr(gates[:, H:]), _ptr(gates), 3 * H, _ptr(st), ld, _ptr(starts), _ptr(slot_ids), _ptr(out), H * P1, count, H, H,
+                         v_head_dim, P1, N, 1 if in_pieces else 0, 1 if from_zero else 0, _ptr(decay), _stream()), "memory_scan")
+
+    n_seqs = seq_start.numel() - 1
+    if pieces is None:
+        scan(state, ld_state, seq_start, slots, y, n_seqs, False, False, None)
+        return y
+    _scan_in_pieces(scan, pieces, n_seqs, H, P1, N, state, ld_state, slots, y)
+    return y
+
+
+# ----------------------------------------------------------------------------------------
+
+def delta_head_prepare(qkv: torch.Tensor, a_pre: torch.Tensor, b_pre: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, n_heads: int,
+                       n_kv_heads: int, dim: int) -> torch.Tensor:
+    """One decay per head: q and k of ``qkv`` float32 [tokens, q (G D) | k (G D) | v ...] become unit vectors in place (q also times
+    D^-1/2); returns float32 [tokens, H, 4] = (exp(-exp(A_log) softplus(a + dt_bias)), sigmoid(b), 0, 0).  a and b float32
+    [tokens, H], possibly column slices."""
+    _need(qkv, "convolved q, k, v", torch.float32, 2)
+    _need(a_pre, "decay input", torch.float32, 2)
+    _need(b_pre, "write strength input", torch.float32, 2)
+    n, C = qkv.shape
+    lda, ldb = _rows_contiguous(a_pre, "decay input"), _rows_contiguous(b_pre, "write strength input")
+    if not qkv.is_contiguous() or C < 2 * n_kv_heads * dim or tuple(a_pre.shape) != (n, n_heads) or tuple(b_pre.shape) != (n, n_heads):
+        raise KernelError("delta_head_prepare: shapes disagree")
+    for t, what in ((a_log, "decay rates"), (dt_bias, "decay bias")):
+        _need(t, what, torch.float32, 1)
+        if t.numel() != n_heads or not t.is_contiguous():
+            raise KernelError(f"delta_head_prepare: one of the {what} per head")
+    gb = torch.empty((n, n_heads, 4), dtype=torch.float32, device=qkv.device)
+    fn = _fn("delta_rule", "lgml_delta_head_prepare", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                                                       c_int, c_void_p])
+    _check("delta_rule", fn(_ptr(qkv), C, _ptr(a_pre), lda, _ptr(b_pre), ldb, _ptr(a_log), _ptr(dt_bias), _ptr(gb), n, n_heads, n_kv_heads, dim,
+                            _stream()), "delta_head_prepare")
+    return gb
+
 
 def delta_prepare(proj: torch.Tensor, a_pre: torch.Tensor, conv_w: torch.Tensor, state: torch.Tensor, conv_off: int,
                   seq_of_token: torch.Tensor, seq_start: torch.Tensor, slots: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
@@ -1430,24 +1652,29 @@ def delta_scan(qkv_c: torch.Tensor, gb: torch.Tensor, state: torch.Tensor, seq_s
     """The recurrence S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q over each request's
     tokens in order, from and into its slot of ``state`` (S of head h at floats [h D Dv, (h + 1) D Dv)).
     ``qkv_c`` [tokens, q | k | v] and ``gb`` [tokens, H, D + 4] (per head the decays, then beta) as
-    ``delta_prepare`` returns them.  Returns o float32 [tokens, H Dv]."""
+    ``delta_prepare`` returns them, or [tokens, H, 4] (one decay per head, beta, zeros) as ``delta_head_prepare`` does.
+    Returns o float32 [tokens, H Dv]."""
     n = qkv_c.shape[0]
+    head_decay = gb.dim() == 3 and gb.shape[2] == 4
     _need(qkv_c, "prepared q, k, v", torch.float32, 2)
     _need(gb, "decays and beta", torch.float32, 3)
     _need(state, "state slots", torch.float32, 2)
-    if qkv_c.shape[1] != 2 * n_kv_heads * dim + n_heads * vdim or tuple(gb.shape) != (n, n_heads, dim + 4) \
-            or state.shape[1] < n_heads * dim * vdim or not (state.is_contiguous() and qkv_c.is_contiguous() and gb.is_contiguous()):
+    if qkv_c.shape[1] != 2 * n_kv_heads * dim + n_heads * vdim or tuple(gb.shape) != (n, n_heads, 4 if head_decay else dim + 4) \
+            or state.shape[1] < n_heads * dim * vdim or state.stride(1) != 1 or not (qkv_c.is_contiguous() and gb.is_contiguous()):
         raise KernelError("delta_scan: shapes disagree")
     o = torch.empty((n, n_heads * vdim), dtype=torch.float32, device=qkv_c.device)
-    fn = _fn("delta_rule", "lgml_delta_scan", [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                               c_int, c_int, c_int, c_void_p])
+    fn = _fn("delta_rule", "lgml_delta_scan_form", [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                                    c_int, c_int, c_int, c_int, c_void_p], label="delta_scan")
     _check("delta_rule", fn(_ptr(qkv_c), _ptr(gb), _ptr(state), state.stride(0), _ptr(seq_start), _ptr(slots), _ptr(o),
-                            slots.numel(), n_heads, n_kv_heads, dim, vdim, _stream()), "delta_scan")
+                            slots.numel(), n_heads, n_kv_heads, dim, vdim, 1 if head_decay else 0, _stream()), "delta_scan")
     return o
 
 
-def delta_output(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, out_dtype: torch.dtype, n_heads: int) -> torch.Tensor:
-    """out[t, h] = o[t, h] / rms(o[t, h]) * weight * sigmoid(gate[t, h]) per head of size Dv = len(weight)."""
+def delta_output(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, out_dtype: torch.dtype, n_heads: int,
+                 act: str = "sigmoid") -> torch.Tensor:
+    """out[t, h] = o[t, h] / rms(o[t, h]) * weight * act(gate[t, h]) per head of size Dv = len(weight); ``act``: "sigmoid" or "silu"."""
+    if act not in ("sigmoid", "silu"):
+        raise KernelError(f"delta_output: unknown gate activation '{act}'")
     _need(o, "read-out", torch.float32, 2)
     _need(weight, "norm weight", torch.float32, 1)
     _need(gate, "gate", torch.float32, 2)
@@ -1456,9 +1683,10 @@ def delta_output(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps:
     if o.shape[1] != n_heads * dv or tuple(gate.shape) != (n, n_heads * dv) or not o.is_contiguous():
         raise KernelError("delta_output: shapes disagree")
     out = torch.empty((n, n_heads * dv), dtype=out_dtype, device=o.device)
-    fn = _fn("delta_rule", "lgml_delta_output", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p])
+    fn = _fn("delta_rule", "lgml_delta_output_act", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
+             label="delta_output")
     _check("delta_rule", fn(_ptr(o), _ptr(weight), _ptr(gate), ldg, _ptr(out), dtype_code(out_dtype), out.stride(0), n, n_heads, dv, float(eps),
-                            _stream()), "delta_output")
+                            1 if act == "silu" else 0, _stream()), "delta_output")
     return out
 
 

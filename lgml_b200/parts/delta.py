@@ -1,4 +1,4 @@
-"""The gated delta rule with a decay per key channel ("channel delta") as a mixer.
+"""The gated delta rule as a mixer: with a decay per key channel ("channel delta") or one per head ("head delta").
 
 Per token, from the mixer's input h (H value heads on G query/key heads; head h reads
 query/key head h // (H / G)):
@@ -9,6 +9,9 @@ query/key head h // (H / G)):
     g         = exp(-exp(A_log) * softplus(W_a2 W_a1 h + dt_bias))   one per head and key channel
     S        <- g * S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q          per head, S [D, Dv]
     out       = W_o (o / rms(o) * w_norm * sigmoid(W_g2 W_g1 h))
+
+With one decay per head, g = exp(-exp(A_log) * softplus(W_a h + dt_bias)) is one number per head, and the output
+gate is silu(W_g h) (no low-rank projections); everything else is the same.
 
 What a request carries from token to token is one float32 vector in its state slot: S of
 every head, then the last taps - 1 inputs of the convolutions.  The four wide projections of h
@@ -79,4 +82,62 @@ class ChannelDelta(Part):
         return rt.linear(y, self.wo, partials_ok=True)
 
 
+class HeadDelta(Part):
+    """One decay per head, a full-rank output gate with silu.  Every projection of h is one product (``in_rows``)."""
+
+    graph_safe = True
+
+    def __init__(self, width: int, n_heads: int, n_kv_heads: int, head_dim: int, v_head_dim: int, taps: int, eps: float):
+        if n_heads % n_kv_heads:
+            raise ValueError(f"{n_heads} heads are no multiple of {n_kv_heads} key heads")
+        if not 1 <= taps <= ops.CONV_MAX_TAPS:
+            raise ValueError(f"a convolution of {taps} taps (1 to {ops.CONV_MAX_TAPS})")
+        self.width, self.n_heads, self.n_kv_heads = width, n_heads, n_kv_heads
+        self.head_dim, self.v_head_dim, self.taps, self.eps = head_dim, v_head_dim, int(taps), float(eps)
+        self.channels = 2 * n_kv_heads * head_dim + n_heads * v_head_dim
+        self.conv_off = -(-(n_heads * head_dim * v_head_dim) // 4) * 4        # S of every head, then the convolutions' inputs (from a 16-byte boundary)
+        self.w_in = self.wo = self.conv_w = self.a_log = self.dt_bias = self.norm_w = None
+
+    def cache_spec(self):
+        return FixedState((-(-(self.conv_off + (self.taps - 1) * self.channels) // 4) * 4,), torch.float32)
+
+    def tensor_specs(self, prefix):
+        H, G, D, Dv, E = self.n_heads, self.n_kv_heads, self.head_dim, self.v_head_dim, self.width
+        conv = lambda n, c: TensorSpec(prefix + n, (c, self.taps), VECTOR, init=(0.0, 10.0))
+        return [
+            TensorSpec(prefix + ".q", (G * D, E)), conv(".q.conv", G * D), TensorSpec(prefix + ".k", (G * D, E)), conv(".k.conv", G * D),
+            TensorSpec(prefix + ".v", (H * Dv, E)), conv(".v.conv", H * Dv), TensorSpec(prefix + ".b", (H, E)), TensorSpec(prefix + ".a", (H, E)),
+            TensorSpec(prefix + ".A_log", (H,), VECTOR), TensorSpec(prefix + ".dt_bias", (H,), VECTOR),
+            TensorSpec(prefix + ".norm", (Dv,), VECTOR, init=(1.0, 1.0)), TensorSpec(prefix + ".g", (H * Dv, E)), TensorSpec(prefix + ".o", (E, H * Dv)),
+        ]
+
+    def bind(self, prefix, tensors, rt):
+        t = lambda n: tensors[prefix + n]
+        self.w_in = torch.cat([t(".q"), t(".k"), t(".v"), t(".g"), t(".b"), t(".a")], dim=0).contiguous()
+        self.conv_w = torch.cat([t(".q.conv"), t(".k.conv"), t(".v.conv")], dim=0).float().t().contiguous()      # [taps, channels]
+        self.wo = t(".o")
+        self.a_log, self.dt_bias, self.norm_w = (t(n).float().contiguous() for n in (".A_log", ".dt_bias", ".norm"))
+
+    def in_rows(self):
+        return self.w_in, None
+
+    def first_weights(self):
+        return [self.w_in]
+
+    def forward_projected(self, rt, proj, batch, cache):
+        H, G, D, Dv, C = self.n_heads, self.n_kv_heads, self.head_dim, self.v_head_dim, self.channels
+        qkv = torch.empty((proj.shape[0], C), dtype=torch.float32, device=proj.device)
+        ops.short_conv(proj[:, :C], self.conv_w, None, cache.state[:, self.conv_off:] if self.taps > 1 else None, batch.seq_of_token, batch.seq_start,
+                       batch.slots, qkv, act="silu")
+        g0, b0, a0 = C, C + H * Dv, C + H * Dv + H
+        gb = ops.delta_head_prepare(qkv, proj[:, a0:a0 + H], proj[:, b0:b0 + H], self.a_log, self.dt_bias, H, G, D)
+        o = ops.delta_scan(qkv, gb, cache.state, batch.seq_start, batch.slots, H, G, D, Dv)
+        y = ops.delta_output(o, self.norm_w, proj[:, g0:g0 + H * Dv], self.eps, rt.dtype, H, act="silu")
+        return rt.linear(y, self.wo, partials_ok=True)
+
+    def forward(self, rt, h, batch, cache):
+        return self.forward_projected(rt, rt.linear(h, self.w_in, out_dtype=torch.float32), batch, cache)
+
+
 register_part("mixer", "channel_delta", ChannelDelta)
+register_part("mixer", "head_delta", HeadDelta)

@@ -12,6 +12,9 @@ Other forms of the same part, by constructor arguments:
 
 * ``router="sigmoid"``: the scores are s = sigmoid(z); the experts with the largest s + bias are chosen (the
   bias corrects the choice only), and w = s of the chosen over their sum (+ 1e-20), times ``route_scale``;
+* ``router="softmax_all"``: the scores are s = softmax(z) over all experts; the experts with the largest s + bias are
+  chosen, and w = s of the chosen, not renormalised;
+* ``n_identity``: that many experts more, behind the others in the router's rows, that have no matrices and return h;
 * ``gated=False``: experts without a gate, W_down,e act(W_up,e h) with act = relu squared;
 * ``shared_inner``: one more expert of that inner width and the same form that every token uses
   (``.shared.up``, ``.shared.down``), added times sigmoid(W_sg h), one number per token (``.shared.sg`` [1, E]);
@@ -30,15 +33,18 @@ class RoutedExperts(Part):
     graph_safe = True
 
     def __init__(self, width: int, inner: int, n_experts: int, top: int, router_bias: bool = True, router: str = "softmax",
-                 route_scale: float = 1.0, gated: bool = True, shared_inner: int = 0, bias_name: str = ".router.b"):
-        if not 0 < top <= n_experts:
-            raise ValueError(f"{top} of {n_experts} experts cannot be chosen")
+                 route_scale: float = 1.0, gated: bool = True, shared_inner: int = 0, bias_name: str = ".router.b",
+                 n_identity: int = 0):
+        if not 0 < top <= n_experts + n_identity:
+            raise ValueError(f"{top} of {n_experts + n_identity} experts cannot be chosen")
+        if shared_inner and n_identity:
+            raise ValueError("a token gets one term beside its experts: a shared expert or identity experts")
         if router not in ops.ROUTER_MODES:
             raise ValueError(f"unknown router '{router}' (known: {', '.join(ops.ROUTER_MODES)})")
         if shared_inner and gated:
             raise ValueError("a shared expert comes only with experts without a gate")
         self.width, self.inner, self.n_experts, self.top = width, inner, n_experts, top
-        self.router_bias = bool(router_bias)
+        self.router_bias, self.n_identity = bool(router_bias), int(n_identity)
         self.router, self.route_scale, self.gated = router, float(route_scale), bool(gated)
         self.shared_inner, self.bias_name = int(shared_inner), bias_name
         self.w_router = self.b_router = self.w_gu = self.wd = self.ws_up = self.ws_down = None
@@ -46,9 +52,9 @@ class RoutedExperts(Part):
     def tensor_specs(self, prefix):
         E, F = self.width, self.inner
         # the router stays float32 (its logits decide which experts run)
-        specs = [TensorSpec(prefix + ".router", (self.n_experts, E), VECTOR)]
+        specs = [TensorSpec(prefix + ".router", (self.n_experts + self.n_identity, E), VECTOR)]
         if self.router_bias:
-            specs.append(TensorSpec(prefix + self.bias_name, (self.n_experts,), VECTOR))
+            specs.append(TensorSpec(prefix + self.bias_name, (self.n_experts + self.n_identity,), VECTOR))
         for e in range(self.n_experts):
             if self.gated:
                 specs.append(TensorSpec(f"{prefix}.e{e}.gate", (F, E)))
@@ -89,6 +95,10 @@ class RoutedExperts(Part):
             else:
                 act = ops.relu_sq(rt.linear(h, self.ws_up))
             also = rt.linear(act, self.ws_down, out_dtype=torch.float32)
+        elif self.n_identity:
+            # the experts that return their input: the token's own row, times the sum of their weights
+            ids, wts, also_w = ops.moe_router(h, self.w_router, self.b_router, self.top, self.router, self.route_scale, n_identity=self.n_identity)
+            also = h
         else:
             ids, wts = ops.moe_router(h, self.w_router, self.b_router, self.top, self.router, self.route_scale)
         return rt.moe_experts(h, ids, wts, self.w_gu, self.wd, gated=self.gated, also=also, also_w=also_w)

@@ -45,23 +45,26 @@ class PendingDelta:
 
 class RMSNorm(Part):
     """``single``: the learned weight is ONE number for all coordinates (a tensor without dimensions);
-    the kernel reads it as a row of equal entries."""
+    the kernel reads it as a row of equal entries.  ``one_plus``: the stored weight is the distance from one
+    (y = x / rms(x) * (1 + w))."""
 
     graph_safe = True
-    def __init__(self, width: int, eps: float, suffix: str = ".weight", single: bool = False):
+    def __init__(self, width: int, eps: float, suffix: str = ".weight", single: bool = False, one_plus: bool = False):
         self.width = width
         self.eps = float(eps)
         self.suffix = suffix        # what the weight's name adds to the part's prefix ("" when the prefix is the name)
-        self.single = bool(single)
+        self.single, self.one_plus = bool(single), bool(one_plus)
         self.weight = None
 
     def tensor_specs(self, prefix):
-        return [TensorSpec(prefix + self.suffix, () if self.single else (self.width,), VECTOR, init=(1.0, 1.0))]
+        return [TensorSpec(prefix + self.suffix, () if self.single else (self.width,), VECTOR, init=(0.0 if self.one_plus else 1.0, 1.0))]
 
     def bind(self, prefix, tensors, rt):
         self.weight = tensors[prefix + self.suffix]
         if self.single:
             self.weight = self.weight.reshape(1).expand(self.width).contiguous()
+        if self.one_plus:
+            self.weight = (1.0 + self.weight.float()).contiguous()
 
     def forward(self, rt, x, out_dtype, delta=None, rows=None, delta_scale: float = 1.0):
         """Norm of x (+ delta_scale * delta).  x is the float32 residual stream; with ``delta`` the sum
