@@ -16,7 +16,7 @@ measured copy bandwidth, and ``roofline_points`` the same fraction for every bat
 
 ``--shape llama32_3b`` runs that shape's own workload (32 prompts of 128 to 4,096 tokens in
 portions of 512 beside decodes, 512 new tokens each) through ``Engine.generate``;
-``--shape llama2_13b`` decodes at batch 16 after 3,584-token prompts; ``--design lefulorn`` (or ``gotulorn``, ``konovik``, ``dizepel``)
+``--shape llama2_13b`` decodes at batch 16 after 3,584-token prompts; ``--design lefulorn`` (or ``gotulorn``, ``konovik``, ``dizepel``, ``tedisun``)
 times that design beside the Llama decoder at equal layer sizes; ``--cpu-baseline`` times the
 plain CPU implementation at the tiny configurations.
 """
@@ -353,7 +353,24 @@ def dizepel_shape(width: int, heads: int, kv_heads: int, head_dim: int, ff: int,
             "layers": [dict(layer) for _ in range(layers)]}
 
 
-DESIGN_SHAPES = {"lefulorn": lefulorn_shape, "gotulorn": gotulorn_shape, "konovik": konovik_shape, "dizepel": dizepel_shape}
+def tedisun_shape(width: int, heads: int, kv_heads: int, head_dim: int, ff: int, layers: int, window: int, vocab: int) -> dict:
+    """Tedisun with layers of a real model's size: two streams; parallel layers (attention with normed heads of ``head_dim``
+    of which half turn, blended frequencies, a window that keeps the first 4 tokens, a sink; beside it a matrix memory of
+    half the model's width: heads of 256 values on keys of 128) and delta layers (``heads`` heads of ``head_dim`` on half as
+    many key heads, four taps) in turn; every one with 8 experts of a quarter of the gated inner width and 2 that return
+    their input, 2 chosen."""
+    inner = (2 * ff // 3 + 255) // 256 * 256
+    mlp = {"kind": "moe", "expert": {"ff": inner // 4}, "router": {"experts": 8, "identity": 2, "top": 2}}
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5, "mask": {"size": window, "keep_first": 4},
+            "rot": {"base": 500000.0, "dims": head_dim // 2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048}}}
+    right = {"heads": width // 512, "dim": 128, "vdim": 256, "gate_cap": 15.0}
+    par = {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 1.0, "right_scale": 1.0}, "mlp": mlp}
+    dl = {"type": "delta", "mixer": {"heads": heads, "kv_heads": heads // 2, "dim": head_dim, "vdim": head_dim, "conv": 4}, "mlp": mlp}
+    return {"architecture": "Tedisun", "vocab": vocab, "width": width, "streams": 2, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "logit_softcap": 30.0, "layers": [dict(par if i % 2 == 0 else dl) for i in range(layers)]}
+
+
+DESIGN_SHAPES = {"lefulorn": lefulorn_shape, "gotulorn": gotulorn_shape, "konovik": konovik_shape, "dizepel": dizepel_shape, "tedisun": tedisun_shape}
 
 DESIGN_SIZES = {          # name -> width, heads, KV heads, head size, dense inner width, layers
     "w2048": (2048, 16, 4, 128, 8192, 4),
@@ -472,7 +489,7 @@ def main() -> int:
     ap.add_argument("--context", type=int, default=0, help="context (tokens a request may hold) instead of the shape's own")
     ap.add_argument("--prefill-tokens", type=int, default=0, help="tokens of the timed prompt instead of 2,048 (read in portions of 2,048)")
     ap.add_argument("--no-kernel-times", action="store_true", help="leave out the per-kernel-class times of a decode step")
-    ap.add_argument("--design", default="", choices=["", "lefulorn", "gotulorn", "konovik", "dizepel"], help="time this design beside the Llama decoder at equal layer sizes "
+    ap.add_argument("--design", default="", choices=["", "lefulorn", "gotulorn", "konovik", "dizepel", "tedisun"], help="time this design beside the Llama decoder at equal layer sizes "
                     "(prefill and decode, with kernel-class times) instead of the headline workload")
     ap.add_argument("--cpu-baseline", action="store_true", help="time the plain CPU implementation at the tiny configurations and stop")
     args = ap.parse_args()

@@ -140,7 +140,7 @@ def rotate_halves(x, rot, positions):
 
 def visible(i, j, size, keep_first):
     """Whether position i sees position j: j is not later, and lies in the window or among the first tokens."""
-    return j <= i and (not size or i - j < size or j < keep_first)
+    return (j <= i) & ((size == 0) | (i - j < size) | (j < keep_first))
 
 
 def sink_window_attention(q, k, v, scale, sink, size, keep_first):
@@ -149,15 +149,13 @@ def sink_window_attention(q, k, v, scale, sink, size, keep_first):
     T, H, _ = q.shape
     G = k.shape[1]
     out = np.zeros((T, H, v.shape[2]))
+    seen = visible(np.arange(T)[:, None], np.arange(T)[None, :], size, keep_first)
     for h in range(H):
         g = h // (H // G)
-        s = (q[:, h] @ k[:, g].T) * scale
-        for t in range(T):
-            js = [j for j in range(t + 1) if visible(t, j, size, keep_first)]
-            row = s[t, js]
-            m = max(row.max(), sink[h])
-            e = np.exp(row - m)
-            out[t, h] = (e @ v[js, g]) / (e.sum() + math.exp(sink[h] - m))
+        s = np.where(seen, (q[:, h] @ k[:, g].T) * scale, -np.inf)
+        m = np.maximum(s.max(axis=1, keepdims=True), sink[h])
+        e = np.exp(s - m)
+        out[:, h] = (e @ v[:, g]) / (e.sum(axis=1, keepdims=True) + np.exp(sink[h] - m))
     return out
 
 
