@@ -51,6 +51,7 @@ LIBRARIES: Dict[str, tuple] = {
     "token_mix": ("token_mix.cu", []),
     "norm_conv": ("norm_conv.cu", []),
     "ssd": ("ssd.cu", []),
+    "chunk_scan": ("chunk_scan.cu", []),
     "matrix_memory": ("matrix_memory.cu", []),
     "streams": ("streams.cu", []),
 }

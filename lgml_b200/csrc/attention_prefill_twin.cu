@@ -223,8 +223,9 @@ __device__ __forceinline__ bool warp_wait(uint64_t *bar, uint32_t parity, volati
 // in the low half.  EDGE: keys outside c_lo..c_hi give 0 (whatever their score, NaN included).
 // The sums are kept as pairs (even keys, odd keys) in four chains; their order is a function of
 // the column only.
-template <bool EDGE>
-__device__ __forceinline__ void write_p(const uint32_t (&r)[PAGE], uint32_t s_addr, float scale_log2, float neg_m, int c_lo, int c_hi,
+// KEEP: columns below c_keep count as inside whatever c_lo.
+template <bool EDGE, bool KEEP>
+__device__ __forceinline__ void write_p(const uint32_t (&r)[PAGE], uint32_t s_addr, float scale_log2, float neg_m, int c_lo, int c_hi, int c_keep,
                                         float2 (&sum4)[4]) {
     const float2 scale2 = make_float2(scale_log2, scale_log2), neg_m2 = make_float2(neg_m, neg_m);
 #pragma unroll
@@ -235,8 +236,8 @@ __device__ __forceinline__ void write_p(const uint32_t (&r)[PAGE], uint32_t s_ad
             const float2 x = fma2(make_float2(__uint_as_float(r[c0 + i]), __uint_as_float(r[c0 + i + 1])), scale2, neg_m2);
             float2 p = make_float2(ex2(x.x), ex2(x.y));
             if (EDGE) {
-                if (c0 + i > c_hi || c0 + i < c_lo) p.x = 0.f;
-                if (c0 + i + 1 > c_hi || c0 + i + 1 < c_lo) p.y = 0.f;
+                if (c0 + i > c_hi || (c0 + i < c_lo && !(KEEP && c0 + i < c_keep))) p.x = 0.f;
+                if (c0 + i + 1 > c_hi || (c0 + i + 1 < c_lo && !(KEEP && c0 + i + 1 < c_keep))) p.y = 0.f;
             }
             sum4[(i >> 1) & 3] = add2(sum4[(i >> 1) & 3], p);
             __nv_bfloat162 h2 = __floats2bfloat162_rn(p.x, p.y);
@@ -251,13 +252,14 @@ __device__ __forceinline__ void write_p(const uint32_t (&r)[PAGE], uint32_t s_ad
 // BIAS: the form with a distance bias, a sink and an output gate.  Head h's scores lose
 // slopes[h] * (query position - key position); its denominator gains exp(sinks[h]) once; the
 // normalised output is multiplied by sigmoid(gate) (float32 [tokens, H D], row stride ldg).  Each
-// of the three pointers may be null.  Without BIAS none of it is compiled in.
+// of the three pointers may be null.  With a window, a request's first keep_first keys stay visible beyond it:
+// the pages that hold them are walked after the window's.  Without BIAS none of it is compiled in.
 template <int D, bool BIAS>
 __global__ void __launch_bounds__(THREADS, 1) prefill_attention_twin_kernel(
     const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const __nv_bfloat16 *__restrict__ q, int ldq,
     const int *__restrict__ positions, const int *__restrict__ tiles, const int *__restrict__ block_table, int max_blocks, int n_pages,
     __nv_bfloat16 *__restrict__ out, int ldo, int H, int Hkv, int hpc, int tt, float scale, int window, int *__restrict__ status,
-    const float *__restrict__ slopes, const float *__restrict__ sinks, const float *__restrict__ gate, int ldg, float softcap) {
+    const float *__restrict__ slopes, const float *__restrict__ sinks, const float *__restrict__ gate, int ldg, float softcap, int keep_first) {
     constexpr int KB = D / 64;                              // 64-element blocks along the head dimension
     constexpr uint32_t TILE_BYTES = KB * ROWS * 128;        // the queries of one tile: [KB][128 rows][128 B]
     constexpr uint32_t PAGE_BYTES = KB * PAGE * 128;        // a page of keys [KB][64 keys][128 B] (K-major: row = key), or of values (N-major: 64 dims per row)
@@ -287,11 +289,14 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attention_twin_kernel(
     const int pos_first = positions[row0], pos_last = pos_first + n_tok - 1;
     const int lo_first = (window > 0 && pos_first - window + 1 > 0) ? pos_first - window + 1 : 0;
     const int pg_lo = lo_first / PAGE, pg_hi = pos_last / PAGE;
-    const int n_steps = pg_hi - pg_lo + 1;                        // a page a step
+    const int n_window = pg_hi - pg_lo + 1;
+    // pages of kept first tokens that lie before the window's pages
+    const int n_kept = BIAS && window > 0 ? min((keep_first + PAGE - 1) / PAGE, pg_lo) : 0;
+    const int n_steps = n_window + n_kept;                        // a page a step
     // BIAS walks the pages from the newest to the oldest: the bias falls with a key's age (by 64
     // slopes a page), so a row's maximum is as good as settled on its first page; walking up,
     // a head with a steep slope would have to correct its output on every page.
-    auto page_index = [&](int j) -> int { return BIAS ? pg_hi - j : pg_lo + j; };
+    auto page_index = [&](int j) -> int { return BIAS ? (j < n_window ? pg_hi - j : n_steps - 1 - j) : pg_lo + j; };
     const int j_fix = BIAS ? 0 : n_steps - 1;                     // the step of the page that holds the last key
     const int n_act = n_tok > tt ? 2 : 1;                         // tiles that hold tokens
     const float scale_log2 = scale * 1.4426950408889634f;
@@ -419,6 +424,7 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attention_twin_kernel(
             const bool edge = key0 + PAGE - 1 > pos_first_t || (window > 0 && key0 < pos_last_t - window + 1);
             const int c_hi = qpos - key0;                                              // qpos = -1 for a row without a token
             const int c_lo = (window > 0) ? qpos - window + 1 - key0 : -(1 << 30);
+            const int c_keep = BIAS ? keep_first - key0 : 0;                           // columns below it are visible whatever the window
             uint32_t r[PAGE];
 #pragma unroll
             for (int c0 = 0; c0 < PAGE; c0 += 16) tcgen05_ld_16(s_addr + (uint32_t)c0, *reinterpret_cast<uint32_t(*)[16]>(&r[c0]));
@@ -454,7 +460,7 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attention_twin_kernel(
             if (edge) {
 #pragma unroll
                 for (int c = 0; c < PAGE; ++c)
-                    if (c <= c_hi && c >= c_lo) mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(r[c]));
+                    if (c <= c_hi && (c >= c_lo || (BIAS && c < c_keep))) mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(r[c]));
             } else {
 #pragma unroll
                 for (int c = 0; c < PAGE; c += 8) {
@@ -498,8 +504,8 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attention_twin_kernel(
             const float neg_m = (m_ref == -INFINITY) ? 0.f : row_bias - m_ref;    // keeps (-inf) - (-inf) out of the exponent
             float2 sum4[4] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
             const float p_scale = BIAS ? 1.f : scale_log2;              // BIAS: r holds scaled scores already
-            if (edge) write_p<true>(r, s_addr, p_scale, neg_m, c_lo, c_hi, sum4);
-            else write_p<false>(r, s_addr, p_scale, neg_m, c_lo, c_hi, sum4);
+            if (edge) write_p<true, BIAS>(r, s_addr, p_scale, neg_m, c_lo, c_hi, c_keep, sum4);
+            else write_p<false, BIAS>(r, s_addr, p_scale, neg_m, c_lo, c_hi, c_keep, sum4);
             const float2 sum2 = add2(add2(sum4[0], sum4[1]), add2(sum4[2], sum4[3]));
             l_run += sum2.x + sum2.y;
             tcgen05_wait_st();
@@ -656,7 +662,7 @@ template <int D, bool BIAS>
 int launch(dim3 grid, const __nv_bfloat16 *q, int ldq, const int *positions, const int *tiles, const int *block_table, int max_blocks,
            const __nv_bfloat16 *k_pages, const __nv_bfloat16 *v_pages, int n_pages, __nv_bfloat16 *out, int ldo, int H, int Hkv, int hpc, int tt,
            float scale, int window, int *status, cudaStream_t stream, const float *slopes = nullptr, const float *sinks = nullptr,
-           const float *gate = nullptr, int ldg = 0, float softcap = 0.f) {
+           const float *gate = nullptr, int ldg = 0, float softcap = 0.f, int keep_first = 0) {
     constexpr int KB = D / 64;
     const size_t smem = 2 * (size_t)KB * ROWS * 128 + 2 * STAGES * (size_t)KB * PAGE * 128 + 1024;
     static bool configured = false;
@@ -670,7 +676,7 @@ int launch(dim3 grid, const __nv_bfloat16 *q, int ldq, const int *positions, con
     if ((rc = lgml_make_page_map(&mk, k_pages, n_pages, Hkv, D, "prefill_attention_twin"))) return rc;
     if ((rc = lgml_make_page_map(&mv, v_pages, n_pages, Hkv, D, "prefill_attention_twin"))) return rc;
     lgml_launch(prefill_attention_twin_kernel<D, BIAS>, grid, THREADS, smem, stream, mk, mv, q, ldq, positions, tiles, block_table, max_blocks, n_pages,
-                out, ldo, H, Hkv, hpc, tt, scale, window, status, slopes, sinks, gate, ldg, softcap);
+                out, ldo, H, Hkv, hpc, tt, scale, window, status, slopes, sinks, gate, ldg, softcap, keep_first);
     return lgml_launch_status("prefill_attention_twin");
 }
 }  // namespace
@@ -713,16 +719,17 @@ LGML_API int lgml_prefill_attention_twin(const void *q, int ldq, const int *posi
 
 // The same kernel with a distance bias (slopes), a sink in the denominator (sinks) and an output
 // gate (float32 [tokens, H D], row stride ldg), each per head and each optional; keys and values
-// of one head size, 64 or 128.
-LGML_API int lgml_sink_attention_twin(const void *q, int ldq, const int *positions, const int *tiles, int n_tiles, const int *block_table,
+// of one head size, 64 or 128.  keep_first: with a window, the first keys that stay visible beyond it.
+LGML_API int lgml_sink_attention_twin_keep(const void *q, int ldq, const int *positions, const int *tiles, int n_tiles, const int *block_table,
                                       int max_blocks, const void *k_pages, const void *v_pages, int n_pages, int page_size,
                                       const float *slopes, const float *sinks, const float *gate, int ldg, void *out, int ldo, int H, int Hkv,
-                                      int D, float scale, float softcap, int window, int *status, cudaStream_t stream) {
+                                      int D, float scale, float softcap, int window, int keep_first, int *status, cudaStream_t stream) {
     LGML_REQUIRE(n_tiles >= 0 && H > 0 && Hkv > 0 && max_blocks > 0 && n_pages > 0, "sink_attention_twin: bad sizes");
     LGML_REQUIRE(page_size == PAGE, "sink_attention_twin: pages of %d tokens, this kernel takes %d", page_size, PAGE);
     LGML_REQUIRE(H % Hkv == 0, "sink_attention_twin: %d heads are no multiple of %d KV heads", H, Hkv);
     LGML_REQUIRE(D == 64 || D == 128, "sink_attention_twin: head_dim %d (this kernel takes 64 and 128)", D);
     LGML_REQUIRE(window >= 0, "sink_attention_twin: bad window");
+    LGML_REQUIRE(keep_first >= 0, "sink_attention_twin: bad number of kept first tokens");
     LGML_REQUIRE(ldq % 8 == 0 && ldo % 8 == 0 && ((uintptr_t)q & 15) == 0 && ((uintptr_t)out & 15) == 0,
                  "sink_attention_twin: q and out must be 16-byte aligned with row strides that are multiples of 8");
     LGML_REQUIRE(((uintptr_t)k_pages & 15) == 0 && ((uintptr_t)v_pages & 15) == 0, "sink_attention_twin: the cache must be 16-byte aligned");
@@ -740,7 +747,15 @@ LGML_API int lgml_sink_attention_twin(const void *q, int ldq, const int *positio
     __nv_bfloat16 *oo = (__nv_bfloat16 *)out;
     if (D == 64)
         return launch<64, true>(grid, qq, ldq, positions, tiles, block_table, max_blocks, kk, vv, n_pages, oo, ldo, H, Hkv, hpc, tile_tokens / 2, scale, window,
-                                status, stream, slopes, sinks, gate, ldg, softcap);
+                                status, stream, slopes, sinks, gate, ldg, softcap, keep_first);
     return launch<128, true>(grid, qq, ldq, positions, tiles, block_table, max_blocks, kk, vv, n_pages, oo, ldo, H, Hkv, hpc, tile_tokens / 2, scale, window,
-                             status, stream, slopes, sinks, gate, ldg, softcap);
+                             status, stream, slopes, sinks, gate, ldg, softcap, keep_first);
+}
+
+LGML_API int lgml_sink_attention_twin(const void *q, int ldq, const int *positions, const int *tiles, int n_tiles, const int *block_table,
+                                      int max_blocks, const void *k_pages, const void *v_pages, int n_pages, int page_size,
+                                      const float *slopes, const float *sinks, const float *gate, int ldg, void *out, int ldo, int H, int Hkv,
+                                      int D, float scale, float softcap, int window, int *status, cudaStream_t stream) {
+    return lgml_sink_attention_twin_keep(q, ldq, positions, tiles, n_tiles, block_table, max_blocks, k_pages, v_pages, n_pages, page_size, slopes, sinks,
+                                         gate, ldg, out, ldo, H, Hkv, D, scale, softcap, window, 0, status, stream);
 }

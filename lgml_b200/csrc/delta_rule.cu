@@ -13,7 +13,8 @@
 //
 // With one decay per head the convolutions are a kernel of their own (short_conv, norm_conv.cu), and
 // delta_head_prepare makes the unit vectors in place and the per-head decay and beta; delta_scan then
-// reads a row of four floats (decay, beta, two zeros) per head.
+// reads a row of four floats (decay, beta, log of the decay, zero) per head.  Many tokens at once take
+// the chunked form in chunk_scan.cu instead.
 //
 // Four kernels a step:
 //   delta_prepare      one block per token, all tokens at once: convolution (the inputs before a
@@ -115,7 +116,7 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_conv_state_kernel(
 }
 
 // One decay per head.  qkv [n, C] (q (G D) | k (G D) | v ...) after convolution and SiLU: q and k become unit vectors per
-// head in place, q also times D^-1/2.  gb [n, H, 4] = (decay, beta, 0, 0) from the projections a and b.  A warp takes a head.
+// head in place, q also times D^-1/2.  gb [n, H, 4] = (decay, beta, log of the decay, 0) from the projections a and b.  A warp takes a head.
 __global__ void __launch_bounds__(PREP_THREADS) delta_head_prepare_kernel(float *__restrict__ qkv, int C, const float *__restrict__ a_pre, int lda,
                                                                           const float *__restrict__ b_pre, int ldb, const float *__restrict__ a_log,
                                                                           const float *__restrict__ dt_bias, float *__restrict__ gb, int n_tokens, int H,
@@ -129,9 +130,9 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_head_prepare_kernel(float 
         const int t = (int)(u / hpt), hd = (int)(u - (long long)t * hpt);
         if (hd == 2 * G) {
             for (int h = lane; h < H; h += 32) {
-                const float g = expf(-expf(a_log[h]) * softplus_f(act_load(a_pre + (size_t)t * lda + h) + dt_bias[h]));
+                const float lg = -expf(a_log[h]) * softplus_f(act_load(a_pre + (size_t)t * lda + h) + dt_bias[h]);
                 const float beta = sigmoid_f(act_load(b_pre + (size_t)t * ldb + h));
-                *reinterpret_cast<float4 *>(gb + ((size_t)t * H + h) * 4) = make_float4(g, beta, 0.f, 0.f);
+                *reinterpret_cast<float4 *>(gb + ((size_t)t * H + h) * 4) = make_float4(expf(lg), beta, lg, 0.f);
             }
             continue;
         }
@@ -177,13 +178,14 @@ template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile(
 // with cp.async (through L2) while this one is computed; else one buffer filled with plain loads.
 // NC columns a thread (column c of a thread lies SCAN_THREADS / R columns after its column c - 1):
 // two independent chains per thread fill the waits of each other, and k, q and the decays are read once for both.
-// HEAD: one decay per head; gb rows are (decay, beta, 0, 0) and a token's row of the decay buffer is those four floats.
+// HEAD: one decay per head; gb rows are (decay, beta, log of the decay, 0) and a token's row of the decay buffer is those four floats.
 template <int NPT, bool ASYNC, int NC, bool HEAD>
 __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
     const float *__restrict__ qkv_c, const float *__restrict__ gb, float *__restrict__ state, long long state_stride,
-    const int *__restrict__ seq_start, const int *__restrict__ slots, float *__restrict__ o_out, int H, int G, int D, int Dv, int R) {
+    const int *__restrict__ seq_start, const int *__restrict__ slots, float *__restrict__ o_out, int H, int G, int D, int Dv, int R, int max_tokens) {
     pdl_trigger();
     pdl_wait();
+    if (max_tokens > 0 && seq_start[blockIdx.x + 1] - seq_start[blockIdx.x] > max_tokens) return;
     extern __shared__ __align__(16) float sm[];
     constexpr int RUN = NPT + 4;                          // floats from one thread's run to the next
     const int DP = RUN * R;
@@ -365,13 +367,13 @@ __global__ void __launch_bounds__(128) delta_output_kernel(const float *__restri
 
 template <int NPT, bool ASYNC, int NC, bool HEAD>
 int launch_scan(dim3 grid, size_t smem, cudaStream_t stream, const float *qkv_c, const float *gb, float *state, long long state_stride,
-                const int *seq_start, const int *slots, float *o_out, int H, int G, int D, int Dv, int R) {
+                const int *seq_start, const int *slots, float *o_out, int H, int G, int D, int Dv, int R, int max_tokens) {
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<NPT, ASYNC, NC, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) LGML_FAIL("delta_scan: cannot have %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
     }
     lgml_launch(delta_scan_kernel<NPT, ASYNC, NC, HEAD>, grid, SCAN_THREADS, smem, stream, qkv_c, gb, state, state_stride, seq_start, slots, o_out, H, G, D,
-                Dv, R);
+                Dv, R, max_tokens);
     return lgml_launch_status("delta_scan");
 }
 }  // namespace
@@ -410,9 +412,10 @@ LGML_API int lgml_delta_head_prepare(float *qkv, int C, const float *a_pre, int 
     return lgml_launch_status("delta_head_prepare");
 }
 
-// gb: float32 [tokens, H, D + 4] as delta_prepare writes it (decays, beta, zeros); head_decay: [tokens, H, 4] (decay, beta, zeros).
+// gb: float32 [tokens, H, D + 4] as delta_prepare writes it (decays, beta, zeros); head_decay: [tokens, H, 4] (decay, beta, log of the decay, zero).
+// max_tokens > 0: requests that bring more tokens are left out.
 LGML_API int lgml_delta_scan_form(const float *qkv_c, const float *gb, float *state, long long state_stride, const int *seq_start,
-                                  const int *slots, float *o_out, int n_seqs, int H, int G, int D, int Dv, int head_decay, cudaStream_t stream) {
+                                  const int *slots, float *o_out, int n_seqs, int H, int G, int D, int Dv, int head_decay, int max_tokens, cudaStream_t stream) {
     LGML_REQUIRE(n_seqs >= 0 && H > 0 && G > 0 && D > 0 && Dv > 0 && H % G == 0, "delta_scan: bad sizes");
     LGML_REQUIRE(D <= 1024, "delta_scan: key size %d is over 1024", D);
     LGML_REQUIRE(H <= 65535, "delta_scan: too many heads");
@@ -437,7 +440,7 @@ LGML_API int lgml_delta_scan_form(const float *qkv_c, const float *gb, float *st
     const bool async = D % 4 == 0 && Dv % 4 == 0 && (((uintptr_t)qkv_c | (uintptr_t)gb) & 15) == 0;
     const size_t smem = sizeof(float) * (size_t)(async ? 2 : 1) * TCH * ((head_decay ? 2 : 3) * (size_t)(npt + 4) * R + 4 + cols);
     dim3 grid(n_seqs, H, (Dv + cols - 1) / cols);
-#define LGML_SCAN_ARGS grid, smem, stream, qkv_c, gb, state, state_stride, seq_start, slots, o_out, H, G, D, Dv, R
+#define LGML_SCAN_ARGS grid, smem, stream, qkv_c, gb, state, state_stride, seq_start, slots, o_out, H, G, D, Dv, R, max_tokens
 #define LGML_SCAN_FORM(N, NC) \
     (head_decay ? (async ? launch_scan<N, true, NC, true>(LGML_SCAN_ARGS) : launch_scan<N, false, NC, true>(LGML_SCAN_ARGS)) \
                 : (async ? launch_scan<N, true, NC, false>(LGML_SCAN_ARGS) : launch_scan<N, false, NC, false>(LGML_SCAN_ARGS)))
@@ -457,7 +460,7 @@ LGML_API int lgml_delta_scan_form(const float *qkv_c, const float *gb, float *st
 
 LGML_API int lgml_delta_scan(const float *qkv_c, const float *gb, float *state, long long state_stride, const int *seq_start,
                              const int *slots, float *o_out, int n_seqs, int H, int G, int D, int Dv, cudaStream_t stream) {
-    return lgml_delta_scan_form(qkv_c, gb, state, state_stride, seq_start, slots, o_out, n_seqs, H, G, D, Dv, 0, stream);
+    return lgml_delta_scan_form(qkv_c, gb, state, state_stride, seq_start, slots, o_out, n_seqs, H, G, D, Dv, 0, 0, stream);
 }
 
 // act 0: the gate is sigmoid(gate); 1: silu(gate)

@@ -23,7 +23,7 @@ __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - l
 
 // Block (request, head).  Every thread takes a run of consecutive tokens: their map m -> max(F + m, I) is composed in order, the
 // runs' maps by a scan over the block, and each thread then walks its run from its true start.
-// gates [n, 3 H]: a | b | exp(-m).
+// gates [n, 4 H]: a | b | exp(-m) | log a.
 __global__ void __launch_bounds__(GATE_THREADS) memory_gates_kernel(const float *__restrict__ zi, const float *__restrict__ zf, int ldz, float cap,
                                                                     float *__restrict__ m_state, long long state_ld, const int *__restrict__ seq_start,
                                                                     const int *__restrict__ slots, float *__restrict__ gates, int H) {
@@ -37,7 +37,7 @@ __global__ void __launch_bounds__(GATE_THREADS) memory_gates_kernel(const float 
     const float m0 = act_load(ms);
     const int per = (n + GATE_THREADS - 1) / GATE_THREADS;
     const int first = min(tid * per, n), last = min(first + per, n);
-    const int ldg = 3 * H;
+    const int ldg = 4 * H;
     float F = 0.f, I = -INFINITY;
     for (int t = first; t < last; ++t) {
         const float i = capped(act_load(zi + (size_t)(t0 + t) * ldz + h), cap);
@@ -76,6 +76,7 @@ __global__ void __launch_bounds__(GATE_THREADS) memory_gates_kernel(const float 
         float *g = gates + (size_t)(t0 + t) * ldg + h;
         const float f = g[0], i = g[H];
         m = fmaxf(f + m, i);
+        g[3 * H] = f + prev - m;
         g[0] = expf(f + prev - m);
         g[H] = expf(i - m);
         g[2 * H] = expf(-m);
@@ -98,7 +99,7 @@ __global__ void __launch_bounds__(128) memory_output_kernel(const float *__restr
         const float *row = y + u * (P + 1);
         const float *gr = gate + (size_t)t * ldg + (size_t)h * P, *wr = w + (size_t)h * P;
         T *orow = out + (size_t)t * ldo + (size_t)h * P;
-        const float den = fmaxf(fabsf(q_scale * act_load(row + P)), act_load(gates + (size_t)t * 3 * H + 2 * H + h)) + 1e-6f;
+        const float den = fmaxf(fabsf(q_scale * act_load(row + P)), act_load(gates + (size_t)t * 4 * H + 2 * H + h)) + 1e-6f;
         const float k = q_scale / den;
         constexpr int KEEP = 8;                 // entries a lane keeps between the two walks
         float v[KEEP], ss = 0.f;
@@ -124,7 +125,7 @@ __global__ void __launch_bounds__(128) memory_output_kernel(const float *__restr
 }
 }  // namespace
 
-// zi, zf: float32 rows of H entries, ldz apart; m_state: the first slot's m of head 0, slots state_ld apart; gates float32 [n, 3 H].
+// zi, zf: float32 rows of H entries, ldz apart; m_state: the first slot's m of head 0, slots state_ld apart; gates float32 [n, 4 H].
 LGML_API int lgml_memory_gates(const float *zi, const float *zf, int ldz, float cap, float *m_state, long long state_ld, const int *seq_start,
                                const int *slots, float *gates, int n_seqs, int H, cudaStream_t stream) {
     LGML_REQUIRE(n_seqs >= 0 && H > 0 && H <= 65535 && ldz >= H && cap > 0.f, "memory_gates: bad sizes");

@@ -41,9 +41,10 @@ __global__ void __launch_bounds__(SCAN_THREADS) ssd_scan_kernel(const float *__r
                                                                 const int *__restrict__ seq_start, const int *__restrict__ slots,
                                                                 float *__restrict__ y, int ldy, int Hs, int G, int P, int N, int LN, int TT,
                                                                 int pieces, int zero_start, float *__restrict__ decay_out, int vec,
-                                                                const float *__restrict__ a_given, int Px) {
+                                                                const float *__restrict__ a_given, int Px, int max_tokens) {
     pdl_trigger();
     pdl_wait();
+    if (max_tokens > 0 && seq_start[blockIdx.z + 1] - seq_start[blockIdx.z] > max_tokens) return;
     extern __shared__ float sm[];
     const int CPB = (SCAN_THREADS / LN) * CQ;          // columns of a block
     const int NS = LN * RN;
@@ -217,7 +218,7 @@ __global__ void __launch_bounds__(NT) ssd_gate_norm_kernel(const float *__restri
 namespace {
 int scan_any(const float *xbc, int ldx, const float *dt_raw, int ldd, const float *dt_bias, const float *a_log, const float *d_skip,
                            float *state, long long state_ld, const int *seq_start, const int *slots, float *y, int ldy, int n_seqs, int Hs, int G,
-                           int P, int N, int pieces, int zero_start, float *decay_out, const float *a_given, int Px, cudaStream_t stream) {
+                           int P, int N, int pieces, int zero_start, float *decay_out, const float *a_given, int Px, int max_tokens, cudaStream_t stream) {
     LGML_REQUIRE(n_seqs >= 0 && Hs > 0 && G > 0 && P > 0 && N > 0 && Px > 0 && Px <= P, "ssd_scan: bad sizes");
     LGML_REQUIRE(Hs % G == 0, "ssd_scan: %d heads are no multiple of %d groups", Hs, G);
     LGML_REQUIRE(N <= 1024, "ssd_scan: a state of %d numbers per column is more than 1024", N);
@@ -247,7 +248,7 @@ int scan_any(const float *xbc, int ldx, const float *dt_raw, int ldd, const floa
     dim3 grid((P + CPB - 1) / CPB, Hs, n_seqs);
     const int vec = N % 4 == 0 && ldx % 4 == 0 && (Hs * Px) % 4 == 0 && ((uintptr_t)xbc & 15) == 0;
 #define LGML_SCAN_K(RN, CQ, GIVEN) lgml_launch(ssd_scan_kernel<RN, CQ, GIVEN>, grid, SCAN_THREADS, smem, stream, xbc, ldx, dt_raw, ldd, dt_bias, a_log, d_skip, \
-                                               state, state_ld, seq_start, slots, y, ldy, Hs, G, P, N, LN, TT, pieces, zero_start, decay_out, vec, a_given, Px)
+                                               state, state_ld, seq_start, slots, y, ldy, Hs, G, P, N, LN, TT, pieces, zero_start, decay_out, vec, a_given, Px, max_tokens)
 #define LGML_SCAN(RN, CQ) do { if (a_given != nullptr) LGML_SCAN_K(RN, CQ, true); else LGML_SCAN_K(RN, CQ, false); } while (0)
     if (quad) {
         switch (best_rn) {
@@ -275,17 +276,19 @@ LGML_API int lgml_ssd_scan(const float *xbc, int ldx, const float *dt_raw, int l
                            float *state, long long state_ld, const int *seq_start, const int *slots, float *y, int ldy, int n_seqs, int Hs, int G,
                            int P, int N, int pieces, int zero_start, float *decay_out, cudaStream_t stream) {
     return scan_any(xbc, ldx, dt_raw, ldd, dt_bias, a_log, d_skip, state, state_ld, seq_start, slots, y, ldy, n_seqs, Hs, G, P, N, pieces, zero_start,
-                    decay_out, nullptr, P, stream);
+                    decay_out, nullptr, P, 0, stream);
 }
 
 // The recurrence with decays and write weights given: decay / weight float32 rows of Hs entries, ldd apart.  x has Px columns per head,
-// the state and y have P >= Px; columns from Px on are written with x = 1.
+// the state and y have P >= Px; columns from Px on are written with x = 1.  max_tokens > 0: requests that bring more
+// tokens are left out.
 LGML_API int lgml_ssd_scan_given(const float *xbc, int ldx, const float *weight, const float *decay, int ldd, float *state, long long state_ld,
                                  const int *seq_start, const int *slots, float *y, int ldy, int n_seqs, int Hs, int G, int Px, int P, int N, int pieces,
-                                 int zero_start, float *decay_out, cudaStream_t stream) {
+                                 int zero_start, float *decay_out, int max_tokens, cudaStream_t stream) {
+    LGML_REQUIRE(max_tokens == 0 || !pieces, "ssd_scan: pieces leave no request out");
     LGML_REQUIRE(decay != nullptr && weight != nullptr, "ssd_scan: decays and write weights are missing");
     return scan_any(xbc, ldx, weight, ldd, nullptr, nullptr, nullptr, state, state_ld, seq_start, slots, y, ldy, n_seqs, Hs, G, P, N, pieces, zero_start,
-                    decay_out, decay, Px, stream);
+                    decay_out, decay, Px, max_tokens, stream);
 }
 
 LGML_API int lgml_ssd_gate_norm(const float *y, int ldy, const float *z, int ldz, const float *w, void *out, int out_dtype, int ldo, int n_tokens,

@@ -50,6 +50,17 @@ def cache_view_of(cm, owner: int, block_tables, writable: bool = True) -> CacheV
     return view
 
 
+@dataclass
+class ScanChunks:
+    """The tokens of a step's requests that bring more than ``longer_than`` of them, in chunks of consecutive tokens."""
+
+    rows: torch.Tensor          # int32 [n_chunks, 2]: first token row, the row past the last; a request's chunks in a row
+    first: torch.Tensor         # int32 [requests + 1]: the first chunk of every one of them
+    requests: torch.Tensor      # int32 [requests]: which requests of the step they are
+    longer_than: int
+    short: bool                 # whether the step holds other requests too
+
+
 class StepBatch:
     """Host lists -> one int32 buffer -> one copy -> device views.
 
@@ -213,6 +224,26 @@ class StepBatch:
             both = self._to_device(np.concatenate([np.asarray(pieces, dtype=np.int32).reshape(-1), np.asarray(first, dtype=np.int32)]))
             cached = (both[:2 * len(pieces)].view(-1, 2), both[2 * len(pieces):])
             self._tiles[("pieces", piece_tokens)] = cached
+        return cached
+
+    def scan_chunks(self, chunk_tokens: int, longer_than: int) -> Optional[ScanChunks]:
+        """The long requests of this step in chunks (None when no request brings more than ``longer_than`` tokens), for a
+        recurrence that takes those as matrix products and the others token by token.  Made once per chunk size."""
+        if self.max_q_len <= longer_than:
+            return None
+        key = ("chunks", chunk_tokens, longer_than)
+        cached = self._tiles.get(key)
+        if cached is None:
+            rows, first, reqs, start = [], [0], [], 0
+            for s, n in enumerate(self.seq_lens):
+                if n > longer_than:
+                    rows += [(start + t0, start + min(t0 + chunk_tokens, n)) for t0 in range(0, n, chunk_tokens)]
+                    first.append(len(rows))
+                    reqs.append(s)
+                start += n
+            flat = self._to_device(np.concatenate([np.asarray(rows, dtype=np.int32).reshape(-1), np.asarray(first, dtype=np.int32), np.asarray(reqs, dtype=np.int32)]))
+            a, b = 2 * len(rows), 2 * len(rows) + len(first)
+            cached = self._tiles[key] = ScanChunks(flat[:a].view(-1, 2), flat[a:b], flat[b:], longer_than, len(reqs) < len(self.seq_lens))
         return cached
 
     @staticmethod

@@ -120,16 +120,16 @@ class Runtime:
         than the keys, or be the first entries of the key cells.  ``softcap`` > 0 caps the scaled scores:
         s -> softcap tanh(s / softcap)."""
         bf16 = self.dtype == torch.bfloat16 and self.attention_backend != "ref" and cache.k.shape[2] == 64
-        # what only this family's own kernels know: kept first tokens, value heads of their own count, values that are a
-        # column range of the key cells, a float32 result
-        plain = not keep_first and cache.v.shape[1] == cache.k.shape[1] and cache.v.is_contiguous() and out.dtype == q.dtype
+        # what only this family's own kernels know: value heads of their own count, values that are a column range of the
+        # key cells, a float32 result
+        plain = cache.v.shape[1] == cache.k.shape[1] and cache.v.is_contiguous() and out.dtype == q.dtype
         if bf16 and batch.max_q_len > ops.DECODE_MAX_Q and cache.k.shape[3] <= 128 and cache.v.shape[3] <= 128:
             if plain and ops.sink_twin_supports(q, out, cache.k, cache.v, gate):
                 # prompts and portions, keys and values of one head size (64 or 128): the two-tile tcgen05 kernel
                 hkv = cache.k.shape[1]
                 tiles = batch.attention_tiles(ops.prefill_twin_tile_tokens(n_heads, hkv))
                 return ops.sink_attention_twin(q, batch.positions, tiles, cache.block_table, cache.k, cache.v, out, n_heads, scale, window,
-                                               self.status, slopes=slopes, sinks=sinks, gate=gate, softcap=softcap)
+                                               self.status, slopes=slopes, sinks=sinks, gate=gate, keep_first=keep_first, softcap=softcap)
             # every other head size up to 128: tiles of 64 tokens, mma.sync
             tiles = batch.attention_tiles(ops.SINK_TILE_TOKENS)
             return ops.sink_attention_mma(q, batch.positions, tiles, cache.block_table, cache.k, cache.v, out, n_heads, scale, window,

@@ -639,7 +639,7 @@ def sink_twin_supports(q: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor
 def sink_attention_twin(q: torch.Tensor, positions: torch.Tensor, tiles: torch.Tensor, block_table: torch.Tensor, k_pages: torch.Tensor,
                         v_pages: torch.Tensor, out: torch.Tensor, n_heads: int, scale: float, window: int, status: torch.Tensor,
                         slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
-                        gate: Optional[torch.Tensor] = None, softcap: float = 0.0) -> torch.Tensor:
+                        gate: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0) -> torch.Tensor:
     """``sink_attention`` for prompts and portions on tcgen05 tensor cores: the two-tile kernel of
     ``prefill_attention_twin`` with the slopes' bias on the scores, the sink in the denominator and
     the gate on the output.  bfloat16, pages of 64, keys and values of one head size (64 or 128).
@@ -670,12 +670,12 @@ def sink_attention_twin(q: torch.Tensor, positions: torch.Tensor, tiles: torch.T
         ldg = _rows_contiguous(gate, "gate")
         if tuple(gate.shape) != (n, n_heads * d):
             raise KernelError(f"sink_attention_twin: gate {tuple(gate.shape)} is not [{n}, {n_heads * d}]")
-    fn = _fn("attention_prefill_twin", "lgml_sink_attention_twin", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
+    fn = _fn("attention_prefill_twin", "lgml_sink_attention_twin_keep", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                                                     c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
-                                                                    c_int, c_float, c_float, c_int, c_void_p, c_void_p])
+                                                                    c_int, c_float, c_float, c_int, c_int, c_void_p, c_void_p], label="sink_attention_twin")
     _check("attention_prefill_twin", fn(_ptr(q), ldq, _ptr(positions), _ptr(tiles), tiles.shape[0], _ptr(block_table), block_table.shape[1],
                                         _ptr(k_pages), _ptr(v_pages), n_pages, page, _ptr(slopes), _ptr(sinks), _ptr(gate), ldg, _ptr(out), ldo,
-                                        n_heads, hkv, d, float(scale), float(softcap or 0.0), int(window or 0), _ptr(status), _stream()), "sink_attention_twin")
+                                        n_heads, hkv, d, float(scale), float(softcap or 0.0), int(window or 0), int(keep_first or 0), _ptr(status), _stream()), "sink_attention_twin")
     return out
 
 
@@ -1518,7 +1518,7 @@ def norm_rope_store(proj: torch.Tensor, q_w: Optional[torch.Tensor], k_w: Option
 def memory_gates(zi: torch.Tensor, zf: torch.Tensor, cap: float, m_state: torch.Tensor, seq_start: torch.Tensor, slots: torch.Tensor) -> torch.Tensor:
     """From the gates' logits zi, zf float32 [tokens, H] (column slices of one projection): i = cap tanh(zi / cap), f =
     logsigmoid(cap tanh(zf / cap)) and, request by request, m <- max(f + m, i) (``m_state`` float32 [slots, H], a column slice of
-    the state rows, holds m between steps).  Returns float32 [tokens, 3 H]: exp(f + m_before - m) | exp(i - m) | exp(-m)."""
+    the state rows, holds m between steps).  Returns float32 [tokens, 4 H]: exp(f + m_before - m) | exp(i - m) | exp(-m) | f + m_before - m."""
     _need(zi, "input gate logits", torch.float32, 2)
     _need(zf, "forget gate logits", torch.float32, 2)
     _need(m_state, "running maxima", torch.float32, 2)
@@ -1526,7 +1526,7 @@ def memory_gates(zi: torch.Tensor, zf: torch.Tensor, cap: float, m_state: torch.
     ldz = _rows_contiguous(zi, "input gate logits") if n else H
     if tuple(zf.shape) != (n, H) or (n and zf.stride(0) != ldz) or zf.stride(1) != 1 or m_state.shape[1] != H or m_state.stride(1) != 1:
         raise KernelError(f"memory_gates: gates {tuple(zi.shape)} / {tuple(zf.shape)} and maxima {tuple(m_state.shape)} do not fit")
-    gates = torch.empty((n, 3 * H), dtype=torch.float32, device=zi.device)
+    gates = torch.empty((n, 4 * H), dtype=torch.float32, device=zi.device)
     fn = _fn("matrix_memory", "lgml_memory_gates", [c_void_p, c_void_p, c_int, c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
     _check("matrix_memory", fn(_ptr(zi), _ptr(zf), ldz, float(cap), _ptr(m_state), m_state.stride(0), _ptr(seq_start), _ptr(slots), _ptr(gates),
                                slots.numel(), H, _stream()), "memory_gates")
@@ -1541,10 +1541,10 @@ def memory_output(y: torch.Tensor, gates: torch.Tensor, q_scale: float, weight: 
     _need(weight, "norm weight", torch.float32, 1)
     _need(gate, "output gate", torch.float32, 2)
     _need(out, "output", ndim=2)
-    n, H = y.shape[0], gates.shape[1] // 3
+    n, H = y.shape[0], gates.shape[1] // 4
     P = y.shape[1] // H - 1
     ldg, ldo = _rows_contiguous(gate, "output gate"), _rows_contiguous(out, "output")
-    if y.shape[1] != H * (P + 1) or tuple(gates.shape) != (n, 3 * H) or weight.numel() != H * P or tuple(gate.shape) != (n, H * P) \
+    if y.shape[1] != H * (P + 1) or tuple(gates.shape) != (n, 4 * H) or weight.numel() != H * P or tuple(gate.shape) != (n, H * P) \
             or tuple(out.shape) != (n, H * P) or not (y.is_contiguous() and gates.is_contiguous() and weight.is_contiguous()):
         raise KernelError(f"memory_output: y {tuple(y.shape)}, gates {tuple(gates.shape)}, weight {tuple(weight.shape)}, out {tuple(out.shape)} do not fit")
     fn = _fn("matrix_memory", "lgml_memory_output", [c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
@@ -1555,27 +1555,34 @@ def memory_output(y: torch.Tensor, gates: torch.Tensor, q_scale: float, weight: 
 
 
 def memory_scan(vkq: torch.Tensor, gates: torch.Tensor, state: torch.Tensor, seq_start: torch.Tensor, slots: torch.Tensor, n_heads: int, head_dim: int,
-                v_head_dim: int, pieces=None) -> torch.Tensor:
+                v_head_dim: int, pieces=None, chunks=None) -> torch.Tensor:
     """S <- a S + b k v^T, n <- a n + b k; y = (S^T q, n . q) per head, over each request's tokens in order.  ``vkq`` float32
     [tokens, v (H P) | k (H N) | q (H N)] (may be a column slice); ``gates`` as ``memory_gates`` returns them; S and n ([P + 1][N] per
-    head, n the last row) live in ``state[slot]``.  Returns y float32 [tokens, H (P + 1)].  ``pieces`` as for ``ssd_scan``."""
+    head, n the last row) live in ``state[slot]``.  Returns y float32 [tokens, H (P + 1)].  ``pieces`` as for ``ssd_scan``; ``chunks`` as
+    for ``chunk_scan``: the requests with many tokens take that form (where the sizes allow), the others the sequential one."""
     _need(vkq, "values, keys and queries", torch.float32, 2)
     _need(gates, "gates", torch.float32, 2)
     H, N, P1 = n_heads, head_dim, v_head_dim + 1
     n = vkq.shape[0]
     ldx = _rows_contiguous(vkq, "values, keys and queries")
-    if vkq.shape[1] != H * (v_head_dim + 2 * N) or tuple(gates.shape) != (n, 3 * H) or not gates.is_contiguous():
+    if vkq.shape[1] != H * (v_head_dim + 2 * N) or tuple(gates.shape) != (n, 4 * H) or not gates.is_contiguous():
         raise KernelError(f"memory_scan: {tuple(vkq.shape)} and gates {tuple(gates.shape)} do not fit {H} heads of {N} and {v_head_dim}")
     ld_state = _state_rows(state, H * P1 * N, "memory_scan")
     y = torch.empty((n, H * P1), dtype=torch.float32, device=vkq.device)
     fn = _fn("ssd", "lgml_ssd_scan_given", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                                            c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p], label="memory_scan")
+                                            c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p], label="memory_scan")
 
-    def scan(st, ld, starts, slot_ids, out, count, in_pieces, from_zero, decay):
-        _check("ssd", fn(_ptr(vkq), ldx, _ptr(gates[:, H:]), _ptr(gates), 3 * H, _ptr(st), ld, _ptr(starts), _ptr(slot_ids), _ptr(out), H * P1, count, H, H,
-                         v_head_dim, P1, N, 1 if in_pieces else 0, 1 if from_zero else 0, _ptr(decay), _stream()), "memory_scan")
+    def scan(st, ld, starts, slot_ids, out, count, in_pieces, from_zero, decay, max_tokens=0):
+        _check("ssd", fn(_ptr(vkq), ldx, _ptr(gates[:, H:]), _ptr(gates), 4 * H, _ptr(st), ld, _ptr(starts), _ptr(slot_ids), _ptr(out), H * P1, count, H, H,
+                         v_head_dim, P1, N, 1 if in_pieces else 0, 1 if from_zero else 0, _ptr(decay), max_tokens, _stream()), "memory_scan")
 
     n_seqs = seq_start.numel() - 1
+    k, q = vkq[:, H * v_head_dim:H * (v_head_dim + N)], vkq[:, H * (v_head_dim + N):]
+    if chunks is not None and n and chunk_scan_supports(q, k, N, False):
+        chunk_scan(q, k, vkq, gates[:, 3 * H:], gates[:, H:], 1, state, 1, N, chunks, slots, y, H, H, N, v_head_dim, P1, False)
+        if chunks.short:
+            scan(state, ld_state, seq_start, slots, y, n_seqs, False, False, None, max_tokens=chunks.longer_than)
+        return y
     if pieces is None:
         scan(state, ld_state, seq_start, slots, y, n_seqs, False, False, None)
         return y
@@ -1585,10 +1592,61 @@ def memory_scan(vkq: torch.Tensor, gates: torch.Tensor, state: torch.Tensor, seq
 
 # ----------------------------------------------------------------------------------------
 
+CHUNK_TOKENS = 64
+CHUNK_FROM = 16           # a request that brings more tokens than this takes the chunked form (a chunk costs about as much as so many steps)
+_chunk_takes = {}
+
+
+def chunk_scan_supports(q: torch.Tensor, k: torch.Tensor, dim: int, delta: bool) -> bool:
+    """Whether ``chunk_scan`` takes these queries and keys: 16-byte aligned rows, heads that are multiples of 4 and fit shared memory."""
+    if dim % 4 or q.stride(0) % 4 or q.stride(0) != k.stride(0) or q.data_ptr() % 16 or k.data_ptr() % 16:
+        return False
+    key = (dim, bool(delta))
+    if key not in _chunk_takes:
+        fn = csrc.load("chunk_scan").lgml_chunk_scan_takes
+        fn.argtypes, fn.restype = [c_int, c_int], c_int
+        _chunk_takes[key] = bool(fn(dim, 1 if delta else 0))
+    return _chunk_takes[key]
+
+
+def chunk_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_a: torch.Tensor, w: torch.Tensor, head_stride: int, state: torch.Tensor,
+               s_row: int, s_col: int, chunks, slots: torch.Tensor, out: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, v_cols: int, cols: int,
+               delta: bool) -> None:
+    """A recurrence with one decay per head over the requests of ``chunks`` that bring many tokens, 64 tokens at a time as matrix
+    products (all float32):
+
+        delta:      S <- a S;  u = w (v - S^T k);  S <- S + k u^T;  o = S^T q
+        otherwise:  S <- a S + w k v^T;                             o = S^T q
+
+    q, k, v: float32 rows of one tensor (equal strides), heads behind each other; ``log_a`` and ``w``: columns of one tensor with
+    ``head_stride`` between heads.  S of head h has ``cols`` columns (the first ``v_cols`` from v, the others written with v = 1) and lies
+    in the slot's row at h dim cols + d s_row + c s_col.  ``chunks``: ``StepBatch.scan_chunks``.  Writes o's rows of those requests into
+    ``out`` [tokens, H cols]."""
+    n_chunks, n_req = chunks.rows.shape[0], chunks.requests.numel()
+    if n_req == 0:
+        return
+    if log_a.stride(0) != w.stride(0) or v.stride(0) != q.stride(0) or not out.is_contiguous() or out.shape[1] != n_heads * cols:
+        raise KernelError("chunk_scan: strides or the output's shape do not fit")
+    ld_state = _state_rows(state, n_heads * dim * cols, "chunk_scan")
+    dev, H = q.device, n_heads
+    T = torch.empty(n_chunks * H * CHUNK_TOKENS ** 2, dtype=torch.float32, device=dev) if delta else None
+    M = torch.empty(n_chunks * H * CHUNK_TOKENS ** 2, dtype=torch.float32, device=dev)
+    fac = torch.empty(n_chunks * H * (2 * CHUNK_TOKENS + 4), dtype=torch.float32, device=dev)
+    fn = _fn("chunk_scan", "lgml_chunk_prepare", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                                                  c_int, c_int, c_int, c_int, c_void_p])
+    _check("chunk_scan", fn(_ptr(q), _ptr(k), q.stride(0), _ptr(log_a), _ptr(w), w.stride(0), head_stride, _ptr(chunks.rows), _ptr(T), _ptr(M), _ptr(fac),
+                            n_chunks, H, n_kv_heads, dim, 1 if delta else 0, _stream()), "chunk_prepare")
+    fn = _fn("chunk_scan", "lgml_chunk_scan", [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                               c_longlong, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check("chunk_scan", fn(_ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(T), _ptr(M), _ptr(fac), _ptr(chunks.rows), _ptr(chunks.first), _ptr(chunks.requests),
+                            _ptr(state), ld_state, s_row, s_col, _ptr(slots), _ptr(out), H * cols, n_req, H, n_kv_heads, dim, v_cols, cols,
+                            1 if delta else 0, _stream()), "chunk_scan")
+
+
 def delta_head_prepare(qkv: torch.Tensor, a_pre: torch.Tensor, b_pre: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, n_heads: int,
                        n_kv_heads: int, dim: int) -> torch.Tensor:
     """One decay per head: q and k of ``qkv`` float32 [tokens, q (G D) | k (G D) | v ...] become unit vectors in place (q also times
-    D^-1/2); returns float32 [tokens, H, 4] = (exp(-exp(A_log) softplus(a + dt_bias)), sigmoid(b), 0, 0).  a and b float32
+    D^-1/2); returns float32 [tokens, H, 4] = (exp(l), sigmoid(b), l, 0), l = -exp(A_log) softplus(a + dt_bias).  a and b float32
     [tokens, H], possibly column slices."""
     _need(qkv, "convolved q, k, v", torch.float32, 2)
     _need(a_pre, "decay input", torch.float32, 2)
@@ -1648,12 +1706,13 @@ def delta_prepare(proj: torch.Tensor, a_pre: torch.Tensor, conv_w: torch.Tensor,
 
 
 def delta_scan(qkv_c: torch.Tensor, gb: torch.Tensor, state: torch.Tensor, seq_start: torch.Tensor, slots: torch.Tensor,
-               n_heads: int, n_kv_heads: int, dim: int, vdim: int) -> torch.Tensor:
+               n_heads: int, n_kv_heads: int, dim: int, vdim: int, chunks=None) -> torch.Tensor:
     """The recurrence S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q over each request's
     tokens in order, from and into its slot of ``state`` (S of head h at floats [h D Dv, (h + 1) D Dv)).
     ``qkv_c`` [tokens, q | k | v] and ``gb`` [tokens, H, D + 4] (per head the decays, then beta) as
-    ``delta_prepare`` returns them, or [tokens, H, 4] (one decay per head, beta, zeros) as ``delta_head_prepare`` does.
-    Returns o float32 [tokens, H Dv]."""
+    ``delta_prepare`` returns them, or [tokens, H, 4] (one decay per head, beta, its logarithm, zero) as ``delta_head_prepare`` does.
+    Returns o float32 [tokens, H Dv].  ``chunks`` (one decay per head) as for ``chunk_scan``: the requests with many tokens take
+    that form (where the sizes allow), the others the sequential one."""
     n = qkv_c.shape[0]
     head_decay = gb.dim() == 3 and gb.shape[2] == 4
     _need(qkv_c, "prepared q, k, v", torch.float32, 2)
@@ -1664,9 +1723,18 @@ def delta_scan(qkv_c: torch.Tensor, gb: torch.Tensor, state: torch.Tensor, seq_s
         raise KernelError("delta_scan: shapes disagree")
     o = torch.empty((n, n_heads * vdim), dtype=torch.float32, device=qkv_c.device)
     fn = _fn("delta_rule", "lgml_delta_scan_form", [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                                    c_int, c_int, c_int, c_int, c_void_p], label="delta_scan")
+                                                    c_int, c_int, c_int, c_int, c_int, c_void_p], label="delta_scan")
+    max_tokens = 0
+    if chunks is not None and head_decay and n:
+        gd = n_kv_heads * dim
+        q, k, rows = qkv_c[:, :gd], qkv_c[:, gd:2 * gd], gb.view(n, 4 * n_heads)
+        if chunk_scan_supports(q, k, dim, True):
+            chunk_scan(q, k, qkv_c[:, 2 * gd:], rows[:, 2:], rows[:, 1:], 4, state, vdim, 1, chunks, slots, o, n_heads, n_kv_heads, dim, vdim, vdim, True)
+            if not chunks.short:
+                return o
+            max_tokens = chunks.longer_than
     _check("delta_rule", fn(_ptr(qkv_c), _ptr(gb), _ptr(state), state.stride(0), _ptr(seq_start), _ptr(slots), _ptr(o),
-                            slots.numel(), n_heads, n_kv_heads, dim, vdim, 1 if head_decay else 0, _stream()), "delta_scan")
+                            slots.numel(), n_heads, n_kv_heads, dim, vdim, 1 if head_decay else 0, max_tokens, _stream()), "delta_scan")
     return o
 
 

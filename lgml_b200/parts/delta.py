@@ -131,7 +131,8 @@ class HeadDelta(Part):
                        batch.slots, qkv, act="silu")
         g0, b0, a0 = C, C + H * Dv, C + H * Dv + H
         gb = ops.delta_head_prepare(qkv, proj[:, a0:a0 + H], proj[:, b0:b0 + H], self.a_log, self.dt_bias, H, G, D)
-        o = ops.delta_scan(qkv, gb, cache.state, batch.seq_start, batch.slots, H, G, D, Dv)
+        chunks = batch.scan_chunks(ops.CHUNK_TOKENS, ops.CHUNK_FROM) if batch.max_q_len > ops.CHUNK_FROM else None
+        o = ops.delta_scan(qkv, gb, cache.state, batch.seq_start, batch.slots, H, G, D, Dv, chunks=chunks)
         y = ops.delta_output(o, self.norm_w, proj[:, g0:g0 + H * Dv], self.eps, rt.dtype, H, act="silu")
         return rt.linear(y, self.wo, partials_ok=True)
 

@@ -325,7 +325,9 @@ class MatrixMemory(_OwnOut):
         gates = ops.memory_gates(proj[:, i0:i0 + H], proj[:, i0 + H:i0 + 2 * H], self.gate_cap, cache.state[:, self.m_off:self.m_off + H],
                                  batch.seq_start, batch.slots)
         pieces = batch.scan_pieces(ops.SSD_PIECE_TOKENS) if batch.max_q_len > SSD_PIECES_FROM else None
-        y = ops.memory_scan(proj[:, :vkq], gates, cache.state, batch.seq_start, batch.slots, H, D, Dv, pieces=pieces)
+        chunks = batch.scan_chunks(ops.CHUNK_TOKENS, ops.CHUNK_FROM) if batch.max_q_len > ops.CHUNK_FROM else None
+        y = ops.memory_scan(proj[:, :vkq], gates, cache.state, batch.seq_start, batch.slots, H, D, Dv, pieces=pieces,
+                            chunks=chunks)
         ops.memory_output(y, gates, D ** -0.5, self.norm_w, proj[:, g0:g0 + H * Dv], self.eps, out)
 
 

@@ -40,6 +40,22 @@ def batch_of(lens):
     return i32([r for r, n in enumerate(lens) for _ in range(n)]), i32(np.concatenate([[0], np.cumsum(lens)]))
 
 
+def chunks_of(lens, longer_than=16):
+    """The description of a step's long requests for the chunked recurrences."""
+    from lgml_b200.engine.batch import ScanChunks
+
+    rows, first, reqs, start = [], [0], [], 0
+    for r, n in enumerate(lens):
+        if n > longer_than:
+            rows += [(start + t, start + min(t + 64, n)) for t in range(0, n, 64)]
+            first.append(len(rows))
+            reqs.append(r)
+        start += n
+    if not reqs:
+        return None
+    return ScanChunks(i32(np.array(rows).reshape(-1)).view(-1, 2), i32(first), i32(reqs), longer_than, len(reqs) < len(lens))
+
+
 def portions_of(total, cuts):
     out, a, i = [], 0, 0
     while a < total:
@@ -254,7 +270,7 @@ def test_delta_rule_with_one_decay_per_head_in_pieces(H_, G, D, Dv):
     want = P.delta_scan(q, k, raw[:, 2 * G * D:].reshape(n, H_, Dv), P.sigmoid(b), g)
     ab = f32(np.concatenate([a, b], axis=1))
     state = torch.zeros((3, off + 8), device=DEV)
-    for cuts in ([330], [64, 2, 130, 3], [1, 2, 70], [33, 31, 65]):
+    for chunked, cuts in [(f, c) for f in (False, True) for c in ([330], [64, 2, 130, 3], [1, 2, 70], [33, 31, 65])]:
         state.zero_()
         other = 0
         got = np.zeros_like(want)
@@ -269,9 +285,9 @@ def test_delta_rule_with_one_decay_per_head_in_pieces(H_, G, D, Dv):
             _, starts = batch_of(lens)
             qkv = f32(rows)
             gb = ops.delta_head_prepare(qkv, gates[:, :H_], gates[:, H_:], f32(a_log), f32(dt_bias), H_, G, D)
-            o = ops.delta_scan(qkv, gb, state, starts, i32(slots), H_, G, D, Dv)
+            o = ops.delta_scan(qkv, gb, state, starts, i32(slots), H_, G, D, Dv, chunks=chunks_of(lens) if chunked else None)
             got[s:e] = o[-(e - s):].cpu().numpy().reshape(-1, H_, Dv)
-        close_to(got, want, 2e-5, str(cuts))
+        close_to(got, want, 2e-5, f"{cuts} {'chunks' if chunked else 'token by token'}")
         assert bool((state[:, off:] == 0).all()) and bool((state[2] == 0).all())
 
 
@@ -288,7 +304,7 @@ def test_output_norm_with_the_silu_gate(out_dtype):
         close_to(y.float().cpu(), want, 1e-5 if out_dtype == torch.float32 else 1e-2, act)
 
 
-@pytest.mark.parametrize("H_,D,Dv", [(2, 16, 24), (1, 5, 9), (3, 64, 64), (2, 128, 130), (4, 33, 7), (1, 300, 20)])
+@pytest.mark.parametrize("H_,D,Dv", [(2, 16, 24), (1, 5, 9), (3, 64, 64), (2, 128, 130), (4, 40, 257), (4, 33, 7), (1, 300, 20)])
 def test_matrix_memory_in_portions_pieces_and_single_tokens(H_, D, Dv):
     """Gates of both signs far into their cap; a head whose input gates are so low that exp(-m) decides the denominator for long;
     a head that never forgets, asked at the end for what the first tokens wrote."""
@@ -307,10 +323,10 @@ def test_matrix_memory_in_portions_pieces_and_single_tokens(H_, D, Dv):
     want = P.rms_unit(o, 1e-6).reshape(n, -1) * w * P.sigmoid(gate)
     # m from 0, not from minus infinity: the first token of head 0 shows it
     assert np.abs(o[0, 0] * (np.exp(-max(f[0, 0], i[0, 0])) + 1e-6) - np.exp(i[0, 0] - max(f[0, 0], i[0, 0])) * v[0, 0] * (q[0, 0] @ k[0, 0]) * D ** -0.5).max() < 1e-9
-    proj = f32(np.concatenate([v.reshape(n, -1), k.reshape(n, -1), q.reshape(n, -1), zi, zf], axis=1))
     wide = H_ * (Dv + 2 * D)
+    proj = f32(np.concatenate([v.reshape(n, -1), k.reshape(n, -1), q.reshape(n, -1), zi, zf, np.zeros((n, -(wide + 2 * H_) % 4))], axis=1))
     m_off = H_ * (Dv + 1) * D
-    for cuts in ([400], [150, 2, 248], [1, 2, 3, 90], [64, 65]):
+    for chunked, cuts in [(f, c) for f in (False, True) for c in ([400], [150, 2, 248], [1, 2, 3, 90], [64, 65])]:
         state = torch.full((3, m_off + H_ + 3), 5.0, device=DEV)
         state[[0, 2], :m_off + H_] = 0.0
         got = np.zeros_like(want)
@@ -320,12 +336,12 @@ def test_matrix_memory_in_portions_pieces_and_single_tokens(H_, D, Dv):
             lens, slots = [m, 4], [2, 0]                     # a second request of four tokens in every step
             rows = torch.cat([proj[s:e], proj[:4]])
             _, starts = batch_of(lens)
-            gates = ops.memory_gates(rows[:, wide:wide + H_], rows[:, wide + H_:], cap, state[:, m_off:m_off + H_], starts, i32(slots))
+            gates = ops.memory_gates(rows[:, wide:wide + H_], rows[:, wide + H_:wide + 2 * H_], cap, state[:, m_off:m_off + H_], starts, i32(slots))
             pieces = None
             if m > 128:
                 cutp = [(t, min(t + 64, m)) for t in range(0, m, 64)] + [(m, m + 4)]
                 pieces = (i32(np.array(cutp).reshape(-1)).view(-1, 2), i32([0, len(cutp) - 1, len(cutp)]))
-            y = ops.memory_scan(rows[:, :wide], gates, state, starts, i32(slots), H_, D, Dv, pieces=pieces)
+            y = ops.memory_scan(rows[:, :wide], gates, state, starts, i32(slots), H_, D, Dv, pieces=pieces, chunks=chunks_of(lens) if chunked else None)
             out = torch.empty((m + 4, H_ * Dv), device=DEV)
             ops.memory_output(y, gates, D ** -0.5, f32(w), torch.cat([f32(gate[s:e]), f32(gate[:4])]), 1e-6, out)
             got[s:e] = out[:m].cpu().numpy()
@@ -333,7 +349,7 @@ def test_matrix_memory_in_portions_pieces_and_single_tokens(H_, D, Dv):
         size = np.sqrt((o ** 2).mean(axis=-1))
         err = np.abs(got - want).reshape(n, H_, Dv).max(axis=-1)
         bound = 3e-4 * (1 + np.abs(want).max()) * np.maximum(1.0, 0.02 / size)
-        assert (err < bound).all(), f"{cuts}: {np.unravel_index(int((err / bound).argmax()), err.shape)} {(err / bound).max():.3g}"
+        assert (err < bound).all(), f"{cuts} {chunked}: {np.unravel_index(int((err / bound).argmax()), err.shape)} {(err / bound).max():.3g}"
         assert bool((state[1] == 5.0).all()) and bool((state[:, m_off + H_:] == 5.0).all())
 
 
@@ -351,7 +367,7 @@ def test_gates_of_a_long_portion_are_those_of_single_tokens():
     i, f, m = P.soft_capped(zi, cap), P.log_sigmoid(P.soft_capped(zf, cap)), np.zeros(H_)
     for t in range(n):
         before, m = m, np.maximum(f[t] + m, i[t])
-        close_to(whole[t].cpu(), np.concatenate([np.exp(f[t] + before - m), np.exp(i[t] - m), np.exp(-m)]), 2e-5, str(t))
+        close_to(whole[t].cpu(), np.concatenate([np.exp(f[t] + before - m), np.exp(i[t] - m), np.exp(-m), f[t] + before - m]), 2e-5, str(t))
 
 
 # ---------------------------------------------------------------------------------------------
