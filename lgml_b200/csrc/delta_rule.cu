@@ -342,26 +342,56 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(
         }
 }
 
+__device__ __forceinline__ void store_quad(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+__device__ __forceinline__ void store_quad(__nv_bfloat16 *p, float4 v) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    float2 raw;
+    raw.x = *reinterpret_cast<float *>(&lo), raw.y = *reinterpret_cast<float *>(&hi);
+    *reinterpret_cast<float2 *>(p) = raw;
+}
+
+// A warp takes a (token, head); vec: 16-byte accesses, heads of up to 512 in registers between the two walks.
 template <typename T>
 __global__ void __launch_bounds__(128) delta_output_kernel(const float *__restrict__ o, const float *__restrict__ weight,
-                                                           const float *__restrict__ gate, int ldg, T *__restrict__ out, int ldo, int H,
-                                                           int Dv, float eps, int act) {
+                                                           const float *__restrict__ gate, int ldg, T *__restrict__ out, int ldo, int n_tokens, int H,
+                                                           int Dv, float eps, int act, int vec) {
     pdl_trigger();
     pdl_wait();
-    __shared__ float red[32];
-    const int t = blockIdx.x, h = blockIdx.y;
-    const float *row = o + ((size_t)t * H + h) * Dv;
-    float ss = 0.f;
-    for (int d = threadIdx.x; d < Dv; d += blockDim.x) {
-        const float v = act_load(row + d);
-        ss = fmaf(v, v, ss);
-    }
-    ss = block_sum(ss, red);
-    const float inv = 1.0f / sqrtf(ss / (float)Dv + eps);
-    for (int d = threadIdx.x; d < Dv; d += blockDim.x) {
-        const float z = act_load(gate + (size_t)t * ldg + (size_t)h * Dv + d);
-        const float v = act_load(row + d) * inv * weight[d] * (act ? z * sigmoid_f(z) : sigmoid_f(z));
-        out[(size_t)t * ldo + (size_t)h * Dv + d] = from_f32<T>(v);
+    const int lane = threadIdx.x & 31;
+    const long long total = (long long)n_tokens * H;
+    for (long long u = (long long)blockIdx.x * 4 + (threadIdx.x >> 5); u < total; u += (long long)gridDim.x * 4) {
+        const int t = (int)(u / H), h = (int)(u - (long long)t * H);
+        const float *row = o + u * Dv, *grow = gate + (size_t)t * ldg + (size_t)h * Dv;
+        T *orow = out + (size_t)t * ldo + (size_t)h * Dv;
+        auto gated = [&](float z) { return act ? z * sigmoid_f(z) : sigmoid_f(z); };
+        float ss = 0.f;
+        if (vec) {
+            float4 v[4], z[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int d = (i * 32 + lane) * 4;
+                v[i] = z[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (d < Dv) v[i] = act_load(reinterpret_cast<const float4 *>(row + d)), z[i] = act_load(reinterpret_cast<const float4 *>(grow + d));
+                ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
+            }
+            const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)Dv + eps);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int d = (i * 32 + lane) * 4;
+                if (d < Dv) {
+                    const float4 w = __ldg(reinterpret_cast<const float4 *>(weight + d));
+                    store_quad(orow + d, make_float4(v[i].x * inv * w.x * gated(z[i].x), v[i].y * inv * w.y * gated(z[i].y), v[i].z * inv * w.z * gated(z[i].z),
+                                                     v[i].w * inv * w.w * gated(z[i].w)));
+                }
+            }
+            continue;
+        }
+        for (int d = lane; d < Dv; d += 32) {
+            const float v = act_load(row + d);
+            ss = fmaf(v, v, ss);
+        }
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)Dv + eps);
+        for (int d = lane; d < Dv; d += 32) orow[d] = from_f32<T>(act_load(row + d) * inv * weight[d] * gated(act_load(grow + d)));
     }
 }
 
@@ -469,11 +499,14 @@ LGML_API int lgml_delta_output_act(const float *o, const float *weight, const fl
     LGML_REQUIRE(n_tokens >= 0 && H > 0 && Dv > 0 && H <= 65535, "delta_output: bad sizes");
     LGML_REQUIRE(ldg >= H * Dv && ldo >= H * Dv, "delta_output: a row stride is below H Dv");
     if (n_tokens == 0) return 0;
-    dim3 grid(n_tokens, H);
+    const long long blocks = ((long long)n_tokens * H + 3) / 4;
+    const int grid = (int)(blocks < 148 * 32 ? blocks : 148 * 32);
+    const int vec = Dv % 4 == 0 && Dv <= 512 && ldg % 4 == 0 && ldo % 4 == 0 &&
+                    (((uintptr_t)o | (uintptr_t)weight | (uintptr_t)gate | (uintptr_t)out) & 15) == 0;
     if (dtype == LGML_F32)
-        lgml_launch(delta_output_kernel<float>, grid, 128, 0, stream, o, weight, gate, ldg, (float *)out, ldo, H, Dv, eps, act);
+        lgml_launch(delta_output_kernel<float>, grid, 128, 0, stream, o, weight, gate, ldg, (float *)out, ldo, n_tokens, H, Dv, eps, act, vec);
     else if (dtype == LGML_BF16)
-        lgml_launch(delta_output_kernel<__nv_bfloat16>, grid, 128, 0, stream, o, weight, gate, ldg, (__nv_bfloat16 *)out, ldo, H, Dv, eps, act);
+        lgml_launch(delta_output_kernel<__nv_bfloat16>, grid, 128, 0, stream, o, weight, gate, ldg, (__nv_bfloat16 *)out, ldo, n_tokens, H, Dv, eps, act, vec);
     else
         LGML_FAIL("delta_output: unknown type %d", dtype);
     return lgml_launch_status("delta_output");

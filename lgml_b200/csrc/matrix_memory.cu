@@ -16,7 +16,7 @@
 LGML_DEFINE_LAST_ERROR(lgml_matrix_memory)
 
 namespace {
-constexpr int GATE_THREADS = 128;
+constexpr int GATE_THREADS = 512;       // at most; fewer when a step brings few tokens a request
 
 __device__ __forceinline__ float capped(float z, float cap) { return cap * tanhf(z / cap); }
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
@@ -30,15 +30,16 @@ __global__ void __launch_bounds__(GATE_THREADS) memory_gates_kernel(const float 
     pdl_trigger();
     pdl_wait();
     __shared__ float Fs[GATE_THREADS], Is[GATE_THREADS], Ms[GATE_THREADS];
-    const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+    const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, threads = blockDim.x;
     const int t0 = seq_start[s], n = seq_start[s + 1] - t0;
     if (n <= 0) return;
     float *ms = m_state + (size_t)slots[s] * state_ld + h;
     const float m0 = act_load(ms);
-    const int per = (n + GATE_THREADS - 1) / GATE_THREADS;
+    const int per = (n + threads - 1) / threads;
     const int first = min(tid * per, n), last = min(first + per, n);
     const int ldg = 4 * H;
     float F = 0.f, I = -INFINITY;
+#pragma unroll 4
     for (int t = first; t < last; ++t) {
         const float i = capped(act_load(zi + (size_t)(t0 + t) * ldz + h), cap);
         const float f = log_sigmoid(capped(act_load(zf + (size_t)(t0 + t) * ldz + h), cap));
@@ -49,7 +50,7 @@ __global__ void __launch_bounds__(GATE_THREADS) memory_gates_kernel(const float 
     }
     Fs[tid] = F, Is[tid] = I;
     __syncthreads();
-    for (int o = 1; o < GATE_THREADS; o <<= 1) {        // inclusive scan: the earlier map first
+    for (int o = 1; o < threads && o < n; o <<= 1) {        // inclusive scan: the earlier map first
         float Fp = 0.f, Ip = -INFINITY;
         const bool have = tid >= o;
         if (have) Fp = Fs[tid - o], Ip = Is[tid - o];
@@ -127,10 +128,11 @@ __global__ void __launch_bounds__(128) memory_output_kernel(const float *__restr
 
 // zi, zf: float32 rows of H entries, ldz apart; m_state: the first slot's m of head 0, slots state_ld apart; gates float32 [n, 4 H].
 LGML_API int lgml_memory_gates(const float *zi, const float *zf, int ldz, float cap, float *m_state, long long state_ld, const int *seq_start,
-                               const int *slots, float *gates, int n_seqs, int H, cudaStream_t stream) {
+                               const int *slots, float *gates, int n_tokens, int n_seqs, int H, cudaStream_t stream) {
     LGML_REQUIRE(n_seqs >= 0 && H > 0 && H <= 65535 && ldz >= H && cap > 0.f, "memory_gates: bad sizes");
     if (n_seqs == 0) return 0;
-    lgml_launch(memory_gates_kernel, dim3(n_seqs, H), GATE_THREADS, 0, stream, zi, zf, ldz, cap, m_state, state_ld, seq_start, slots, gates, H);
+    const int threads = n_tokens == n_seqs ? 32 : (n_tokens / n_seqs <= 256 ? 128 : GATE_THREADS);
+    lgml_launch(memory_gates_kernel, dim3(n_seqs, H), threads, 0, stream, zi, zf, ldz, cap, m_state, state_ld, seq_start, slots, gates, H);
     return lgml_launch_status("memory_gates");
 }
 

@@ -26,53 +26,11 @@ LGML_DEFINE_LAST_ERROR(lgml_moe)
 
 namespace {
 
-template <typename T>
-__global__ void __launch_bounds__(128) moe_router_kernel(const T *__restrict__ h, int ldh, const float *__restrict__ wr, const float *__restrict__ br,
-                                                         int *__restrict__ ids, float *__restrict__ wts, int E, int X, int top, int mode,
-                                                         float route_scale, int n_extra, float *__restrict__ extra, int n_identity,
-                                                         float *__restrict__ identity_w) {
-    pdl_trigger();
-    pdl_wait();
-    // X choice values (+ n_extra logits of rows that are no experts), X scores (mode 1), then the token's row (E floats, from a 16-byte boundary)
-    extern __shared__ __align__(16) float rsm[];
-    const int zn = (X + n_extra + 3) & ~3;
-    float *z = rsm, *sc = rsm + zn, *hs = rsm + 2 * zn;
-    const int t = blockIdx.x;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
-    const T *row = h + (size_t)t * ldh;
-    for (int k = threadIdx.x; k < E; k += blockDim.x) hs[k] = to_f32(act_load(row + k));
-    __syncthreads();
-    // one order of summation whatever the batch: lane l takes elements 4 l .. 4 l + 3 of every run of 128, then the warp's tree
-    const bool vec = (E % 4 == 0) && ((reinterpret_cast<uintptr_t>(wr) & 15) == 0);
-    for (int e = warp; e < X + n_extra; e += n_warps) {
-        const float *w = wr + (size_t)e * E;
-        float dot = 0.f;
-        if (vec) {
-#pragma unroll 4
-            for (int k = lane * 4; k < E; k += 128) {
-                const float4 a = *reinterpret_cast<const float4 *>(hs + k), b = __ldg(reinterpret_cast<const float4 *>(w + k));
-                dot = fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, dot))));
-            }
-        } else {
-            for (int k = lane; k < E; k += 32) dot = fmaf(hs[k], w[k], dot);
-        }
-        dot = warp_sum(dot);
-        if (lane == 0) {
-            if (e >= X) {
-                // rows behind the experts': a gate of the token (sigmoid of its logit), for the caller
-                extra[(size_t)t * n_extra + (e - X)] = 1.0f / (1.0f + expf(-dot));
-            } else if (mode == 1) {
-                // scores are sigmoids; the bias only corrects the choice, the weights use the plain scores
-                const float sg = 1.0f / (1.0f + expf(-dot));
-                sc[e] = sg;
-                z[e] = sg + (br ? br[e] : 0.f);
-            } else {
-                z[e] = dot + (br && mode == 0 ? br[e] : 0.f);
-            }
-        }
-    }
-    __syncthreads();
-    if (warp != 0) return;
+// One warp chooses a token's experts.  z: mode 0 and 1 the choice values, mode 2 the logits (z and sc are used up); sc: mode 1 the
+// scores, mode 2 room for them.
+__device__ __forceinline__ void select_experts(float *z, float *sc, const float *__restrict__ br, int *__restrict__ ids, float *__restrict__ wts, int t, int X,
+                                               int top, int mode, float route_scale, int n_identity, float *__restrict__ identity_w) {
+    const int lane = threadIdx.x & 31;
     float zmax = 0.f, sum = 0.f, own = 0.f;
     if (mode == 2) {
         // scores over all logits (z holds them without the bias)
@@ -122,6 +80,71 @@ __global__ void __launch_bounds__(128) moe_router_kernel(const T *__restrict__ h
     if (identity_w != nullptr && lane == 0) identity_w[t] = own * inv;
     __syncwarp();
     for (int s = lane; s < top; s += 32) wts[(size_t)t * top + s] *= inv;
+}
+
+// The choice alone, from logits that a product has computed (mode 2): z_in rows of X floats, ldz apart.  A warp a token.
+constexpr int SEL_WARPS = 4;
+__global__ void __launch_bounds__(SEL_WARPS * 32) moe_select_kernel(const float *__restrict__ z_in, int ldz, const float *__restrict__ br, int *__restrict__ ids,
+                                                                    float *__restrict__ wts, int n_tokens, int X, int top, float route_scale, int n_identity,
+                                                                    float *__restrict__ identity_w) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ __align__(16) float ssm[];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = blockIdx.x * SEL_WARPS + warp;
+    if (t >= n_tokens) return;
+    float *z = ssm + (size_t)warp * 2 * X, *sc = z + X;
+    for (int e = lane; e < X; e += 32) z[e] = act_load(z_in + (size_t)t * ldz + e);
+    __syncwarp();
+    select_experts(z, sc, br, ids, wts, t, X, top, 2, route_scale, n_identity, identity_w);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) moe_router_kernel(const T *__restrict__ h, int ldh, const float *__restrict__ wr, const float *__restrict__ br,
+                                                         int *__restrict__ ids, float *__restrict__ wts, int E, int X, int top, int mode,
+                                                         float route_scale, int n_extra, float *__restrict__ extra, int n_identity,
+                                                         float *__restrict__ identity_w) {
+    pdl_trigger();
+    pdl_wait();
+    // X choice values (+ n_extra logits of rows that are no experts), X scores (mode 1), then the token's row (E floats, from a 16-byte boundary)
+    extern __shared__ __align__(16) float rsm[];
+    const int zn = (X + n_extra + 3) & ~3;
+    float *z = rsm, *sc = rsm + zn, *hs = rsm + 2 * zn;
+    const int t = blockIdx.x;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+    const T *row = h + (size_t)t * ldh;
+    for (int k = threadIdx.x; k < E; k += blockDim.x) hs[k] = to_f32(act_load(row + k));
+    __syncthreads();
+    // one order of summation whatever the batch: lane l takes elements 4 l .. 4 l + 3 of every run of 128, then the warp's tree
+    const bool vec = (E % 4 == 0) && ((reinterpret_cast<uintptr_t>(wr) & 15) == 0);
+    for (int e = warp; e < X + n_extra; e += n_warps) {
+        const float *w = wr + (size_t)e * E;
+        float dot = 0.f;
+        if (vec) {
+#pragma unroll 4
+            for (int k = lane * 4; k < E; k += 128) {
+                const float4 a = *reinterpret_cast<const float4 *>(hs + k), b = __ldg(reinterpret_cast<const float4 *>(w + k));
+                dot = fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, dot))));
+            }
+        } else {
+            for (int k = lane; k < E; k += 32) dot = fmaf(hs[k], w[k], dot);
+        }
+        dot = warp_sum(dot);
+        if (lane == 0) {
+            if (e >= X) {
+                // rows behind the experts': a gate of the token (sigmoid of its logit), for the caller
+                extra[(size_t)t * n_extra + (e - X)] = 1.0f / (1.0f + expf(-dot));
+            } else if (mode == 1) {
+                // scores are sigmoids; the bias only corrects the choice, the weights use the plain scores
+                const float sg = 1.0f / (1.0f + expf(-dot));
+                sc[e] = sg;
+                z[e] = sg + (br ? br[e] : 0.f);
+            } else {
+                z[e] = dot + (br && mode == 0 ? br[e] : 0.f);
+            }
+        }
+    }
+    __syncthreads();
+    if (warp == 0) select_experts(z, sc, br, ids, wts, t, X, top, mode, route_scale, n_identity, identity_w);
 }
 
 // dot products of `NF` weight rows (bfloat16, 16-byte loads) with one float32 vector in shared memory: the loads of all rows of a
@@ -315,6 +338,18 @@ LGML_API int lgml_moe_router_form(const void *h, int dtype, int ldh, const float
     else
         LGML_FAIL("moe_router: unknown type %d", dtype);
     return lgml_launch_status("moe_router");
+}
+
+// The choice from ready logits: z float32 rows of X entries, ldz apart; scores = softmax over all of them, as mode 2 above.
+LGML_API int lgml_moe_select(const float *z, int ldz, const float *br, int *ids, float *wts, int n_tokens, int X, int top, int n_identity, float *identity_w,
+                             cudaStream_t stream) {
+    LGML_REQUIRE(n_tokens >= 0 && X > 0 && X <= 4096 && top > 0 && top <= X && ldz >= X && n_identity >= 0 && n_identity <= X, "moe_select: bad sizes");
+    if (n_tokens == 0) return 0;
+    const size_t smem = sizeof(float) * 2 * SEL_WARPS * (size_t)X;
+    if (need_smem(moe_select_kernel, smem, "moe_select")) return -1;
+    lgml_launch(moe_select_kernel, (n_tokens + SEL_WARPS - 1) / SEL_WARPS, SEL_WARPS * 32, smem, stream, z, ldz, br, ids, wts, n_tokens, X, top, 1.0f,
+                n_identity, identity_w);
+    return lgml_launch_status("moe_select");
 }
 
 LGML_API int lgml_moe_router_mode(const void *h, int dtype, int ldh, const float *wr, const float *br, int *ids, float *wts, int n_tokens, int E, int X,

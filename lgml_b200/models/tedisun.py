@@ -47,7 +47,7 @@ def feed_forward_of(cfg: TedisunConfig, mlp):
         return None
     r = mlp["router"]
     return make_part("feed_forward", "routed_experts", width=cfg.width, inner=mlp["expert"]["ff"], n_experts=r["experts"], top=r["top"],
-                     router="softmax_all", n_identity=r.get("identity", 0), bias_name=".correction")
+                     router="softmax_all", n_identity=r.get("identity", 0), bias_name=".correction", router_rows=True)
 
 
 def build_tedisun(cfg: TedisunConfig) -> DecoderModel:

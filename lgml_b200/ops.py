@@ -868,6 +868,26 @@ def moe_router(h: torch.Tensor, w_router: torch.Tensor, b_router: Optional[torch
     return (ids, wts, extra) if n_extra else (ids, wts)
 
 
+def moe_select(z: torch.Tensor, b_router: Optional[torch.Tensor], top: int, n_identity: int = 0):
+    """The choice of ``moe_router`` in mode "softmax_all" from logits that a product has computed: z float32 [tokens, X] (may be a
+    column slice).  Returns what ``moe_router`` does."""
+    _need(z, "router logits", torch.float32, 2)
+    ldz = _rows_contiguous(z, "router logits")
+    n, X = z.shape
+    if not 0 < top <= X or not 0 <= n_identity <= X:
+        raise KernelError(f"moe_select: {top} of {X} experts, {n_identity} of them identities")
+    if b_router is not None:
+        _need(b_router, "router bias", torch.float32, 1)
+        if b_router.numel() != X:
+            raise KernelError("moe_select: one bias per expert")
+    ids = torch.empty((n, top), dtype=torch.int32, device=z.device)
+    wts = torch.empty((n, top), dtype=torch.float32, device=z.device)
+    own = torch.empty(n, dtype=torch.float32, device=z.device) if n_identity else None
+    fn = _fn("moe", "lgml_moe_select", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
+    _check("moe", fn(_ptr(z), ldz, _ptr(b_router), _ptr(ids), _ptr(wts), n, X, int(top), int(n_identity), _ptr(own), _stream()), "moe_select")
+    return (ids, wts, own) if n_identity else (ids, wts)
+
+
 def _also(also, also_w, n: int, E: int, dtype: torch.dtype, who: str):
     """A term every token gets beside its experts' (float32 or the compute type, [tokens, E]) and the token's weight on it
     (float32 [tokens]).  Returns (1 if the term is bfloat16, its row stride)."""
@@ -1527,8 +1547,9 @@ def memory_gates(zi: torch.Tensor, zf: torch.Tensor, cap: float, m_state: torch.
     if tuple(zf.shape) != (n, H) or (n and zf.stride(0) != ldz) or zf.stride(1) != 1 or m_state.shape[1] != H or m_state.stride(1) != 1:
         raise KernelError(f"memory_gates: gates {tuple(zi.shape)} / {tuple(zf.shape)} and maxima {tuple(m_state.shape)} do not fit")
     gates = torch.empty((n, 4 * H), dtype=torch.float32, device=zi.device)
-    fn = _fn("matrix_memory", "lgml_memory_gates", [c_void_p, c_void_p, c_int, c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
-    _check("matrix_memory", fn(_ptr(zi), _ptr(zf), ldz, float(cap), _ptr(m_state), m_state.stride(0), _ptr(seq_start), _ptr(slots), _ptr(gates),
+    fn = _fn("matrix_memory", "lgml_memory_gates", [c_void_p, c_void_p, c_int, c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                                                    c_void_p])
+    _check("matrix_memory", fn(_ptr(zi), _ptr(zf), ldz, float(cap), _ptr(m_state), m_state.stride(0), _ptr(seq_start), _ptr(slots), _ptr(gates), n,
                                slots.numel(), H, _stream()), "memory_gates")
     return gates
 

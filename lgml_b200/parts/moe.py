@@ -18,6 +18,8 @@ Other forms of the same part, by constructor arguments:
 * ``gated=False``: experts without a gate, W_down,e act(W_up,e h) with act = relu squared;
 * ``shared_inner``: one more expert of that inner width and the same form that every token uses
   (``.shared.up``, ``.shared.down``), added times sigmoid(W_sg h), one number per token (``.shared.sg`` [1, E]);
+* ``router_rows``: the router's matrix is a matrix like the others (the compute type; its products are summed in float32) and
+  its rows are offered to the block for a product they can share (``in_rows`` / ``forward_projected``); softmax_all only;
 * ``bias_name``: what the bias's name adds to the part's prefix.
 """
 from __future__ import annotations
@@ -25,7 +27,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from ..weights import VECTOR, TensorSpec
+from ..weights import MATRIX, VECTOR, TensorSpec
 from .base import Part, register_part
 
 
@@ -34,7 +36,7 @@ class RoutedExperts(Part):
 
     def __init__(self, width: int, inner: int, n_experts: int, top: int, router_bias: bool = True, router: str = "softmax",
                  route_scale: float = 1.0, gated: bool = True, shared_inner: int = 0, bias_name: str = ".router.b",
-                 n_identity: int = 0):
+                 n_identity: int = 0, router_rows: bool = False):
         if not 0 < top <= n_experts + n_identity:
             raise ValueError(f"{top} of {n_experts + n_identity} experts cannot be chosen")
         if shared_inner and n_identity:
@@ -43,6 +45,11 @@ class RoutedExperts(Part):
             raise ValueError(f"unknown router '{router}' (known: {', '.join(ops.ROUTER_MODES)})")
         if shared_inner and gated:
             raise ValueError("a shared expert comes only with experts without a gate")
+        if router_rows and router != "softmax_all":
+            raise ValueError("only the softmax over all experts can be taken from ready logits")
+        self.router_rows = bool(router_rows)
+        if router_rows:
+            self.in_rows = self._in_rows
         self.width, self.inner, self.n_experts, self.top = width, inner, n_experts, top
         self.router_bias, self.n_identity = bool(router_bias), int(n_identity)
         self.router, self.route_scale, self.gated = router, float(route_scale), bool(gated)
@@ -52,7 +59,7 @@ class RoutedExperts(Part):
     def tensor_specs(self, prefix):
         E, F = self.width, self.inner
         # the router stays float32 (its logits decide which experts run)
-        specs = [TensorSpec(prefix + ".router", (self.n_experts + self.n_identity, E), VECTOR)]
+        specs = [TensorSpec(prefix + ".router", (self.n_experts + self.n_identity, E), MATRIX if self.router_rows else VECTOR)]
         if self.router_bias:
             specs.append(TensorSpec(prefix + self.bias_name, (self.n_experts + self.n_identity,), VECTOR))
         for e in range(self.n_experts):
@@ -86,7 +93,20 @@ class RoutedExperts(Part):
     def first_weights(self):
         return [self.w_router]
 
+    def _in_rows(self):
+        """The router's rows, padded with zero rows to a multiple of 8."""
+        pad = -self.w_router.shape[0] % 8
+        return torch.cat([self.w_router, self.w_router.new_zeros((pad, self.width))], dim=0), None
+
+    def forward_projected(self, rt, h, proj):
+        """``proj``: float32 [tokens, >= experts], the router's logits in its first columns."""
+        chosen = ops.moe_select(proj[:, :self.n_experts + self.n_identity], self.b_router, self.top, self.n_identity)
+        also, also_w = (h, chosen[2]) if self.n_identity else (None, None)
+        return rt.moe_experts(h, chosen[0], chosen[1], self.w_gu, self.wd, gated=self.gated, also=also, also_w=also_w)
+
     def forward(self, rt, h):
+        if self.router_rows:
+            return self.forward_projected(rt, h, rt.linear(h, self.w_router, out_dtype=torch.float32))
         also = also_w = None
         if self.shared_inner:
             ids, wts, also_w = ops.moe_router(h, self.w_router, self.b_router, self.top, self.router, self.route_scale, n_extra=1)

@@ -154,7 +154,8 @@ class HyperBlock(Part):
     def forward(self, rt, x, pending, batch, cache):
         h = self.mixer_norm.forward(rt, x, rt.dtype, delta=pending, w_in=self.mixer_hyper.w_in)
         if self.ffn is not None:
-            rt.ahead(self.ffn.first_weights())
+            stacked = self._in.get("ffn")
+            rt.ahead([stacked[0]] if stacked is not None else self.ffn.first_weights())       # read after the mixer: L2 may fetch it meanwhile
         y, gate = self._sublayer(rt, "mixer", self.mixer, h, batch, cache)
         pending = PendingStreams(delta=y, gate=gate, w_out=self.mixer_hyper.w_out, mix=self.mixer_hyper.mix)
         if self.ffn is not None:

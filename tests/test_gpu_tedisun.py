@@ -392,7 +392,12 @@ def test_router_and_experts_some_of_which_return_their_input(dtype, X, I, top, E
     dev = lambda a: torch.tensor(a, dtype=dtype, device=DEV)
     ids, wts = P.route(h, W, "p", top)
     got = ops.moe_router(dev(h), f32(W["p.router"]), f32(W["p.correction"]), top, "softmax_all", n_identity=I)
+    z = torch.zeros((n, X + I + 3), device=DEV)
+    z[:, 1:1 + X + I] = f32(h @ W["p.router"].T)
+    ready = ops.moe_select(z[:, 1:1 + X + I], f32(W["p.correction"]), top, n_identity=I)       # the same choice from ready logits
     margin = P.choice_margin(h, W, "p", top) > 1e-5
+    for a, b in zip(got, ready):
+        assert np.allclose(np.sort(a.cpu().numpy().reshape(n, -1)[margin], axis=1), np.sort(b.cpu().numpy().reshape(n, -1)[margin], axis=1), atol=1e-5)
     want_ids = np.where(ids >= X, -1, ids)
     # (the order of the chosen is by falling choice score, but two of them may lie as close as rounding)
     assert np.array_equal(np.sort(got[0].cpu().numpy()[margin], axis=1), np.sort(want_ids[margin], axis=1))
