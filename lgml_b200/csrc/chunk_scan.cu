@@ -29,7 +29,7 @@ LGML_DEFINE_LAST_ERROR(lgml_chunk_scan)
 namespace {
 constexpr int CT = 64;              // tokens of a chunk
 constexpr int LDC = CT + 4;         // floats between rows of a 64-wide matrix in shared memory
-constexpr int THREADS = 256;
+constexpr int PREP_THREADS = 256, SCAN_THREADS = 512;
 constexpr int FAC = 2 * CT + 4;     // per (chunk, head): e^G (64), e^(G_last - G) w (64), e^(G_last), zeros
 
 __device__ __forceinline__ void cp16(float *dst, const float *src, bool valid) {
@@ -39,13 +39,23 @@ __device__ __forceinline__ void cp16(float *dst, const float *src, bool valid) {
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
+// two float32 products-and-sums in one instruction
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+    uint64_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(*reinterpret_cast<uint64_t *>(&a)), "l"(*reinterpret_cast<uint64_t *>(&b)), "l"(*reinterpret_cast<uint64_t *>(&c)));
+    return *reinterpret_cast<float2 *>(&d);
+}
+
 // nt rows of D floats (ld apart) into rows of LD floats; rows nt .. 63 become zeros
+template <int THREADS>
 __device__ __forceinline__ void stage_rows(float *dst, int LD, const float *src, long long ld, int nt, int D, int tid) {
-    const int d4 = D / 4;
-    for (int e = tid; e < CT * d4; e += THREADS) {
-        const int i = e / d4, d = (e - i * d4) * 4;
+    const int d4 = D / 4, di = THREADS / d4, dc = THREADS - di * d4;
+    int i = tid / d4, c = tid - i * d4;
+    while (i < CT) {                            // (one division per call: rows and columns then advance by steps)
         const bool ok = i < nt;
-        cp16(dst + i * LD + d, src + (ok ? (long long)i * ld : 0) + d, ok);
+        cp16(dst + i * LD + c * 4, src + (ok ? (long long)i * ld : 0) + c * 4, ok);
+        i += di, c += dc;
+        if (c >= d4) c -= d4, ++i;
     }
 }
 
@@ -87,7 +97,7 @@ __device__ __forceinline__ void dots_64(const float *A0, const float *A1, const 
 }
 
 template <bool DELTA>
-__global__ void __launch_bounds__(THREADS) chunk_prepare_kernel(const PrepArgs p) {
+__global__ void __launch_bounds__(PREP_THREADS) chunk_prepare_kernel(const PrepArgs p) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float sm[];
@@ -97,8 +107,8 @@ __global__ void __launch_bounds__(THREADS) chunk_prepare_kernel(const PrepArgs p
     float *Ks = sm, *Qs = Ks + CT * LD;
     __shared__ double Gs[2][CT];
     __shared__ float ws[2][CT];
-    stage_rows(Ks, LD, p.k + (size_t)t0 * p.ldx + (size_t)g * D, p.ldx, nt, D, tid);
-    stage_rows(Qs, LD, p.q + (size_t)t0 * p.ldx + (size_t)g * D, p.ldx, nt, D, tid);
+    stage_rows<PREP_THREADS>(Ks, LD, p.k + (size_t)t0 * p.ldx + (size_t)g * D, p.ldx, nt, D, tid);
+    stage_rows<PREP_THREADS>(Qs, LD, p.q + (size_t)t0 * p.ldx + (size_t)g * D, p.ldx, nt, D, tid);
     cp_commit();
     cp_wait<0>();
     __syncthreads();
@@ -152,7 +162,7 @@ __global__ void __launch_bounds__(THREADS) chunk_prepare_kernel(const PrepArgs p
         const int nh = min(2, per - h0);
         for (int hh = 0; hh < nh; ++hh) {
             float *Mo = p.M + ((size_t)c * p.H + g * per + h0 + hh) * CT * CT;
-            for (int e = tid; e < CT * CT; e += THREADS) {
+            for (int e = tid; e < CT * CT; e += PREP_THREADS) {
                 const int i = e >> 6, j = e & 63;
                 float m = 0.f, a = 0.f;
                 if (j <= i && i < nt) {
@@ -207,77 +217,66 @@ struct ScanArgs {
     int v_vec;
 };
 
-// acc[n][r][c] (+)= A_n[row r][k] Bt[col c][k] over this thread's share of k, then added up over the SPLIT lanes that share the
-// tile: the thread ends with TC / SPLIT of the columns.  Rows rg + 16 r.
-template <int NA, int TC, int SPLIT> struct Tile {
-    int rg, cg, sp;
-    __device__ __forceinline__ explicit Tile(int tid) {
-        constexpr int LS = SPLIT == 4 ? 2 : 1;
-        sp = (tid >> 3) & (SPLIT - 1);
-        const int rest = tid >> (3 + LS);
-        rg = (tid & 7) + 8 * (rest & 1);
-        cg = rest >> 1;
-    }
+// own[r][c] = A[row r] . Bt[col c], each lane over its share of the contraction, then added up over the SPLIT lanes that share the
+// tile: a thread ends with TC / SPLIT of the tile's columns.  A thread's rows are rg + (64 / RT) r.
+template <int RT, int TC, int SPLIT> struct Tile {
+    static constexpr int GROUPS = CT / RT;          // row groups
     static constexpr int OWN = TC / SPLIT;
-    __device__ __forceinline__ int col(int c) const {      // the thread's c-th own column
-        return cg * TC + (SPLIT == 4 ? (sp >> 1) * (TC / 2) + (sp & 1) * (TC / 4) : sp * (TC / 2)) + c;
+    static_assert(SPLIT == 4 && TC % 4 == 0, "four lanes share a tile");
+    int rg, cg, sp;
+    __device__ __forceinline__ explicit Tile(int i) {
+        sp = (i >> 3) & 3;
+        const int rest = i >> 5;
+        rg = (i & 7) + 8 * (rest % (GROUPS / 8));
+        cg = rest / (GROUPS / 8);
     }
-    __device__ __forceinline__ void run(const float *A0, const float *A1, int lda, const float *Bt, int ldb, int quads, float (&own)[NA][4][OWN]) const {
-        float acc[NA][4][TC];
+    __device__ __forceinline__ int row(int r) const { return rg + GROUPS * r; }
+    __device__ __forceinline__ int col(int c) const { return cg * TC + (sp >> 1) * (TC / 2) + (sp & 1) * (TC / 4) + c; }      // the thread's c-th own column
+    __device__ __forceinline__ void run(const float *A, int lda, const float *Bt, int ldb, int quads, float (&own)[RT][OWN]) const {
+        float2 acc2[RT][TC];                         // even and odd places of the contraction
 #pragma unroll
-        for (int n = 0; n < NA; ++n)
+        for (int r = 0; r < RT; ++r)
 #pragma unroll
-            for (int r = 0; r < 4; ++r)
-#pragma unroll
-                for (int c = 0; c < TC; ++c) acc[n][r][c] = 0.f;
-        const float *b0 = Bt + (size_t)(cg * TC) * ldb, *a0 = A0 + rg * lda, *a1 = NA > 1 ? A1 + rg * lda : nullptr;
+            for (int c = 0; c < TC; ++c) acc2[r][c] = make_float2(0.f, 0.f);
+        const float *b0 = Bt + (size_t)(cg * TC) * ldb, *a0 = A + rg * lda;
         for (int kq = sp; kq < quads; kq += SPLIT) {
-            float4 a[NA][4];
+            float4 a[RT];
 #pragma unroll
-            for (int r = 0; r < 4; ++r) {
-                a[0][r] = *reinterpret_cast<const float4 *>(a0 + 16 * r * lda + kq * 4);
-                if (NA > 1) a[NA - 1][r] = *reinterpret_cast<const float4 *>(a1 + 16 * r * lda + kq * 4);
-            }
+            for (int r = 0; r < RT; ++r) a[r] = *reinterpret_cast<const float4 *>(a0 + GROUPS * r * lda + kq * 4);
 #pragma unroll
             for (int c = 0; c < TC; ++c) {
                 const float4 b = *reinterpret_cast<const float4 *>(b0 + c * ldb + kq * 4);
 #pragma unroll
-                for (int n = 0; n < NA; ++n)
-#pragma unroll
-                    for (int r = 0; r < 4; ++r)
-                        acc[n][r][c] = fmaf(a[n][r].x, b.x, fmaf(a[n][r].y, b.y, fmaf(a[n][r].z, b.z, fmaf(a[n][r].w, b.w, acc[n][r][c]))));
+                for (int r = 0; r < RT; ++r)
+                    acc2[r][c] = fma2(make_float2(a[r].x, a[r].y), make_float2(b.x, b.y), fma2(make_float2(a[r].z, a[r].w), make_float2(b.z, b.w), acc2[r][c]));
             }
         }
-        constexpr int H1 = TC / 2;
-        const bool up1 = SPLIT == 4 ? (sp >> 1) : sp;
+        float acc[RT][TC];
 #pragma unroll
-        for (int n = 0; n < NA; ++n)
+        for (int r = 0; r < RT; ++r)
 #pragma unroll
-            for (int r = 0; r < 4; ++r) {
-                float half[H1];
+            for (int c = 0; c < TC; ++c) acc[r][c] = acc2[r][c].x + acc2[r][c].y;
+        constexpr int H1 = TC / 2, H2 = TC / 4;
+        const bool up1 = sp >> 1, up2 = sp & 1;
 #pragma unroll
-                for (int c = 0; c < H1; ++c) {
-                    const float send = up1 ? acc[n][r][c] : acc[n][r][c + H1], keep = up1 ? acc[n][r][c + H1] : acc[n][r][c];
-                    half[c] = keep + __shfl_xor_sync(0xffffffffu, send, SPLIT == 4 ? 16 : 8);
-                }
-                if (SPLIT == 4) {
-                    constexpr int H2 = TC / 4;
-                    const bool up2 = sp & 1;
+        for (int r = 0; r < RT; ++r) {
+            float half[H1];
 #pragma unroll
-                    for (int c = 0; c < H2; ++c) {
-                        const float send = up2 ? half[c] : half[c + H2], keep = up2 ? half[c + H2] : half[c];
-                        own[n][r][c] = keep + __shfl_xor_sync(0xffffffffu, send, 8);
-                    }
-                } else {
-#pragma unroll
-                    for (int c = 0; c < OWN; ++c) own[n][r][c] = half[c];
-                }
+            for (int c = 0; c < H1; ++c) {
+                const float send = up1 ? acc[r][c] : acc[r][c + H1], keep = up1 ? acc[r][c + H1] : acc[r][c];
+                half[c] = keep + __shfl_xor_sync(0xffffffffu, send, 16);
             }
+#pragma unroll
+            for (int c = 0; c < H2; ++c) {
+                const float send = up2 ? half[c] : half[c + H2], keep = up2 ? half[c + H2] : half[c];
+                own[r][c] = keep + __shfl_xor_sync(0xffffffffu, send, 8);
+            }
+        }
     }
 };
 
 template <bool DELTA, int CB>
-__global__ void __launch_bounds__(THREADS, 1) chunk_scan_kernel(const ScanArgs p) {
+__global__ void __launch_bounds__(SCAN_THREADS, 1) chunk_scan_kernel(const ScanArgs p) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float sm[];
@@ -296,7 +295,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_scan_kernel(const ScanArgs p
     const int r = blockIdx.z, h = blockIdx.y, g = h / (p.H / p.G), col0 = blockIdx.x * CB;
     const int c0 = p.first_piece[r], c1 = p.first_piece[r + 1];
     float *S_base = p.state + (size_t)p.slots[p.req[r]] * p.state_ld + (size_t)h * D * p.P;
-    for (int e = tid; e < D * CB; e += THREADS) {
+    for (int e = tid; e < D * CB; e += SCAN_THREADS) {
         // (neighbouring threads along the direction in which the state is contiguous)
         const int d = p.s_row == 1 ? e % D : e / CB, c = p.s_row == 1 ? e / D : e % CB;
         St[c * LD + d] = col0 + c < p.P ? act_load(S_base + (size_t)d * p.s_row + (size_t)(col0 + c) * p.s_col) : 0.f;
@@ -304,7 +303,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_scan_kernel(const ScanArgs p
     auto stage_k = [&](int c) {
         if (c < c1) {
             const int t0 = p.pieces[2 * c], nt = p.pieces[2 * c + 1] - t0;
-            stage_rows(Kb + ((c - c0) & 1) * CT * LD, LD, p.k + (size_t)t0 * p.ldx + (size_t)g * D, p.ldx, nt, D, tid);
+            stage_rows<SCAN_THREADS>(Kb + ((c - c0) & 1) * CT * LD, LD, p.k + (size_t)t0 * p.ldx + (size_t)g * D, p.ldx, nt, D, tid);
             const float *f = p.fac + ((size_t)c * p.H + h) * FAC;
             if (tid < FAC / 4) cp16(Fs + ((c - c0) & 1) * FAC + tid * 4, f + tid * 4, true);
         }
@@ -313,16 +312,16 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_scan_kernel(const ScanArgs p
     auto stage_qv = [&](int c) {
         if (c < c1) {
             const int t0 = p.pieces[2 * c], nt = p.pieces[2 * c + 1] - t0;
-            stage_rows(Qs, LD, p.q + (size_t)t0 * p.ldx + (size_t)g * D, p.ldx, nt, D, tid);
+            stage_rows<SCAN_THREADS>(Qs, LD, p.q + (size_t)t0 * p.ldx + (size_t)g * D, p.ldx, nt, D, tid);
             const float *v = p.v + (size_t)t0 * p.ldx + (size_t)h * p.Pv + col0;
             if (p.v_vec && col0 + CB <= p.Pv) {
-                for (int e = tid; e < CT * (CB / 4); e += THREADS) {
+                for (int e = tid; e < CT * (CB / 4); e += SCAN_THREADS) {
                     const int i = e / (CB / 4), cc = (e - i * (CB / 4)) * 4;
                     const bool ok = i < nt;
                     cp16(Vs + i * LV + cc, v + (ok ? (size_t)i * p.ldx : 0) + cc, ok);
                 }
             } else {
-                for (int e = tid; e < CT * CB; e += THREADS) {
+                for (int e = tid; e < CT * CB; e += SCAN_THREADS) {
                     const int i = e / CB, cc = e - i * CB;
                     Vs[i * LV + cc] = i < nt && col0 + cc < p.P ? (col0 + cc < p.Pv ? act_load(v + (size_t)i * p.ldx + cc) : 1.f) : 0.f;
                 }
@@ -333,7 +332,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_scan_kernel(const ScanArgs p
     auto stage_sq = [&](float *dst, const float *src, int c) {
         if (c < c1) {
             const float *m = src + ((size_t)c * p.H + h) * CT * CT;
-            for (int e = tid; e < CT * (CT / 4); e += THREADS) cp16(dst + (e >> 4) * LDC + (e & 15) * 4, m + e * 4, true);
+            for (int e = tid; e < CT * (CT / 4); e += SCAN_THREADS) cp16(dst + (e >> 4) * LDC + (e & 15) * 4, m + e * 4, true);
         }
         cp_commit();
     };
@@ -349,73 +348,76 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_scan_kernel(const ScanArgs p
         cp_wait<3>();                            // this chunk's K, factors, Q and V
         __syncthreads();
         {
-            constexpr int NA = DELTA ? 2 : 1, TC = CB / 4;
-            const Tile<NA, TC, 4> tile(tid);
-            float own[NA][4][TC / 4];
-            tile.run(Qs, Ks, LD, St, LD, D / 4, own);
+            // half of the threads Q S0, half K S0 (delta) or V's columns as rows
+            const int half = tid / (SCAN_THREADS / 2), i0 = tid % (SCAN_THREADS / 2);
+            constexpr int TC = CB / 4;
+            const Tile<4, TC, 4> tile(i0);
+            if (half == 0) {
+                float own[4][TC / 4];
+                tile.run(Qs, LD, St, LD, D / 4, own);
 #pragma unroll
-            for (int u = 0; u < TC / 4; ++u) {
-                const int cc = tile.col(u);
+                for (int u = 0; u < TC / 4; ++u)
 #pragma unroll
-                for (int q = 0; q < 4; ++q) {
-                    const int i = tile.rg + 16 * q;
-                    const float eg = F[i];
-                    Ot[cc * LDC + i] = eg * own[0][q][u];
-                    if (DELTA) {
-                        Xt[cc * LDC + i] = fmaf(-eg, own[NA - 1][q][u], Vs[i * LV + cc]);
-                    } else {
-                        const float v = Vs[i * LV + cc];
-                        Ut[cc * LDC + i] = v;
-                        Wt[cc * LDC + i] = v * F[CT + i];
+                    for (int q = 0; q < 4; ++q) Ot[tile.col(u) * LDC + tile.row(q)] = F[tile.row(q)] * own[q][u];
+            } else if (DELTA) {
+                float own[4][TC / 4];
+                tile.run(Ks, LD, St, LD, D / 4, own);
+#pragma unroll
+                for (int u = 0; u < TC / 4; ++u)
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) {
+                        const int i = tile.row(q), cc = tile.col(u);
+                        Xt[cc * LDC + i] = fmaf(-F[i], own[q][u], Vs[i * LV + cc]);
                     }
+            } else {
+                for (int e = i0; e < CT * CB; e += SCAN_THREADS / 2) {
+                    const int cc = e >> 6, i = e & 63;
+                    const float v = Vs[i * LV + cc];
+                    Ut[cc * LDC + i] = v;
+                    Wt[cc * LDC + i] = v * F[CT + i];
                 }
             }
         }
         cp_wait<2>();                            // T
         __syncthreads();
         stage_qv(c + 1);
-        using Sq = Tile<1, 4, CB == 32 ? 2 : 4>;
+        constexpr int RT = CB == 32 ? 4 : 2;
+        using Sq = Tile<RT, 4, 4>;
         const Sq sq(tid);
         if (DELTA) {
-            float own[1][4][Sq::OWN];
-            sq.run(Ts, nullptr, LDC, Xt, LDC, CT / 4, own);
+            float own[RT][1];
+            sq.run(Ts, LDC, Xt, LDC, CT / 4, own);
 #pragma unroll
-            for (int u = 0; u < Sq::OWN; ++u)
-#pragma unroll
-                for (int q = 0; q < 4; ++q) {
-                    const int i = sq.rg + 16 * q, at = sq.col(u) * LDC + i;
-                    Ut[at] = own[0][q][u];
-                    Wt[at] = own[0][q][u] * F[CT + i];
-                }
+            for (int q = 0; q < RT; ++q) {
+                const int i = sq.row(q), at = sq.col(0) * LDC + i;
+                Ut[at] = own[q][0];
+                Wt[at] = own[q][0] * F[CT + i];
+            }
         }
         cp_wait<2>();                            // M
         __syncthreads();
         if (DELTA) stage_sq(Ts, p.T, c + 1);
         else cp_commit();
         {
-            float own[1][4][Sq::OWN];
-            sq.run(Ms, nullptr, LDC, Ut, LDC, CT / 4, own);
+            float own[RT][1];
+            sq.run(Ms, LDC, Ut, LDC, CT / 4, own);
 #pragma unroll
-            for (int u = 0; u < Sq::OWN; ++u)
-#pragma unroll
-                for (int q = 0; q < 4; ++q) Ot[sq.col(u) * LDC + sq.rg + 16 * q] += own[0][q][u];      // (the same thread's own element)
+            for (int q = 0; q < RT; ++q) Ot[sq.col(0) * LDC + sq.row(q)] += own[q][0];      // (the same thread's own element)
         }
-        // S = e^(G_last) S + K^T W: a thread has four rows and four columns; with few of them, two threads share the tokens
+        // S = e^(G_last) S + K^T W: a thread has four rows and four columns; with few of them, two or four threads share the tokens
         {
             const int d4 = D / 4, items = d4 * (CB / 4);
-            const bool two = 2 * items <= THREADS;
+            const int parts = 4 * items <= SCAN_THREADS ? 4 : (2 * items <= SCAN_THREADS ? 2 : 1);
             const float eg_last = F[2 * CT];
-            for (int it0 = 0; it0 < items; it0 += THREADS) {
-                const int it = it0 + (two ? tid % items : tid), half = two ? tid / items : 0;
-                const bool on = it < items && half < 2;
+            for (int it0 = 0; it0 < items; it0 += SCAN_THREADS) {
+                const int it = it0 + (parts > 1 ? tid % items : tid), part = parts > 1 ? tid / items : 0;
+                const bool on = it < items && part < parts;
                 const int dq = it % d4, cq = it / d4;
-                float acc[4][4];             // [column][row]
+                float2 acc[4][2];            // [column][two rows]
 #pragma unroll
-                for (int x = 0; x < 4; ++x)
-#pragma unroll
-                    for (int y = 0; y < 4; ++y) acc[x][y] = 0.f;
+                for (int x = 0; x < 4; ++x) acc[x][0] = acc[x][1] = make_float2(0.f, 0.f);
                 if (on) {
-                    const int j0 = two ? half * (CT / 2) : 0, j1 = two ? j0 + CT / 2 : CT;
+                    const int j0 = part * (CT / parts), j1 = j0 + CT / parts;
                     for (int j = j0; j < j1; j += 4) {
                         float4 w4[4];
 #pragma unroll
@@ -426,21 +428,21 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_scan_kernel(const ScanArgs p
 #pragma unroll
                             for (int x = 0; x < 4; ++x) {
                                 const float w = y == 0 ? w4[x].x : y == 1 ? w4[x].y : y == 2 ? w4[x].z : w4[x].w;
-                                acc[x][0] = fmaf(kk.x, w, acc[x][0]), acc[x][1] = fmaf(kk.y, w, acc[x][1]);
-                                acc[x][2] = fmaf(kk.z, w, acc[x][2]), acc[x][3] = fmaf(kk.w, w, acc[x][3]);
+                                acc[x][0] = fma2(make_float2(kk.x, kk.y), make_float2(w, w), acc[x][0]);
+                                acc[x][1] = fma2(make_float2(kk.z, kk.w), make_float2(w, w), acc[x][1]);
                             }
                         }
                     }
                 }
-                for (int turn = 0; turn < (two ? 2 : 1); ++turn) {
-                    if (turn == 1) __syncthreads();
-                    if (on && half == turn)
+                for (int turn = 0; turn < parts; ++turn) {
+                    if (turn > 0) __syncthreads();
+                    if (on && part == turn)
 #pragma unroll
                         for (int x = 0; x < 4; ++x) {
                             float4 *s = reinterpret_cast<float4 *>(St + (cq * 4 + x) * LD + dq * 4);
                             float4 v = *s;
                             const float f = turn == 0 ? eg_last : 1.f;
-                            v.x = fmaf(f, v.x, acc[x][0]), v.y = fmaf(f, v.y, acc[x][1]), v.z = fmaf(f, v.z, acc[x][2]), v.w = fmaf(f, v.w, acc[x][3]);
+                            v.x = fmaf(f, v.x, acc[x][0].x), v.y = fmaf(f, v.y, acc[x][0].y), v.z = fmaf(f, v.z, acc[x][1].x), v.w = fmaf(f, v.w, acc[x][1].y);
                             *s = v;
                         }
                 }
@@ -448,13 +450,13 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_scan_kernel(const ScanArgs p
         }
         __syncthreads();
         stage_sq(Ms, p.M, c + 1);
-        for (int e = tid; e < nt * CB; e += THREADS) {
+        for (int e = tid; e < nt * CB; e += SCAN_THREADS) {
             const int i = e / CB, cc = e - i * CB;
             if (col0 + cc < p.P) p.o[(size_t)(t0 + i) * p.ldo + (size_t)h * p.P + col0 + cc] = Ot[cc * LDC + i];
         }
     }
     cp_wait<0>();
-    for (int e = tid; e < D * CB; e += THREADS) {
+    for (int e = tid; e < D * CB; e += SCAN_THREADS) {
         const int d = p.s_row == 1 ? e % D : e / CB, c = p.s_row == 1 ? e / D : e % CB;
         if (col0 + c < p.P) S_base[(size_t)d * p.s_row + (size_t)(col0 + c) * p.s_col] = St[c * LD + d];
     }
@@ -497,10 +499,10 @@ LGML_API int lgml_chunk_prepare(const float *q, const float *k, int ldx, const f
     dim3 grid(n_chunks, G);
     if (delta) {
         if (allow(chunk_prepare_kernel<true>, smem, "chunk_prepare")) return -1;
-        lgml_launch(chunk_prepare_kernel<true>, grid, THREADS, smem, stream, a);
+        lgml_launch(chunk_prepare_kernel<true>, grid, PREP_THREADS, smem, stream, a);
     } else {
         if (allow(chunk_prepare_kernel<false>, smem, "chunk_prepare")) return -1;
-        lgml_launch(chunk_prepare_kernel<false>, grid, THREADS, smem, stream, a);
+        lgml_launch(chunk_prepare_kernel<false>, grid, PREP_THREADS, smem, stream, a);
     }
     return lgml_launch_status("chunk_prepare");
 }
@@ -526,7 +528,7 @@ LGML_API int lgml_chunk_scan(const float *q, const float *k, const float *v, int
 #define LGML_CS(DELTA, CB)                                                            \
     do {                                                                              \
         if (allow(chunk_scan_kernel<DELTA, CB>, smem, "chunk_scan")) return -1;       \
-        lgml_launch(chunk_scan_kernel<DELTA, CB>, grid, THREADS, smem, stream, a);    \
+        lgml_launch(chunk_scan_kernel<DELTA, CB>, grid, SCAN_THREADS, smem, stream, a);    \
     } while (0)
     if (delta) { if (wide) LGML_CS(true, 32); else LGML_CS(true, 16); }
     else { if (wide) LGML_CS(false, 32); else LGML_CS(false, 16); }

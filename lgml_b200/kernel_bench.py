@@ -7,6 +7,8 @@
     python -m lgml_b200.kernel_bench token_shift --rows 2048 --width 4096
     python -m lgml_b200.kernel_bench mingru --rows 2048 --width 4096 [--requests 8]
     python -m lgml_b200.kernel_bench token_side --rows 8 --width 4096 --dim 64
+    python -m lgml_b200.kernel_bench chunk_scan --rows 2048 --heads 16 --kv-heads 8 --dim 128 --vdim 128 [--memory]
+    python -m lgml_b200.kernel_bench stream_norm --rows 2048 --width 4096 --streams 2
 
 Each case is run over a ring of input buffers larger than the L2 cache, so that weights and
 cache pages come from HBM as they do in a decode step; warm-up launches first, then the timed
@@ -219,6 +221,49 @@ def case_token_side(a) -> None:
     print(f"side_add rows={rows} width={width}: {us:.2f} us, {rows * width * 12 / us / 1e3:.0f} GB/s")
 
 
+def case_chunk_scan(a) -> None:
+    """A recurrence with one decay per head over one request's tokens, 64 at a time (the row factors' kernel and the scan): the delta
+    rule, or the matrix memory with its extra column (``--memory``)."""
+    from .engine.batch import ScanChunks
+
+    n, H, G, D, Dv = a.rows, a.heads, (a.heads if a.memory else a.kv_heads), a.dim, a.vdim
+    P = Dv + 1 if a.memory else Dv
+    C = 2 * G * D + H * Dv
+    nb = min(ring(n * C * 4), 8)
+    bufs = [torch.nn.functional.normalize(torch.randn(n, C // 4, 4, device=DEV), dim=1).view(n, C) for _ in range(nb)]
+    gb = torch.rand(n, 4 * H, device=DEV) * 0.5
+    gb[:, 3::4] = -gb[:, 3::4]
+    gb[:, 2::4] = -gb[:, 2::4]
+    state = torch.zeros(1, H * D * P, device=DEV)
+    rows = torch.tensor([(t, min(t + 64, n)) for t in range(0, n, 64)], dtype=torch.int32, device=DEV)
+    i32 = lambda *v: torch.tensor(v, dtype=torch.int32, device=DEV)
+    chunks = ScanChunks(rows, i32(0, rows.shape[0]), i32(0), 16, False)
+    out = torch.empty(n, H * P, device=DEV)
+    slots = i32(0)
+
+    def run(i):
+        x = bufs[i]
+        v, k, q = x[:, :H * Dv], x[:, H * Dv:H * Dv + G * D], x[:, H * Dv + G * D:]
+        ops.chunk_scan(q, k, v, gb[:, 2:], gb[:, 1:], 4, state, *((1, D) if a.memory else (P, 1)), chunks, slots, out, H, G, D, Dv, P, not a.memory)
+
+    us = timed(run, nb, a.warmup, a.iters)
+    seq = 2.0 * n * H * P * D * (2 if a.memory else 3)         # the recurrence's own multiply-adds, token by token
+    print(f"chunk_scan {'memory' if a.memory else 'delta'} rows={n} heads={H}/{G} dim={D} vdim={Dv}: {us:.2f} us, {seq / us / 1e6:.2f} TFLOP/s of the recurrence itself")
+
+
+def case_stream_norm(a) -> None:
+    n, E, R = a.rows, a.width, a.streams
+    nb = min(ring(n * E * 4 * (R + 2)), 8)
+    xs = [torch.randn(n, R, E, device=DEV) for _ in range(nb)]
+    ds = [torch.randn(n, E, device=DEV) for _ in range(nb)]
+    gs = [torch.randn(n, E, device=DEV) for _ in range(nb)]
+    w, w_in, w_out, mix = torch.ones(E, device=DEV), torch.ones(R, device=DEV), torch.ones(R, device=DEV), torch.eye(R, device=DEV)
+    out = torch.empty(n, E, dtype=torch.bfloat16, device=DEV)
+    us = timed(lambda i: ops.stream_norm(xs[i], 1e-6, out, w, w_in=w_in, delta=ds[i], gate=gs[i], w_out=w_out, mix=mix), nb, a.warmup, a.iters)
+    byts = n * E * (8 * R + 8 + 2)
+    print(f"stream_norm rows={n} width={E} streams={R}: {us:.2f} us, {byts / us / 1e3:.0f} GB/s")
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="python -m lgml_b200.kernel_bench")
     ap.add_argument("--warmup", type=int, default=5)
@@ -259,6 +304,13 @@ def main(argv=None) -> int:
         t.add_argument("--width", type=int, default=4096)
         t.add_argument("--requests", type=int, default=1)
         t.add_argument("--dim", type=int, default=64)
+    c = sub.add_parser("chunk_scan")
+    for name, size in (("rows", 2048), ("heads", 16), ("kv-heads", 8), ("dim", 128), ("vdim", 128)):
+        c.add_argument("--" + name, type=int, default=size)
+    c.add_argument("--memory", action="store_true", help="the matrix memory instead of the delta rule")
+    c = sub.add_parser("stream_norm")
+    for name, size in (("rows", 2048), ("width", 4096), ("streams", 2)):
+        c.add_argument("--" + name, type=int, default=size)
     a = ap.parse_args(argv)
     global USE_GRAPH
     USE_GRAPH = not a.no_graph
@@ -266,7 +318,8 @@ def main(argv=None) -> int:
         print("kernel_bench needs a CUDA device", file=sys.stderr)
         return 1
     {"gemm": case_gemm, "decode_attention": case_decode_attention, "prefill_attention": case_prefill_attention, "rmsnorm": case_rmsnorm,
-     "token_shift": case_token_shift, "mingru": case_mingru, "token_side": case_token_side}[a.case](a)
+     "token_shift": case_token_shift, "mingru": case_mingru, "token_side": case_token_side, "chunk_scan": case_chunk_scan,
+     "stream_norm": case_stream_norm}[a.case](a)
     return 0
 
 
