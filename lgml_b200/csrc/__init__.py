@@ -54,6 +54,8 @@ LIBRARIES: Dict[str, tuple] = {
     "chunk_scan": ("chunk_scan.cu", []),
     "matrix_memory": ("matrix_memory.cu", []),
     "streams": ("streams.cu", []),
+    "scaled_norm": ("scaled_norm.cu", []),
+    "rglru": ("rglru.cu", []),
 }
 
 _HEADERS = ["common.cuh", "page_map.cuh"]
@@ -137,6 +139,8 @@ def _digest(name: str) -> str:
 # extra headers a library includes (its hash covers them)
 LIBRARY_HEADERS: Dict[str, List[str]] = {
     "attention_decode_noalloc": ["attention_decode.cu", "attention_decode_noalloc.h"],
+    "attention_heads": ["few_rows.cuh"],
+    "rglru": ["few_rows.cuh"],
 }
 
 

@@ -518,9 +518,11 @@ __global__ void __launch_bounds__(THREADS, 1) prefill_attention_twin_kernel(
             tcgen05_fence_after();
             // the sink: a term of the denominator without a key or a value
             if (BIAS && sinks && m_ref != -INFINITY) l_run += ex2(sinks[my_head] * 1.4426950408889634f - m_ref);
-            const float inv = l_run > 0.f && l_run < INFINITY ? 1.f / l_run : 0.f;
+            float inv = l_run > 0.f && l_run < INFINITY ? 1.f / l_run : 0.f;
             const bool store = row_valid && alive;
-            const float *grow = (BIAS && gate && store) ? gate + (size_t)(row0 + t * tt + my_tok) * ldg + (size_t)my_head * D : nullptr;
+            // the gate: a logit per value, or (ldg negative, rows -ldg apart) one for the whole head, which joins the row's factor
+            const float *grow = (BIAS && gate && store && ldg > 0) ? gate + (size_t)(row0 + t * tt + my_tok) * ldg + (size_t)my_head * D : nullptr;
+            if (BIAS && gate && store && ldg < 0) inv *= 1.0f / (1.0f + __expf(-act_load(gate + (size_t)(row0 + t * tt + my_tok) * (size_t)(-ldg) + my_head)));
             // (every lane takes part in the loads from tensor memory, which are for whole warps; rows
             //  without a token only skip the stores)
             __nv_bfloat16 *dst = out + (size_t)(row0 + (store ? t * tt + my_tok : 0)) * ldo + (size_t)(kvh * group + g0 + (store ? my_g : 0)) * D;
@@ -718,7 +720,7 @@ LGML_API int lgml_prefill_attention_twin(const void *q, int ldq, const int *posi
 }
 
 // The same kernel with a distance bias (slopes), a sink in the denominator (sinks) and an output
-// gate (float32 [tokens, H D], row stride ldg), each per head and each optional; keys and values
+// gate (float32 [tokens, H D], row stride ldg; or [tokens, H], row stride -ldg: one per head), each optional; keys and values
 // of one head size, 64 or 128.  keep_first: with a window, the first keys that stay visible beyond it.
 LGML_API int lgml_sink_attention_twin_keep(const void *q, int ldq, const int *positions, const int *tiles, int n_tiles, const int *block_table,
                                       int max_blocks, const void *k_pages, const void *v_pages, int n_pages, int page_size,
@@ -733,8 +735,8 @@ LGML_API int lgml_sink_attention_twin_keep(const void *q, int ldq, const int *po
     LGML_REQUIRE(ldq % 8 == 0 && ldo % 8 == 0 && ((uintptr_t)q & 15) == 0 && ((uintptr_t)out & 15) == 0,
                  "sink_attention_twin: q and out must be 16-byte aligned with row strides that are multiples of 8");
     LGML_REQUIRE(((uintptr_t)k_pages & 15) == 0 && ((uintptr_t)v_pages & 15) == 0, "sink_attention_twin: the cache must be 16-byte aligned");
-    LGML_REQUIRE(gate == nullptr || (ldg >= H * D && ldg % 4 == 0 && ((uintptr_t)gate & 15) == 0),
-                 "sink_attention_twin: the gate must be 16-byte aligned with a row stride that is a multiple of 4 and at least H D");
+    LGML_REQUIRE(gate == nullptr || ldg <= -H || (ldg >= H * D && ldg % 4 == 0 && ((uintptr_t)gate & 15) == 0),
+                 "sink_attention_twin: a gate per value must be 16-byte aligned with a row stride that is a multiple of 4 and at least H D");
     if (n_tiles == 0) return 0;
     const int group = H / Hkv;
     int hpc, tile_tokens;

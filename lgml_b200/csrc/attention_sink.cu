@@ -32,10 +32,16 @@ __device__ __forceinline__ float capped_score(float dot, float scale, float cap)
 __device__ __forceinline__ float capped_score2(float dot, float scale, float cap) {
     return cap * 1.4426950408889634f * tanhf(dot * scale / cap);
 }
+// The output gate's logit for head h, value d of token t: one per value (gate[t, h Dv + d], rows ldg apart), or, with a
+// negative ldg, one per head (gate[t, h], rows -ldg apart).
+__device__ __forceinline__ float gate_logit(const float *gate, int ldg, size_t t, int h, int Dv, int d) {
+    return act_load(ldg > 0 ? gate + t * ldg + (size_t)h * Dv + d : gate + t * (size_t)(-ldg) + h);
+}
+static inline bool gate_stride_ok(const float *gate, int ldg, int H, int Dv) { return gate == nullptr || ldg >= H * Dv || ldg <= -H; }
 constexpr int ITEMS = 256;
 constexpr int WARPS = 4;
 constexpr int MAX_D = 256;        // the split decode forms (a lane holds 8 value columns)
-constexpr int GEN_MAX_D = 512;    // the general form
+constexpr int GEN_MAX_D = 1024;   // the general form (built for 512 and for 1,024)
 
 // v_mode: 0 store v as it is; 1 also keep it in v_keep (float32 [tokens, Hkv Dv]); 2 mix with v_keep first
 template <typename T>
@@ -80,7 +86,7 @@ __global__ void __launch_bounds__(ITEMS) sink_qkv_store_kernel(
     v_pages[(((size_t)page * Hv + g) * page_size + (size_t)(pos % page_size)) * Dv + d] = from_f32<T>(val);
 }
 
-template <typename T, typename TO>
+template <typename T, typename TO, int MAXD>
 __global__ void __launch_bounds__(WARPS * 32) sink_attention_kernel(
     const T *__restrict__ q, int ldq, const int *__restrict__ positions, const int *__restrict__ seq_of_token,
     const int *__restrict__ block_table, int max_blocks, const T *__restrict__ k_pages, const T *__restrict__ v_pages,
@@ -89,8 +95,8 @@ __global__ void __launch_bounds__(WARPS * 32) sink_attention_kernel(
     int window, int keep_first, int *__restrict__ status) {
     pdl_trigger();
     pdl_wait();
-    __shared__ float qs[GEN_MAX_D];
-    __shared__ float acc_w[WARPS][GEN_MAX_D];
+    __shared__ float qs[MAXD];
+    __shared__ float acc_w[WARPS][MAXD];
     __shared__ float m_w[WARPS], l_w[WARPS];
     const int t = blockIdx.x, h = blockIdx.y;
     const int g = h / (H / Hkv);
@@ -108,9 +114,9 @@ __global__ void __launch_bounds__(WARPS * 32) sink_attention_kernel(
     __syncthreads();
 
     float m = -INFINITY, l = 0.f;
-    float acc[GEN_MAX_D / 32];
+    float acc[MAXD / 32];
 #pragma unroll
-    for (int i = 0; i < GEN_MAX_D / 32; ++i) acc[i] = 0.f;
+    for (int i = 0; i < MAXD / 32; ++i) acc[i] = 0.f;
 
     // the visible keys in order: the kept first tokens, then the window; warp w takes every WARPS-th
     for (int i = warp; i < n_keys; i += WARPS) {
@@ -131,7 +137,7 @@ __global__ void __launch_bounds__(WARPS * 32) sink_attention_kernel(
         const float p = expf(s - m_new);
         l = l * corr + p;
 #pragma unroll
-        for (int i2 = 0; i2 < GEN_MAX_D / 32; ++i2) {
+        for (int i2 = 0; i2 < MAXD / 32; ++i2) {
             const int d = lane + 32 * i2;
             if (d < Dv) acc[i2] = acc[i2] * corr + p * to_f32(act_load(v_pages + vcell * ldv + d));
         }
@@ -142,7 +148,7 @@ __global__ void __launch_bounds__(WARPS * 32) sink_attention_kernel(
         l_w[warp] = l;
     }
 #pragma unroll
-    for (int i = 0; i < GEN_MAX_D / 32; ++i) {
+    for (int i = 0; i < MAXD / 32; ++i) {
         const int d = lane + 32 * i;
         if (d < Dv) acc_w[warp][d] = acc[i];
     }
@@ -160,7 +166,7 @@ __global__ void __launch_bounds__(WARPS * 32) sink_attention_kernel(
         float o = 0.f;
         for (int w = 0; w < WARPS; ++w) o += acc_w[w][d] * f[w];
         o = lsum > 0.f ? o / lsum : 0.f;
-        if (gate) o *= 1.0f / (1.0f + expf(-act_load(gate + (size_t)t * ldg + (size_t)h * Dv + d)));
+        if (gate) o *= 1.0f / (1.0f + expf(-gate_logit(gate, ldg, (size_t)t, h, Dv, d)));
         out[(size_t)t * ldo + (size_t)h * Dv + d] = from_f32<TO>(o);
     }
 }
@@ -438,7 +444,7 @@ __global__ void __launch_bounds__(128, 3) sink_attention_mma_kernel(
                 const int d = nv * 8 + (lane & 3) * 2 + e;
                 if (d >= Dv) continue;
                 float o = oacc[nv][rr * 2 + e] * inv;
-                if (gate) o *= 1.0f / (1.0f + __expf(-act_load(gate + t * ldg + (size_t)h * Dv + d)));
+                if (gate) o *= 1.0f / (1.0f + __expf(-gate_logit(gate, ldg, t, h, Dv, d)));
                 store_out(out, out_f32, t * ldo + (size_t)h * Dv + d, o);
             }
     }
@@ -716,7 +722,7 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) sink_decode_kernel(
             const float f = (m == -INFINITY) ? 0.f : exp2f(m - m_all);
             const float den = l * f + (sinks ? exp2f(sink2 - m_all) : 0.f);
             float r = den > 0.f ? o * f / den : 0.f;
-            if (gate) r *= 1.0f / (1.0f + __expf(-act_load(gate + (size_t)t * ldg + (size_t)h * Dv + d)));
+            if (gate) r *= 1.0f / (1.0f + __expf(-gate_logit(gate, ldg, (size_t)t, h, Dv, d)));
             store_out(out, out_f32, (size_t)t * ldo + (size_t)h * Dv + d, r);
         } else {
             part_o[(((size_t)t * H + h) * n_splits + split) * Dv + d] = o;
@@ -754,7 +760,7 @@ __global__ void __launch_bounds__(128) sink_decode_combine_kernel(const float *_
         float o = 0.f;
         for (int i = 0; i < n_splits; ++i) o += act_load(po + (size_t)i * Dv + d) * f_s[i];
         o *= inv_s;
-        if (gate) o *= 1.0f / (1.0f + __expf(-act_load(gate + (size_t)t * ldg + (size_t)h * Dv + d)));
+        if (gate) o *= 1.0f / (1.0f + __expf(-gate_logit(gate, ldg, (size_t)t, h, Dv, d)));
         store_out(out, out_f32, (size_t)t * ldo + (size_t)h * Dv + d, o);
     }
 }
@@ -967,7 +973,7 @@ __global__ void __launch_bounds__(DEC_WARPS * 32) sink_decode_mma_kernel(
             const float f = (m == -INFINITY) ? 0.f : exp2f(m - m_all);
             const float den = l * f + (sinks ? exp2f(sink2 - m_all) : 0.f);
             float r = den > 0.f ? o * f / den : 0.f;
-            if (gate) r *= 1.0f / (1.0f + __expf(-act_load(gate + (size_t)t * ldg + (size_t)h * DV + d)));
+            if (gate) r *= 1.0f / (1.0f + __expf(-gate_logit(gate, ldg, (size_t)t, h, DV, d)));
             store_out(out, out_f32, (size_t)t * ldo + (size_t)h * DV + d, r);
         } else {
             part_o[(((size_t)t * H + h) * n_splits + split) * DV + d] = o;
@@ -1044,7 +1050,8 @@ LGML_API int lgml_sink_qkv_store(const float *proj, int ldp, void *q_out, int dt
     return lgml_launch_status("sink_qkv_store");
 }
 
-// slopes, sinks: float32 [H] or null (no bias, no sink); gate: float32 [n_tokens, ldg] (column h Dv + d) or null.
+// slopes, sinks: float32 [H] or null (no bias, no sink); gate: float32 [n_tokens, ldg] (column h Dv + d), or [n_tokens, -ldg] (column h: one gate per
+// head), or null.
 // Hv value heads (Hkv a multiple of it: key heads g Hkv / Hv ... share value head g), value rows ldv elements apart
 // (values that are a column range of wider cells), keep_first: the first tokens of a request that stay visible
 // beyond the window; out_dtype: the output's type (float32 for a caller that combines heads afterwards).
@@ -1059,24 +1066,26 @@ LGML_API int lgml_sink_attention(const void *q, int dtype, int ldq, const int *p
     LGML_REQUIRE(ldv >= Dv, "sink_attention: value rows %d apart hold no %d values", ldv, Dv);
     LGML_REQUIRE(H <= 65535, "sink_attention: too many heads");
     LGML_REQUIRE(window >= 0 && keep_first >= 0, "sink_attention: bad window");
-    LGML_REQUIRE(gate == nullptr || ldg >= H * Dv, "sink_attention: the gate's row stride %d is below H Dv", ldg);
+    LGML_REQUIRE(gate_stride_ok(gate, ldg, H, Dv), "sink_attention: the gate's row stride %d is below its row", ldg);
     LGML_REQUIRE(out_dtype == dtype || out_dtype == LGML_F32, "sink_attention: the output is the inputs' type or float32");
     if (n_tokens == 0) return 0;
     dim3 grid(n_tokens, H);
-    if (dtype == LGML_F32)
-        lgml_launch(sink_attention_kernel<float, float>, grid, WARPS * 32, 0, stream, (const float *)q, ldq, positions, seq_of_token, block_table,
-                    max_blocks, (const float *)k_pages, (const float *)v_pages, n_pages, page_size, slopes, sinks, gate, ldg, (float *)out, ldo, H,
-                    Hkv, Hv, D, Dv, ldv, scale, softcap, window, keep_first, status);
-    else if (dtype == LGML_BF16 && out_dtype == LGML_F32)
-        lgml_launch(sink_attention_kernel<__nv_bfloat16, float>, grid, WARPS * 32, 0, stream, (const __nv_bfloat16 *)q, ldq, positions, seq_of_token,
-                    block_table, max_blocks, (const __nv_bfloat16 *)k_pages, (const __nv_bfloat16 *)v_pages, n_pages, page_size, slopes, sinks,
-                    gate, ldg, (float *)out, ldo, H, Hkv, Hv, D, Dv, ldv, scale, softcap, window, keep_first, status);
-    else if (dtype == LGML_BF16)
-        lgml_launch(sink_attention_kernel<__nv_bfloat16, __nv_bfloat16>, grid, WARPS * 32, 0, stream, (const __nv_bfloat16 *)q, ldq, positions, seq_of_token,
-                    block_table, max_blocks, (const __nv_bfloat16 *)k_pages, (const __nv_bfloat16 *)v_pages, n_pages, page_size, slopes, sinks,
-                    gate, ldg, (__nv_bfloat16 *)out, ldo, H, Hkv, Hv, D, Dv, ldv, scale, softcap, window, keep_first, status);
-    else
-        LGML_FAIL("sink_attention: unknown type %d", dtype);
+#define LGML_GEN(T, TO)                                                                                                                              \
+    do {                                                                                                                                             \
+        if (D <= 512 && Dv <= 512)                                                                                                                   \
+            lgml_launch(sink_attention_kernel<T, TO, 512>, grid, WARPS * 32, 0, stream, (const T *)q, ldq, positions, seq_of_token, block_table,     \
+                        max_blocks, (const T *)k_pages, (const T *)v_pages, n_pages, page_size, slopes, sinks, gate, ldg, (TO *)out, ldo, H, Hkv,    \
+                        Hv, D, Dv, ldv, scale, softcap, window, keep_first, status);                                                                 \
+        else                                                                                                                                         \
+            lgml_launch(sink_attention_kernel<T, TO, GEN_MAX_D>, grid, WARPS * 32, 0, stream, (const T *)q, ldq, positions, seq_of_token,            \
+                        block_table, max_blocks, (const T *)k_pages, (const T *)v_pages, n_pages, page_size, slopes, sinks, gate, ldg, (TO *)out,    \
+                        ldo, H, Hkv, Hv, D, Dv, ldv, scale, softcap, window, keep_first, status);                                                    \
+    } while (0)
+    if (dtype == LGML_F32) LGML_GEN(float, float);
+    else if (dtype == LGML_BF16 && out_dtype == LGML_F32) LGML_GEN(__nv_bfloat16, float);
+    else if (dtype == LGML_BF16) LGML_GEN(__nv_bfloat16, __nv_bfloat16);
+    else LGML_FAIL("sink_attention: unknown type %d", dtype);
+#undef LGML_GEN
     return lgml_launch_status("sink_attention");
 }
 
@@ -1094,7 +1103,7 @@ LGML_API int lgml_sink_attention_mma(const void *q, int ldq, const int *position
     LGML_REQUIRE(H % Hkv == 0 && H <= 65535, "sink_attention_mma: %d heads on %d KV heads", H, Hkv);
     LGML_REQUIRE(D <= 128 && Dv <= 128, "sink_attention_mma: head sizes %d and %d must be at most 128", D, Dv);
     LGML_REQUIRE(window >= 0, "sink_attention_mma: bad window");
-    LGML_REQUIRE(gate == nullptr || ldg >= H * Dv, "sink_attention_mma: the gate's row stride %d is below H Dv", ldg);
+    LGML_REQUIRE(gate_stride_ok(gate, ldg, H, Dv), "sink_attention_mma: the gate's row stride %d is below its row", ldg);
     if (n_tiles == 0) return 0;
     dim3 grid(n_tiles, H);
     const int ks = D <= 32 ? 2 : D <= 64 ? 4 : D <= 96 ? 6 : 8;
@@ -1130,7 +1139,7 @@ LGML_API int lgml_sink_decode(const void *q, int ldq, const int *positions, cons
     LGML_REQUIRE(n_splits >= 1 && n_splits <= DEC_MAX_SPLITS, "sink_decode: %d key ranges (1 to %d)", n_splits, DEC_MAX_SPLITS);
     LGML_REQUIRE(n_splits == 1 || scratch != nullptr, "sink_decode: %d ranges need scratch memory", n_splits);
     LGML_REQUIRE(window >= 0, "sink_decode: bad window");
-    LGML_REQUIRE(gate == nullptr || ldg >= H * Dv, "sink_decode: the gate's row stride %d is below H Dv", ldg);
+    LGML_REQUIRE(gate_stride_ok(gate, ldg, H, Dv), "sink_decode: the gate's row stride %d is below its row", ldg);
     if (n_tokens == 0) return 0;
     const int group = H / Hkv;
     float *part_o = scratch;

@@ -10,9 +10,9 @@ LGML_DEFINE_LAST_ERROR(lgml_elementwise)
 // ---------------------------------------------------------------------------------------
 // x[t, :] = table[ids[t], :]            (lua/lgml/transformer.lua:2303: get_rows, no scale)
 // ---------------------------------------------------------------------------------------
-template <typename TW>
+template <typename TW, typename TO>
 __global__ void embed_rows_kernel(const TW *__restrict__ table, const int *__restrict__ ids,
-                                  float *__restrict__ out, int width, int vocab, int *__restrict__ status) {
+                                  TO *__restrict__ out, int width, int vocab, int *__restrict__ status) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
@@ -23,21 +23,25 @@ __global__ void embed_rows_kernel(const TW *__restrict__ table, const int *__res
     const int i0 = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-        if (i0 + j < width) out[(size_t)t * width + i0 + j] = ok ? to_f32(row[i0 + j]) : 0.f;
+        if (i0 + j < width) out[(size_t)t * width + i0 + j] = from_f32<TO>(ok ? to_f32(row[i0 + j]) : 0.f);
 }
 
-LGML_API int lgml_embed_rows(const void *table, int table_dtype, const int *ids, float *out, int n_tokens,
-                             int width, int vocab, int *status, cudaStream_t stream) {
+// out_dtype: float32, or the table's own type
+LGML_API int lgml_embed_rows_as(const void *table, int table_dtype, const int *ids, void *out, int out_dtype, int n_tokens,
+                                int width, int vocab, int *status, cudaStream_t stream) {
     LGML_REQUIRE(n_tokens >= 0 && width > 0 && vocab > 0, "embed_rows: bad sizes");
     if (n_tokens == 0) return 0;
     const int threads = 128;
     dim3 grid(n_tokens, (width + threads * 4 - 1) / (threads * 4));
-    if (table_dtype == LGML_F32)
-        lgml_launch(embed_rows_kernel<float>, grid, threads, 0, stream, (const float *)table, ids, out, width, vocab, status);
+    if (table_dtype == LGML_F32 && out_dtype == LGML_F32)
+        lgml_launch(embed_rows_kernel<float, float>, grid, threads, 0, stream, (const float *)table, ids, (float *)out, width, vocab, status);
+    else if (table_dtype == LGML_BF16 && out_dtype == LGML_BF16)
+        lgml_launch(embed_rows_kernel<__nv_bfloat16, __nv_bfloat16>, grid, threads, 0, stream, (const __nv_bfloat16 *)table, ids, (__nv_bfloat16 *)out, width,
+                    vocab, status);
     else if (table_dtype == LGML_BF16)
-        lgml_launch(embed_rows_kernel<__nv_bfloat16>, grid, threads, 0, stream, (const __nv_bfloat16 *)table, ids, out, width, vocab, status);
+        lgml_launch(embed_rows_kernel<__nv_bfloat16, float>, grid, threads, 0, stream, (const __nv_bfloat16 *)table, ids, (float *)out, width, vocab, status);
     else
-        LGML_FAIL("embed_rows: unknown table type %d", table_dtype);
+        LGML_FAIL("embed_rows: types %d -> %d are not built", table_dtype, out_dtype);
     return lgml_launch_status("embed_rows");
 }
 

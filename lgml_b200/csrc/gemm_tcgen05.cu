@@ -1096,16 +1096,18 @@ LGML_API int lgml_gemm_tcgen05_glu_clamped(const void *x, const void *w, void *y
 // A grouped product: x [max_tiles * 128, K] holds tiles of 128 rows, tile t of them multiplied by the rows
 // group[3 t] * N ... + N - 1 of w [n_groups * N, K] (the matrices of n_groups experts stacked); group[3 max_tiles] is the
 // number of tiles in use, read on the device (the list is written by the kernel ahead).  y [max_tiles * 128, N], or
-// [.., N / 2] with swiglu = 1 (rows of w in (gate, up) pairs, y = silu(gate) * up).  The single-CTA persistent kernel with
+// [.., N / 2] with swiglu = 1 (rows of w in (gate, up) pairs, y = silu(gate) * up) or 3 (the same pairs, the clamped activation with
+// act_alpha and act_limit).  The single-CTA persistent kernel with
 // 128 x 256 tiles (128 x 128 where those would be fewer than the SMs); rows of a tile past an expert's last feature are computed from the next expert's rows and not stored.
-LGML_API int lgml_gemm_tcgen05_grouped(const void *x, const void *w, void *y, int y_f32, int max_tiles, int N, int K, int n_groups, int ldy,
-                                       const int *group, int swiglu, int *status, cudaStream_t stream) {
+LGML_API int lgml_gemm_tcgen05_grouped_act(const void *x, const void *w, void *y, int y_f32, int max_tiles, int N, int K, int n_groups, int ldy,
+                                           const int *group, int swiglu, float act_alpha, float act_limit, int *status, cudaStream_t stream) {
     LGML_REQUIRE(max_tiles > 0 && N > 0 && K > 0 && n_groups > 0 && group != nullptr, "gemm_tcgen05_grouped: bad sizes");
-    LGML_REQUIRE(swiglu >= 0 && swiglu <= 2, "gemm_tcgen05_grouped: unknown epilogue %d", swiglu);
-    LGML_REQUIRE(swiglu != 1 || N % 2 == 0, "gemm_tcgen05_grouped: the gated epilogue needs an even N");
+    LGML_REQUIRE(swiglu >= 0 && swiglu <= 3, "gemm_tcgen05_grouped: unknown epilogue %d", swiglu);
+    const bool paired = swiglu == 1 || swiglu == 3;
+    LGML_REQUIRE(!paired || N % 2 == 0, "gemm_tcgen05_grouped: the gated epilogue needs an even N");
     LGML_REQUIRE(K % 8 == 0, "gemm_tcgen05_grouped: K = %d must be a multiple of 8 elements (16 bytes) for TMA", K);
     LGML_REQUIRE(((uintptr_t)x & 15) == 0 && ((uintptr_t)w & 15) == 0, "gemm_tcgen05_grouped: operands must be 16-byte aligned for TMA");
-    LGML_REQUIRE(ldy >= (swiglu == 1 ? N / 2 : N), "gemm_tcgen05_grouped: the output's rows are too short");
+    LGML_REQUIRE(ldy >= (paired ? N / 2 : N), "gemm_tcgen05_grouped: the output's rows are too short");
     Params p;
     p.k_blocks = (K + BK - 1) / BK;
     p.kb_per_split = p.k_blocks;
@@ -1116,7 +1118,7 @@ LGML_API int lgml_gemm_tcgen05_grouped(const void *x, const void *w, void *y, in
     p.bias = nullptr;
     p.status = status;
     p.swiglu = swiglu;
-    p.act_alpha = p.act_limit = 0.f;
+    p.act_alpha = act_alpha, p.act_limit = act_limit;
     p.transposed = 0;
     p.rows_a = max_tiles * BM;
     p.rows_b = N;
@@ -1133,4 +1135,10 @@ LGML_API int lgml_gemm_tcgen05_grouped(const void *x, const void *w, void *y, in
     dim3 grid(n_tiles < 148 ? n_tiles : 148, 1, 1);
     if (bn == 128) return launch<128, 6, 1>(ma, mb, p, grid, stream);
     return launch<256, 4, 2>(ma, mb, p, grid, stream);
+}
+
+LGML_API int lgml_gemm_tcgen05_grouped(const void *x, const void *w, void *y, int y_f32, int max_tiles, int N, int K, int n_groups, int ldy,
+                                       const int *group, int swiglu, int *status, cudaStream_t stream) {
+    LGML_REQUIRE(swiglu >= 0 && swiglu <= 2, "gemm_tcgen05_grouped: unknown epilogue %d", swiglu);
+    return lgml_gemm_tcgen05_grouped_act(x, w, y, y_f32, max_tiles, N, K, n_groups, ldy, group, swiglu, 0.f, 0.f, status, stream);
 }

@@ -170,11 +170,20 @@ __device__ __forceinline__ void rows_dot_bf16(const __nv_bfloat16 *const (&rows)
     for (int i = 0; i < NF; ++i) out[i] = warp_sum(out[i]);
 }
 
-// act[(t top + s), f] = silu(Wg[e] h_t)[f] * (Wu[e] h_t)[f], e = ids[t, s].  A warp takes GU_PER_WARP features at once.
+// the activation of a (gate, up) pair: silu(gate) * up, or (form 2) g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, +-limit)
+__device__ __forceinline__ float pair_act(float gate, float up, int form, float alpha, float limit) {
+    if (form == 2) {
+        const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+        return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+    }
+    return gate / (1.0f + expf(-gate)) * up;
+}
+
+// act[(t top + s), f] = silu(Wg[e] h_t)[f] * (Wu[e] h_t)[f] (or the clamped form), e = ids[t, s].  A warp takes GU_PER_WARP features at once.
 constexpr int GU_WARPS = 4, GU_PER_WARP = 4;
 template <typename T>
 __global__ void __launch_bounds__(GU_WARPS * 32) moe_gate_up_kernel(const T *__restrict__ h, int ldh, const int *__restrict__ ids, const T *__restrict__ wgu,
-                                                                    T *__restrict__ act, int E, int F, int X, int top, int plain) {
+                                                                    T *__restrict__ act, int E, int F, int X, int top, int plain, float alpha, float limit) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float hs[];       // the token's row
@@ -187,7 +196,7 @@ __global__ void __launch_bounds__(GU_WARPS * 32) moe_gate_up_kernel(const T *__r
     __syncthreads();
     const int f0 = (blockIdx.y * GU_WARPS + warp) * GU_PER_WARP;
     if (f0 >= F) return;
-    if (plain) {
+    if (plain == 1) {
         // experts without a gate: wgu is [X, F, E] and act = relu(W_up h)^2
         const T *we = wgu + (size_t)e * F * E;
         if (sizeof(T) == 2 && (E % 8 == 0) && (reinterpret_cast<uintptr_t>(wgu) & 15) == 0) {
@@ -229,7 +238,7 @@ __global__ void __launch_bounds__(GU_WARPS * 32) moe_gate_up_kernel(const T *__r
         if (lane == 0)
 #pragma unroll
             for (int i = 0; i < GU_PER_WARP; ++i)
-                if (f0 + i < F) act[(size_t)row * F + f0 + i] = from_f32<T>(r[i] / (1.0f + expf(-r[i])) * r[GU_PER_WARP + i]);
+                if (f0 + i < F) act[(size_t)row * F + f0 + i] = from_f32<T>(pair_act(r[i], r[GU_PER_WARP + i], plain, alpha, limit));
         return;
     }
     for (int f = f0; f < f0 + GU_PER_WARP && f < F; ++f) {
@@ -242,7 +251,7 @@ __global__ void __launch_bounds__(GU_WARPS * 32) moe_gate_up_kernel(const T *__r
         }
         g = warp_sum(g);
         u = warp_sum(u);
-        if (lane == 0) act[(size_t)row * F + f] = from_f32<T>(g / (1.0f + expf(-g)) * u);
+        if (lane == 0) act[(size_t)row * F + f] = from_f32<T>(pair_act(g, u, plain, alpha, limit));
     }
 }
 
@@ -271,7 +280,7 @@ __global__ void __launch_bounds__(DN_WARPS * 32) moe_down_kernel(const T *__rest
         int e = act_load(ids + (size_t)t * top + s);
         if (e < 0) continue;                    // a slot without an expert
         e = e >= X ? X - 1 : e;
-        const float w = act_load(wts + (size_t)t * top + s);
+        const float w = wts != nullptr ? act_load(wts + (size_t)t * top + s) : 1.0f / (float)top;      // null: every expert counts the same
         float r[DN_PER_WARP];
         if (vec) {
             const __nv_bfloat16 *rows[DN_PER_WARP];
@@ -365,9 +374,10 @@ LGML_API int lgml_moe_router(const void *h, int dtype, int ldh, const float *wr,
 // The row form: act [n top, F] in the compute type (scratch of the caller), out float32 [n, E].
 // plain = 1: experts without a gate (wgu is [X, F, E], act = relu(W_up h)^2).  also / also_w: rows of E entries, lda apart, float32 or (also_own = 1) in the
 // compute type, and float32 [n]: out += also_w[t] also[t] (or null).
-LGML_API int lgml_moe_experts_rows_form(const void *h, int dtype, int ldh, const int *ids, const float *wts, const void *wgu, const void *wd,
-                                        void *act, float *out, int n_tokens, int E, int F, int X, int top, int plain, const void *also,
-                                        int also_own, int lda, const float *also_w, cudaStream_t stream) {
+// plain = 2: gated experts with the clamped activation (alpha, limit).  wts null: a token's experts count the same, 1 / top each.
+LGML_API int lgml_moe_experts_rows_act(const void *h, int dtype, int ldh, const int *ids, const float *wts, const void *wgu, const void *wd,
+                                       void *act, float *out, int n_tokens, int E, int F, int X, int top, int plain, float alpha, float limit,
+                                       const void *also, int also_own, int lda, const float *also_w, cudaStream_t stream) {
     LGML_REQUIRE(n_tokens >= 0 && E > 0 && F > 0 && X > 0 && top > 0, "moe_experts_rows: bad sizes");
     if (n_tokens == 0) return 0;
     const size_t smem_gu = sizeof(float) * (size_t)E, smem_dn = sizeof(float) * (size_t)top * F;
@@ -377,7 +387,7 @@ LGML_API int lgml_moe_experts_rows_form(const void *h, int dtype, int ldh, const
     if (dtype == LGML_F32) {
         if (need_smem(moe_gate_up_kernel<float>, smem_gu, "moe_experts_rows") || need_smem(moe_down_kernel<float, float>, smem_dn, "moe_experts_rows")) return -1;
         lgml_launch(moe_gate_up_kernel<float>, grid_gu, GU_WARPS * 32, smem_gu, stream, (const float *)h, ldh, ids, (const float *)wgu, (float *)act, E, F, X,
-                    top, plain);
+                    top, plain, alpha, limit);
         lgml_launch(moe_down_kernel<float, float>, grid_dn, DN_WARPS * 32, smem_dn, stream, (const float *)act, ids, wts, (const float *)wd, out, E, F, X, top,
                     (const float *)also, lda, also_w);
     } else if (dtype == LGML_BF16) {
@@ -386,7 +396,7 @@ LGML_API int lgml_moe_experts_rows_form(const void *h, int dtype, int ldh, const
             need_smem(moe_down_kernel<__nv_bfloat16, __nv_bfloat16>, smem_dn, "moe_experts_rows"))
             return -1;
         lgml_launch(moe_gate_up_kernel<__nv_bfloat16>, grid_gu, GU_WARPS * 32, smem_gu, stream, (const __nv_bfloat16 *)h, ldh, ids,
-                    (const __nv_bfloat16 *)wgu, (__nv_bfloat16 *)act, E, F, X, top, plain);
+                    (const __nv_bfloat16 *)wgu, (__nv_bfloat16 *)act, E, F, X, top, plain, alpha, limit);
         if (also_own)
             lgml_launch(moe_down_kernel<__nv_bfloat16, __nv_bfloat16>, grid_dn, DN_WARPS * 32, smem_dn, stream, (const __nv_bfloat16 *)act, ids, wts,
                         (const __nv_bfloat16 *)wd, out, E, F, X, top, (const __nv_bfloat16 *)also, lda, also_w);
@@ -397,6 +407,13 @@ LGML_API int lgml_moe_experts_rows_form(const void *h, int dtype, int ldh, const
         LGML_FAIL("moe_experts_rows: unknown type %d", dtype);
     }
     return lgml_launch_status("moe_experts_rows");
+}
+
+LGML_API int lgml_moe_experts_rows_form(const void *h, int dtype, int ldh, const int *ids, const float *wts, const void *wgu, const void *wd,
+                                        void *act, float *out, int n_tokens, int E, int F, int X, int top, int plain, const void *also,
+                                        int also_own, int lda, const float *also_w, cudaStream_t stream) {
+    LGML_REQUIRE(plain == 0 || plain == 1, "moe_experts_rows: unknown form %d", plain);
+    return lgml_moe_experts_rows_act(h, dtype, ldh, ids, wts, wgu, wd, act, out, n_tokens, E, F, X, top, plain, 0.f, 0.f, also, also_own, lda, also_w, stream);
 }
 
 LGML_API int lgml_moe_experts_rows(const void *h, int dtype, int ldh, const int *ids, const float *wts, const void *wgu, const void *wd,
@@ -753,4 +770,73 @@ LGML_API int lgml_moe_weighted_sum_form(const float *y, const int *pos, const in
 
 LGML_API int lgml_moe_weighted_sum(const float *y, const int *pos, const float *wts, float *out, int n_tokens, int E, int top, cudaStream_t stream) {
     return lgml_moe_weighted_sum_form(y, pos, nullptr, wts, out, n_tokens, E, top, nullptr, 0, E, nullptr, stream);
+}
+
+// ---------------------------------------------------------------------------------------------
+// Experts that stand in a table: a token's id names them, so what runs is known before the first layer.  One launch per step
+// does it for the tables of all layers, a block a table: the experts of every (token, slot) row, the tiles of 128 rows of
+// one expert, and the row's place among the tiles (its tile times 128 + its place in it).
+//   desc int32 [n_tables, 3]: experts X, slots a token `top`, first entry of the table in `tables` ([vocab, top] each)
+//   out: per table, one behind the other: ids [n top] | places [n top] | tiles [3 max_tiles] | number of tiles, with
+//   max_tiles = ceil(n top / 128) + min(X, n top)
+// ---------------------------------------------------------------------------------------------
+namespace {
+__global__ void __launch_bounds__(1024) table_route_kernel(const int *__restrict__ token_ids, int n, int vocab, const int *__restrict__ tables,
+                                                           const int *__restrict__ desc, int *__restrict__ out, int max_x) {
+    pdl_trigger();
+    extern __shared__ int sh[];         // counts[X], cursor[X], tile0[X]
+    __shared__ long long base_s;
+    int *counts = sh, *cursor = sh + max_x, *tile0 = sh + 2 * max_x;
+    const int X = desc[3 * blockIdx.x], top = desc[3 * blockIdx.x + 1];
+    const int *table = tables + desc[3 * blockIdx.x + 2];
+    if (threadIdx.x == 0) {
+        long long b = 0;
+        for (int l = 0; l < (int)blockIdx.x; ++l) {
+            const int rows = n * desc[3 * l + 1];
+            b += 2LL * rows + 3LL * ((rows + G_TM - 1) / G_TM + min(desc[3 * l], rows)) + 1;
+        }
+        base_s = b;
+    }
+    for (int e = threadIdx.x; e < X; e += blockDim.x) counts[e] = 0, cursor[e] = 0;
+    pdl_wait();
+    __syncthreads();
+    const int rows = n * top, max_tiles = (rows + G_TM - 1) / G_TM + min(X, rows);
+    int *ids = out + base_s, *pos = ids + rows, *tiles = pos + rows;
+    for (int r = threadIdx.x; r < rows; r += blockDim.x) {
+        const int t = r / top, id = min(max(act_load(token_ids + t), 0), vocab - 1);      // the embedding kernel has flagged an id outside the vocabulary
+        const int e = min(max(__ldg(table + (size_t)id * top + (r - t * top)), 0), X - 1);
+        ids[r] = e;
+        atomicAdd(&counts[e], 1);
+    }
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        int tl = 0;
+        for (int e = 0; e < X; ++e) {
+            tile0[e] = tl;
+            tl += (counts[e] + G_TM - 1) / G_TM;
+        }
+        tiles[3 * max_tiles] = tl;
+    }
+    __syncthreads();
+    for (int r = threadIdx.x; r < rows; r += blockDim.x) {
+        const int e = ids[r];           // this thread wrote it
+        const int c = atomicAdd(&cursor[e], 1);
+        pos[r] = (tile0[e] + c / G_TM) * G_TM + c % G_TM;
+    }
+    for (int e = threadIdx.x; e < X; e += blockDim.x)
+        for (int i = 0; i * G_TM < counts[e]; ++i) {
+            int *tl = tiles + 3 * (tile0[e] + i);
+            tl[0] = e, tl[1] = 0, tl[2] = min(G_TM, counts[e] - i * G_TM);
+        }
+}
+}  // namespace
+
+LGML_API int lgml_table_route(const int *token_ids, int n_tokens, int vocab, const int *tables, const int *desc, int n_tables, int max_x, int *out,
+                              cudaStream_t stream) {
+    LGML_REQUIRE(n_tokens >= 0 && vocab > 0 && n_tables > 0 && max_x > 0 && max_x <= 8192, "table_route: bad sizes");
+    if (n_tokens == 0) return 0;
+    const size_t smem = sizeof(int) * 3 * (size_t)max_x;
+    if (need_smem(table_route_kernel, smem, "table_route")) return -1;
+    lgml_launch(table_route_kernel, n_tables, 1024, smem, stream, token_ids, n_tokens, vocab, tables, desc, out, max_x);
+    return lgml_launch_status("table_route");
 }

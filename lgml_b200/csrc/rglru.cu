@@ -1,0 +1,530 @@
+// A real-gated linear recurrent unit behind a short convolution, per channel c of request s:
+//
+//   u_t   = bias_c + sum_j w[j, c] x_(t - taps + 1 + j)              (inputs before the start are zero)
+//   r_t   = sigmoid((Ra[b] u_t,b + ra_b)_c),  i_t = sigmoid((Ri[b] u_t,b + ri_b)_c)      b: the part of the channels that holds c
+//   a_t   = exp(-8 r_t softplus(lam_c));      S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t
+//   out_t = S_t gelu_tanh(y_t)
+//
+// x | y are the columns of one projection, proj float32 [n, 2 C].  A request's state row, float32: S [C], then a ring of the
+// last `taps` inputs, [taps, C], the input of position p in row p mod taps (absent with one tap): what a step of one token
+// writes is then not what anyone reads, and every block of channels may work on its own.
+//
+//   rglru_step    one token a request: convolution, both gates, recurrence and output in one kernel, a block per (8 tokens, 32 channels)
+//   rglru_conv    the convolution alone for longer portions; also brings the ring up to date
+//   rglru_gates   a_t and the pushed term sqrt(1 - a^2) i u for many tokens: in bfloat16 on tensor cores with u in three
+//                 bfloat16 pieces (24 bits: what is multiplied is the float32 number), else as products of 8 rows
+//   rglru_scan    S_t = a_t S_(t-1) + push_t and the output, a thread a channel of a request
+//   rglru_chunks  the same for long portions in three passes: every chunk's (product of a, scan from zero), the chain over
+//                 a request's chunks, every chunk again from its true start
+//
+// Everything here is float32 arithmetic in both compute types (the gates' matrices are in the compute type); only out, which
+// feeds a matrix product, is stored in the compute type.
+#include <math.h>
+
+#include "common.cuh"
+#include "few_rows.cuh"
+
+LGML_DEFINE_LAST_ERROR(lgml_rglru)
+
+namespace {
+constexpr int NT = 8;            // tokens a block of the row forms takes
+constexpr int CH = 32;           // channels a block of the row forms takes: eight warps of four
+constexpr int CHUNK = 32;        // tokens of a chunk of a long portion
+constexpr int MAX_TAPS = 16;
+
+__device__ __forceinline__ float sigmoid_(float v) { return 1.0f / (1.0f + expf(-v)); }
+__device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+
+// a and the pushed term from the gates' logits; sp8 = 8 softplus(lam)
+__device__ __forceinline__ void gate_pair(float zr, float zi, float sp8, float u, float &a, float &push) {
+    const float log_a = -sigmoid_(zr) * sp8;
+    a = expf(log_a);
+    push = sqrtf(-expm1f(2.0f * log_a)) * sigmoid_(zi) * u;
+}
+
+// One result of the convolution: the inputs in order, oldest first.  Token t of the step at position pos, its request's first token
+// t0; inputs of earlier steps come from the ring.
+__device__ __forceinline__ float conv_at(const float *__restrict__ x, int ldx, const float *__restrict__ w, float bias, const float *ring, int C, int taps,
+                                         int t, int t0, int pos, int c) {
+    float v = bias;
+    for (int j = 0; j < taps; ++j) {
+        const int back = taps - 1 - j;
+        if (pos - back < 0) continue;
+        const float in = t - back >= t0 ? act_load(x + (size_t)(t - back) * ldx + c) : act_load(ring + (size_t)((pos - back) % taps) * C + c);
+        v = fmaf(__ldg(w + (size_t)j * C + c), in, v);
+    }
+    return v;
+}
+
+// ---- one token a request ---------------------------------------------------------------------------
+template <typename T, typename TO>
+__global__ void __launch_bounds__(256) rglru_step_kernel(const float *__restrict__ proj, int ldp, const float *__restrict__ conv_w,
+                                                         const float *__restrict__ conv_b, float *__restrict__ state, long long state_ld,
+                                                         const int *__restrict__ slots, const int *__restrict__ positions, const T *__restrict__ ra,
+                                                         const float *__restrict__ ra_b, const T *__restrict__ ri, const float *__restrict__ ri_b,
+                                                         const float *__restrict__ sp8, TO *__restrict__ out, int n, int C, int P, int taps, int lanes, int vec) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ __align__(16) float us[];        // u of up to 8 tokens, the whole part of the channels
+    const int ldu = (P + 3) & ~3;
+    const int b = blockIdx.y, t0 = blockIdx.z * NT, nt = min(NT, n - t0);
+    for (int e = threadIdx.x; e < NT * ldu; e += blockDim.x) {
+        const int j = e / ldu, k = e - j * ldu;
+        float u = 0.f;
+        if (j < nt && k < P) {
+            const int t = t0 + j, c = b * P + k;
+            const float *ring = state + (size_t)slots[t] * state_ld + C;
+            u = conv_at(proj, ldp, conv_w, conv_b[c], ring, C, taps, t, t, positions[t], c);
+        }
+        us[e] = u;
+    }
+    __syncthreads();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, per = 32 / lanes, sub = lane % lanes;
+    for (int j0 = 0; j0 < 4; j0 += per) {
+        const int q = j0 + lane / lanes, k = blockIdx.x * CH + warp * 4 + q;       // this lane group's channel of the part
+        const bool mine = q < 4 && k < P;
+        float zr[NT], zi[NT];
+#pragma unroll
+        for (int j = 0; j < NT; ++j) zr[j] = zi[j] = 0.f;
+        if (mine) {
+            few_rows_share<T, NT>(ra + ((size_t)b * P + k) * P, us, ldu, P, sub, lanes, vec != 0, zr);
+            few_rows_share<T, NT>(ri + ((size_t)b * P + k) * P, us, ldu, P, sub, lanes, vec != 0, zi);
+        }
+        few_rows_reduce<NT>(zr, lanes);
+        few_rows_reduce<NT>(zi, lanes);
+        if (!mine) continue;
+        const int c = b * P + k;
+        // the lanes of a channel share its tokens
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+            if (j % lanes != sub || j >= nt) continue;
+            const int t = t0 + j;
+            float *row = state + (size_t)slots[t] * state_ld;
+            float a, push;
+            gate_pair(zr[j] + ra_b[c], zi[j] + ri_b[c], sp8[c], us[j * ldu + k], a, push);
+            const float S = fmaf(a, act_load(row + c), push);
+            row[c] = S;
+            out[(size_t)t * C + c] = from_f32<TO>(S * gelu_tanh(act_load(proj + (size_t)t * ldp + C + c)));
+            if (taps > 1) row[C + (size_t)(positions[t] % taps) * C + c] = act_load(proj + (size_t)t * ldp + c);
+        }
+    }
+}
+
+// ---- the convolution of longer portions ----------------------------------------------------------------
+// A thread takes one channel of one token.  The thread of a request's first token computes every token that reaches into
+// the ring and then writes the step's last taps - 1 inputs there; nobody else touches those floats.
+__global__ void __launch_bounds__(256) rglru_conv_kernel(const float *__restrict__ proj, int ldp, const float *__restrict__ conv_w,
+                                                         const float *__restrict__ conv_b, float *__restrict__ state, long long state_ld,
+                                                         const int *__restrict__ seq_of_token, const int *__restrict__ seq_start,
+                                                         const int *__restrict__ slots, const int *__restrict__ positions, float *__restrict__ u, int n, int C,
+                                                         int taps) {
+    pdl_trigger();
+    pdl_wait();
+    const size_t total = (size_t)n * C;
+    for (size_t it = (size_t)blockIdx.x * blockDim.x + threadIdx.x; it < total; it += (size_t)gridDim.x * blockDim.x) {
+        const int t = (int)(it / C), c = (int)(it - (size_t)t * C);
+        const int s = seq_of_token[t], t0 = seq_start[s];
+        const float bias = __ldg(conv_b + c);
+        if (t == t0) {
+            float *ring = state + (size_t)slots[s] * state_ld + C;
+            const int t1 = seq_start[s + 1], last = min(t1, t0 + max(taps - 1, 1)), pos0 = positions[t0];
+            for (int i = t0; i < last; ++i) u[(size_t)i * C + c] = conv_at(proj, ldp, conv_w, bias, ring, C, taps, i, t0, pos0 + i - t0, c);
+            if (taps > 1)
+                for (int i = max(t0, t1 - (taps - 1)); i < t1; ++i) ring[(size_t)((pos0 + i - t0) % taps) * C + c] = act_load(proj + (size_t)i * ldp + c);
+        } else if (t - t0 >= taps - 1) {
+            u[it] = conv_at(proj, ldp, conv_w, bias, nullptr, C, taps, t, t0, positions[t], c);
+        }
+    }
+}
+
+// The same for many tokens, four channels a thread and four tokens in a row (a row of inputs is read once for four results): tokens
+// 4 i .. 4 i + 3 of the step, whichever requests they belong to.  Taps at compile time, C a multiple of 4.
+template <int TAPS>
+__global__ void __launch_bounds__(256) rglru_conv_runs_kernel(const float *__restrict__ proj, int ldp, const float *__restrict__ conv_w,
+                                                              const float *__restrict__ conv_b, float *__restrict__ state, long long state_ld,
+                                                              const int *__restrict__ seq_of_token, const int *__restrict__ seq_start,
+                                                              const int *__restrict__ slots, const int *__restrict__ positions, float *__restrict__ u, int n,
+                                                              int C) {
+    pdl_trigger();
+    pdl_wait();
+    constexpr int RUN = 4;
+    const int quads = C / 4;
+    const size_t total = (size_t)((n + RUN - 1) / RUN) * quads;
+    for (size_t it = (size_t)blockIdx.x * blockDim.x + threadIdx.x; it < total; it += (size_t)gridDim.x * blockDim.x) {
+        const int ta = (int)(it / quads) * RUN, c = (int)(it - (size_t)(ta / RUN) * quads) * 4, tb = min(n, ta + RUN);
+        float4 w[TAPS];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[j] = __ldg(reinterpret_cast<const float4 *>(conv_w + (size_t)j * C + c));
+        const float4 bias = __ldg(reinterpret_cast<const float4 *>(conv_b + c));
+        float4 in[RUN + TAPS - 1];
+#pragma unroll
+        for (int k = 0; k < RUN + TAPS - 1; ++k) {
+            const int t = ta - (TAPS - 1) + k;
+            in[k] = t >= 0 && t < tb ? act_load(reinterpret_cast<const float4 *>(proj + (size_t)t * ldp + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int i = 0; i < RUN; ++i) {
+            const int t = ta + i;
+            if (t >= tb) break;
+            const int s = seq_of_token[t], t0 = seq_start[s];
+            if (t - t0 >= TAPS - 1) {
+                float4 v = bias;
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) {
+                    v.x = fmaf(w[j].x, in[i + j].x, v.x), v.y = fmaf(w[j].y, in[i + j].y, v.y);
+                    v.z = fmaf(w[j].z, in[i + j].z, v.z), v.w = fmaf(w[j].w, in[i + j].w, v.w);
+                }
+                *reinterpret_cast<float4 *>(u + (size_t)t * C + c) = v;
+            } else if (t == t0) {
+                float *ring = state + (size_t)slots[s] * state_ld + C;
+                const int t1 = seq_start[s + 1], last = min(t1, t0 + max(TAPS - 1, 1)), pos0 = positions[t0];
+                for (int e = 0; e < 4; ++e) {
+                    for (int k = t0; k < last; ++k)
+                        u[(size_t)k * C + c + e] = conv_at(proj, ldp, conv_w, __ldg(conv_b + c + e), ring, C, TAPS, k, t0, pos0 + k - t0, c + e);
+                    if (TAPS > 1)
+                        for (int k = max(t0, t1 - (TAPS - 1)); k < t1; ++k)
+                            ring[(size_t)((pos0 + k - t0) % TAPS) * C + c + e] = act_load(proj + (size_t)k * ldp + c + e);
+                }
+            }
+        }
+    }
+}
+
+// ---- the gates of longer portions -------------------------------------------------------------------------
+// u float32 [n, C] -> ab float32 [2, n, C]: a, then the pushed term
+template <typename T>
+__global__ void __launch_bounds__(256) rglru_gates_rows_kernel(const float *__restrict__ u, const T *__restrict__ ra, const float *__restrict__ ra_b,
+                                                               const T *__restrict__ ri, const float *__restrict__ ri_b, const float *__restrict__ sp8,
+                                                               float *__restrict__ ab, int n, int C, int P, int lanes, int vec) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ __align__(16) float us[];
+    const int ldu = (P + 3) & ~3;
+    const int b = blockIdx.y, t0 = blockIdx.x * NT, nt = min(NT, n - t0);
+    for (int e = threadIdx.x; e < NT * ldu; e += blockDim.x) {
+        const int j = e / ldu, k = e - j * ldu;
+        us[e] = j < nt && k < P ? act_load(u + (size_t)(t0 + j) * C + b * P + k) : 0.f;
+    }
+    __syncthreads();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, per = 32 / lanes, sub = lane % lanes;
+    for (int j0 = 0; j0 < 4; j0 += per) {
+        const int q = j0 + lane / lanes, k = blockIdx.z * CH + warp * 4 + q;
+        const bool mine = q < 4 && k < P;
+        float zr[NT], zi[NT];
+#pragma unroll
+        for (int j = 0; j < NT; ++j) zr[j] = zi[j] = 0.f;
+        if (mine) {
+            few_rows_share<T, NT>(ra + ((size_t)b * P + k) * P, us, ldu, P, sub, lanes, vec != 0, zr);
+            few_rows_share<T, NT>(ri + ((size_t)b * P + k) * P, us, ldu, P, sub, lanes, vec != 0, zi);
+        }
+        few_rows_reduce<NT>(zr, lanes);
+        few_rows_reduce<NT>(zi, lanes);
+        if (!mine) continue;
+        const int c = b * P + k;
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+            if (j % lanes != sub || j >= nt) continue;
+            float a, push;
+            gate_pair(zr[j] + ra_b[c], zi[j] + ri_b[c], sp8[c], us[j * ldu + k], a, push);
+            ab[(size_t)(t0 + j) * C + c] = a;
+            ab[(size_t)(n + t0 + j) * C + c] = push;
+        }
+    }
+}
+
+// Many tokens in bfloat16 (mma.sync m16n8k16, float32 accumulation): a block of four warps takes 64 tokens x 64 channels of one part, both
+// gates at once (128 columns), a warp 16 tokens.  u goes into shared memory as three bfloat16 numbers whose sum is the float32 number
+// (8 + 8 + 8 bits), each multiplied by the same matrix piece: bfloat16 products are exact in float32, so only the sums round.
+constexpr int GT = 64, GK = 64, GLD = GK + 8;
+__device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void load_matrix(uint32_t (&r)[4], const __nv_bfloat16 *p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)));
+}
+__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__global__ void __launch_bounds__(128) rglru_gates_mma_kernel(const float *__restrict__ u, const __nv_bfloat16 *__restrict__ ra, const float *__restrict__ ra_b,
+                                                              const __nv_bfloat16 *__restrict__ ri, const float *__restrict__ ri_b,
+                                                              const float *__restrict__ sp8, float *__restrict__ ab, int n, int C, int P) {
+    pdl_trigger();
+    pdl_wait();
+    extern __shared__ __align__(16) __nv_bfloat16 gm[];
+    __nv_bfloat16 *As = gm, *Bs = gm + 3 * GT * GLD;          // three pieces of u; 64 rows of Ra and 64 of Ri
+    const int t0 = blockIdx.x * GT, b = blockIdx.z, k_out = blockIdx.y * 64;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int mat = lane >> 3, mrow = lane & 7;
+    float acc[16][4];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    for (int k0 = 0; k0 < P; k0 += GK) {
+        for (int e = threadIdx.x; e < 128 * (GK / 8); e += 128) {
+            const int r = e / (GK / 8), col = (e - r * (GK / 8)) * 8, o = k_out + (r & 63);
+            const bool ok = o < P && k0 + col < P;
+            const __nv_bfloat16 *src = (r < 64 ? ra : ri) + ((size_t)b * P + (ok ? o : 0)) * P + (ok ? k0 + col : 0);
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(Bs + r * GLD + col)), "l"(src), "r"(ok ? 16 : 0) : "memory");
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        for (int e = threadIdx.x; e < GT * (GK / 4); e += 128) {
+            const int r = e / (GK / 4), col = (e - r * (GK / 4)) * 4;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (t0 + r < n && k0 + col < P) v = act_load(reinterpret_cast<const float4 *>(u + (size_t)(t0 + r) * C + b * P + k0 + col));
+            float x[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (int piece = 0; piece < 3; ++piece) {
+                __nv_bfloat162 lo = __floats2bfloat162_rn(x[0], x[1]), hi = __floats2bfloat162_rn(x[2], x[3]);
+                *reinterpret_cast<uint2 *>(As + (piece * GT + r) * GLD + col) = make_uint2(*reinterpret_cast<unsigned *>(&lo), *reinterpret_cast<unsigned *>(&hi));
+                x[0] -= __low2float(lo), x[1] -= __high2float(lo), x[2] -= __low2float(hi), x[3] -= __high2float(hi);
+            }
+        }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+#pragma unroll
+        for (int ks = 0; ks < GK / 16; ++ks) {
+            uint32_t a[3][4];
+#pragma unroll
+            for (int piece = 0; piece < 3; ++piece)
+                load_matrix(a[piece], As + (piece * GT + warp * 16 + (mat & 1) * 8 + mrow) * GLD + ks * 16 + (mat >> 1) * 8);
+#pragma unroll
+            for (int np = 0; np < 8; ++np) {
+                uint32_t q[4];
+                load_matrix(q, Bs + (np * 16 + (mat >> 1) * 8 + mrow) * GLD + ks * 16 + (mat & 1) * 8);
+#pragma unroll
+                for (int piece = 2; piece >= 0; --piece) {         // the small pieces first
+                    mma_bf16(acc[2 * np], a[piece], q[0], q[1]);
+                    mma_bf16(acc[2 * np + 1], a[piece], q[2], q[3]);
+                }
+            }
+        }
+        __syncthreads();
+    }
+    // accumulators 0..7: Ra's columns, 8..15: Ri's, the same channels in the same thread
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt) {
+        const int k = k_out + nt * 8 + (lane & 3) * 2;
+        if (k >= P) continue;
+        const int c = b * P + k;          // P and so k and c are even
+        const float2 br = __ldg(reinterpret_cast<const float2 *>(ra_b + c)), bi = __ldg(reinterpret_cast<const float2 *>(ri_b + c));
+        const float2 sp = __ldg(reinterpret_cast<const float2 *>(sp8 + c));
+#pragma unroll
+        for (int rr = 0; rr < 2; ++rr) {
+            const int t = t0 + warp * 16 + (lane >> 2) + rr * 8;
+            if (t >= n) continue;
+            const float2 uv = act_load(reinterpret_cast<const float2 *>(u + (size_t)t * C + c));
+            float2 a, p;
+            gate_pair(acc[nt][rr * 2] + br.x, acc[nt + 8][rr * 2] + bi.x, sp.x, uv.x, a.x, p.x);
+            gate_pair(acc[nt][rr * 2 + 1] + br.y, acc[nt + 8][rr * 2 + 1] + bi.y, sp.y, uv.y, a.y, p.y);
+            *reinterpret_cast<float2 *>(ab + (size_t)t * C + c) = a;
+            *reinterpret_cast<float2 *>(ab + (size_t)(n + t) * C + c) = p;
+        }
+    }
+}
+
+// ---- the recurrence ---------------------------------------------------------------------------------------
+// ab float32 [2, n, C]; y: columns C .. 2 C - 1 of proj.  A thread owns one channel of one request (or of one chunk, from S0) and walks
+// its tokens in order; the loads of AHEAD tokens are in flight at a time.
+constexpr int AHEAD = 8;
+template <typename TO>
+__device__ __forceinline__ float walk(const float *__restrict__ ab, const float *__restrict__ proj, int ldp, TO *__restrict__ out, int n, int C, int c, int t0,
+                                      int t1, float S) {
+    for (int t = t0; t < t1; t += AHEAD) {
+        float a[AHEAD], b[AHEAD], y[AHEAD];
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i)
+            if (t + i < t1) {
+                a[i] = act_load(ab + (size_t)(t + i) * C + c), b[i] = act_load(ab + (size_t)(n + t + i) * C + c);
+                y[i] = act_load(proj + (size_t)(t + i) * ldp + C + c);
+            }
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i)
+            if (t + i < t1) {
+                S = fmaf(a[i], S, b[i]);
+                out[(size_t)(t + i) * C + c] = from_f32<TO>(S * gelu_tanh(y[i]));
+            }
+    }
+    return S;
+}
+
+template <typename TO>
+__global__ void __launch_bounds__(128) rglru_scan_kernel(const float *__restrict__ ab, const float *__restrict__ proj, int ldp, float *__restrict__ state,
+                                                         long long state_ld, const int *__restrict__ seq_start, const int *__restrict__ slots,
+                                                         TO *__restrict__ out, int n, int C) {
+    pdl_trigger();
+    pdl_wait();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, s = blockIdx.y;
+    if (c >= C) return;
+    float *st = state + (size_t)slots[s] * state_ld + c;
+    *st = walk<TO>(ab, proj, ldp, out, n, C, c, seq_start[s], seq_start[s + 1], act_load(st));
+}
+
+// pass 1: per (chunk, channel): A = prod a, B = the scan's end from S = 0
+__global__ void __launch_bounds__(128) rglru_chunk_ends_kernel(const float *__restrict__ ab, const int *__restrict__ chunks, float *__restrict__ A,
+                                                               float *__restrict__ B, int n, int C) {
+    pdl_trigger();
+    pdl_wait();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, k = blockIdx.y;
+    if (c >= C) return;
+    const int t0 = chunks[2 * k], t1 = chunks[2 * k + 1];
+    float prod = 1.f, S = 0.f;
+    for (int t = t0; t < t1; t += AHEAD) {
+        float a[AHEAD], b[AHEAD];
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i)
+            if (t + i < t1) a[i] = act_load(ab + (size_t)(t + i) * C + c), b[i] = act_load(ab + (size_t)(n + t + i) * C + c);
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i)
+            if (t + i < t1) S = fmaf(a[i], S, b[i]), prod *= a[i];
+    }
+    A[(size_t)k * C + c] = prod, B[(size_t)k * C + c] = S;
+}
+
+// pass 2: per (request, channel): S at the start of every chunk (written over B), and the slot's new state
+__global__ void __launch_bounds__(128) rglru_chain_kernel(const float *__restrict__ A, float *__restrict__ B, const int *__restrict__ chunk_start,
+                                                          float *__restrict__ state, long long state_ld, const int *__restrict__ slots, int C) {
+    pdl_trigger();
+    pdl_wait();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, s = blockIdx.y;
+    if (c >= C) return;
+    float *st = state + (size_t)slots[s] * state_ld + c;
+    float S = act_load(st);
+    const int k1 = chunk_start[s + 1];
+    for (int k = chunk_start[s]; k < k1; k += AHEAD) {
+        float a[AHEAD], b[AHEAD];
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i)
+            if (k + i < k1) a[i] = act_load(A + (size_t)(k + i) * C + c), b[i] = act_load(B + (size_t)(k + i) * C + c);
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i)
+            if (k + i < k1) {
+                B[(size_t)(k + i) * C + c] = S;
+                S = fmaf(a[i], S, b[i]);
+            }
+    }
+    *st = S;
+}
+
+// pass 3: every chunk from its true start
+template <typename TO>
+__global__ void __launch_bounds__(128) rglru_chunk_scan_kernel(const float *__restrict__ ab, const float *__restrict__ proj, int ldp,
+                                                               const int *__restrict__ chunks, const float *__restrict__ S0, TO *__restrict__ out, int n, int C) {
+    pdl_trigger();
+    pdl_wait();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, k = blockIdx.y;
+    if (c >= C) return;
+    walk<TO>(ab, proj, ldp, out, n, C, c, chunks[2 * k], chunks[2 * k + 1], act_load(S0 + (size_t)k * C + c));
+}
+}  // namespace
+
+LGML_API int lgml_rglru_chunk_tokens(void) { return CHUNK; }
+
+#define RGLRU_SIZES(who)                                                                                                                       \
+    LGML_REQUIRE(n_tokens >= 0 && C > 0 && P > 0 && C % P == 0 && C / P <= 65535, who ": %d channels in parts of %d", C, P);                   \
+    LGML_REQUIRE(dtype == LGML_F32 || dtype == LGML_BF16, who ": unknown type %d", dtype)
+
+// One token a request, n_tokens of them.  ra, ri: [C / P, P, P] in `dtype`; ra_b, ri_b, sp8 (8 softplus(lam)), conv_b float32 [C]; conv_w float32 [taps, C];
+// state rows: C floats, then the ring.
+LGML_API int lgml_rglru_step(const float *proj, int ldp, const float *conv_w, const float *conv_b, float *state, long long state_ld, const int *slots,
+                             const int *positions, const void *ra, const float *ra_b, const void *ri, const float *ri_b, const float *sp8, void *out, int dtype,
+                             int n_tokens, int C, int P, int taps, cudaStream_t stream) {
+    RGLRU_SIZES("rglru_step");
+    LGML_REQUIRE(taps >= 1 && taps <= MAX_TAPS && ldp >= 2 * C && state_ld >= C + (taps > 1 ? (long long)taps * C : 0), "rglru_step: bad strides or taps");
+    const size_t smem = sizeof(float) * NT * (size_t)((P + 3) & ~3);
+    LGML_REQUIRE(smem <= 48 * 1024, "rglru_step: parts of %d channels are too wide", P);
+    LGML_REQUIRE((n_tokens + NT - 1) / NT <= 65535, "rglru_step: too many tokens");
+    if (n_tokens == 0) return 0;
+    dim3 grid((P + CH - 1) / CH, C / P, (n_tokens + NT - 1) / NT);
+    if (dtype == LGML_F32)
+        lgml_launch(rglru_step_kernel<float, float>, grid, 256, smem, stream, proj, ldp, conv_w, conv_b, state, state_ld, slots, positions, (const float *)ra, ra_b,
+                    (const float *)ri, ri_b, sp8, (float *)out, n_tokens, C, P, taps, few_rows_lanes<float>(P),
+                    few_rows_vec<float>(ra, P) && few_rows_vec<float>(ri, P) ? 1 : 0);
+    else
+        lgml_launch(rglru_step_kernel<__nv_bfloat16, __nv_bfloat16>, grid, 256, smem, stream, proj, ldp, conv_w, conv_b, state, state_ld, slots, positions,
+                    (const __nv_bfloat16 *)ra, ra_b, (const __nv_bfloat16 *)ri, ri_b, sp8, (__nv_bfloat16 *)out, n_tokens, C, P, taps,
+                    few_rows_lanes<__nv_bfloat16>(P), few_rows_vec<__nv_bfloat16>(ra, P) && few_rows_vec<__nv_bfloat16>(ri, P) ? 1 : 0);
+    return lgml_launch_status("rglru_step");
+}
+
+// u float32 [n, C]
+LGML_API int lgml_rglru_conv(const float *proj, int ldp, const float *conv_w, const float *conv_b, float *state, long long state_ld, const int *seq_of_token,
+                             const int *seq_start, const int *slots, const int *positions, float *u, int n_tokens, int C, int taps, cudaStream_t stream) {
+    LGML_REQUIRE(n_tokens >= 0 && C > 0 && taps >= 1 && taps <= MAX_TAPS && ldp >= C && state_ld >= C + (taps > 1 ? (long long)taps * C : 0), "rglru_conv: bad sizes");
+    if (n_tokens == 0) return 0;
+    const bool vec = C % 4 == 0 && ldp % 4 == 0 && (((uintptr_t)proj | (uintptr_t)conv_w | (uintptr_t)conv_b | (uintptr_t)u) & 15) == 0;
+    if (vec && n_tokens >= 64 && taps >= 2 && taps <= 4) {
+        const size_t items = (size_t)((n_tokens + 3) / 4) * (C / 4);
+        const int blocks = (int)((items + 255) / 256 < 148 * 16 ? (items + 255) / 256 : 148 * 16);
+#define RGLRU_RUNS(TT) lgml_launch(rglru_conv_runs_kernel<TT>, blocks, 256, 0, stream, proj, ldp, conv_w, conv_b, state, state_ld, seq_of_token, seq_start, slots, positions, u, n_tokens, C)
+        if (taps == 2) RGLRU_RUNS(2);
+        else if (taps == 3) RGLRU_RUNS(3);
+        else RGLRU_RUNS(4);
+#undef RGLRU_RUNS
+        return lgml_launch_status("rglru_conv");
+    }
+    const size_t items = (size_t)n_tokens * C;
+    const int blocks = (int)((items + 255) / 256 < 148 * 16 ? (items + 255) / 256 : 148 * 16);
+    lgml_launch(rglru_conv_kernel, blocks, 256, 0, stream, proj, ldp, conv_w, conv_b, state, state_ld, seq_of_token, seq_start, slots, positions, u, n_tokens, C,
+                taps);
+    return lgml_launch_status("rglru_conv");
+}
+
+// ab float32 [2, n, C].  form 0: choose; 1: products of 8 rows; 2: tensor cores (bfloat16, parts that are multiples of 8)
+LGML_API int lgml_rglru_gates(const float *u, const void *ra, const float *ra_b, const void *ri, const float *ri_b, const float *sp8, float *ab, int dtype,
+                              int n_tokens, int C, int P, int form, cudaStream_t stream) {
+    RGLRU_SIZES("rglru_gates");
+    LGML_REQUIRE(form >= 0 && form <= 2, "rglru_gates: unknown form %d", form);
+    if (n_tokens == 0) return 0;
+    const bool fits = dtype == LGML_BF16 && P % 8 == 0 && C % 4 == 0 &&
+                      (((uintptr_t)u | (uintptr_t)ra | (uintptr_t)ri | (uintptr_t)ra_b | (uintptr_t)ri_b | (uintptr_t)sp8 | (uintptr_t)ab) & 15) == 0;
+    LGML_REQUIRE(form != 2 || fits, "rglru_gates: the tensor-core form takes bfloat16 matrices and parts that are multiples of 8");
+    if (fits && (form == 2 || (form == 0 && n_tokens >= 32))) {
+        const size_t smem = sizeof(__nv_bfloat16) * (3 * GT + 128) * GLD;
+        cudaError_t e = cudaFuncSetAttribute(rglru_gates_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) LGML_FAIL("rglru_gates: cannot have %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
+        dim3 grid((n_tokens + GT - 1) / GT, (P + 63) / 64, C / P);
+        lgml_launch(rglru_gates_mma_kernel, grid, 128, smem, stream, u, (const __nv_bfloat16 *)ra, ra_b, (const __nv_bfloat16 *)ri, ri_b, sp8, ab, n_tokens, C, P);
+        return lgml_launch_status("rglru_gates");
+    }
+    const size_t smem = sizeof(float) * NT * (size_t)((P + 3) & ~3);
+    LGML_REQUIRE(smem <= 48 * 1024, "rglru_gates: parts of %d channels are too wide", P);
+    dim3 grid((n_tokens + NT - 1) / NT, C / P, (P + CH - 1) / CH);
+    if (dtype == LGML_F32)
+        lgml_launch(rglru_gates_rows_kernel<float>, grid, 256, smem, stream, u, (const float *)ra, ra_b, (const float *)ri, ri_b, sp8, ab, n_tokens, C, P,
+                    few_rows_lanes<float>(P), few_rows_vec<float>(ra, P) && few_rows_vec<float>(ri, P) ? 1 : 0);
+    else
+        lgml_launch(rglru_gates_rows_kernel<__nv_bfloat16>, grid, 256, smem, stream, u, (const __nv_bfloat16 *)ra, ra_b, (const __nv_bfloat16 *)ri, ri_b, sp8, ab,
+                    n_tokens, C, P, few_rows_lanes<__nv_bfloat16>(P), few_rows_vec<__nv_bfloat16>(ra, P) && few_rows_vec<__nv_bfloat16>(ri, P) ? 1 : 0);
+    return lgml_launch_status("rglru_gates");
+}
+
+LGML_API int lgml_rglru_scan(const float *ab, const float *proj, int ldp, float *state, long long state_ld, const int *seq_start, const int *slots, void *out,
+                             int dtype, int n_tokens, int n_seqs, int C, cudaStream_t stream) {
+    LGML_REQUIRE(n_tokens >= 0 && n_seqs >= 0 && n_seqs <= 65535 && C > 0 && ldp >= 2 * C && state_ld >= C, "rglru_scan: bad sizes");
+    if (n_tokens == 0 || n_seqs == 0) return 0;
+    dim3 grid((C + 127) / 128, n_seqs);
+    if (dtype == LGML_F32)
+        lgml_launch(rglru_scan_kernel<float>, grid, 128, 0, stream, ab, proj, ldp, state, state_ld, seq_start, slots, (float *)out, n_tokens, C);
+    else if (dtype == LGML_BF16)
+        lgml_launch(rglru_scan_kernel<__nv_bfloat16>, grid, 128, 0, stream, ab, proj, ldp, state, state_ld, seq_start, slots, (__nv_bfloat16 *)out, n_tokens, C);
+    else
+        LGML_FAIL("rglru_scan: unknown type %d", dtype);
+    return lgml_launch_status("rglru_scan");
+}
+
+// chunks int32 [n_chunks, 2]: token rows [first, past the last), a request's chunks in a row; chunk_start int32 [n_seqs + 1]; scratch float32 [2, n_chunks, C]
+LGML_API int lgml_rglru_chunks(const float *ab, const float *proj, int ldp, float *state, long long state_ld, const int *chunks, const int *chunk_start,
+                               int n_chunks, const int *slots, float *scratch, void *out, int dtype, int n_tokens, int n_seqs, int C, cudaStream_t stream) {
+    LGML_REQUIRE(n_tokens >= 0 && n_chunks >= 0 && n_chunks <= 65535 && n_seqs >= 0 && n_seqs <= 65535 && C > 0 && ldp >= 2 * C && state_ld >= C, "rglru_chunks: bad sizes");
+    if (n_chunks == 0) return 0;
+    float *A = scratch, *B = scratch + (size_t)n_chunks * C;
+    dim3 grid((C + 127) / 128, n_chunks), chain((C + 127) / 128, n_seqs);
+    lgml_launch(rglru_chunk_ends_kernel, grid, 128, 0, stream, ab, chunks, A, B, n_tokens, C);
+    lgml_launch(rglru_chain_kernel, chain, 128, 0, stream, (const float *)A, B, chunk_start, state, state_ld, slots, C);
+    if (dtype == LGML_F32)
+        lgml_launch(rglru_chunk_scan_kernel<float>, grid, 128, 0, stream, ab, proj, ldp, chunks, (const float *)B, (float *)out, n_tokens, C);
+    else if (dtype == LGML_BF16)
+        lgml_launch(rglru_chunk_scan_kernel<__nv_bfloat16>, grid, 128, 0, stream, ab, proj, ldp, chunks, (const float *)B, (__nv_bfloat16 *)out, n_tokens, C);
+    else
+        LGML_FAIL("rglru_chunks: unknown type %d", dtype);
+    return lgml_launch_status("rglru_chunks");
+}

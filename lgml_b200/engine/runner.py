@@ -89,8 +89,8 @@ class ModelRunner:
         """Random weights without a folder: drawn on the device, or on the host; either way
         the values of ``write_random_model(folder, cfg, seed)``, bit for bit (one generator)."""
         from .. import ops
-        from ..weights.loader import target_dtype
-        from ..weights.random_init import tensor_key
+        from ..weights.loader import INT_TABLE, target_dtype
+        from ..weights.random_init import random_table, tensor_key
 
         rt = Runtime(device, dtype)
         model = build_model(cfg)
@@ -98,6 +98,9 @@ class ModelRunner:
         if on_device:
             tensors = {}
             for s in specs:
+                if s.kind == INT_TABLE:
+                    tensors[s.name] = random_table(s, seed).to(rt.device)
+                    continue
                 t = torch.empty(s.shape, dtype=target_dtype(s.kind, dtype), device=rt.device)
                 ops.fill_normal(t, s.init[0], s.init[1] * std, tensor_key(seed, s.name))
                 tensors[s.name] = t

@@ -145,6 +145,11 @@ class Runtime:
                                   window, self.status, slopes=slopes, sinks=sinks, gate=gate, keep_first=keep_first, softcap=softcap)
 
     # ---- mixture of experts ------------------------------------------------------------
+    def experts_in_tiles(self, n_rows: int, w_gu) -> bool:
+        """Whether the experts of a step with that many (token, expert) rows run as grouped products over tiles of one
+        expert's rows (their matrices ``w_gu`` [experts, 2 F, E], bfloat16, widths that are multiples of 8)."""
+        return n_rows >= MOE_GROUPED_ROWS and self.dtype == torch.bfloat16 and w_gu.shape[1] % 16 == 0 and w_gu.shape[2] % 8 == 0
+
     def moe_experts(self, h, ids, wts, w_gu, w_down, gated: bool = True, also=None, also_w=None) -> torch.Tensor:
         """The chosen experts' weighted outputs, float32 [tokens, width]: a block per (token, expert) for few
         tokens and on the 32-bit path; for many, tiles of one expert's rows as grouped products on tcgen05

@@ -7,6 +7,7 @@ from . import gotulorn  # noqa: F401  (registers Gotulorn)
 from . import konovik  # noqa: F401  (registers Konovik)
 from . import dizepel  # noqa: F401  (registers Dizepel)
 from . import tedisun  # noqa: F401  (registers Tedisun)
+from . import nelosun  # noqa: F401  (registers Nelosun)
 
 
 def build_model(config):

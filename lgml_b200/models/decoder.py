@@ -20,7 +20,7 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from .. import ops
-from ..parts.norm import PendingDelta, UnitMix
+from ..parts.norm import PendingDelta, ScaledTerms, UnitMix
 from ..parts.streams import PendingStreams
 from ..weights import VECTOR, TensorSpec
 
@@ -31,6 +31,7 @@ class LayerCall:
     cache: Optional[int] = None   # index of the call that owns the cache used; None = this call
     add_input: bool = False       # the residual stream as it was before the first call is added to it before this call
     add_row: Optional[int] = None  # this row of the model's table of pass vectors is added to every token's x before this call
+    begins_pass: Optional[int] = None  # this pass of a loop begins here: the model's ``pass_input`` makes x anew before this call
 
 
 class DecoderModel:
@@ -38,7 +39,8 @@ class DecoderModel:
                  block_prefix: str = "model.layers.{}", final_norm_prefix: str = "model.norm",
                  embed_scale: Optional[float] = None, logit_scale: Optional[float] = None, logit_softcap: Optional[float] = None,
                  ignored_tensors: Sequence[str] = (), embed_norm=None, embed_norm_prefix: str = "model.embed_norm",
-                 delta_dtype: Optional[torch.dtype] = None, pass_rows: Optional[str] = None, streams: int = 0):
+                 delta_dtype: Optional[torch.dtype] = None, pass_rows: Optional[str] = None, streams: int = 0,
+                 pass_input=None, step_parts: Sequence = ()):
         self.config = config
         # the residual in this many streams (``parts/streams.py``; the blocks and the final norm are made for them); 0: one x
         self.streams = int(streams)
@@ -46,6 +48,10 @@ class DecoderModel:
         self.delta_dtype = delta_dtype
         # the name of a tensor [rows, width] whose rows schedule entries add to x (``LayerCall.add_row``)
         self.pass_rows_name, self.pass_rows = pass_rows, None
+        # what makes x anew at the start of a pass (``LayerCall.begins_pass``; ``parts/token_mix.py``: ``PassInput``)
+        self.pass_input = pass_input
+        # things with ``begin(rt, batch)`` that settle something for the whole step before its first layer
+        self.step_parts = tuple(step_parts)
         self.embedding = embedding
         self.blocks = list(blocks)
         self.final_norm = final_norm
@@ -71,11 +77,15 @@ class DecoderModel:
                     raise ValueError(f"schedule entry {ci} reads the cache of entry {call.cache}, which has none of its own")
             if call.add_row is not None and pass_rows is None:
                 raise ValueError(f"schedule entry {ci} adds a pass vector, but the model names no table of them")
+            if call.begins_pass is not None and ci == 0 and embed_norm is not None:
+                raise ValueError("a pass that starts the model reads the embedding's rows, not a norm of them")
+            if call.begins_pass is not None and (pass_input is None or self.streams):
+                raise ValueError(f"schedule entry {ci} begins a pass, but the model has no part that makes x anew")
             if self.streams and (call.add_row is not None or call.add_input):
                 raise ValueError(f"schedule entry {ci} adds a row to x, which is {self.streams} streams")
         self.n_pass_rows = 1 + max((call.add_row for call in self.schedule if call.add_row is not None), default=-1)
         self.vocab_size = head.vocab
-        parts = [embedding, final_norm, head] + self.blocks + ([embed_norm] if embed_norm is not None else [])
+        parts = [embedding, final_norm, head] + self.blocks + [p for p in (embed_norm, pass_input) if p is not None]
         self.graph_safe = all(getattr(p, "graph_safe", False) for p in parts)
         self.max_position = getattr(config, "max_position_embeddings", None)
 
@@ -86,6 +96,8 @@ class DecoderModel:
             specs += self.embed_norm.tensor_specs(self.embed_norm_prefix)
         for i, b in enumerate(self.blocks):
             specs += b.tensor_specs(self.block_prefix.format(i))
+        if self.pass_input is not None:
+            specs += self.pass_input.tensor_specs("")
         specs += self.final_norm.tensor_specs(self.final_norm_prefix)
         specs += self.head.tensor_specs("")
         if self.pass_rows_name is not None and self.n_pass_rows:
@@ -101,6 +113,8 @@ class DecoderModel:
             self.embed_norm.bind(self.embed_norm_prefix, tensors, rt)
         for i, b in enumerate(self.blocks):
             b.bind(self.block_prefix.format(i), tensors, rt)
+        if self.pass_input is not None:
+            self.pass_input.bind("", tensors, rt)
         self.final_norm.bind(self.final_norm_prefix, tensors, rt)
         self.head.bind("", tensors, rt)
         if self.pass_rows_name is not None and self.n_pass_rows:
@@ -130,7 +144,9 @@ class DecoderModel:
     @staticmethod
     def _fold(x, pending) -> None:
         """x += what is pending, now, by a kernel of its own."""
-        if isinstance(pending, PendingDelta):
+        if isinstance(pending, ScaledTerms):
+            ops.scaled_norm(x, pending.terms, keep=pending.keep)
+        elif isinstance(pending, PendingDelta):
             d = pending.delta
             if isinstance(d, UnitMix):
                 ops.sandwich_norm(x, None, pending.eps, None, delta=(d.a, d.b), units=(d.u_a, d.u_b), w_post=pending.w_post, row_add=pending.row_add)
@@ -143,8 +159,15 @@ class DecoderModel:
     # ---- the forward pass of one step --------------------------------------------------
     def forward(self, rt, batch) -> torch.Tensor:
         """float32 logits [len(batch.logit_rows), vocab] for the tokens of ``batch``."""
-        x = self.embedding.forward(rt, batch.token_ids)
-        if self.embed_scale is not None and not (self.streams and self.embed_norm is None):
+        for part in self.step_parts:
+            part.begin(rt, batch)
+        # a pass that starts the model reads the embedding itself
+        starts = self.schedule[0].begins_pass is not None
+        if starts:
+            x = torch.empty((batch.token_ids.numel(), self.embedding.width), dtype=torch.float32, device=batch.token_ids.device)
+        else:
+            x = self.embedding.forward(rt, batch.token_ids)
+        if self.embed_scale is not None and not starts and not (self.streams and self.embed_norm is None):
             ops.scale_cap(x, self.embed_scale)
         if self.embed_norm is not None:
             x = self.embed_norm.forward(rt, x, torch.float32)
@@ -160,6 +183,8 @@ class DecoderModel:
                     self._fold(x, pending)
                     pending = None
                 ops.residual_fold(x, x_in)
+            if call.begins_pass is not None:
+                pending = self.pass_input.forward(rt, x, pending, batch, call.begins_pass, starts_model=ci == 0)
             if call.add_row is not None:
                 pending = self._with_row(x, pending, self.pass_rows[call.add_row], self.blocks[call.block])
             owner = ci if call.cache is None else call.cache

@@ -171,17 +171,19 @@ def _check(lib_name: str, rc: int, what: str) -> None:
 # ----------------------------------------------------------------------------------------
 
 def embed_rows(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, status: torch.Tensor) -> torch.Tensor:
-    """out[t] = table[ids[t]] as float32."""
+    """out[t] = table[ids[t]] as float32 (or in the table's own type)."""
     _need(table, "embedding table", ndim=2)
     _need(ids, "token ids", torch.int32, 1)
-    _need(out, "embedding output", torch.float32, 2)
+    _need(out, "embedding output", ndim=2)
+    if out.dtype not in (torch.float32, table.dtype):
+        raise KernelError(f"embed_rows: rows of {table.dtype} come out as float32 or as they are, not as {out.dtype}")
     if not table.is_contiguous() or not out.is_contiguous():
         raise KernelError("embedding table and output must be contiguous")
     n, width = out.shape
     if ids.numel() != n or table.shape[1] != width:
         raise KernelError(f"embed_rows: shapes disagree: table {tuple(table.shape)}, ids {tuple(ids.shape)}, out {tuple(out.shape)}")
-    fn = _fn("elementwise", "lgml_embed_rows", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p])
-    _check("elementwise", fn(_ptr(table), dtype_code(table.dtype), _ptr(ids), _ptr(out), n, width, table.shape[0], _ptr(status), _stream()), "embed_rows")
+    fn = _fn("elementwise", "lgml_embed_rows_as", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p], label="embed_rows")
+    _check("elementwise", fn(_ptr(table), dtype_code(table.dtype), _ptr(ids), _ptr(out), dtype_code(out.dtype), n, width, table.shape[0], _ptr(status), _stream()), "embed_rows")
     return out
 
 
@@ -534,6 +536,20 @@ def _value_pages(v_pages: torch.Tensor, k_pages: torch.Tensor, who: str):
     return hv, dv, ldv
 
 
+def _gate_stride(gate: Optional[torch.Tensor], n: int, n_heads: int, dv: int, who: str) -> int:
+    """The row stride of an output gate's logits as the kernels want it: positive for a logit per value
+    ([tokens, H Dv]), negative for one per head ([tokens, H])."""
+    if gate is None:
+        return 0
+    _need(gate, "gate", torch.float32, 2)
+    ldg = _rows_contiguous(gate, "gate")
+    if tuple(gate.shape) == (n, n_heads * dv):
+        return ldg
+    if tuple(gate.shape) == (n, n_heads):
+        return -ldg
+    raise KernelError(f"{who}: gate {tuple(gate.shape)} is neither [{n}, {n_heads * dv}] nor [{n}, {n_heads}]")
+
+
 def sink_attention(q: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Tensor, block_table: torch.Tensor,
                    k_pages: torch.Tensor, v_pages: torch.Tensor, out: torch.Tensor, n_heads: int, scale: float, window: int,
                    status: torch.Tensor, slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
@@ -543,7 +559,7 @@ def sink_attention(q: torch.Tensor, positions: torch.Tensor, seq_of_token: torch
     w_j = exp(s_j) / (exp(sink_h) + sum exp(s)), s_j = cap((q . k_j) scale) - slope_h (p - j), cap(s) = softcap tanh(s / softcap)
     (``softcap`` 0: s itself);
     then times sigmoid(gate[t, h]) element by element when ``gate`` (float32, pre-sigmoid; may be a
-    column slice) is given.  Keys have head size D, values Dv.  The value pages may have fewer heads than the
+    column slice) is given, or, with a gate of one column per head, head by head.  Keys have head size D, values Dv.  The value pages may have fewer heads than the
     key pages (key heads g Hkv / Hv ... share value head g) and may be a column range of wider cells.
     ``out`` has the queries' type or is float32."""
     _need(q, "queries", ndim=2)
@@ -566,12 +582,7 @@ def sink_attention(q: torch.Tensor, positions: torch.Tensor, seq_of_token: torch
             _need(t, what, torch.float32, 1)
             if t.numel() != n_heads or not t.is_contiguous():
                 raise KernelError(f"sink_attention: one of the {what} per head")
-    ldg = 0
-    if gate is not None:
-        _need(gate, "gate", torch.float32, 2)
-        ldg = _rows_contiguous(gate, "gate")
-        if tuple(gate.shape) != (n, n_heads * dv):
-            raise KernelError(f"sink_attention: gate {tuple(gate.shape)} is not [{n}, {n_heads * dv}]")
+    ldg = _gate_stride(gate, n, n_heads, dv, "sink_attention")
     fn = _fn("attention_sink", "lgml_sink_attention", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
                                                        c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                                        c_int, c_int, c_float, c_float, c_int, c_int, c_void_p, c_void_p])
@@ -612,12 +623,7 @@ def sink_attention_mma(q: torch.Tensor, positions: torch.Tensor, tiles: torch.Te
             _need(t, what, torch.float32, 1)
             if t.numel() != n_heads or not t.is_contiguous():
                 raise KernelError(f"sink_attention_mma: one of the {what} per head")
-    ldg = 0
-    if gate is not None:
-        _need(gate, "gate", torch.float32, 2)
-        ldg = _rows_contiguous(gate, "gate")
-        if tuple(gate.shape) != (n, n_heads * dv):
-            raise KernelError(f"sink_attention_mma: gate {tuple(gate.shape)} is not [{n}, {n_heads * dv}]")
+    ldg = _gate_stride(gate, n, n_heads, dv, "sink_attention_mma")
     fn = _fn("attention_sink", "lgml_sink_attention_mma", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int,
                                                            c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                            c_int, c_int, c_float, c_float, c_int, c_int, c_void_p, c_void_p])
@@ -633,7 +639,8 @@ def sink_twin_supports(q: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor
     size, 64 or 128, and q, out and the gate readable in 16-byte pieces."""
     return (PREFILL_ATTENTION == "tcgen05" and k_pages.shape[2] == 64 and k_pages.shape[3] in (64, 128) and v_pages.shape[3] == k_pages.shape[3]
             and prefill_tc_supports(q, out)
-            and (gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.stride(0) % 4 == 0 and gate.data_ptr() % 16 == 0)))
+            and (gate is None or gate.shape[1] * k_pages.shape[3] == out.shape[1]        # a gate per head is read number by number
+                 or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.stride(0) % 4 == 0 and gate.data_ptr() % 16 == 0)))
 
 
 def sink_attention_twin(q: torch.Tensor, positions: torch.Tensor, tiles: torch.Tensor, block_table: torch.Tensor, k_pages: torch.Tensor,
@@ -664,12 +671,7 @@ def sink_attention_twin(q: torch.Tensor, positions: torch.Tensor, tiles: torch.T
             _need(t, what, torch.float32, 1)
             if t.numel() != n_heads or not t.is_contiguous():
                 raise KernelError(f"sink_attention_twin: one of the {what} per head")
-    ldg = 0
-    if gate is not None:
-        _need(gate, "gate", torch.float32, 2)
-        ldg = _rows_contiguous(gate, "gate")
-        if tuple(gate.shape) != (n, n_heads * d):
-            raise KernelError(f"sink_attention_twin: gate {tuple(gate.shape)} is not [{n}, {n_heads * d}]")
+    ldg = _gate_stride(gate, n, n_heads, d, "sink_attention_twin")
     fn = _fn("attention_prefill_twin", "lgml_sink_attention_twin_keep", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                                                     c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
                                                                     c_int, c_float, c_float, c_int, c_int, c_void_p, c_void_p], label="sink_attention_twin")
@@ -716,12 +718,7 @@ def sink_decode(q: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Te
             _need(t, what, torch.float32, 1)
             if t.numel() != n_heads or not t.is_contiguous():
                 raise KernelError(f"sink_decode: one of the {what} per head")
-    ldg = 0
-    if gate is not None:
-        _need(gate, "gate", torch.float32, 2)
-        ldg = _rows_contiguous(gate, "gate")
-        if tuple(gate.shape) != (n, n_heads * dv):
-            raise KernelError(f"sink_decode: gate {tuple(gate.shape)} is not [{n}, {n_heads * dv}]")
+    ldg = _gate_stride(gate, n, n_heads, dv, "sink_decode")
     scratch = torch.empty(n * n_heads * n_splits * (dv + 2), dtype=torch.float32, device=q.device) if n_splits > 1 else None
     fn = _fn("attention_sink", "lgml_sink_decode", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p,
                                                     c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
@@ -757,7 +754,8 @@ def diff_combine(maps: torch.Tensor, out: torch.Tensor, n_heads: int, n_key_head
 
 def latent_prepare(q_proj: torch.Tensor, down: torch.Tensor, norm_w: torch.Tensor, eps: float, inv_freq: torch.Tensor, n_rot: int,
                    positions: torch.Tensor, seq_of_token: torch.Tensor, block_table: torch.Tensor, cells: torch.Tensor, n_heads: int,
-                   head_dim: int, rot_dim: int, rank: int, status: torch.Tensor, write_kv: bool = True, rot_mag: float = 1.0):
+                   head_dim: int, rot_dim: int, rank: int, status: torch.Tensor, write_kv: bool = True, rot_mag: float = 1.0,
+                   halves: bool = False):
     """Latent attention between its projections and attention.  ``q_proj`` float32 [tokens, H (D + Dr)]
     (per head D plain, then Dr rotated entries), ``down`` float32 [tokens, R + Dr].  The first R columns
     of ``down``, over their root mean square, times ``norm_w``, are the latent c; the last Dr are a key
@@ -766,7 +764,7 @@ def latent_prepare(q_proj: torch.Tensor, down: torch.Tensor, norm_w: torch.Tenso
     cell of ``cells`` [pages, 1, page, R + Dr].  Returns (q_plain [tokens, H D], q_full [tokens,
     H (R + Dr)]) in the cells' type; of q_full only the rotated Dr entries behind each head's first R
     are written (``head_linear`` fills those).  ``rot_mag`` multiplies every cosine and sine (a frequency
-    scaling that lengthens the rotated vectors)."""
+    scaling that lengthens the rotated vectors); ``halves``: the pairs are (i, i + n_rot / 2)."""
     _need(q_proj, "query projection", torch.float32, 2)
     _need(down, "down projection", torch.float32, 2)
     _need(cells, "latent cells", ndim=4)
@@ -790,12 +788,69 @@ def latent_prepare(q_proj: torch.Tensor, down: torch.Tensor, norm_w: torch.Tenso
     q_full = torch.empty((n, n_heads * (rank + rot_dim)), dtype=cells.dtype, device=cells.device)
     fn = _fn("attention_heads", "lgml_latent_prepare", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int, c_void_p,
                                                         c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int,
-                                                        c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
+                                                        c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p])
     _check("attention_heads", fn(_ptr(q_proj), ldq, _ptr(down), ldd, _ptr(norm_w), float(eps), _ptr(inv_freq[0]), _ptr(inv_freq[1]), int(n_rot),
                                  _ptr(positions), _ptr(seq_of_token), _ptr(block_table), block_table.shape[1], _ptr(cells), dtype_code(cells.dtype),
                                  n_pages, page, _ptr(q_plain), q_plain.stride(0), _ptr(q_full), q_full.stride(0), n, n_heads, head_dim, rot_dim,
-                                 rank, 1 if write_kv else 0, float(rot_mag), _ptr(status), _stream()), "latent_prepare")
+                                 rank, 1 if write_kv else 0, float(rot_mag), 1 if halves else 0, _ptr(status), _stream()), "latent_prepare")
     return q_plain, q_full
+
+
+def latent_down(down: torch.Tensor, q_norm_w: torch.Tensor, norm_w: torch.Tensor, eps: float, inv_freq: torch.Tensor, n_rot: int, positions: torch.Tensor,
+                seq_of_token: torch.Tensor, block_table: torch.Tensor, cells: torch.Tensor, q_rank: int, rank: int, rot_dim: int, status: torch.Tensor,
+                rot_mag: float = 1.0, halves: bool = False):
+    """Latent attention whose queries have a latent of their own, behind the down-projection.  ``down`` float32 [tokens,
+    Rq | R | Dr]: the first Rq over their root mean square, times ``q_norm_w``, are returned in the cells' type ([tokens, Rq]);
+    the next R, normed with ``norm_w``, and the last Dr, rotated as in ``latent_prepare``, go into the token's cell.  Second
+    result: the cosines and sines of the step's positions, float32 [tokens, n_rot], for ``latent_query``."""
+    _need(down, "down projection", torch.float32, 2)
+    _need(cells, "latent cells", ndim=4)
+    _need(q_norm_w, "query latent's norm weight", torch.float32, 1)
+    _need(norm_w, "latent norm weight", torch.float32, 1)
+    _need(inv_freq, "frequencies", torch.float32, 2)
+    n = down.shape[0]
+    n_pages, one, page, width = cells.shape
+    if one != 1 or width != rank + rot_dim or not cells.is_contiguous():
+        raise KernelError(f"latent_down: cells {tuple(cells.shape)} are not [pages, 1, page, {rank + rot_dim}]")
+    if down.shape[1] != q_rank + rank + rot_dim or q_norm_w.numel() != q_rank or norm_w.numel() != rank:
+        raise KernelError(f"latent_down: down {tuple(down.shape)} does not hold {q_rank} + {rank} + {rot_dim} columns")
+    if n_rot % 2 or n_rot > rot_dim or tuple(inv_freq.shape) != (2, max(n_rot // 2, 1)) or not inv_freq.is_contiguous():
+        raise KernelError(f"latent_down: {n_rot} rotated entries of {rot_dim}, frequencies {tuple(inv_freq.shape)}")
+    _need(positions, "positions", torch.int32, 1)
+    _need(seq_of_token, "request index of tokens", torch.int32, 1)
+    _need(block_table, "block table", torch.int32, 2)
+    if positions.numel() != n or seq_of_token.numel() != n or not block_table.is_contiguous():
+        raise KernelError("latent_down: one position and one request index per token, and a contiguous block table")
+    ldd = _rows_contiguous(down, "down projection")
+    cq = torch.empty((n, q_rank), dtype=cells.dtype, device=cells.device)
+    cos_sin = torch.empty((n, max(n_rot, 1)), dtype=torch.float32, device=cells.device)
+    fn = _fn("attention_heads", "lgml_latent_down", [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
+                                                     c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
+                                                     c_void_p])
+    _check("attention_heads", fn(_ptr(down), ldd, _ptr(q_norm_w), _ptr(norm_w), float(eps), _ptr(inv_freq[0]), _ptr(inv_freq[1]), int(n_rot), _ptr(positions),
+                                 _ptr(seq_of_token), _ptr(block_table), block_table.shape[1], _ptr(cells), dtype_code(cells.dtype), n_pages, page, _ptr(cq),
+                                 _ptr(cos_sin), n, int(q_rank), int(rank), int(rot_dim), float(rot_mag), 1 if halves else 0, _ptr(status), _stream()), "latent_down")
+    return cq, cos_sin
+
+
+def latent_query(q: torch.Tensor, w_uk_t: torch.Tensor, cos_sin: torch.Tensor, n_rot: int, rot_dim: int, halves: bool = False) -> torch.Tensor:
+    """The queries of latent attention on the latent's side: ``q`` float32 [tokens, H (D + Dr)] (per head D plain, Dr rotated
+    entries), ``w_uk_t`` [H, R, D]; returns [tokens, H (R + Dr)] in the matrix's type, per head W q_plain and the rotated part
+    (``cos_sin`` as ``latent_down`` gives it)."""
+    _need(q, "queries", torch.float32, 2)
+    _need(w_uk_t, "up-projection", ndim=3)
+    _need(cos_sin, "cosines and sines", torch.float32, 2)
+    n = q.shape[0]
+    H, R, D = w_uk_t.shape
+    ldq = _rows_contiguous(q, "queries")
+    if q.shape[1] != H * (D + rot_dim) or not w_uk_t.is_contiguous() or tuple(cos_sin.shape) != (n, max(n_rot, 1)) or not cos_sin.is_contiguous():
+        raise KernelError(f"latent_query: queries {tuple(q.shape)} / matrices {tuple(w_uk_t.shape)} / cosines {tuple(cos_sin.shape)} do not fit")
+    out = torch.empty((n, H * (R + rot_dim)), dtype=w_uk_t.dtype, device=q.device)
+    fn = _fn("attention_heads", "lgml_latent_query", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                                                      c_int, c_void_p])
+    _check("attention_heads", fn(_ptr(q), ldq, _ptr(w_uk_t), _ptr(cos_sin), int(n_rot), _ptr(out), out.stride(0), dtype_code(out.dtype), n, H, D, int(rot_dim), R,
+                                 1 if halves else 0, _stream()), "latent_query")
+    return out
 
 
 def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_head_stride: int, out_head_stride: int,
@@ -906,34 +961,41 @@ def _moe_shapes(h, ids, wts, w_gu, w_down, who: str, gated: bool = True):
         if not t.is_contiguous():
             raise KernelError(f"{who}: the {what} matrices must be contiguous")
     _need(ids, "chosen experts", torch.int32, 2)
-    _need(wts, "experts' weights", torch.float32, 2)
+    if wts is not None:
+        _need(wts, "experts' weights", torch.float32, 2)
     n, E = h.shape
     X, F2, _ = w_gu.shape
     F, top = (F2 // 2 if gated else F2), ids.shape[1]
     if tuple(w_gu.shape) != (X, 2 * F if gated else F, E) or tuple(w_down.shape) != (X, E, F) or tuple(ids.shape) != (n, top) \
-            or tuple(wts.shape) != (n, top) or not ids.is_contiguous() or not wts.is_contiguous():
+            or not ids.is_contiguous() or (wts is not None and (tuple(wts.shape) != (n, top) or not wts.is_contiguous())):
         raise KernelError(f"{who}: shapes disagree: h {tuple(h.shape)}, gate|up {tuple(w_gu.shape)}, down {tuple(w_down.shape)}, ids {tuple(ids.shape)}")
     return n, E, F, X, top
 
 
-def moe_experts_rows(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, gated: bool = True,
-                     also: Optional[torch.Tensor] = None, also_w: Optional[torch.Tensor] = None) -> torch.Tensor:
+def moe_experts_rows(h: torch.Tensor, ids: torch.Tensor, wts: Optional[torch.Tensor], w_gu: torch.Tensor, w_down: torch.Tensor, gated: bool = True,
+                     also: Optional[torch.Tensor] = None, also_w: Optional[torch.Tensor] = None, clamp=None) -> torch.Tensor:
     """out[t] = sum_s wts[t, s] W_down[e] (silu(W_gate[e] h_t) * (W_up[e] h_t)), e = ids[t, s]: float32
     [tokens, E].  The experts' matrices stacked: ``w_gu`` [X, 2 F, E] with the gate row of a feature followed
     by its up row, ``w_down`` [X, E, F].  A block per (token, chosen expert): the form for few tokens and for
     the 32-bit path.  ``gated`` False: experts without a gate, ``w_gu`` [X, F, E] and the activation relu squared.
     ``also`` / ``also_w``: out += also_w[t] * also[t] (a shared expert's output and the token's gate on it; the token's own row
-    and the weight of its identity experts).  A slot whose id is -1 holds no expert."""
+    and the weight of its identity experts).  A slot whose id is -1 holds no expert.  ``clamp`` = (alpha, limit): gated experts with
+    the clamped activation (``glu_clamped``) in place of silu(gate) * up.  ``wts`` None: 1 / top each."""
     _need(h, "experts' input", ndim=2)
     ldh = _rows_contiguous(h, "experts' input")
     n, E, F, X, top = _moe_shapes(h, ids, wts, w_gu, w_down, "moe_experts_rows", gated)
     also_own, lda = _also(also, also_w, n, E, h.dtype, "moe_experts_rows")
     act = torch.empty((n * top, F), dtype=h.dtype, device=h.device)
     out = torch.empty((n, E), dtype=torch.float32, device=h.device)
-    fn = _fn("moe", "lgml_moe_experts_rows_form", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                                   c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p])
+    if clamp is not None and not gated:
+        raise KernelError("moe_experts_rows: the clamped activation is a gated one")
+    alpha, limit = clamp if clamp is not None else (0.0, 0.0)
+    fn = _fn("moe", "lgml_moe_experts_rows_act", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                                  c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_int, c_void_p, c_void_p],
+             label="moe_experts_rows_form")
     _check("moe", fn(_ptr(h), dtype_code(h.dtype), ldh, _ptr(ids), _ptr(wts), _ptr(w_gu), _ptr(w_down), _ptr(act), _ptr(out), n, E, F, X,
-                     top, 0 if gated else 1, _ptr(also), also_own, lda, _ptr(also_w), _stream()), "moe_experts_rows")
+                     top, 2 if clamp is not None else (0 if gated else 1), float(alpha), float(limit), _ptr(also), also_own, lda, _ptr(also_w), _stream()),
+           "moe_experts_rows")
     return out
 
 
@@ -996,23 +1058,320 @@ def moe_experts_tcgen05(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w
     pos = torch.empty(n_rows, dtype=torch.int32, device=dev)
     tiles = torch.empty(3 * max_tiles + 1, dtype=torch.int32, device=dev)
     a_perm = torch.empty((max_tiles * MOE_TILE_ROWS, E), dtype=torch.bfloat16, device=dev)
-    act = torch.empty((max_tiles * MOE_TILE_ROWS, F), dtype=torch.bfloat16, device=dev)
-    y = torch.empty((max_tiles * MOE_TILE_ROWS, E), dtype=torch.float32, device=dev)
     out = torch.empty((n, E), dtype=torch.float32, device=dev)
     stream = _stream()
     fn = _fn("moe", "lgml_moe_group_rows", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
     _check("moe", fn(_ptr(ids), _ptr(rows), _ptr(tiles), max_tiles, n, X, top, stream), "moe_group_rows")
     fn = _fn("moe", "lgml_moe_gather_rows", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p])
     _check("moe", fn(_ptr(h), ldh, _ptr(rows), _ptr(tiles), max_tiles, _ptr(a_perm), _ptr(pos), E, top, stream), "moe_gather_rows")
-    fn = _fn("gemm_tcgen05", "lgml_gemm_tcgen05_grouped", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
-                                                           c_void_p, c_void_p])
-    _check("gemm_tcgen05", fn(_ptr(a_perm), _ptr(w_gu), _ptr(act), 0, max_tiles, 2 * F if gated else F, E, X, F, _ptr(tiles), 1 if gated else 2,
-                              _ptr(status), stream), "gemm_tcgen05_grouped")
-    _check("gemm_tcgen05", fn(_ptr(act), _ptr(w_down), _ptr(y), 1, max_tiles, E, F, X, E, _ptr(tiles), 0, _ptr(status), stream),
-           "gemm_tcgen05_grouped")
+    y = moe_tile_products(a_perm, tiles, w_gu, w_down, status, gated=gated)
     fn = _fn("moe", "lgml_moe_weighted_sum_form", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p,
                                                    c_void_p], label="moe_weighted_sum")
     _check("moe", fn(_ptr(y), _ptr(pos), _ptr(ids), _ptr(wts), _ptr(out), n, E, top, _ptr(also), also_bf16, lda, _ptr(also_w), stream), "moe_weighted_sum")
+    return out
+
+
+def moe_tile_products(a_perm: torch.Tensor, tiles: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, status: torch.Tensor, gated: bool = True,
+                      clamp=None) -> torch.Tensor:
+    """The experts' two products over tiles of 128 rows of one expert, bfloat16 on tcgen05: ``a_perm`` [max_tiles 128, E],
+    ``tiles`` int32 [3 max_tiles + 1] (per tile: expert, -, rows; the last word: how many tiles there are); float32 [max_tiles 128, E].
+    The first product's epilogue is silu(gate) * up, with ``clamp`` = (alpha, limit) the clamped activation, without a gate relu
+    squared.  Rows of a tile that hold no token come out as whatever they are."""
+    _need(a_perm, "experts' rows", torch.bfloat16, 2)
+    _need(tiles, "tiles", torch.int32, 1)
+    X, F2, E = w_gu.shape
+    F = F2 // 2 if gated else F2
+    max_tiles = a_perm.shape[0] // MOE_TILE_ROWS
+    if a_perm.shape != (max_tiles * MOE_TILE_ROWS, E) or not a_perm.is_contiguous() or tiles.numel() != 3 * max_tiles + 1 or not tiles.is_contiguous():
+        raise KernelError(f"moe_tile_products: rows {tuple(a_perm.shape)} / tiles {tuple(tiles.shape)} do not fit matrices {tuple(w_gu.shape)}")
+    if tuple(w_down.shape) != (X, E, F) or (clamp is not None and not gated):
+        raise KernelError(f"moe_tile_products: matrices {tuple(w_gu.shape)} and {tuple(w_down.shape)} do not go together")
+    alpha, limit = clamp if clamp is not None else (0.0, 0.0)
+    act = torch.empty((max_tiles * MOE_TILE_ROWS, F), dtype=torch.bfloat16, device=a_perm.device)
+    y = torch.empty((max_tiles * MOE_TILE_ROWS, E), dtype=torch.float32, device=a_perm.device)
+    stream = _stream()
+    fn = _fn("gemm_tcgen05", "lgml_gemm_tcgen05_grouped_act", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
+                                                               c_float, c_float, c_void_p, c_void_p], label="gemm_tcgen05_grouped")
+    _check("gemm_tcgen05", fn(_ptr(a_perm), _ptr(w_gu), _ptr(act), 0, max_tiles, F2, E, X, F, _ptr(tiles), (3 if clamp is not None else 1) if gated else 2,
+                              float(alpha), float(limit), _ptr(status), stream), "gemm_tcgen05_grouped")
+    _check("gemm_tcgen05", fn(_ptr(act), _ptr(w_down), _ptr(y), 1, max_tiles, E, F, X, E, _ptr(tiles), 0, 0.0, 0.0, _ptr(status), stream),
+           "gemm_tcgen05_grouped")
+    return y
+
+
+class TableRoute:
+    """Where the rows of one table's experts go in a step: ``ids`` int32 [tokens, top], ``places`` int32 [tokens, top] (the row
+    among the tiles), ``tiles`` int32 [3 max_tiles + 1]."""
+
+    def __init__(self, ids: torch.Tensor, places: torch.Tensor, tiles: torch.Tensor):
+        self.ids, self.places, self.tiles = ids, places, tiles
+
+    @property
+    def max_tiles(self) -> int:
+        return self.tiles.numel() // 3
+
+
+def table_route(token_ids: torch.Tensor, vocab: int, tables: torch.Tensor, desc: torch.Tensor, shapes):
+    """The experts of every token of a step by tables that the token's id indexes, for all tables in one launch.
+    ``tables`` int32: the tables [vocab, top] one behind the other; ``desc`` int32 [n_tables, 3] on the device: experts, top, first
+    entry; ``shapes``: the same experts and tops on the host.  Returns a ``TableRoute`` per table."""
+    _need(token_ids, "token ids", torch.int32, 1)
+    _need(tables, "expert tables", torch.int32, 1)
+    _need(desc, "tables' description", torch.int32, 2)
+    n = token_ids.numel()
+    if tuple(desc.shape) != (len(shapes), 3) or not desc.is_contiguous() or not tables.is_contiguous():
+        raise KernelError("table_route: one row (experts, top, first entry) per table")
+    if tables.numel() != sum(vocab * top for _, top in shapes):
+        raise KernelError(f"table_route: {tables.numel()} entries are not those of the tables")
+    sizes = [(n * top, _moe_tiles(n * top, X)) for X, top in shapes]
+    out = torch.empty(sum(2 * r + 3 * t + 1 for r, t in sizes), dtype=torch.int32, device=token_ids.device)
+    fn = _fn("moe", "lgml_table_route", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p])
+    _check("moe", fn(_ptr(token_ids), n, int(vocab), _ptr(tables), _ptr(desc), len(shapes), max(X for X, _ in shapes), _ptr(out), _stream()), "table_route")
+    routes, at = [], 0
+    for (r, t), (_, top) in zip(sizes, shapes):
+        routes.append(TableRoute(out[at:at + r].view(n, top), out[at + r:at + 2 * r].view(n, top), out[at + 2 * r:at + 2 * r + 3 * t + 1]))
+        at += 2 * r + 3 * t + 1
+    return routes
+
+
+# ----------------------------------------------------------------------------------------
+# results scaled channel by channel on their way into the residual stream
+# ----------------------------------------------------------------------------------------
+
+class ExpertRows:
+    """A token's experts' outputs, not yet added up: rows ``places[t, :]`` of ``data`` (float32 [rows, E]), each counting ``weight``."""
+
+    def __init__(self, data: torch.Tensor, places: torch.Tensor, weight: float):
+        self.data, self.places, self.weight = data, places, float(weight)
+
+
+class Term:
+    """Something to be added to the residual stream: ``value`` (a float32 tensor [tokens, E] with dense rows, ``Partials``, or
+    ``ExpertRows``) times ``mul`` times ``scale`` (float32 [E], channel by channel; None: ones).  ``stacked``: the value has two rows per
+    token, t and tokens + t, that are added (the two halves of a product over x in two bfloat16 pieces)."""
+
+    def __init__(self, value, scale: Optional[torch.Tensor] = None, mul: float = 1.0, stacked: bool = False):
+        self.value, self.scale, self.mul, self.stacked = value, scale, float(mul), bool(stacked)
+
+
+def scaled_norm(x: torch.Tensor, terms, eps: float = 0.0, weight: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, keep: bool = True,
+                rows: Optional[torch.Tensor] = None, tiles: Optional[torch.Tensor] = None, places: Optional[torch.Tensor] = None,
+                split: Optional[torch.Tensor] = None):
+    """x <- keep x + the terms (at most one ``Partials`` or stacked one and one other); with ``weight`` also out = x / rms(x) *
+    weight, its rows again at ``places`` [tokens, top] of ``tiles`` (bfloat16) when those are given; ``rows`` (int32) picks the rows
+    to norm (x is then not written).  ``split`` (bfloat16 [2 tokens, E]): x rounded, then what the rounding lost."""
+    _need(x, "residual stream", torch.float32, 2)
+    n, E = x.shape
+    if not x.is_contiguous():
+        raise KernelError("scaled_norm: the residual stream must be contiguous")
+    a = b = None
+    for term in terms:
+        plain = not isinstance(term.value, (Partials, ExpertRows)) and not term.stacked
+        if isinstance(term.value, ExpertRows) or (plain and a is not None):
+            if b is not None:
+                raise KernelError("scaled_norm: one tensor or experts' rows beside one product")
+            b = term
+        elif a is None:
+            a = term
+        elif b is None and not isinstance(a.value, Partials) and not a.stacked:
+            a, b = term, a
+        else:
+            raise KernelError("scaled_norm: at most one product in parts")
+    for term in (a, b):
+        if term is not None and term.scale is not None:
+            _need(term.scale, "channel scale", torch.float32, 1)
+            if term.scale.numel() != E or not term.scale.is_contiguous():
+                raise KernelError(f"scaled_norm: a channel scale of {term.scale.numel()} for rows of {E}")
+    ap, n_parts, a_stride, lda, second, bias = None, 1, 0, E, 0, None
+    if a is not None:
+        m = 2 * n if a.stacked else n
+        if isinstance(a.value, Partials):
+            ap, bias = a.value.data, a.value.bias
+            _need(ap, "product's parts", torch.float32, 3)
+            if tuple(ap.shape[1:]) != (m, E) or not ap.is_contiguous():
+                raise KernelError(f"scaled_norm: parts {tuple(ap.shape)} do not fit [{m}, {E}]")
+            n_parts, a_stride = ap.shape[0], m * E
+        else:
+            ap = a.value
+            _need(ap, "residual term", torch.float32, 2)
+            lda = _rows_contiguous(ap, "residual term")
+            if tuple(ap.shape) != (m, E):
+                raise KernelError(f"scaled_norm: a term of {tuple(ap.shape)} does not fit [{m}, {E}]")
+        second = n * lda if a.stacked else 0
+        if bias is not None:
+            _need(bias, "product's bias", torch.float32, 1)
+            if bias.numel() != E:
+                raise KernelError("scaled_norm: one bias per channel")
+    bp, ldb, bpos, btop, bmul = None, E, None, 0, 0.0
+    if b is not None:
+        bmul = b.mul
+        if isinstance(b.value, ExpertRows):
+            bp, bpos = b.value.data, b.value.places
+            bmul *= b.value.weight
+            _need(bpos, "experts' rows", torch.int32, 2)
+            if bpos.shape[0] != n or not bpos.is_contiguous() or bp.shape[1] != E:
+                raise KernelError(f"scaled_norm: experts' rows {tuple(bpos.shape)} / outputs {tuple(bp.shape)} do not fit [{n}, {E}]")
+            btop = bpos.shape[1]
+        else:
+            bp = b.value
+            if tuple(bp.shape) != (n, E):
+                raise KernelError(f"scaled_norm: a term of {tuple(bp.shape)} does not fit [{n}, {E}]")
+        _need(bp, "residual term", torch.float32, 2)
+        ldb = _rows_contiguous(bp, "residual term")
+    n_rows = n if rows is None else rows.numel()
+    if rows is not None:
+        _need(rows, "row list", torch.int32, 1)
+        if n_rows == 0:             # no row is wanted
+            return out
+    if (weight is None) != (out is None):
+        raise KernelError("scaled_norm: a norm has a weight and an output")
+    if out is not None:
+        _need(weight, "norm weight", torch.float32, 1)
+        _need(out, "norm output", ndim=2)
+        if tuple(out.shape) != (n_rows, E) or not out.is_contiguous() or weight.numel() != E:
+            raise KernelError(f"scaled_norm: output {tuple(out.shape)} does not fit [{n_rows}, {E}]")
+    if tiles is not None:
+        _need(tiles, "experts' tiles", torch.bfloat16, 2)
+        _need(places, "experts' rows", torch.int32, 2)
+        if tiles.shape[1] != E or not tiles.is_contiguous() or places.shape[0] != n or not places.is_contiguous():
+            raise KernelError(f"scaled_norm: tiles {tuple(tiles.shape)} with places {tuple(places.shape)} do not fit [{n}, {E}]")
+    if split is not None:
+        _need(split, "split rows", torch.bfloat16, 2)
+        if tuple(split.shape) != (2 * n, E) or not split.is_contiguous():
+            raise KernelError(f"scaled_norm: split rows {tuple(split.shape)} are not [{2 * n}, {E}]")
+    fn = _fn("scaled_norm", "lgml_scaled_norm", [c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_int,
+                                                 c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int,
+                                                 c_void_p, c_int, c_int, c_int, c_void_p])
+    _check("scaled_norm", fn(_ptr(x), 1 if keep else 0, _ptr(ap), n_parts, a_stride, lda, second, _ptr(bias), _ptr(a.scale if a is not None else None),
+                             a.mul if a is not None else 0.0, _ptr(bp), ldb, _ptr(bpos), btop, _ptr(b.scale if b is not None else None), bmul, _ptr(rows),
+                             _ptr(weight), float(eps), _ptr(out), dtype_code(out.dtype) if out is not None else F32, _ptr(tiles), _ptr(places),
+                             places.shape[1] if tiles is not None else 0, _ptr(split), n, n_rows, E, _stream()), "scaled_norm")
+    return out
+
+
+# ----------------------------------------------------------------------------------------
+# the real-gated linear recurrent unit
+# ----------------------------------------------------------------------------------------
+
+def rglru_chunk_tokens() -> int:
+    fn = getattr(csrc.load("rglru"), "lgml_rglru_chunk_tokens")
+    fn.argtypes, fn.restype = [], c_int
+    return fn()
+
+
+def _rglru_shapes(proj, ra, ra_b, ri, ri_b, sp8, who: str):
+    _need(proj, "projections", torch.float32, 2)
+    B, P, P2 = ra.shape
+    C = B * P
+    for t, what in ((ra, "decay gate"), (ri, "input gate")):
+        _need(t, f"{what}'s matrices", ra.dtype, 3)
+        if tuple(t.shape) != (B, P, P) or not t.is_contiguous():
+            raise KernelError(f"{who}: the {what}'s matrices {tuple(t.shape)} are not [{B}, {P}, {P}]")
+    for t, what in ((ra_b, "decay gate's bias"), (ri_b, "input gate's bias"), (sp8, "decay rates")):
+        _need(t, what, torch.float32)
+        if t.numel() != C or not t.is_contiguous():
+            raise KernelError(f"{who}: the {what} hold one number per channel")
+    return C, P
+
+
+def _conv_shapes(conv_w, conv_b, C: int, who: str) -> int:
+    _need(conv_w, "convolution weights", torch.float32, 2)
+    _need(conv_b, "convolution bias", torch.float32, 1)
+    if conv_w.shape[1] != C or not conv_w.is_contiguous() or conv_b.numel() != C:
+        raise KernelError(f"{who}: convolution weights {tuple(conv_w.shape)} are not [taps, {C}]")
+    return conv_w.shape[0]
+
+
+def rglru_state_floats(channels: int, taps: int) -> int:
+    """Floats of a request's state: S, and the ring of the convolution's last inputs."""
+    return channels + (taps * channels if taps > 1 else 0)
+
+
+def rglru_step(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, state: torch.Tensor, slots: torch.Tensor, positions: torch.Tensor,
+               ra: torch.Tensor, ra_b: torch.Tensor, ri: torch.Tensor, ri_b: torch.Tensor, sp8: torch.Tensor) -> torch.Tensor:
+    """One token of every request through the convolution, the gates, the recurrence and the output branch, in one kernel.
+    ``proj`` float32 [tokens, x | y] (2 C columns); conv_w float32 [taps, C]; ra, ri [parts, P, P]; ``sp8`` = 8 softplus(lam); ``state`` float32
+    [slots, >= ``rglru_state_floats``].  Returns S gelu_tanh(y) in the matrices' type, [tokens, C]."""
+    C, P = _rglru_shapes(proj, ra, ra_b, ri, ri_b, sp8, "rglru_step")
+    taps = _conv_shapes(conv_w, conv_b, C, "rglru_step")
+    n, ldp = proj.shape[0], _rows_contiguous(proj, "projections")
+    if proj.shape[1] != 2 * C or slots.numel() != n or positions.numel() != n:
+        raise KernelError(f"rglru_step: projections {tuple(proj.shape)}, {slots.numel()} slots and {positions.numel()} positions do not fit {C} channels")
+    ld = _state_rows(state, rglru_state_floats(C, taps), "rglru_step")
+    out = torch.empty((n, C), dtype=ra.dtype, device=proj.device)
+    fn = _fn("rglru", "lgml_rglru_step", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                          c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check("rglru", fn(_ptr(proj), ldp, _ptr(conv_w), _ptr(conv_b), _ptr(state), ld, _ptr(slots), _ptr(positions), _ptr(ra), _ptr(ra_b), _ptr(ri), _ptr(ri_b),
+                       _ptr(sp8), _ptr(out), dtype_code(out.dtype), n, C, P, taps, _stream()), "rglru_step")
+    return out
+
+
+def rglru_conv(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, state: torch.Tensor, seq_of_token: torch.Tensor, seq_start: torch.Tensor,
+               slots: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+    """The causal convolution of ``proj``'s first C columns, float32 [tokens, C]; the inputs of earlier steps come from the ring in
+    the request's state, which takes the step's last ones."""
+    _need(proj, "projections", torch.float32, 2)
+    C = conv_b.numel()
+    taps = _conv_shapes(conv_w, conv_b, C, "rglru_conv")
+    n, ldp = proj.shape[0], _rows_contiguous(proj, "projections")
+    if proj.shape[1] < C or positions.numel() != n or seq_of_token.numel() != n:
+        raise KernelError(f"rglru_conv: projections {tuple(proj.shape)} hold no {C} channels")
+    ld = _state_rows(state, rglru_state_floats(C, taps), "rglru_conv")
+    u = torch.empty((n, C), dtype=torch.float32, device=proj.device)
+    fn = _fn("rglru", "lgml_rglru_conv", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                          c_int, c_void_p])
+    _check("rglru", fn(_ptr(proj), ldp, _ptr(conv_w), _ptr(conv_b), _ptr(state), ld, _ptr(seq_of_token), _ptr(seq_start), _ptr(slots), _ptr(positions), _ptr(u),
+                       n, C, taps, _stream()), "rglru_conv")
+    return u
+
+
+RGLRU_FORMS = {"auto": 0, "rows": 1, "mma": 2}
+
+
+def rglru_gates(u: torch.Tensor, ra: torch.Tensor, ra_b: torch.Tensor, ri: torch.Tensor, ri_b: torch.Tensor, sp8: torch.Tensor, form: str = "auto") -> torch.Tensor:
+    """From the convolved inputs ``u`` float32 [tokens, C]: float32 [2, tokens, C], the decay a = exp(-sigmoid(Ra u + ra_b) sp8) and the
+    pushed term sqrt(1 - a^2) sigmoid(Ri u + ri_b) u, Ra and Ri block-diagonal [parts, P, P].  The products are true 32-bit
+    sums over the float32 u in every form."""
+    C, P = _rglru_shapes(u, ra, ra_b, ri, ri_b, sp8, "rglru_gates")
+    n = u.shape[0]
+    if u.shape[1] != C or not u.is_contiguous():
+        raise KernelError(f"rglru_gates: inputs {tuple(u.shape)} do not fit {C} channels")
+    ab = torch.empty((2, n, C), dtype=torch.float32, device=u.device)
+    fn = _fn("rglru", "lgml_rglru_gates", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check("rglru", fn(_ptr(u), _ptr(ra), _ptr(ra_b), _ptr(ri), _ptr(ri_b), _ptr(sp8), _ptr(ab), dtype_code(ra.dtype), n, C, P, RGLRU_FORMS[form], _stream()),
+           "rglru_gates")
+    return ab
+
+
+def rglru_scan(ab: torch.Tensor, proj: torch.Tensor, state: torch.Tensor, seq_start: torch.Tensor, slots: torch.Tensor, out: torch.Tensor,
+               chunks: Optional[torch.Tensor] = None, chunk_start: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """S <- a S + push over every request's tokens of this step, from ``state[slot]`` (which takes the last S); out[t] = S_t *
+    gelu_tanh(y_t), y the columns C .. 2 C - 1 of ``proj``.  ``ab`` as ``rglru_gates`` gives it.  With ``chunks`` and ``chunk_start``
+    (``StepBatch.scan_pieces``) the pieces of a request's portion run side by side."""
+    _need(ab, "decays and pushed terms", torch.float32, 3)
+    _need(proj, "projections", torch.float32, 2)
+    _need(out, "recurrence output", ndim=2)
+    two, n, C = ab.shape
+    ldp = _rows_contiguous(proj, "projections")
+    if two != 2 or not ab.is_contiguous() or tuple(proj.shape) != (n, 2 * C) or tuple(out.shape) != (n, C) or not out.is_contiguous():
+        raise KernelError(f"rglru_scan: {tuple(ab.shape)}, projections {tuple(proj.shape)} and output {tuple(out.shape)} do not fit")
+    ld = _state_rows(state, C, "rglru_scan")
+    n_seqs = slots.numel()
+    if chunks is None:
+        fn = _fn("rglru", "lgml_rglru_scan", [c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+        _check("rglru", fn(_ptr(ab), _ptr(proj), ldp, _ptr(state), ld, _ptr(seq_start), _ptr(slots), _ptr(out), dtype_code(out.dtype), n, n_seqs, C, _stream()),
+               "rglru_scan")
+        return out
+    _need(chunks, "chunks", torch.int32, 2)
+    _need(chunk_start, "chunk starts", torch.int32, 1)
+    n_chunks = chunks.shape[0]
+    if chunks.shape[1] != 2 or not chunks.is_contiguous() or chunk_start.numel() != n_seqs + 1:
+        raise KernelError("rglru_scan: chunks are [n, 2] and chunk starts one more than the requests")
+    scratch = torch.empty((2, n_chunks, C), dtype=torch.float32, device=ab.device)
+    fn = _fn("rglru", "lgml_rglru_chunks", [c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                            c_int, c_int, c_void_p])
+    _check("rglru", fn(_ptr(ab), _ptr(proj), ldp, _ptr(state), ld, _ptr(chunks), _ptr(chunk_start), n_chunks, _ptr(slots), _ptr(scratch), _ptr(out),
+                       dtype_code(out.dtype), n, n_seqs, C, _stream()), "rglru_chunks")
     return out
 
 

@@ -23,8 +23,9 @@ import torch
 
 from .. import ops
 from ..cache import FixedState
+from ..weights import VECTOR, TensorSpec
 from .base import Part, register_part
-from .norm import PendingDelta
+from .norm import PendingDelta, ScaledTerms
 
 
 class PreNormBlock(Part):
@@ -185,5 +186,58 @@ class SandwichBlock(Part):
         return x, pending
 
 
+class ParallelBlock(Part):
+    """A layer whose two sublayers read the same norm, and whose results are scaled channel by channel:
+
+        h = norm(x);   x = x + (s1 mixer(h) + s2 ffn(h))
+
+    The two scales are vectors of the layer (``scale1``, ``scale2``).  Both sums ride in the next norm's kernel, which must take
+    ``ScaledTerms``.  A feed-forward with ``routes_ahead`` says before the norm where its rows go, and the norm's kernel puts
+    them there."""
+
+    def __init__(self, norm, mixer, ffn, width: int, names=None):
+        self.norm, self.mixer, self.ffn, self.width = norm, mixer, ffn, width
+        self.names = {"norm": "norm1", "mixer": "mix", "ffn": "mlp", "scale1": "ls1", "scale2": "ls2"}
+        self.names.update(names or {})
+        self.scale1 = self.scale2 = None
+
+    def _parts(self, prefix):
+        for key in ("norm", "mixer", "ffn"):
+            part = getattr(self, key)
+            if part is not None:
+                yield part, f"{prefix}.{self.names[key]}"
+
+    def tensor_specs(self, prefix):
+        scale = lambda key, optional: TensorSpec(f"{prefix}.{self.names[key]}", (self.width,), VECTOR, optional=optional, init=(1.0, 1.0))
+        # a layer without a feed-forward may carry the vector of one unread
+        return [s for part, p in self._parts(prefix) for s in part.tensor_specs(p)] + [scale("scale1", False), scale("scale2", self.ffn is None)]
+
+    def bind(self, prefix, tensors, rt):
+        for part, p in self._parts(prefix):
+            part.bind(p, tensors, rt)
+        self.scale1 = tensors[f"{prefix}.{self.names['scale1']}"].contiguous()
+        self.scale2 = tensors[f"{prefix}.{self.names['scale2']}"].contiguous() if self.ffn is not None else None
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    @property
+    def graph_safe(self):
+        return all(getattr(part, "graph_safe", False) for part, _ in self._parts(""))
+
+    def forward(self, rt, x, pending, batch, cache):
+        routed = self.ffn.route(rt, batch) if getattr(self.ffn, "routes_ahead", False) else None
+        if routed is not None and routed.tiles is not None:
+            h = self.norm.forward(rt, x, rt.dtype, delta=pending, tiles=routed.tiles, places=routed.places)
+        else:
+            h = self.norm.forward(rt, x, rt.dtype, delta=pending)
+        terms = (ops.Term(self.mixer.forward(rt, h, batch, cache), self.scale1),)
+        if self.ffn is not None:
+            out = self.ffn.forward(rt, h) if routed is None else self.ffn.forward(rt, h, routed)
+            terms += (ops.Term(out.sum() if isinstance(out, ops.Partials) else out, self.scale2),)
+        return x, ScaledTerms(terms)
+
+
+register_part("block", "parallel", ParallelBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "sandwich", SandwichBlock)

@@ -29,6 +29,11 @@ class TokenEmbedding(Part):
         out = torch.empty((token_ids.numel(), self.width), dtype=torch.float32, device=token_ids.device)
         return ops.embed_rows(self.table, token_ids, out, rt.status)
 
+    def rows(self, rt, token_ids):
+        """The table's rows in the table's own type (for a product that reads them)."""
+        out = torch.empty((token_ids.numel(), self.width), dtype=self.table.dtype, device=token_ids.device)
+        return ops.embed_rows(self.table, token_ids, out, rt.status)
+
 
 class LMHead(Part):
     graph_safe = True

@@ -20,6 +20,9 @@ Options: ``window`` (a token sees itself and the window - 1 before it; the cache
 longer than ``original``: with n(t) = rope_dims ln(original / (2 pi t)) / (2 ln base), lo = max(floor(n(fast)), 0),
 hi = min(ceil(n(slow)), rope_dims - 1) and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the frequency
 is f_i / factor * r_i + f_i (1 - r_i), and cosines and sines are multiplied by 0.1 ln(factor) + 1.
+``q_rank``: the queries go through a latent of their own, q = W_uq c_q with c_q = W_dq h over its root mean square times a
+weight (tensors ``.dq``, ``.dq.norm``, ``.uq`` in place of ``.q``); both down-projections are then one product.  ``halves``: the
+pairs that turn are (i, i + rope_dims / 2).
 """
 from __future__ import annotations
 
@@ -58,7 +61,10 @@ class LatentAttention(Part):
 
     def __init__(self, width: int, n_heads: int, head_dim: int, rot_dim: int, v_head_dim: int, rank: int, scale: float, eps: float,
                  rope_base: float, rope_dims: Optional[int] = None, window: Optional[int] = None, out_gate: bool = False,
-                 rope_scaling: Optional[Dict[str, float]] = None):
+                 rope_scaling: Optional[Dict[str, float]] = None, q_rank: Optional[int] = None, halves: bool = False):
+        if q_rank and out_gate:
+            raise ValueError("an output gate comes with queries that are projected directly")
+        self.q_rank, self.halves = int(q_rank) if q_rank else 0, bool(halves)
         self.width, self.n_heads, self.head_dim, self.rot_dim = width, n_heads, head_dim, rot_dim
         self.v_head_dim, self.rank = v_head_dim, rank
         self.scale, self.eps = float(scale), float(eps)
@@ -70,7 +76,7 @@ class LatentAttention(Part):
         self.out_gate = bool(out_gate)
         self.rope_scaling = dict(rope_scaling) if rope_scaling else None
         self.rot_mag = 1.0
-        self.w_in = self.w_uk_t = self.w_uv = self.wo = self.norm_w = self.inv_freq = None
+        self.w_in = self.w_uq = self.w_uk_t = self.w_uv = self.wo = self.norm_w = self.q_norm_w = self.inv_freq = None
 
     def cache_spec(self):
         return PagedKV(1, self.rank + self.rot_dim, self.window, self.rank, v_in_k=True)
@@ -78,14 +84,20 @@ class LatentAttention(Part):
     def tensor_specs(self, prefix):
         H, D, Dr, Dv, R, E = self.n_heads, self.head_dim, self.rot_dim, self.v_head_dim, self.rank, self.width
         gate = [TensorSpec(prefix + ".g", (H * Dv, E))] if self.out_gate else []
-        return [TensorSpec(prefix + ".q", (H * (D + Dr), E)), TensorSpec(prefix + ".dkv", (R + Dr, E)),
+        q = [TensorSpec(prefix + ".q", (H * (D + Dr), E))]
+        if self.q_rank:
+            q = [TensorSpec(prefix + ".dq", (self.q_rank, E)), TensorSpec(prefix + ".dq.norm", (self.q_rank,), VECTOR, init=(1.0, 1.0)),
+                 TensorSpec(prefix + ".uq", (H * (D + Dr), self.q_rank))]
+        return q + [TensorSpec(prefix + ".dkv", (R + Dr, E)),
                 TensorSpec(prefix + ".dkv.norm", (R,), VECTOR, init=(1.0, 1.0)), TensorSpec(prefix + ".uk", (H * D, R)),
                 TensorSpec(prefix + ".uv", (H * Dv, R)), TensorSpec(prefix + ".o", (E, H * Dv))] + gate
 
     def bind(self, prefix, tensors, rt):
         H, D, Dv, R = self.n_heads, self.head_dim, self.v_head_dim, self.rank
-        # one product for everything that reads the mixer's input: queries, the down-projection, the output gate's logits
-        self.w_in = torch.cat([tensors[prefix + ".q"], tensors[prefix + ".dkv"]] + ([tensors[prefix + ".g"]] if self.out_gate else []),
+        # one product for everything that reads the mixer's input: queries (or their latent), the down-projection, the output gate's logits
+        if self.q_rank:
+            self.q_norm_w, self.w_uq = tensors[prefix + ".dq.norm"], tensors[prefix + ".uq"]
+        self.w_in = torch.cat([tensors[prefix + (".dq" if self.q_rank else ".q")], tensors[prefix + ".dkv"]] + ([tensors[prefix + ".g"]] if self.out_gate else []),
                               dim=0).contiguous()
         self.norm_w = tensors[prefix + ".dkv.norm"]
         self.w_uk_t = tensors[prefix + ".uk"].view(H, D, R).transpose(1, 2).contiguous()       # [H, R, D]: q_plain -> the latent's side
@@ -103,13 +115,18 @@ class LatentAttention(Part):
         H, D, Dr, Dv, R = self.n_heads, self.head_dim, self.rot_dim, self.v_head_dim, self.rank
         n = h.shape[0]
         proj = rt.linear(h, self.w_in, out_dtype=torch.float32)
-        nq = H * (D + Dr)
-        q_plain, q_full = ops.latent_prepare(proj[:, :nq], proj[:, nq:nq + R + Dr], self.norm_w, self.eps, self.inv_freq, self.rope_dims, batch.positions,
-                                             batch.seq_of_token, cache.block_table, cache.k, H, D, Dr, R, rt.status, write_kv=cache.writable,
-                                             rot_mag=self.rot_mag)
-        gate = proj[:, nq + R + Dr:] if self.out_gate else None
-        window = self.window or 0
-        ops.head_linear(q_plain, self.w_uk_t, q_full, D, R + Dr)
+        window, gate = self.window or 0, None
+        if self.q_rank:
+            cq, cos_sin = ops.latent_down(proj, self.q_norm_w, self.norm_w, self.eps, self.inv_freq, self.rope_dims, batch.positions, batch.seq_of_token,
+                                          cache.block_table, cache.k, self.q_rank, R, Dr, rt.status, rot_mag=self.rot_mag, halves=self.halves)
+            q_full = ops.latent_query(rt.linear(cq, self.w_uq, out_dtype=torch.float32), self.w_uk_t, cos_sin, self.rope_dims, Dr, halves=self.halves)
+        else:
+            nq = H * (D + Dr)
+            q_plain, q_full = ops.latent_prepare(proj[:, :nq], proj[:, nq:nq + R + Dr], self.norm_w, self.eps, self.inv_freq, self.rope_dims,
+                                                 batch.positions, batch.seq_of_token, cache.block_table, cache.k, H, D, Dr, R, rt.status,
+                                                 write_kv=cache.writable, rot_mag=self.rot_mag, halves=self.halves)
+            gate = proj[:, nq + R + Dr:] if self.out_gate else None
+            ops.head_linear(q_plain, self.w_uk_t, q_full, D, R + Dr)
         o = torch.empty((n, H * Dv), dtype=h.dtype, device=h.device)
         if rt.dtype == torch.bfloat16 and (R + Dr) in (64, 128):
             # A cell of 64 or 128 numbers is a head size the plain causal attention kernels are built for (tcgen05 for

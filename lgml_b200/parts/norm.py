@@ -43,6 +43,15 @@ class PendingDelta:
     eps: float = 0.0            # of the norm with ``w_post``
 
 
+@dataclass
+class ScaledTerms:
+    """What a layer has computed but not yet added to the residual stream: ``ops.Term``s, each a result with a scale per
+    channel.  ``keep`` False: x is replaced by their sum."""
+
+    terms: tuple = ()
+    keep: bool = True
+
+
 class RMSNorm(Part):
     """``single``: the learned weight is ONE number for all coordinates (a tensor without dimensions);
     the kernel reads it as a row of equal entries.  ``one_plus``: the stored weight is the distance from one
@@ -66,11 +75,16 @@ class RMSNorm(Part):
         if self.one_plus:
             self.weight = (1.0 + self.weight.float()).contiguous()
 
-    def forward(self, rt, x, out_dtype, delta=None, rows=None, delta_scale: float = 1.0):
-        """Norm of x (+ delta_scale * delta).  x is the float32 residual stream; with ``delta`` the sum
-        is written back to x.  ``rows`` (int32 on the device) picks the rows to norm."""
+    def forward(self, rt, x, out_dtype, delta=None, rows=None, delta_scale: float = 1.0, tiles=None, places=None):
+        """Norm of x (+ delta_scale * delta).  x is the float32 residual stream; with ``delta`` (a tensor, ``ops.Partials`` or
+        ``ScaledTerms``) the sum is written back to x.  ``rows`` (int32 on the device) picks the rows to norm; ``tiles`` and
+        ``places``: the normed rows go there as well (``ops.scaled_norm``)."""
         n = x.shape[0] if rows is None else rows.numel()
         out = torch.empty((n, self.width), dtype=out_dtype, device=x.device)
+        if isinstance(delta, ScaledTerms) or tiles is not None:
+            if not isinstance(delta, ScaledTerms):
+                delta = ScaledTerms(() if delta is None else (ops.Term(delta, mul=delta_scale),))
+            return ops.scaled_norm(x, delta.terms, self.eps, self.weight, out, keep=delta.keep, rows=rows, tiles=tiles, places=places)
         return ops.rmsnorm(x, self.weight, self.eps, out, delta=delta, rows=rows, delta_scale=delta_scale)
 
 

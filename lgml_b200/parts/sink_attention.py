@@ -17,6 +17,9 @@ the mixing layers read them there; the mixed values are what the cache holds.  T
 learned number per head that only adds to the softmax's denominator.  Each constant is a
 constructor argument; ``slope_base`` None, ``sink`` False, ``gate`` False, ``temperature`` None
 switch a mechanism off.
+
+Other forms: ``sink`` a number: that score for every head, nothing learned (0: one is added to the denominator); ``gate`` "head": one
+logit per head, sigmoid(W_g h)_h on the whole head's output; ``out_bias``: W_o has a bias.
 """
 from __future__ import annotations
 
@@ -35,7 +38,7 @@ class SinkAttention(Part):
 
     def __init__(self, width: int, n_heads: int, n_kv_heads: int, head_dim: int, v_head_dim: int, scale: float,
                  window: Optional[int] = None, temperature: Optional[Tuple[float, int]] = None, slope_base: Optional[float] = 8.0,
-                 sink: bool = True, gate: bool = True, bias: bool = True, v_mix: Optional[str] = None, v_mix_key: str = "v_first"):
+                 sink=True, gate=True, bias: bool = True, out_bias: bool = False, v_mix: Optional[str] = None, v_mix_key: str = "v_first"):
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} heads are no multiple of {n_kv_heads} KV heads")
         if v_mix not in (None, "keep", "mix"):
@@ -46,9 +49,14 @@ class SinkAttention(Part):
         self.window = int(window) if window else None
         self.temp_coef, self.temp_every = (float(temperature[0]), int(temperature[1])) if temperature else (0.0, 1)
         self.slope_base = slope_base
-        self.has_sink, self.has_gate, self.bias = bool(sink), bool(gate), bool(bias)
+        # a learned sink (True), none (False), or one fixed score for every head
+        self.sink_score = None if isinstance(sink, bool) else float(sink)
+        self.has_sink, self.has_gate, self.bias, self.out_bias = sink is True, bool(gate), bool(bias), bool(out_bias)
+        if gate not in (True, False, "head"):
+            raise ValueError(f"gate must be True, False or 'head', not {gate!r}")
+        self.gate_cols = n_heads if gate == "head" else n_heads * v_head_dim
         self.v_mix, self.v_mix_key = v_mix, v_mix_key
-        self.w_in = self.b_in = self.wo = self.sinks = self.slopes = self.lam = None
+        self.w_in = self.b_in = self.wo = self.bo = self.sinks = self.slopes = self.lam = None
 
     def cache_spec(self):
         return PagedKV(self.n_kv_heads, self.head_dim, self.window, self.v_head_dim)
@@ -61,7 +69,9 @@ class SinkAttention(Part):
             specs += [TensorSpec(prefix + ".q.b", (H * D,), VECTOR), TensorSpec(prefix + ".k.b", (G * D,), VECTOR),
                       TensorSpec(prefix + ".v.b", (G * Dv,), VECTOR)]
         if self.has_gate:
-            specs.append(TensorSpec(prefix + ".g", (H * Dv, E)))
+            specs.append(TensorSpec(prefix + ".g", (self.gate_cols, E)))
+        if self.out_bias:
+            specs.append(TensorSpec(prefix + ".o.b", (E,), VECTOR))
         if self.has_sink:
             specs.append(TensorSpec(prefix + ".sink", (H,), VECTOR))
         # only a mixing layer reads the weight; the layer that keeps its values may carry one unread
@@ -69,7 +79,7 @@ class SinkAttention(Part):
         return specs
 
     def bind(self, prefix, tensors, rt):
-        H, Dv = self.n_heads, self.v_head_dim
+        H = self.n_heads
         mats = [tensors[prefix + ".q"], tensors[prefix + ".k"], tensors[prefix + ".v"]]
         if self.has_gate:
             mats.append(tensors[prefix + ".g"])
@@ -77,10 +87,13 @@ class SinkAttention(Part):
         if self.bias:
             vecs = [tensors[prefix + ".q.b"], tensors[prefix + ".k.b"], tensors[prefix + ".v.b"]]
             if self.has_gate:
-                vecs.append(torch.zeros(H * Dv, dtype=torch.float32, device=vecs[0].device))
+                vecs.append(torch.zeros(self.gate_cols, dtype=torch.float32, device=vecs[0].device))
             self.b_in = torch.cat(vecs, dim=0).contiguous()
         self.wo = tensors[prefix + ".o"]
+        self.bo = tensors[prefix + ".o.b"].contiguous() if self.out_bias else None
         self.sinks = tensors[prefix + ".sink"].contiguous() if self.has_sink else None
+        if self.sink_score is not None:
+            self.sinks = torch.full((H,), self.sink_score, dtype=torch.float32, device=rt.device)
         if self.slope_base is not None:
             self.slopes = torch.tensor([2.0 ** (-float(self.slope_base) * (h + 1) / H) for h in range(H)], dtype=torch.float64) \
                 .to(torch.float32).to(rt.device)
@@ -107,10 +120,10 @@ class SinkAttention(Part):
                                temp_coef=self.temp_coef, temp_every=self.temp_every, v_mode=v_mode, v_keep=kept, v_lambda=self.lam,
                                write_kv=cache.writable)
         lo = H * D + G * (D + Dv)
-        gate = proj[:, lo:lo + H * Dv] if self.has_gate else None
+        gate = proj[:, lo:lo + self.gate_cols] if self.has_gate else None
         o = torch.empty((n, H * Dv), dtype=h.dtype, device=h.device)
         rt.sink_attention(q, batch, cache, o, H, self.scale, self.window or 0, self.slopes, self.sinks, gate)
-        return rt.linear(o, self.wo, partials_ok=True)
+        return rt.linear(o, self.wo, bias=self.bo, partials_ok=True)
 
 
 register_part("mixer", "sink_attention", SinkAttention)

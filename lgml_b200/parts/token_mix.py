@@ -1,4 +1,4 @@
-"""Two small parts that sit around a layer's mixer and feed-forward.
+"""Small parts that sit around a layer's mixer and feed-forward.
 
 ``TokenShift``: what the mixer reads moves towards the previous token's, per channel:
 
@@ -13,6 +13,15 @@ float32 rows (the norm before it writes them so) and gives rows in the compute t
 
 x is the residual stream itself (not a norm of it).  For a few tokens one kernel does all of it
 (and the residual sum before it); for many, in bfloat16, the two products run as matrix products.
+
+``PassInput``: before a pass of a loop over layers, the residual stream is made anew from itself and the embedding's output:
+
+    x <- W [x; x0],    W [E, 2 E],  x0 = scale * (the token's row of the embedding's table)
+
+The half that reads x0 is the same in every pass and is computed once a step, from the table's rows themselves (the
+scale multiplies the float32 result).  A pass that starts the model has x = x0: both halves are then one product.  Later x enters its
+half in two bfloat16 pieces, as twice as many rows, so that no pass rounds the stream to bfloat16 (the piece that rounding
+lost is a row of its own; the kernel that adds the halves adds the pieces).
 """
 from __future__ import annotations
 
@@ -22,6 +31,7 @@ from .. import ops
 from ..cache import FixedState
 from ..weights import MATRIX, VECTOR, TensorSpec
 from .base import Part, register_part
+from .norm import ScaledTerms
 
 # tokens of a step from which the token input's two products run as matrix products
 SIDE_PRODUCTS_FROM = 64
@@ -79,6 +89,39 @@ class TokenSide(Part):
         return ops.side_add(x, y, self.norm_w, self.eps, scale)
 
 
+class PassInput(Part):
+    graph_safe = True
+
+    def __init__(self, width: int, embedding, scale: float = 1.0, name: str = "loop.in"):
+        self.width, self.embedding, self.scale, self.name = width, embedding, float(scale), name
+        self.w_both = None
+
+    def tensor_specs(self, prefix=""):
+        return [TensorSpec(self.name, (self.width, 2 * self.width), MATRIX)]
+
+    def bind(self, prefix, tensors, rt):
+        w, E = tensors[self.name], self.width
+        self.w_both = torch.cat([w[:, :E], w[:, E:]], dim=0).contiguous()       # rows for x, then rows for x0
+
+    def forward(self, rt, x, pending, batch, number: int, starts_model: bool):
+        """What is pending for x once pass ``number`` of the loop begins (``pending`` included); ``starts_model``: nothing ran
+        before, and x is not read."""
+        E = self.width
+        if number == 0:
+            rows = self.embedding.rows(rt, batch.token_ids)
+            both = rt.linear(rows, self.w_both if starts_model else self.w_both[E:], out_dtype=torch.float32)
+            batch.shared[self] = ops.Term(both[:, E:] if starts_model else both, mul=self.scale)
+            if starts_model:
+                return ScaledTerms((ops.Term(both[:, :E], mul=self.scale), batch.shared[self]), keep=False)
+        if not isinstance(pending, ScaledTerms):
+            pending = ScaledTerms(() if pending is None else (ops.Term(pending),))
+        split = torch.empty((2 * x.shape[0], E), dtype=rt.dtype, device=x.device) if rt.dtype == torch.bfloat16 else None
+        if split is not None or pending.terms:
+            ops.scaled_norm(x, pending.terms, keep=pending.keep, split=split)
+        half = rt.linear(x if split is None else split, self.w_both[:E], out_dtype=torch.float32, partials_ok=True)
+        return ScaledTerms((ops.Term(half, stacked=split is not None), batch.shared[self]), keep=False)
+
+
 class InputConv(Part):
     """What a sublayer reads gains a causal convolution of itself over time, per channel:
 
@@ -114,3 +157,4 @@ class InputConv(Part):
 register_part("token_input", "token_shift", TokenShift)
 register_part("token_input", "input_conv", InputConv)
 register_part("token_input", "token_side", TokenSide)
+register_part("token_input", "pass_input", PassInput)

@@ -28,13 +28,14 @@ MATRIX, VECTOR, INT_TABLE = "matrix", "vector", "int"
 @dataclass(frozen=True)
 class TensorSpec:
     """One tensor a part needs.  ``init`` = (mean, scale): random-weights mode
-    draws N(mean, (scale * std)^2)."""
+    draws N(mean, (scale * std)^2); an integer table's rows are different numbers below ``below``."""
 
     name: str
     shape: Tuple[int, ...]
     kind: str = MATRIX
     optional: bool = False
     init: Tuple[float, float] = (0.0, 1.0)
+    below: int = 0
 
 
 class WeightError(ValueError):

@@ -97,6 +97,16 @@ def fill_normal_host(shape, mean: float, sd: float, key: int, chunk: int = 1 << 
     return torch.from_numpy(out.reshape(tuple(shape)))
 
 
+def random_table(spec: TensorSpec, seed: int) -> torch.Tensor:
+    """An integer table [rows, n] whose rows hold n different numbers below ``spec.below``: the places of the n smallest of that
+    many values of the tensor's stream."""
+    if len(spec.shape) != 2 or spec.below < spec.shape[1]:
+        raise ValueError(f"random-weights mode cannot draw the integer table '{spec.name}'")
+    rows, n = spec.shape
+    z = seeded_normal(tensor_key(seed, spec.name), rows * spec.below).reshape(rows, spec.below)
+    return torch.from_numpy(np.argsort(z, axis=1, kind="stable")[:, :n].astype(np.int32))
+
+
 def random_tensors(specs: Iterable[TensorSpec], seed: int, std: float = 0.02,
                    matrix_dtype: torch.dtype = torch.float32) -> Dict[str, torch.Tensor]:
     """Host tensors for every non-optional spec."""
@@ -105,7 +115,8 @@ def random_tensors(specs: Iterable[TensorSpec], seed: int, std: float = 0.02,
         if s.optional:
             continue
         if s.kind == INT_TABLE:
-            raise ValueError(f"random-weights mode cannot draw the integer table '{s.name}'")
+            out[s.name] = random_table(s, seed)
+            continue
         mean, scale = s.init
         t = fill_normal_host(s.shape, mean, scale * std, tensor_key(seed, s.name))
         out[s.name] = t.to(matrix_dtype) if s.kind == MATRIX else t
