@@ -16,7 +16,8 @@ measured copy bandwidth, and ``roofline_points`` the same fraction for every bat
 
 ``--shape llama32_3b`` runs that shape's own workload (32 prompts of 128 to 4,096 tokens in
 portions of 512 beside decodes, 512 new tokens each) through ``Engine.generate``;
-``--shape llama2_13b`` decodes at batch 16 after 3,584-token prompts; ``--design lefulorn`` (or ``gotulorn``, ``konovik``, ``dizepel``, ``tedisun``)
+``--shape llama2_13b`` decodes at batch 16 after 3,584-token prompts; ``--design lefulorn`` (or ``gotulorn``, ``konovik``, ``dizepel``, ``tedisun``,
+``nelosun``)
 times that design beside the Llama decoder at equal layer sizes; ``--cpu-baseline`` times the
 plain CPU implementation at the tiny configurations.
 """
@@ -370,7 +371,26 @@ def tedisun_shape(width: int, heads: int, kv_heads: int, head_dim: int, ff: int,
             "logit_softcap": 30.0, "layers": [dict(par if i % 2 == 0 else dl) for i in range(layers)]}
 
 
-DESIGN_SHAPES = {"lefulorn": lefulorn_shape, "gotulorn": gotulorn_shape, "konovik": konovik_shape, "dizepel": dizepel_shape, "tedisun": tedisun_shape}
+def nelosun_shape(width: int, heads: int, kv_heads: int, head_dim: int, ff: int, layers: int, window: int, vocab: int) -> dict:
+    """Nelosun with layers of a real model's size: attention, latent attention, attention and the gated linear recurrence in turn (attention:
+    ``heads`` heads of ``head_dim`` on ``kv_heads`` key heads; latent: heads of half that size, latents of width / 4 for the queries and 96
+    for keys and values, a rotated part of 32; the recurrence as wide as the model, gate matrices of 256, four taps), every one beside 8
+    experts of a quarter of the gated inner width of which a token's row of the table names 2; one pass of a loop over all layers (its
+    product over the stream and the embedding once; the Llama decoder beside it runs every layer once)."""
+    inner = (2 * ff // 3 + 255) // 256 * 256
+    mlp = {"kind": "moe", "expert": {"ff": inner // 4, "limit": 7.0}, "router": {"experts": 8, "top": 2}}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5, "q_temp": {"coef": 0.1, "every": 1024}}
+    lat = {"heads": heads, "dim": head_dim // 2, "rot_dim": 32, "vdim": head_dim // 2, "q_rank": width // 4, "kv_rank": 96,
+           "scale": (head_dim // 2 + 32) ** -0.5, "rot": {"base": 10000.0, "dims": 32}}
+    rec = {"width": width, "blocks": width // 256, "conv": 4}
+    kinds = [("attention", att), ("latent_attention", lat), ("attention", att), ("rglru", rec)]
+    return {"architecture": "Nelosun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "loop": {"start": 0, "stop": layers, "times": 1},
+            "layers": [{"type": kinds[i % 4][0], "mixer": dict(kinds[i % 4][1]), "mlp": mlp} for i in range(layers)]}
+
+
+DESIGN_SHAPES = {"lefulorn": lefulorn_shape, "gotulorn": gotulorn_shape, "konovik": konovik_shape, "dizepel": dizepel_shape, "tedisun": tedisun_shape,
+                 "nelosun": nelosun_shape}
 
 DESIGN_SIZES = {          # name -> width, heads, KV heads, head size, dense inner width, layers
     "w2048": (2048, 16, 4, 128, 8192, 4),
@@ -489,7 +509,7 @@ def main() -> int:
     ap.add_argument("--context", type=int, default=0, help="context (tokens a request may hold) instead of the shape's own")
     ap.add_argument("--prefill-tokens", type=int, default=0, help="tokens of the timed prompt instead of 2,048 (read in portions of 2,048)")
     ap.add_argument("--no-kernel-times", action="store_true", help="leave out the per-kernel-class times of a decode step")
-    ap.add_argument("--design", default="", choices=["", "lefulorn", "gotulorn", "konovik", "dizepel", "tedisun"], help="time this design beside the Llama decoder at equal layer sizes "
+    ap.add_argument("--design", default="", choices=["", "lefulorn", "gotulorn", "konovik", "dizepel", "tedisun", "nelosun"], help="time this design beside the Llama decoder at equal layer sizes "
                     "(prefill and decode, with kernel-class times) instead of the headline workload")
     ap.add_argument("--cpu-baseline", action="store_true", help="time the plain CPU implementation at the tiny configurations and stop")
     args = ap.parse_args()

@@ -86,6 +86,60 @@ __global__ void __launch_bounds__(ITEMS) sink_qkv_store_kernel(
     v_pages[(((size_t)page * Hv + g) * page_size + (size_t)(pos % page_size)) * Dv + d] = from_f32<T>(val);
 }
 
+// The same, four entries a thread in 16-byte reads (head sizes and the row stride multiples of 4).
+template <typename T> __device__ __forceinline__ void store_quad(T *p, const float4 &v);
+template <> __device__ __forceinline__ void store_quad<float>(float *p, const float4 &v) { *reinterpret_cast<float4 *>(p) = v; }
+template <> __device__ __forceinline__ void store_quad<__nv_bfloat16>(__nv_bfloat16 *p, const float4 &v) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<unsigned *>(&lo), *reinterpret_cast<unsigned *>(&hi));
+}
+template <typename T>
+__global__ void __launch_bounds__(ITEMS) sink_qkv_store_quads_kernel(
+    const float *__restrict__ proj, int ldp, T *__restrict__ q_out, int ldq, const int *__restrict__ positions,
+    const int *__restrict__ seq_of_token, const int *__restrict__ block_table, int max_blocks, T *__restrict__ k_pages,
+    T *__restrict__ v_pages, int n_pages, int page_size, int H, int Hkv, int Hv, int D, int Dv, float temp_coef, int temp_every,
+    int v_mode, float *__restrict__ v_keep, const float *__restrict__ v_lambda, int write_kv, int *__restrict__ status) {
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const int nq = H * D, nk = Hkv * D, nv = Hv * Dv;
+    const int e = (blockIdx.y * ITEMS + threadIdx.x) * 4;
+    if (e >= nq + (write_kv ? nk + nv : 0)) return;
+    const int pos = positions[t];
+    float4 val = act_load(reinterpret_cast<const float4 *>(proj + (size_t)t * ldp + e));
+    if (e < nq) {
+        if (temp_coef != 0.f) {
+            const float f = 1.0f + temp_coef * logf((float)((pos + 1) / temp_every) + 1.0f);
+            val.x *= f, val.y *= f, val.z *= f, val.w *= f;
+        }
+        store_quad<T>(q_out + (size_t)t * ldq + e, val);
+        return;
+    }
+    const int seq = seq_of_token[t];
+    const int blk = pos / page_size;
+    int page = -1;
+    if (pos >= 0 && blk < max_blocks) page = block_table[(size_t)seq * max_blocks + blk];
+    if (page < 0 || page >= n_pages) {   // the host reserves pages first; never write outside the pool
+        if (e == nq) atomicExch(status, 2);
+        return;
+    }
+    if (e < nq + nk) {
+        const int c = e - nq, g = c / D, d = c - g * D;
+        store_quad<T>(k_pages + (((size_t)page * Hkv + g) * page_size + (size_t)(pos % page_size)) * D + d, val);
+        return;
+    }
+    const int c = e - nq - nk, g = c / Dv, d = c - g * Dv;
+    if (v_mode == 1) {
+        *reinterpret_cast<float4 *>(v_keep + (size_t)t * nv + c) = val;
+    } else if (v_mode == 2) {
+        const float lam = v_lambda[0];
+        const float4 k = act_load(reinterpret_cast<const float4 *>(v_keep + (size_t)t * nv + c));
+        val.x = (1.0f - lam) * val.x + lam * k.x, val.y = (1.0f - lam) * val.y + lam * k.y;
+        val.z = (1.0f - lam) * val.z + lam * k.z, val.w = (1.0f - lam) * val.w + lam * k.w;
+    }
+    store_quad<T>(v_pages + (((size_t)page * Hv + g) * page_size + (size_t)(pos % page_size)) * Dv + d, val);
+}
+
 template <typename T, typename TO, int MAXD>
 __global__ void __launch_bounds__(WARPS * 32) sink_attention_kernel(
     const T *__restrict__ q, int ldq, const int *__restrict__ positions, const int *__restrict__ seq_of_token,
@@ -1036,17 +1090,20 @@ LGML_API int lgml_sink_qkv_store(const float *proj, int ldp, void *q_out, int dt
     LGML_REQUIRE(v_mode != 2 || v_lambda != nullptr, "sink_qkv_store: mixing needs its weight");
     if (n_tokens == 0) return 0;
     const int items = H * D + (write_kv ? Hkv * D + Hv * Dv : 0);
-    dim3 grid(n_tokens, (items + ITEMS - 1) / ITEMS);
-    if (dtype == LGML_F32)
-        lgml_launch(sink_qkv_store_kernel<float>, grid, ITEMS, 0, stream, proj, ldp, (float *)q_out, ldq, positions, seq_of_token, block_table,
-                    max_blocks, (float *)k_pages, (float *)v_pages, n_pages, page_size, H, Hkv, Hv, D, Dv, temp_coef, temp_every, v_mode, v_keep,
-                    v_lambda, write_kv, status);
-    else if (dtype == LGML_BF16)
-        lgml_launch(sink_qkv_store_kernel<__nv_bfloat16>, grid, ITEMS, 0, stream, proj, ldp, (__nv_bfloat16 *)q_out, ldq, positions, seq_of_token,
-                    block_table, max_blocks, (__nv_bfloat16 *)k_pages, (__nv_bfloat16 *)v_pages, n_pages, page_size, H, Hkv, Hv, D, Dv, temp_coef,
-                    temp_every, v_mode, v_keep, v_lambda, write_kv, status);
+    const bool quads = D % 4 == 0 && Dv % 4 == 0 && ldp % 4 == 0 && ldq % 4 == 0 &&
+                       (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)v_keep) & 15) == 0;
+    const int per = quads ? 4 * ITEMS : ITEMS;
+    dim3 grid(n_tokens, (items + per - 1) / per);
+#define LGML_QKV(KERNEL, T)                                                                                                                         \
+    lgml_launch(KERNEL<T>, grid, ITEMS, 0, stream, proj, ldp, (T *)q_out, ldq, positions, seq_of_token, block_table, max_blocks, (T *)k_pages,     \
+                (T *)v_pages, n_pages, page_size, H, Hkv, Hv, D, Dv, temp_coef, temp_every, v_mode, v_keep, v_lambda, write_kv, status)
+    if (dtype == LGML_F32 && quads) LGML_QKV(sink_qkv_store_quads_kernel, float);
+    else if (dtype == LGML_F32) LGML_QKV(sink_qkv_store_kernel, float);
+    else if (dtype == LGML_BF16 && quads) LGML_QKV(sink_qkv_store_quads_kernel, __nv_bfloat16);
+    else if (dtype == LGML_BF16) LGML_QKV(sink_qkv_store_kernel, __nv_bfloat16);
     else
         LGML_FAIL("sink_qkv_store: unknown type %d", dtype);
+#undef LGML_QKV
     return lgml_launch_status("sink_qkv_store");
 }
 

@@ -142,6 +142,8 @@ struct Params {
     // A grouped product (null: none): the rows of A come in tiles of BM rows, tile t of them against the rows
     // group[3 t] * group_rows_b ... of B (the matrices of several experts stacked); group[3 group_max_tiles] says
     // how many tiles there are.  The list is written on the device by the kernel ahead, so it is read after the wait.
+    // With `transposed` the weights are the tile's rows: tiles of BN rows of B (tokens) come one per list entry, tile t of them
+    // against the rows group[3 t] * group_rows_b ... of A.
     const int *group;
     int group_max_tiles, group_rows_b;
 };
@@ -297,7 +299,7 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_tcgen05_kernel(const __grid_c
     const int kb1 = min(kb0 + p.kb_per_split, p.k_blocks);
     const int n_kb = max(kb1 - kb0, 0);
     const bool grouped = p.group != nullptr;
-    int ta = p.tiles_a;                // tiles along A: fewer in a grouped product, once its tile list is there
+    int ta = p.tiles_a;                // tiles along A (in a grouped product along the tokens: fewer, once its tile list is there)
     int n_tiles = ta * p.tiles_b;
     constexpr uint32_t ACC_COLS = BN <= 32 ? 32 : (BN <= 64 ? 64 : (BN <= 128 ? 128 : 256));
     constexpr uint32_t TMEM_COLS = ACC_COLS * NACC;
@@ -330,8 +332,12 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_tcgen05_kernel(const __grid_c
             // stages at once, then wait for the earlier kernels, then fetch the activations.
             if (grouped) {          // which weights a tile reads is in the list the kernel ahead wrote: nothing is fetched before the wait
                 pdl_wait();
-                ta = min(p.tiles_a, act_load(p.group + 3 * p.group_max_tiles));
-                n_tiles = ta * p.tiles_b;
+                if (p.transposed) {
+                    n_tiles = ta * min(p.tiles_b, act_load(p.group + 3 * p.group_max_tiles));
+                } else {
+                    ta = min(p.tiles_a, act_load(p.group + 3 * p.group_max_tiles));
+                    n_tiles = ta * p.tiles_b;
+                }
             }
             const int first = blockIdx.x;
             const int pre = (!grouped && first < n_tiles) ? min(n_kb, STAGES) : 0;
@@ -354,7 +360,9 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_tcgen05_kernel(const __grid_c
             bool ok = true;
             for (int tile = first; tile < n_tiles && ok; tile += gridDim.x) {
                 const int tile_a = tile % ta, tile_b = tile / ta;
-                const int b_row = tile_b * BN + (grouped ? act_load(p.group + 3 * tile_a) * p.group_rows_b : 0);
+                // where the stacked matrices of this tile's group begin
+                const int off = grouped ? act_load(p.group + 3 * (p.transposed ? tile_b : tile_a)) * p.group_rows_b : 0;
+                const int a_row = tile_a * BM + (p.transposed ? off : 0), b_row = tile_b * BN + (p.transposed ? 0 : off);
                 for (int i = (tile == first ? pre : 0); i < n_kb; ++i, ++it) {
                     const int s = it % STAGES;
                     if (!mbar_wait(&empty_bar[s], ((it / STAGES) - 1) & 1, abort_flag, p.status) || *abort_flag) {
@@ -364,7 +372,7 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_tcgen05_kernel(const __grid_c
                     uint8_t *a_dst = tiles + (size_t)s * Smem<BN>::STAGE_BYTES;
                     uint8_t *b_dst = a_dst + Smem<BN>::A_BYTES;
                     mbar_expect_tx(&full_bar[s], Smem<BN>::STAGE_BYTES);
-                    tma_load_2d(a_dst, &map_a, (kb0 + i) * BK, tile_a * BM, &full_bar[s]);
+                    tma_load_2d(a_dst, &map_a, (kb0 + i) * BK, a_row, &full_bar[s]);
                     tma_load_2d(b_dst, &map_b, (kb0 + i) * BK, b_row, &full_bar[s]);
                     issued = it + 1;
                 }
@@ -388,8 +396,12 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_tcgen05_kernel(const __grid_c
             int it = 0, j = 0;
             if (grouped) {
                 pdl_wait();
-                ta = min(p.tiles_a, act_load(p.group + 3 * p.group_max_tiles));
-                n_tiles = ta * p.tiles_b;
+                if (p.transposed) {
+                    n_tiles = ta * min(p.tiles_b, act_load(p.group + 3 * p.group_max_tiles));
+                } else {
+                    ta = min(p.tiles_a, act_load(p.group + 3 * p.group_max_tiles));
+                    n_tiles = ta * p.tiles_b;
+                }
             }
             for (int tile = blockIdx.x; tile < n_tiles && ok; tile += gridDim.x, ++j) {
                 const int acc = j % NACC;
@@ -426,8 +438,12 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_tcgen05_kernel(const __grid_c
         const bool f32 = p.out_f32 || p.split_stride != 0;
         int j = 0;
         if (grouped) {
-            ta = min(p.tiles_a, act_load(p.group + 3 * p.group_max_tiles));
-            n_tiles = ta * p.tiles_b;
+            if (p.transposed) {
+                n_tiles = ta * min(p.tiles_b, act_load(p.group + 3 * p.group_max_tiles));
+            } else {
+                ta = min(p.tiles_a, act_load(p.group + 3 * p.group_max_tiles));
+                n_tiles = ta * p.tiles_b;
+            }
         }
         for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x, ++j) {
         const int tile_a = tile % ta, tile_b = tile / ta;
@@ -1099,8 +1115,11 @@ LGML_API int lgml_gemm_tcgen05_glu_clamped(const void *x, const void *w, void *y
 // [.., N / 2] with swiglu = 1 (rows of w in (gate, up) pairs, y = silu(gate) * up) or 3 (the same pairs, the clamped activation with
 // act_alpha and act_limit).  The single-CTA persistent kernel with
 // 128 x 256 tiles (128 x 128 where those would be fewer than the SMs); rows of a tile past an expert's last feature are computed from the next expert's rows and not stored.
-LGML_API int lgml_gemm_tcgen05_grouped_act(const void *x, const void *w, void *y, int y_f32, int max_tiles, int N, int K, int n_groups, int ldy,
-                                           const int *group, int swiglu, float act_alpha, float act_limit, int *status, cudaStream_t stream) {
+// tile_rows: 128, or for few rows a group 16, 32 or 64 (x and y then have max_tiles * tile_rows rows): the weights are the tile's 128
+// rows and the tokens its columns, two CTAs an SM, so that what is streamed is the weights and not padding.
+LGML_API int lgml_gemm_tcgen05_grouped_tiles(const void *x, const void *w, void *y, int y_f32, int max_tiles, int tile_rows, int N, int K, int n_groups,
+                                             int ldy, const int *group, int swiglu, float act_alpha, float act_limit, int *status, cudaStream_t stream) {
+    LGML_REQUIRE(tile_rows == 16 || tile_rows == 32 || tile_rows == 64 || tile_rows == BM, "gemm_tcgen05_grouped: tiles of %d rows", tile_rows);
     LGML_REQUIRE(max_tiles > 0 && N > 0 && K > 0 && n_groups > 0 && group != nullptr, "gemm_tcgen05_grouped: bad sizes");
     LGML_REQUIRE(swiglu >= 0 && swiglu <= 3, "gemm_tcgen05_grouped: unknown epilogue %d", swiglu);
     const bool paired = swiglu == 1 || swiglu == 3;
@@ -1119,6 +1138,23 @@ LGML_API int lgml_gemm_tcgen05_grouped_act(const void *x, const void *w, void *y
     p.status = status;
     p.swiglu = swiglu;
     p.act_alpha = act_alpha, p.act_limit = act_limit;
+    if (tile_rows != BM) {
+        p.transposed = 1;
+        p.rows_a = N;
+        p.rows_b = max_tiles * tile_rows;
+        p.tiles_a = (N + BM - 1) / BM;
+        p.tiles_b = max_tiles;
+        p.group = group, p.group_max_tiles = max_tiles, p.group_rows_b = N;
+        CUtensorMap ma, mb;
+        int rc;
+        if ((rc = make_map(&ma, w, (long long)n_groups * N, K, K, BM))) return rc;
+        if ((rc = make_map(&mb, x, (long long)max_tiles * tile_rows, K, K, tile_rows))) return rc;
+        const long long n_tiles = (long long)p.tiles_a * p.tiles_b;
+        dim3 grid((unsigned)(n_tiles < 2 * 148 ? n_tiles : 2 * 148), 1, 1);
+        if (tile_rows == 16) return launch<16, 6, 2>(ma, mb, p, grid, stream);
+        if (tile_rows == 32) return launch<32, 5, 2>(ma, mb, p, grid, stream);
+        return launch<64, 4, 2>(ma, mb, p, grid, stream);
+    }
     p.transposed = 0;
     p.rows_a = max_tiles * BM;
     p.rows_b = N;
@@ -1135,6 +1171,11 @@ LGML_API int lgml_gemm_tcgen05_grouped_act(const void *x, const void *w, void *y
     dim3 grid(n_tiles < 148 ? n_tiles : 148, 1, 1);
     if (bn == 128) return launch<128, 6, 1>(ma, mb, p, grid, stream);
     return launch<256, 4, 2>(ma, mb, p, grid, stream);
+}
+
+LGML_API int lgml_gemm_tcgen05_grouped_act(const void *x, const void *w, void *y, int y_f32, int max_tiles, int N, int K, int n_groups, int ldy,
+                                           const int *group, int swiglu, float act_alpha, float act_limit, int *status, cudaStream_t stream) {
+    return lgml_gemm_tcgen05_grouped_tiles(x, w, y, y_f32, max_tiles, BM, N, K, n_groups, ldy, group, swiglu, act_alpha, act_limit, status, stream);
 }
 
 LGML_API int lgml_gemm_tcgen05_grouped(const void *x, const void *w, void *y, int y_f32, int max_tiles, int N, int K, int n_groups, int ldy,

@@ -440,7 +440,7 @@ namespace {
 constexpr int G_TM = 128, G_TN = 128, G_TK = 32, G_LD = G_TK + 8;
 
 __global__ void __launch_bounds__(1024) moe_group_kernel(const int *__restrict__ ids, int n_rows, int X, int *__restrict__ rows,
-                                                         int *__restrict__ tiles, int *__restrict__ n_tiles, int max_tiles) {
+                                                         int *__restrict__ tiles, int *__restrict__ n_tiles, int max_tiles, int tm) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ int sh[];         // counts[X], first[X], cursor[X], tile0[X]
@@ -459,7 +459,7 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int *__restrict__
         for (int e = 0; e < X; ++e) {
             first[e] = at, tile0[e] = tl;
             at += counts[e];
-            tl += (counts[e] + G_TM - 1) / G_TM;
+            tl += (counts[e] + tm - 1) / tm;
         }
         *n_tiles = tl < max_tiles ? tl : max_tiles;
     }
@@ -471,13 +471,13 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(const int *__restrict__
         rows[first[e] + atomicAdd(&cursor[e], 1)] = r;
     }
     for (int e = threadIdx.x; e < X; e += blockDim.x) {
-        const int nt = (counts[e] + G_TM - 1) / G_TM;
+        const int nt = (counts[e] + tm - 1) / tm;
         for (int i = 0; i < nt; ++i) {
             const int tl = tile0[e] + i;
             if (tl >= max_tiles) break;
             tiles[tl * 3] = e;
-            tiles[tl * 3 + 1] = first[e] + i * G_TM;
-            tiles[tl * 3 + 2] = min(G_TM, counts[e] - i * G_TM);
+            tiles[tl * 3 + 1] = first[e] + i * tm;
+            tiles[tl * 3 + 2] = min(tm, counts[e] - i * tm);
         }
     }
 }
@@ -647,7 +647,7 @@ LGML_API int lgml_moe_experts_grouped(const void *h, int ldh, const int *ids, co
     LGML_REQUIRE(max_tiles >= need, "moe_experts_grouped: room for %d tiles, %d may be needed", max_tiles, need);
     int *n_tiles = tiles + 3 * max_tiles;
     if (need_smem(moe_group_kernel, sizeof(int) * 4 * (size_t)X, "moe_experts_grouped")) return -1;
-    lgml_launch(moe_group_kernel, 1, 1024, sizeof(int) * 4 * (size_t)X, stream, ids, n_rows, X, rows, tiles, n_tiles, max_tiles);
+    lgml_launch(moe_group_kernel, 1, 1024, sizeof(int) * 4 * (size_t)X, stream, ids, n_rows, X, rows, tiles, n_tiles, max_tiles, G_TM);
     dim3 g0(max_tiles, (F + G_TN / 2 - 1) / (G_TN / 2)), g1(max_tiles, (E + G_TN - 1) / G_TN);
     LGML_REQUIRE(g0.y <= 65535 && g1.y <= 65535, "moe_experts_grouped: too many columns");
     const size_t smem = (size_t)G_STAGES * G_STAGE_ELEMS * 2 + sizeof(int) * G_TM;
@@ -672,10 +672,10 @@ LGML_API int lgml_moe_experts_grouped(const void *h, int ldh, const int *ids, co
 namespace {
 __global__ void __launch_bounds__(128) moe_gather_rows_kernel(const __nv_bfloat16 *__restrict__ h, int ldh, const int *__restrict__ rows,
                                                               const int *__restrict__ tiles, int max_tiles, __nv_bfloat16 *__restrict__ a_perm,
-                                                              int *__restrict__ pos, int E, int top) {
+                                                              int *__restrict__ pos, int E, int top, int tm) {
     pdl_trigger();
     pdl_wait();
-    const int pr = blockIdx.x, tile = pr / G_TM, i = pr - tile * G_TM;
+    const int pr = blockIdx.x, tile = pr / tm, i = pr - tile * tm;
     if (tile >= act_load(tiles + 3 * max_tiles) || i >= act_load(tiles + 3 * tile + 2)) return;
     const int r = act_load(rows + act_load(tiles + 3 * tile + 1) + i);
     if (threadIdx.x == 0) pos[r] = pr;
@@ -732,25 +732,37 @@ __global__ void __launch_bounds__(256) moe_weighted_sum_kernel(const float *__re
 }
 }  // namespace
 
+// The rows of a tile for n_rows (token, expert) rows over X experts: 128 (the tokens are the product's tile rows), or, where an expert gets few
+// rows, 16, 32 or 64 (the weights are the tile's rows then).
+static __host__ __device__ inline int tile_rows_of(int n_rows, int X) {
+    const int per = (n_rows + X - 1) / (X > 0 ? X : 1);
+    if (n_rows <= 16 || per <= 8) return 16;
+    if (n_rows <= 32 || per <= 20) return 32;
+    if (n_rows <= 64 || per <= 44) return 64;
+    return G_TM;
+}
+LGML_API int lgml_moe_tile_rows(int n_rows, int X) { return tile_rows_of(n_rows, X); }
+
 // rows int32 [n top]; tiles int32 [3 max_tiles + 1] (the last word: the number of tiles)
-LGML_API int lgml_moe_group_rows(const int *ids, int *rows, int *tiles, int max_tiles, int n_tokens, int X, int top, cudaStream_t stream) {
+LGML_API int lgml_moe_group_rows(const int *ids, int *rows, int *tiles, int max_tiles, int tile_rows, int n_tokens, int X, int top, cudaStream_t stream) {
+    LGML_REQUIRE(tile_rows > 0, "moe_group_rows: bad tile");
     LGML_REQUIRE(n_tokens >= 0 && X > 0 && X <= 8192 && top > 0, "moe_group_rows: bad sizes");
     const int n_rows = n_tokens * top;
-    const int need = (n_rows + G_TM - 1) / G_TM + (X < n_rows ? X : n_rows);
+    const int need = (n_rows + tile_rows - 1) / tile_rows + (X < n_rows ? X : n_rows);
     LGML_REQUIRE(max_tiles >= need, "moe_group_rows: room for %d tiles, %d may be needed", max_tiles, need);
     if (n_tokens == 0) return 0;
     if (need_smem(moe_group_kernel, sizeof(int) * 4 * (size_t)X, "moe_group_rows")) return -1;
-    lgml_launch(moe_group_kernel, 1, 1024, sizeof(int) * 4 * (size_t)X, stream, ids, n_rows, X, rows, tiles, tiles + 3 * max_tiles, max_tiles);
+    lgml_launch(moe_group_kernel, 1, 1024, sizeof(int) * 4 * (size_t)X, stream, ids, n_rows, X, rows, tiles, tiles + 3 * max_tiles, max_tiles, tile_rows);
     return lgml_launch_status("moe_group_rows");
 }
 
-// a_perm bfloat16 [max_tiles 128, E]; pos int32 [n top]
-LGML_API int lgml_moe_gather_rows(const void *h, int ldh, const int *rows, const int *tiles, int max_tiles, void *a_perm, int *pos, int E, int top,
+// a_perm bfloat16 [max_tiles tile_rows, E]; pos int32 [n top]
+LGML_API int lgml_moe_gather_rows(const void *h, int ldh, const int *rows, const int *tiles, int max_tiles, int tile_rows, void *a_perm, int *pos, int E, int top,
                                   cudaStream_t stream) {
-    LGML_REQUIRE(max_tiles > 0 && E > 0 && E % 8 == 0 && ldh % 8 == 0 && top > 0, "moe_gather_rows: bad sizes");
+    LGML_REQUIRE(max_tiles > 0 && tile_rows > 0 && E > 0 && E % 8 == 0 && ldh % 8 == 0 && top > 0, "moe_gather_rows: bad sizes");
     LGML_REQUIRE((((uintptr_t)h | (uintptr_t)a_perm) & 15) == 0, "moe_gather_rows: operands must be 16-byte aligned");
-    lgml_launch(moe_gather_rows_kernel, max_tiles * G_TM, 128, 0, stream, (const __nv_bfloat16 *)h, ldh, rows, tiles, max_tiles, (__nv_bfloat16 *)a_perm, pos,
-                E, top);
+    lgml_launch(moe_gather_rows_kernel, max_tiles * tile_rows, 128, 0, stream, (const __nv_bfloat16 *)h, ldh, rows, tiles, max_tiles, (__nv_bfloat16 *)a_perm, pos,
+                E, top, tile_rows);
     return lgml_launch_status("moe_gather_rows");
 }
 
@@ -774,11 +786,12 @@ LGML_API int lgml_moe_weighted_sum(const float *y, const int *pos, const float *
 
 // ---------------------------------------------------------------------------------------------
 // Experts that stand in a table: a token's id names them, so what runs is known before the first layer.  One launch per step
-// does it for the tables of all layers, a block a table: the experts of every (token, slot) row, the tiles of 128 rows of
-// one expert, and the row's place among the tiles (its tile times 128 + its place in it).
-//   desc int32 [n_tables, 3]: experts X, slots a token `top`, first entry of the table in `tables` ([vocab, top] each)
+// does it for the tables of all layers, a block a table: the experts of every (token, slot) row, the tiles of rows of one
+// expert (of `tile_rows` rows: desc says so), and the row's place among the tiles (its tile times the tile's rows + its place in it).
+//   desc int32 [n_tables, 3]: experts X, slots a token `top`, first entry of the table in `tables` ([vocab, top] each);
+//   a tile has lgml_moe_tile_rows(n top, X) rows
 //   out: per table, one behind the other: ids [n top] | places [n top] | tiles [3 max_tiles] | number of tiles, with
-//   max_tiles = ceil(n top / 128) + min(X, n top)
+//   max_tiles = ceil(n top / tile rows) + min(X, n top)
 // ---------------------------------------------------------------------------------------------
 namespace {
 __global__ void __launch_bounds__(1024) table_route_kernel(const int *__restrict__ token_ids, int n, int vocab, const int *__restrict__ tables,
@@ -793,14 +806,15 @@ __global__ void __launch_bounds__(1024) table_route_kernel(const int *__restrict
         long long b = 0;
         for (int l = 0; l < (int)blockIdx.x; ++l) {
             const int rows = n * desc[3 * l + 1];
-            b += 2LL * rows + 3LL * ((rows + G_TM - 1) / G_TM + min(desc[3 * l], rows)) + 1;
+            const int m = tile_rows_of(rows, desc[3 * l]);
+            b += 2LL * rows + 3LL * ((rows + m - 1) / m + min(desc[3 * l], rows)) + 1;
         }
         base_s = b;
     }
     for (int e = threadIdx.x; e < X; e += blockDim.x) counts[e] = 0, cursor[e] = 0;
     pdl_wait();
     __syncthreads();
-    const int rows = n * top, max_tiles = (rows + G_TM - 1) / G_TM + min(X, rows);
+    const int rows = n * top, tm = tile_rows_of(rows, X), max_tiles = (rows + tm - 1) / tm + min(X, rows);
     int *ids = out + base_s, *pos = ids + rows, *tiles = pos + rows;
     for (int r = threadIdx.x; r < rows; r += blockDim.x) {
         const int t = r / top, id = min(max(act_load(token_ids + t), 0), vocab - 1);      // the embedding kernel has flagged an id outside the vocabulary
@@ -813,7 +827,7 @@ __global__ void __launch_bounds__(1024) table_route_kernel(const int *__restrict
         int tl = 0;
         for (int e = 0; e < X; ++e) {
             tile0[e] = tl;
-            tl += (counts[e] + G_TM - 1) / G_TM;
+            tl += (counts[e] + tm - 1) / tm;
         }
         tiles[3 * max_tiles] = tl;
     }
@@ -821,12 +835,12 @@ __global__ void __launch_bounds__(1024) table_route_kernel(const int *__restrict
     for (int r = threadIdx.x; r < rows; r += blockDim.x) {
         const int e = ids[r];           // this thread wrote it
         const int c = atomicAdd(&cursor[e], 1);
-        pos[r] = (tile0[e] + c / G_TM) * G_TM + c % G_TM;
+        pos[r] = (tile0[e] + c / tm) * tm + c % tm;
     }
     for (int e = threadIdx.x; e < X; e += blockDim.x)
-        for (int i = 0; i * G_TM < counts[e]; ++i) {
+        for (int i = 0; i * tm < counts[e]; ++i) {
             int *tl = tiles + 3 * (tile0[e] + i);
-            tl[0] = e, tl[1] = 0, tl[2] = min(G_TM, counts[e] - i * G_TM);
+            tl[0] = e, tl[1] = 0, tl[2] = min(tm, counts[e] - i * tm);
         }
 }
 }  // namespace

@@ -11,8 +11,8 @@
 //
 //   rglru_step    one token a request: convolution, both gates, recurrence and output in one kernel, a block per (8 tokens, 32 channels)
 //   rglru_conv    the convolution alone for longer portions; also brings the ring up to date
-//   rglru_gates   a_t and the pushed term sqrt(1 - a^2) i u for many tokens: in bfloat16 on tensor cores with u in three
-//                 bfloat16 pieces (24 bits: what is multiplied is the float32 number), else as products of 8 rows
+//   rglru_gates   a_t and the pushed term sqrt(1 - a^2) i u of longer portions: on tensor cores with u in three bfloat16
+//                 pieces (24 bits: what is multiplied is the float32 number), else as products of 8 rows
 //   rglru_scan    S_t = a_t S_(t-1) + push_t and the output, a thread a channel of a request
 //   rglru_chunks  the same for long portions in three passes: every chunk's (product of a, scan from zero), the chain over
 //                 a request's chunks, every chunk again from its true start
@@ -56,32 +56,14 @@ __device__ __forceinline__ float conv_at(const float *__restrict__ x, int ldx, c
     return v;
 }
 
-// ---- one token a request ---------------------------------------------------------------------------
-template <typename T, typename TO>
-__global__ void __launch_bounds__(256) rglru_step_kernel(const float *__restrict__ proj, int ldp, const float *__restrict__ conv_w,
-                                                         const float *__restrict__ conv_b, float *__restrict__ state, long long state_ld,
-                                                         const int *__restrict__ slots, const int *__restrict__ positions, const T *__restrict__ ra,
-                                                         const float *__restrict__ ra_b, const T *__restrict__ ri, const float *__restrict__ ri_b,
-                                                         const float *__restrict__ sp8, TO *__restrict__ out, int n, int C, int P, int taps, int lanes, int vec) {
-    pdl_trigger();
-    pdl_wait();
-    extern __shared__ __align__(16) float us[];        // u of up to 8 tokens, the whole part of the channels
-    const int ldu = (P + 3) & ~3;
-    const int b = blockIdx.y, t0 = blockIdx.z * NT, nt = min(NT, n - t0);
-    for (int e = threadIdx.x; e < NT * ldu; e += blockDim.x) {
-        const int j = e / ldu, k = e - j * ldu;
-        float u = 0.f;
-        if (j < nt && k < P) {
-            const int t = t0 + j, c = b * P + k;
-            const float *ring = state + (size_t)slots[t] * state_ld + C;
-            u = conv_at(proj, ldp, conv_w, conv_b[c], ring, C, taps, t, t, positions[t], c);
-        }
-        us[e] = u;
-    }
-    __syncthreads();
+// The logits of both gates for the 8 tokens in `us` and the 32 channels from k_out on of part b: zs [2][NT][CH].  A warp takes four
+// channels, lane groups of `lanes` a channel at a time.
+template <typename T>
+__device__ __forceinline__ void gate_logits(const T *__restrict__ ra, const T *__restrict__ ri, const float *us, int ldu, int b, int P, int k_out, int lanes, int vec,
+                                            float *zs) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, per = 32 / lanes, sub = lane % lanes;
     for (int j0 = 0; j0 < 4; j0 += per) {
-        const int q = j0 + lane / lanes, k = blockIdx.x * CH + warp * 4 + q;       // this lane group's channel of the part
+        const int q = j0 + lane / lanes, ch = warp * 4 + q, k = k_out + ch;       // this lane group's channel of the part
         const bool mine = q < 4 && k < P;
         float zr[NT], zi[NT];
 #pragma unroll
@@ -92,31 +74,138 @@ __global__ void __launch_bounds__(256) rglru_step_kernel(const float *__restrict
         }
         few_rows_reduce<NT>(zr, lanes);
         few_rows_reduce<NT>(zi, lanes);
-        if (!mine) continue;
-        const int c = b * P + k;
-        // the lanes of a channel share its tokens
+        if (mine && sub == 0) {
 #pragma unroll
-        for (int j = 0; j < NT; ++j) {
-            if (j % lanes != sub || j >= nt) continue;
-            const int t = t0 + j;
-            float *row = state + (size_t)slots[t] * state_ld;
-            float a, push;
-            gate_pair(zr[j] + ra_b[c], zi[j] + ri_b[c], sp8[c], us[j * ldu + k], a, push);
-            const float S = fmaf(a, act_load(row + c), push);
-            row[c] = S;
-            out[(size_t)t * C + c] = from_f32<TO>(S * gelu_tanh(act_load(proj + (size_t)t * ldp + C + c)));
-            if (taps > 1) row[C + (size_t)(positions[t] % taps) * C + c] = act_load(proj + (size_t)t * ldp + c);
+            for (int j = 0; j < NT; ++j) zs[j * CH + ch] = zr[j], zs[(NT + j) * CH + ch] = zi[j];
         }
     }
 }
 
+// ---- one token a request ---------------------------------------------------------------------------
+// TAPS: the taps at compile time (0: any number).
+template <typename T, typename TO, int TAPS>
+__global__ void __launch_bounds__(256) rglru_step_kernel(const float *__restrict__ proj, int ldp, const float *__restrict__ conv_w,
+                                                         const float *__restrict__ conv_b, float *__restrict__ state, long long state_ld,
+                                                         const int *__restrict__ slots, const int *__restrict__ positions, const T *__restrict__ ra,
+                                                         const float *__restrict__ ra_b, const T *__restrict__ ri, const float *__restrict__ ri_b,
+                                                         const float *__restrict__ sp8, TO *__restrict__ out, int n, int C, int P, int any_taps, int lanes,
+                                                         int vec) {
+    pdl_trigger();
+    // the gates' matrices depend on no earlier kernel: have this block's rows of them in L2 by the time it may go on
+    {
+        const size_t first = ((size_t)blockIdx.y * P + blockIdx.x * CH) * P, bytes = (size_t)min(CH, P - (int)blockIdx.x * CH) * P * sizeof(T);
+        for (size_t o = (size_t)threadIdx.x * 128; o < bytes; o += (size_t)blockDim.x * 128) {
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char *>(ra + first) + o));
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char *>(ri + first) + o));
+        }
+    }
+    pdl_wait();
+    extern __shared__ __align__(16) float us[];        // u of up to 8 tokens, the whole part of the channels
+    __shared__ float zs[2 * NT * CH];
+    const int ldu = (P + 3) & ~3, taps = TAPS > 0 ? TAPS : any_taps;
+    const int b = blockIdx.y, t0 = blockIdx.z * NT, nt = min(NT, n - t0);
+    if (TAPS > 0) {
+        // a thread a channel: the inputs of all its tokens are in flight together
+        const float *ring[NT];
+        int pos[NT];
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+            const int t = t0 + min(j, nt - 1);
+            ring[j] = state + (size_t)slots[t] * state_ld + C, pos[j] = positions[t];
+        }
+        for (int k = threadIdx.x; k < ldu; k += blockDim.x) {
+            const int c = b * P + k;
+            float in[NT][TAPS > 0 ? TAPS : 1], w[TAPS > 0 ? TAPS : 1];
+#pragma unroll
+            for (int j = 0; j < NT; ++j)
+#pragma unroll
+                for (int i = 0; i < TAPS; ++i) {
+                    const int back = TAPS - 1 - i;
+                    const bool there = j < nt && k < P && pos[j] >= back;
+                    in[j][i] = !there ? 0.f : (back == 0 ? act_load(proj + (size_t)(t0 + j) * ldp + c) : act_load(ring[j] + (size_t)((pos[j] - back) % TAPS) * C + c));
+                }
+#pragma unroll
+            for (int i = 0; i < TAPS; ++i) w[i] = k < P ? __ldg(conv_w + (size_t)i * C + c) : 0.f;
+            const float bias = k < P ? __ldg(conv_b + c) : 0.f;
+#pragma unroll
+            for (int j = 0; j < NT; ++j) {
+                float v = bias;
+#pragma unroll
+                for (int i = 0; i < TAPS; ++i) v = fmaf(w[i], in[j][i], v);
+                us[j * ldu + k] = j < nt ? v : 0.f;
+            }
+        }
+    } else {
+        for (int e = threadIdx.x; e < NT * ldu; e += blockDim.x) {
+            const int j = e / ldu, k = e - j * ldu;
+            float u = 0.f;
+            if (j < nt && k < P) {
+                const int t = t0 + j, c = b * P + k;
+                u = conv_at(proj, ldp, conv_w, conv_b[c], state + (size_t)slots[t] * state_ld + C, C, taps, t, t, positions[t], c);
+            }
+            us[e] = u;
+        }
+    }
+    // a thread finishes one channel of one token: what it needs beside the logits is on its way meanwhile
+    const int my_j = threadIdx.x / CH, my_k = blockIdx.x * CH + threadIdx.x % CH;
+    const bool mine = my_j < nt && my_k < P;
+    const int t = t0 + my_j, c = b * P + my_k;
+    float *row = nullptr;
+    float s_old = 0.f, y = 0.f, x_in = 0.f;
+    int pos_t = 0;
+    if (mine) {
+        row = state + (size_t)slots[t] * state_ld, pos_t = positions[t];
+        s_old = act_load(row + c), y = act_load(proj + (size_t)t * ldp + C + c), x_in = act_load(proj + (size_t)t * ldp + c);
+    }
+    __syncthreads();
+    gate_logits<T>(ra, ri, us, ldu, b, P, blockIdx.x * CH, lanes, vec, zs);
+    __syncthreads();
+    if (!mine) return;
+    float a, push;
+    gate_pair(zs[my_j * CH + threadIdx.x % CH] + ra_b[c], zs[(NT + my_j) * CH + threadIdx.x % CH] + ri_b[c], sp8[c], us[my_j * ldu + my_k], a, push);
+    const float S = fmaf(a, s_old, push);
+    row[c] = S;
+    out[(size_t)t * C + c] = from_f32<TO>(S * gelu_tanh(y));
+    if (taps > 1) row[C + (size_t)(pos_t % taps) * C + c] = x_in;
+}
+
+// A convolved input on its way out: a float32 number, or three bfloat16 numbers whose sum it is (8 + 8 + 8 bits), in three planes
+// of `plane` numbers (what the gates' tensor-core form multiplies).
+struct AsFloat {
+    float *u;
+    __device__ __forceinline__ void put(size_t i, float v) const { u[i] = v; }
+    __device__ __forceinline__ void put4(size_t i, const float4 &v) const { *reinterpret_cast<float4 *>(u + i) = v; }
+};
+struct AsPieces {
+    __nv_bfloat16 *u;
+    size_t plane;
+    __device__ __forceinline__ void put(size_t i, float v) const {
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {
+            const __nv_bfloat16 h = __float2bfloat16_rn(v);
+            u[k * plane + i] = h;
+            v -= __bfloat162float(h);
+        }
+    }
+    __device__ __forceinline__ void put4(size_t i, const float4 &v) const {
+        float x[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(x[0], x[1]), hi = __floats2bfloat162_rn(x[2], x[3]);
+            *reinterpret_cast<uint2 *>(u + k * plane + i) = make_uint2(*reinterpret_cast<unsigned *>(&lo), *reinterpret_cast<unsigned *>(&hi));
+            x[0] -= __low2float(lo), x[1] -= __high2float(lo), x[2] -= __low2float(hi), x[3] -= __high2float(hi);
+        }
+    }
+};
+
 // ---- the convolution of longer portions ----------------------------------------------------------------
 // A thread takes one channel of one token.  The thread of a request's first token computes every token that reaches into
 // the ring and then writes the step's last taps - 1 inputs there; nobody else touches those floats.
+template <typename OUT>
 __global__ void __launch_bounds__(256) rglru_conv_kernel(const float *__restrict__ proj, int ldp, const float *__restrict__ conv_w,
                                                          const float *__restrict__ conv_b, float *__restrict__ state, long long state_ld,
                                                          const int *__restrict__ seq_of_token, const int *__restrict__ seq_start,
-                                                         const int *__restrict__ slots, const int *__restrict__ positions, float *__restrict__ u, int n, int C,
+                                                         const int *__restrict__ slots, const int *__restrict__ positions, const OUT u, int n, int C,
                                                          int taps) {
     pdl_trigger();
     pdl_wait();
@@ -128,22 +217,22 @@ __global__ void __launch_bounds__(256) rglru_conv_kernel(const float *__restrict
         if (t == t0) {
             float *ring = state + (size_t)slots[s] * state_ld + C;
             const int t1 = seq_start[s + 1], last = min(t1, t0 + max(taps - 1, 1)), pos0 = positions[t0];
-            for (int i = t0; i < last; ++i) u[(size_t)i * C + c] = conv_at(proj, ldp, conv_w, bias, ring, C, taps, i, t0, pos0 + i - t0, c);
+            for (int i = t0; i < last; ++i) u.put((size_t)i * C + c, conv_at(proj, ldp, conv_w, bias, ring, C, taps, i, t0, pos0 + i - t0, c));
             if (taps > 1)
                 for (int i = max(t0, t1 - (taps - 1)); i < t1; ++i) ring[(size_t)((pos0 + i - t0) % taps) * C + c] = act_load(proj + (size_t)i * ldp + c);
         } else if (t - t0 >= taps - 1) {
-            u[it] = conv_at(proj, ldp, conv_w, bias, nullptr, C, taps, t, t0, positions[t], c);
+            u.put(it, conv_at(proj, ldp, conv_w, bias, nullptr, C, taps, t, t0, positions[t], c));
         }
     }
 }
 
 // The same for many tokens, four channels a thread and four tokens in a row (a row of inputs is read once for four results): tokens
 // 4 i .. 4 i + 3 of the step, whichever requests they belong to.  Taps at compile time, C a multiple of 4.
-template <int TAPS>
+template <int TAPS, typename OUT>
 __global__ void __launch_bounds__(256) rglru_conv_runs_kernel(const float *__restrict__ proj, int ldp, const float *__restrict__ conv_w,
                                                               const float *__restrict__ conv_b, float *__restrict__ state, long long state_ld,
                                                               const int *__restrict__ seq_of_token, const int *__restrict__ seq_start,
-                                                              const int *__restrict__ slots, const int *__restrict__ positions, float *__restrict__ u, int n,
+                                                              const int *__restrict__ slots, const int *__restrict__ positions, const OUT u, int n,
                                                               int C) {
     pdl_trigger();
     pdl_wait();
@@ -174,13 +263,13 @@ __global__ void __launch_bounds__(256) rglru_conv_runs_kernel(const float *__res
                     v.x = fmaf(w[j].x, in[i + j].x, v.x), v.y = fmaf(w[j].y, in[i + j].y, v.y);
                     v.z = fmaf(w[j].z, in[i + j].z, v.z), v.w = fmaf(w[j].w, in[i + j].w, v.w);
                 }
-                *reinterpret_cast<float4 *>(u + (size_t)t * C + c) = v;
+                u.put4((size_t)t * C + c, v);
             } else if (t == t0) {
                 float *ring = state + (size_t)slots[s] * state_ld + C;
                 const int t1 = seq_start[s + 1], last = min(t1, t0 + max(TAPS - 1, 1)), pos0 = positions[t0];
                 for (int e = 0; e < 4; ++e) {
                     for (int k = t0; k < last; ++k)
-                        u[(size_t)k * C + c + e] = conv_at(proj, ldp, conv_w, __ldg(conv_b + c + e), ring, C, TAPS, k, t0, pos0 + k - t0, c + e);
+                        u.put((size_t)k * C + c + e, conv_at(proj, ldp, conv_w, __ldg(conv_b + c + e), ring, C, TAPS, k, t0, pos0 + k - t0, c + e));
                     if (TAPS > 1)
                         for (int k = max(t0, t1 - (TAPS - 1)); k < t1; ++k)
                             ring[(size_t)((pos0 + k - t0) % TAPS) * C + c + e] = act_load(proj + (size_t)k * ldp + c + e);
@@ -199,6 +288,7 @@ __global__ void __launch_bounds__(256) rglru_gates_rows_kernel(const float *__re
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(16) float us[];
+    __shared__ float zs[2 * NT * CH];
     const int ldu = (P + 3) & ~3;
     const int b = blockIdx.y, t0 = blockIdx.x * NT, nt = min(NT, n - t0);
     for (int e = threadIdx.x; e < NT * ldu; e += blockDim.x) {
@@ -206,36 +296,20 @@ __global__ void __launch_bounds__(256) rglru_gates_rows_kernel(const float *__re
         us[e] = j < nt && k < P ? act_load(u + (size_t)(t0 + j) * C + b * P + k) : 0.f;
     }
     __syncthreads();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, per = 32 / lanes, sub = lane % lanes;
-    for (int j0 = 0; j0 < 4; j0 += per) {
-        const int q = j0 + lane / lanes, k = blockIdx.z * CH + warp * 4 + q;
-        const bool mine = q < 4 && k < P;
-        float zr[NT], zi[NT];
-#pragma unroll
-        for (int j = 0; j < NT; ++j) zr[j] = zi[j] = 0.f;
-        if (mine) {
-            few_rows_share<T, NT>(ra + ((size_t)b * P + k) * P, us, ldu, P, sub, lanes, vec != 0, zr);
-            few_rows_share<T, NT>(ri + ((size_t)b * P + k) * P, us, ldu, P, sub, lanes, vec != 0, zi);
-        }
-        few_rows_reduce<NT>(zr, lanes);
-        few_rows_reduce<NT>(zi, lanes);
-        if (!mine) continue;
-        const int c = b * P + k;
-#pragma unroll
-        for (int j = 0; j < NT; ++j) {
-            if (j % lanes != sub || j >= nt) continue;
-            float a, push;
-            gate_pair(zr[j] + ra_b[c], zi[j] + ri_b[c], sp8[c], us[j * ldu + k], a, push);
-            ab[(size_t)(t0 + j) * C + c] = a;
-            ab[(size_t)(n + t0 + j) * C + c] = push;
-        }
-    }
+    gate_logits<T>(ra, ri, us, ldu, b, P, blockIdx.z * CH, lanes, vec, zs);
+    __syncthreads();
+    const int j = threadIdx.x / CH, ch = threadIdx.x % CH, k = blockIdx.z * CH + ch, c = b * P + k;
+    if (j >= nt || k >= P) return;
+    float a, push;
+    gate_pair(zs[j * CH + ch] + ra_b[c], zs[(NT + j) * CH + ch] + ri_b[c], sp8[c], us[j * ldu + k], a, push);
+    ab[(size_t)(t0 + j) * C + c] = a;
+    ab[(size_t)(n + t0 + j) * C + c] = push;
 }
 
-// Many tokens in bfloat16 (mma.sync m16n8k16, float32 accumulation): a block of four warps takes 64 tokens x 64 channels of one part, both
-// gates at once (128 columns), a warp 16 tokens.  u goes into shared memory as three bfloat16 numbers whose sum is the float32 number
-// (8 + 8 + 8 bits), each multiplied by the same matrix piece: bfloat16 products are exact in float32, so only the sums round.
-constexpr int GT = 64, GK = 64, GLD = GK + 8;
+// Many tokens in bfloat16 (mma.sync m16n8k16, float32 accumulation): a block of eight warps takes 128 tokens x 64 channels of one part, both
+// gates at once (128 columns), a warp 32 tokens x 32 channels.  u comes as three bfloat16 planes whose sum is the float32 number, each
+// multiplied by the same matrix piece: bfloat16 products are exact in float32, so only the sums round.  Two stages of cp.async.
+constexpr int GT = 128, GK = 32, GLD = GK + 8, GSTAGE = (3 * GT + 128) * GLD;
 __device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void load_matrix(uint32_t (&r)[4], const __nv_bfloat16 *p) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)));
@@ -245,79 +319,103 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__global__ void __launch_bounds__(128) rglru_gates_mma_kernel(const float *__restrict__ u, const __nv_bfloat16 *__restrict__ ra, const float *__restrict__ ra_b,
-                                                              const __nv_bfloat16 *__restrict__ ri, const float *__restrict__ ri_b,
-                                                              const float *__restrict__ sp8, float *__restrict__ ab, int n, int C, int P) {
+__device__ __forceinline__ void copy16(const __nv_bfloat16 *dst, const __nv_bfloat16 *src, bool ok) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+__global__ void __launch_bounds__(256, 2) rglru_gates_mma_kernel(const __nv_bfloat16 *__restrict__ u, const __nv_bfloat16 *__restrict__ ra,
+                                                                 const float *__restrict__ ra_b, const __nv_bfloat16 *__restrict__ ri,
+                                                                 const float *__restrict__ ri_b, const float *__restrict__ sp8, float *__restrict__ ab, int n,
+                                                                 int C, int P) {
     pdl_trigger();
-    pdl_wait();
     extern __shared__ __align__(16) __nv_bfloat16 gm[];
-    __nv_bfloat16 *As = gm, *Bs = gm + 3 * GT * GLD;          // three pieces of u; 64 rows of Ra and 64 of Ri
     const int t0 = blockIdx.x * GT, b = blockIdx.z, k_out = blockIdx.y * 64;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, wm = warp & 3, wn = warp >> 2;
     const int mat = lane >> 3, mrow = lane & 7;
-    float acc[16][4];
+    const size_t plane = (size_t)n * C;
+    auto matrices = [&](int k0, int buf) {
+        __nv_bfloat16 *Bs = gm + (size_t)buf * GSTAGE + 3 * GT * GLD;
 #pragma unroll
-    for (int i = 0; i < 16; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-    for (int k0 = 0; k0 < P; k0 += GK) {
-        for (int e = threadIdx.x; e < 128 * (GK / 8); e += 128) {
-            const int r = e / (GK / 8), col = (e - r * (GK / 8)) * 8, o = k_out + (r & 63);
+        for (int i = 0; i < 2; ++i) {
+            const int e = threadIdx.x + 256 * i, r = e / (GK / 8), col = (e % (GK / 8)) * 8, o = k_out + (r & 63);
             const bool ok = o < P && k0 + col < P;
-            const __nv_bfloat16 *src = (r < 64 ? ra : ri) + ((size_t)b * P + (ok ? o : 0)) * P + (ok ? k0 + col : 0);
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(Bs + r * GLD + col)), "l"(src), "r"(ok ? 16 : 0) : "memory");
+            copy16(Bs + r * GLD + col, (r < 64 ? ra : ri) + ((size_t)b * P + (ok ? o : 0)) * P + (ok ? k0 + col : 0), ok);
+        }
+    };
+    auto inputs = [&](int k0, int buf) {
+        __nv_bfloat16 *As = gm + (size_t)buf * GSTAGE;
+#pragma unroll
+        for (int i = 0; i < 6; ++i) {
+            const int e = threadIdx.x + 256 * i, r = e / (GK / 8), col = (e % (GK / 8)) * 8, piece = r / GT, t = t0 + r % GT;
+            const bool ok = t < n && k0 + col < P;
+            copy16(As + r * GLD + col, u + piece * plane + (ok ? (size_t)t * C + b * P + k0 + col : 0), ok);
+        }
+    };
+    matrices(0, 0);                 // the matrices depend on no earlier kernel
+    pdl_wait();
+    inputs(0, 0);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    float acc[2][8][4];
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) acc[m][i][0] = acc[m][i][1] = acc[m][i][2] = acc[m][i][3] = 0.f;
+    const int n_k = (P + GK - 1) / GK;
+    for (int kt = 0; kt < n_k; ++kt) {
+        if (kt + 1 < n_k) {
+            matrices((kt + 1) * GK, (kt + 1) & 1);
+            inputs((kt + 1) * GK, (kt + 1) & 1);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
-        for (int e = threadIdx.x; e < GT * (GK / 4); e += 128) {
-            const int r = e / (GK / 4), col = (e - r * (GK / 4)) * 4;
-            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (t0 + r < n && k0 + col < P) v = act_load(reinterpret_cast<const float4 *>(u + (size_t)(t0 + r) * C + b * P + k0 + col));
-            float x[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-            for (int piece = 0; piece < 3; ++piece) {
-                __nv_bfloat162 lo = __floats2bfloat162_rn(x[0], x[1]), hi = __floats2bfloat162_rn(x[2], x[3]);
-                *reinterpret_cast<uint2 *>(As + (piece * GT + r) * GLD + col) = make_uint2(*reinterpret_cast<unsigned *>(&lo), *reinterpret_cast<unsigned *>(&hi));
-                x[0] -= __low2float(lo), x[1] -= __high2float(lo), x[2] -= __low2float(hi), x[3] -= __high2float(hi);
-            }
-        }
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
         __syncthreads();
+        const __nv_bfloat16 *As = gm + (size_t)(kt & 1) * GSTAGE, *Bs = As + 3 * GT * GLD;
 #pragma unroll
         for (int ks = 0; ks < GK / 16; ++ks) {
-            uint32_t a[3][4];
+            uint32_t q[4][4];
 #pragma unroll
-            for (int piece = 0; piece < 3; ++piece)
-                load_matrix(a[piece], As + (piece * GT + warp * 16 + (mat & 1) * 8 + mrow) * GLD + ks * 16 + (mat >> 1) * 8);
+            for (int np = 0; np < 4; ++np)          // 0, 1: Ra's rows of this warp's channels; 2, 3: Ri's
+                load_matrix(q[np], Bs + ((np >> 1) * 64 + wn * 32 + (np & 1) * 16 + (mat >> 1) * 8 + mrow) * GLD + ks * 16 + (mat & 1) * 8);
 #pragma unroll
-            for (int np = 0; np < 8; ++np) {
-                uint32_t q[4];
-                load_matrix(q, Bs + (np * 16 + (mat >> 1) * 8 + mrow) * GLD + ks * 16 + (mat & 1) * 8);
+            for (int piece = 2; piece >= 0; --piece)         // the small pieces first
 #pragma unroll
-                for (int piece = 2; piece >= 0; --piece) {         // the small pieces first
-                    mma_bf16(acc[2 * np], a[piece], q[0], q[1]);
-                    mma_bf16(acc[2 * np + 1], a[piece], q[2], q[3]);
+                for (int m = 0; m < 2; ++m) {
+                    uint32_t a[4];
+                    load_matrix(a, As + (piece * GT + wm * 32 + m * 16 + (mat & 1) * 8 + mrow) * GLD + ks * 16 + (mat >> 1) * 8);
+#pragma unroll
+                    for (int np = 0; np < 4; ++np) {
+                        mma_bf16(acc[m][2 * np], a, q[np][0], q[np][1]);
+                        mma_bf16(acc[m][2 * np + 1], a, q[np][2], q[np][3]);
+                    }
                 }
-            }
         }
-        __syncthreads();
+        __syncthreads();            // everyone is done with this buffer before it is filled again
     }
-    // accumulators 0..7: Ra's columns, 8..15: Ri's, the same channels in the same thread
+    // accumulators 0..3: Ra's columns, 4..7: Ri's, the same channels in the same thread
 #pragma unroll
-    for (int nt = 0; nt < 8; ++nt) {
-        const int k = k_out + nt * 8 + (lane & 3) * 2;
+    for (int nt = 0; nt < 4; ++nt) {
+        const int k = k_out + wn * 32 + nt * 8 + (lane & 3) * 2;
         if (k >= P) continue;
         const int c = b * P + k;          // P and so k and c are even
         const float2 br = __ldg(reinterpret_cast<const float2 *>(ra_b + c)), bi = __ldg(reinterpret_cast<const float2 *>(ri_b + c));
         const float2 sp = __ldg(reinterpret_cast<const float2 *>(sp8 + c));
 #pragma unroll
-        for (int rr = 0; rr < 2; ++rr) {
-            const int t = t0 + warp * 16 + (lane >> 2) + rr * 8;
-            if (t >= n) continue;
-            const float2 uv = act_load(reinterpret_cast<const float2 *>(u + (size_t)t * C + c));
-            float2 a, p;
-            gate_pair(acc[nt][rr * 2] + br.x, acc[nt + 8][rr * 2] + bi.x, sp.x, uv.x, a.x, p.x);
-            gate_pair(acc[nt][rr * 2 + 1] + br.y, acc[nt + 8][rr * 2 + 1] + bi.y, sp.y, uv.y, a.y, p.y);
-            *reinterpret_cast<float2 *>(ab + (size_t)t * C + c) = a;
-            *reinterpret_cast<float2 *>(ab + (size_t)(n + t) * C + c) = p;
-        }
+        for (int m = 0; m < 2; ++m)
+#pragma unroll
+            for (int rr = 0; rr < 2; ++rr) {
+                const int t = t0 + wm * 32 + m * 16 + (lane >> 2) + rr * 8;
+                if (t >= n) continue;
+                float2 uv = make_float2(0.f, 0.f);
+#pragma unroll
+                for (int piece = 2; piece >= 0; --piece) {
+                    const unsigned raw = act_load(reinterpret_cast<const unsigned *>(u + piece * plane + (size_t)t * C + c));
+                    uv.x += __uint_as_float(raw << 16), uv.y += __uint_as_float(raw & 0xffff0000u);
+                }
+                float2 a, p;
+                gate_pair(acc[m][nt][rr * 2] + br.x, acc[m][nt + 4][rr * 2] + bi.x, sp.x, uv.x, a.x, p.x);
+                gate_pair(acc[m][nt][rr * 2 + 1] + br.y, acc[m][nt + 4][rr * 2 + 1] + bi.y, sp.y, uv.y, a.y, p.y);
+                *reinterpret_cast<float2 *>(ab + (size_t)t * C + c) = a;
+                *reinterpret_cast<float2 *>(ab + (size_t)(n + t) * C + c) = p;
+            }
     }
 }
 
@@ -434,27 +532,30 @@ LGML_API int lgml_rglru_step(const float *proj, int ldp, const float *conv_w, co
     LGML_REQUIRE((n_tokens + NT - 1) / NT <= 65535, "rglru_step: too many tokens");
     if (n_tokens == 0) return 0;
     dim3 grid((P + CH - 1) / CH, C / P, (n_tokens + NT - 1) / NT);
-    if (dtype == LGML_F32)
-        lgml_launch(rglru_step_kernel<float, float>, grid, 256, smem, stream, proj, ldp, conv_w, conv_b, state, state_ld, slots, positions, (const float *)ra, ra_b,
-                    (const float *)ri, ri_b, sp8, (float *)out, n_tokens, C, P, taps, few_rows_lanes<float>(P),
-                    few_rows_vec<float>(ra, P) && few_rows_vec<float>(ri, P) ? 1 : 0);
-    else
-        lgml_launch(rglru_step_kernel<__nv_bfloat16, __nv_bfloat16>, grid, 256, smem, stream, proj, ldp, conv_w, conv_b, state, state_ld, slots, positions,
-                    (const __nv_bfloat16 *)ra, ra_b, (const __nv_bfloat16 *)ri, ri_b, sp8, (__nv_bfloat16 *)out, n_tokens, C, P, taps,
-                    few_rows_lanes<__nv_bfloat16>(P), few_rows_vec<__nv_bfloat16>(ra, P) && few_rows_vec<__nv_bfloat16>(ri, P) ? 1 : 0);
+#define RGLRU_STEP(T, TAPS)                                                                                                                        \
+    lgml_launch(rglru_step_kernel<T, T, TAPS>, grid, 256, smem, stream, proj, ldp, conv_w, conv_b, state, state_ld, slots, positions, (const T *)ra, \
+                ra_b, (const T *)ri, ri_b, sp8, (T *)out, n_tokens, C, P, taps, few_rows_lanes<T>(P), few_rows_vec<T>(ra, P) && few_rows_vec<T>(ri, P) ? 1 : 0)
+#define RGLRU_STEP_TAPS(T)                 \
+    switch (taps) {                        \
+        case 2: RGLRU_STEP(T, 2); break;   \
+        case 3: RGLRU_STEP(T, 3); break;   \
+        case 4: RGLRU_STEP(T, 4); break;   \
+        default: RGLRU_STEP(T, 0);         \
+    }
+    if (dtype == LGML_F32) { RGLRU_STEP_TAPS(float) } else { RGLRU_STEP_TAPS(__nv_bfloat16) }
+#undef RGLRU_STEP_TAPS
+#undef RGLRU_STEP
     return lgml_launch_status("rglru_step");
 }
 
-// u float32 [n, C]
-LGML_API int lgml_rglru_conv(const float *proj, int ldp, const float *conv_w, const float *conv_b, float *state, long long state_ld, const int *seq_of_token,
-                             const int *seq_start, const int *slots, const int *positions, float *u, int n_tokens, int C, int taps, cudaStream_t stream) {
-    LGML_REQUIRE(n_tokens >= 0 && C > 0 && taps >= 1 && taps <= MAX_TAPS && ldp >= C && state_ld >= C + (taps > 1 ? (long long)taps * C : 0), "rglru_conv: bad sizes");
-    if (n_tokens == 0) return 0;
-    const bool vec = C % 4 == 0 && ldp % 4 == 0 && (((uintptr_t)proj | (uintptr_t)conv_w | (uintptr_t)conv_b | (uintptr_t)u) & 15) == 0;
+template <typename OUT>
+static int conv_run(const float *proj, int ldp, const float *conv_w, const float *conv_b, float *state, long long state_ld, const int *seq_of_token,
+                    const int *seq_start, const int *slots, const int *positions, const OUT &u, bool vec, int n_tokens, int C, int taps, cudaStream_t stream) {
     if (vec && n_tokens >= 64 && taps >= 2 && taps <= 4) {
         const size_t items = (size_t)((n_tokens + 3) / 4) * (C / 4);
         const int blocks = (int)((items + 255) / 256 < 148 * 16 ? (items + 255) / 256 : 148 * 16);
-#define RGLRU_RUNS(TT) lgml_launch(rglru_conv_runs_kernel<TT>, blocks, 256, 0, stream, proj, ldp, conv_w, conv_b, state, state_ld, seq_of_token, seq_start, slots, positions, u, n_tokens, C)
+#define RGLRU_RUNS(TT) \
+    lgml_launch(rglru_conv_runs_kernel<TT, OUT>, blocks, 256, 0, stream, proj, ldp, conv_w, conv_b, state, state_ld, seq_of_token, seq_start, slots, positions, u, n_tokens, C)
         if (taps == 2) RGLRU_RUNS(2);
         else if (taps == 3) RGLRU_RUNS(3);
         else RGLRU_RUNS(4);
@@ -463,28 +564,42 @@ LGML_API int lgml_rglru_conv(const float *proj, int ldp, const float *conv_w, co
     }
     const size_t items = (size_t)n_tokens * C;
     const int blocks = (int)((items + 255) / 256 < 148 * 16 ? (items + 255) / 256 : 148 * 16);
-    lgml_launch(rglru_conv_kernel, blocks, 256, 0, stream, proj, ldp, conv_w, conv_b, state, state_ld, seq_of_token, seq_start, slots, positions, u, n_tokens, C,
-                taps);
+    lgml_launch(rglru_conv_kernel<OUT>, blocks, 256, 0, stream, proj, ldp, conv_w, conv_b, state, state_ld, seq_of_token, seq_start, slots, positions, u, n_tokens,
+                C, taps);
     return lgml_launch_status("rglru_conv");
 }
 
-// ab float32 [2, n, C].  form 0: choose; 1: products of 8 rows; 2: tensor cores (bfloat16, parts that are multiples of 8)
-LGML_API int lgml_rglru_gates(const float *u, const void *ra, const float *ra_b, const void *ri, const float *ri_b, const float *sp8, float *ab, int dtype,
-                              int n_tokens, int C, int P, int form, cudaStream_t stream) {
-    RGLRU_SIZES("rglru_gates");
-    LGML_REQUIRE(form >= 0 && form <= 2, "rglru_gates: unknown form %d", form);
+// u: float32 [n, C], or (pieces = 1) bfloat16 [3, n, C], three numbers whose sum is the float32 one
+LGML_API int lgml_rglru_conv(const float *proj, int ldp, const float *conv_w, const float *conv_b, float *state, long long state_ld, const int *seq_of_token,
+                             const int *seq_start, const int *slots, const int *positions, void *u, int pieces, int n_tokens, int C, int taps, cudaStream_t stream) {
+    LGML_REQUIRE(n_tokens >= 0 && C > 0 && taps >= 1 && taps <= MAX_TAPS && ldp >= C && state_ld >= C + (taps > 1 ? (long long)taps * C : 0), "rglru_conv: bad sizes");
     if (n_tokens == 0) return 0;
-    const bool fits = dtype == LGML_BF16 && P % 8 == 0 && C % 4 == 0 &&
-                      (((uintptr_t)u | (uintptr_t)ra | (uintptr_t)ri | (uintptr_t)ra_b | (uintptr_t)ri_b | (uintptr_t)sp8 | (uintptr_t)ab) & 15) == 0;
-    LGML_REQUIRE(form != 2 || fits, "rglru_gates: the tensor-core form takes bfloat16 matrices and parts that are multiples of 8");
-    if (fits && (form == 2 || (form == 0 && n_tokens >= 32))) {
-        const size_t smem = sizeof(__nv_bfloat16) * (3 * GT + 128) * GLD;
+    const bool vec = C % 4 == 0 && ldp % 4 == 0 && (((uintptr_t)proj | (uintptr_t)conv_w | (uintptr_t)conv_b | (uintptr_t)u) & 15) == 0;
+    if (pieces)
+        return conv_run(proj, ldp, conv_w, conv_b, state, state_ld, seq_of_token, seq_start, slots, positions, AsPieces{(__nv_bfloat16 *)u, (size_t)n_tokens * C},
+                        vec, n_tokens, C, taps, stream);
+    return conv_run(proj, ldp, conv_w, conv_b, state, state_ld, seq_of_token, seq_start, slots, positions, AsFloat{(float *)u}, vec, n_tokens, C, taps, stream);
+}
+
+// ab float32 [2, n, C].  u float32 [n, C] (products of 8 rows), or (pieces = 1) bfloat16 [3, n, C] (tensor cores: bfloat16 matrices, parts and
+// channels that are multiples of 8).
+LGML_API int lgml_rglru_gates(const void *u_any, int pieces, const void *ra, const float *ra_b, const void *ri, const float *ri_b, const float *sp8, float *ab,
+                              int dtype, int n_tokens, int C, int P, cudaStream_t stream) {
+    RGLRU_SIZES("rglru_gates");
+    if (n_tokens == 0) return 0;
+    if (pieces) {
+        LGML_REQUIRE(dtype == LGML_BF16 && P % 8 == 0 &&
+                         (((uintptr_t)u_any | (uintptr_t)ra | (uintptr_t)ri | (uintptr_t)ra_b | (uintptr_t)ri_b | (uintptr_t)sp8 | (uintptr_t)ab) & 15) == 0,
+                     "rglru_gates: the tensor-core form takes bfloat16 matrices and parts that are multiples of 8, on 16-byte borders");
+        const size_t smem = sizeof(__nv_bfloat16) * 2 * (size_t)GSTAGE;
         cudaError_t e = cudaFuncSetAttribute(rglru_gates_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) LGML_FAIL("rglru_gates: cannot have %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
         dim3 grid((n_tokens + GT - 1) / GT, (P + 63) / 64, C / P);
-        lgml_launch(rglru_gates_mma_kernel, grid, 128, smem, stream, u, (const __nv_bfloat16 *)ra, ra_b, (const __nv_bfloat16 *)ri, ri_b, sp8, ab, n_tokens, C, P);
+        lgml_launch(rglru_gates_mma_kernel, grid, 256, smem, stream, (const __nv_bfloat16 *)u_any, (const __nv_bfloat16 *)ra, ra_b, (const __nv_bfloat16 *)ri, ri_b,
+                    sp8, ab, n_tokens, C, P);
         return lgml_launch_status("rglru_gates");
     }
+    const float *u = (const float *)u_any;
     const size_t smem = sizeof(float) * NT * (size_t)((P + 3) & ~3);
     LGML_REQUIRE(smem <= 48 * 1024, "rglru_gates: parts of %d channels are too wide", P);
     dim3 grid((n_tokens + NT - 1) / NT, C / P, (P + CH - 1) / CH);

@@ -79,8 +79,10 @@ __device__ __forceinline__ void store4(__nv_bfloat16 *p, int i, int E, int vec, 
 
 // A block a row; thread i holds the quads i, i + threads, ... of it (NQ of them).  The number of threads is the width's, so that a
 // row's sums are formed in one order whatever else is in the batch.
-template <typename TO, int NQ>
-__global__ void __launch_bounds__(NQ > 4 ? 1024 : 512) scaled_norm_kernel(const Args a) {
+// PARTS: A comes in several parts (or halves): up to eight of them are in flight at a time.  Without them, for many rows, a
+// thread needs few enough registers for two blocks or more an SM.
+template <typename TO, int NQ, bool PARTS>
+__global__ void __launch_bounds__(NQ > 4 ? 1024 : 512, NQ > 2 || PARTS ? 1 : 2) scaled_norm_kernel(const Args a) {
     pdl_trigger();
     pdl_wait();
     __shared__ float red[32];
@@ -89,11 +91,12 @@ __global__ void __launch_bounds__(NQ > 4 ? 1024 : 512) scaled_norm_kernel(const 
     float *xr = a.x + t * E;
     constexpr bool AHEAD = NQ <= 4;         // very wide rows load as they go
     constexpr int ND = AHEAD ? NQ : 1;
-    float v[NQ][4], da[ND][4], db[ND][4];
+    float v[NQ][4], da[ND][4], db[ND][4], dc[ND][4];
     const float *ar = a.a ? a.a + t * a.lda : nullptr;
-    const float *br = nullptr;
+    const float *br = nullptr, *cr = nullptr;           // B, and a token's second expert
     if (a.b) br = a.b + (a.b_pos ? (size_t)act_load(a.b_pos + t * a.b_top) : t) * a.ldb;
-    // the first loads of all three before any is used
+    if (a.b && a.b_pos && a.b_top > 1) cr = a.b + (size_t)act_load(a.b_pos + t * a.b_top + 1) * a.ldb;
+    // the first loads of all of them before any is used
 #pragma unroll
     for (int q = 0; q < NQ; ++q) {
         const int i = 4 * (q * T + threadIdx.x);
@@ -102,6 +105,7 @@ __global__ void __launch_bounds__(NQ > 4 ? 1024 : 512) scaled_norm_kernel(const 
         if (a.keep) load4(xr, i, E, a.vec, v[q]);
         if (AHEAD && ar) load4(ar, i, E, a.vec, da[q % ND]);
         if (AHEAD && br) load4(br, i, E, a.vec, db[q % ND]);
+        if (AHEAD && cr) load4(cr, i, E, a.vec, dc[q % ND]);
     }
     float ss = 0.f;
 #pragma unroll
@@ -109,29 +113,30 @@ __global__ void __launch_bounds__(NQ > 4 ? 1024 : 512) scaled_norm_kernel(const 
         const int i = 4 * (q * T + threadIdx.x);
         if (i >= E) continue;
         float s[4];
-        float (&ad)[4] = da[q % ND], (&bd)[4] = db[q % ND];
+        float (&ad)[4] = da[q % ND], (&bd)[4] = db[q % ND], (&cd)[4] = dc[q % ND];
         if (!AHEAD && ar) load4(ar, i, E, a.vec, ad);
         if (!AHEAD && br) load4(br, i, E, a.vec, bd);
+        if (!AHEAD && cr) load4(cr, i, E, a.vec, cd);
         if (ar) {
-            // the other parts, four at a time in flight, added in their order
-            for (int p = 1; p < a.n_parts; p += 4) {
-                float o[4][4];
+            if (PARTS) {
+                // the other parts (a row's halves one after the other), added in their order
+                constexpr int W = NQ > 4 ? 2 : 8;
+                const int total = a.a_second ? 2 * a.n_parts : a.n_parts;
+                for (int p = 1; p < total; p += W) {
+                    float o[W][4];
 #pragma unroll
-                for (int k = 0; k < 4; ++k)
-                    if (p + k < a.n_parts) load4(ar + (size_t)(p + k) * a.a_stride, i, E, a.vec, o[k]);
+                    for (int k = 0; k < W; ++k)
+                        if (p + k < total) {
+                            const int m = p + k;
+                            load4(ar + (size_t)(m < a.n_parts ? m : m - a.n_parts) * a.a_stride + (m < a.n_parts ? 0 : a.a_second), i, E, a.vec, o[k]);
+                        }
 #pragma unroll
-                for (int k = 0; k < 4; ++k)
-                    if (p + k < a.n_parts)
+                    for (int k = 0; k < W; ++k)
+                        if (p + k < total)
 #pragma unroll
-                        for (int e = 0; e < 4; ++e) ad[e] += o[k][e];
-            }
-            if (a.a_second)
-                for (int p = 0; p < a.n_parts; ++p) {
-                    float o[4];
-                    load4(ar + (size_t)p * a.a_stride + a.a_second, i, E, a.vec, o);
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) ad[e] += o[e];
+                            for (int e = 0; e < 4; ++e) ad[e] += o[k][e];
                 }
+            }
             if (a.a_bias) {
                 const4(a.a_bias, i, E, a.vec, s);
 #pragma unroll
@@ -147,8 +152,12 @@ __global__ void __launch_bounds__(NQ > 4 ? 1024 : 512) scaled_norm_kernel(const 
             }
         }
         if (br) {
+            if (cr) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) bd[e] += cd[e];
+            }
             if (a.b_pos)
-                for (int k = 1; k < a.b_top; ++k) {
+                for (int k = 2; k < a.b_top; ++k) {
                     load4(a.b + (size_t)act_load(a.b_pos + t * a.b_top + k) * a.ldb, i, E, a.vec, s);
 #pragma unroll
                     for (int e = 0; e < 4; ++e) bd[e] += s[e];
@@ -195,11 +204,18 @@ template <typename TO>
 int launch(const Args &a, int n_rows, cudaStream_t stream) {
     const int quads = (a.E + 3) / 4;
     auto threads = [&](int nq) { return ((quads + nq - 1) / nq + 31) / 32 * 32; };
-    if (quads <= 256) lgml_launch(scaled_norm_kernel<TO, 1>, n_rows, threads(1), 0, stream, a);
-    else if (quads <= 1024) lgml_launch(scaled_norm_kernel<TO, 2>, n_rows, threads(2), 0, stream, a);
-    else if (quads <= 2048) lgml_launch(scaled_norm_kernel<TO, 4>, n_rows, threads(4), 0, stream, a);
-    else if (quads <= 8192) lgml_launch(scaled_norm_kernel<TO, 8>, n_rows, threads(8), 0, stream, a);
+    const bool parts = a.a != nullptr && (a.n_parts > 1 || a.a_second != 0);
+#define LGML_SN(NQ)                                                                                              \
+    do {                                                                                                         \
+        if (parts) lgml_launch(scaled_norm_kernel<TO, NQ, true>, n_rows, threads(NQ), 0, stream, a);             \
+        else lgml_launch(scaled_norm_kernel<TO, NQ, false>, n_rows, threads(NQ), 0, stream, a);                  \
+    } while (0)
+    if (quads <= 256) LGML_SN(1);
+    else if (quads <= 1024) LGML_SN(2);
+    else if (quads <= 2048) LGML_SN(4);
+    else if (quads <= 8192) LGML_SN(8);
     else LGML_FAIL("scaled_norm: rows of %d are too wide", a.E);
+#undef LGML_SN
     return lgml_launch_status("scaled_norm");
 }
 }  // namespace

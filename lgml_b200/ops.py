@@ -1008,8 +1008,22 @@ def moe_grouped_supports(h: torch.Tensor, w_gu: torch.Tensor, gated: bool = True
             and w_gu.shape[1] % (16 if gated else 8) == 0 and w_gu.shape[2] % 8 == 0)
 
 
-def _moe_tiles(n_rows: int, X: int) -> int:
-    return -(-n_rows // MOE_TILE_ROWS) + min(X, n_rows)
+def _moe_tiles(n_rows: int, X: int, tile_rows: int = MOE_TILE_ROWS) -> int:
+    return -(-n_rows // tile_rows) + min(X, n_rows)
+
+
+_tile_rows_memo = {}
+
+
+def moe_tile_rows(n_rows: int, X: int) -> int:
+    """Rows of a tile of the grouped products for ``n_rows`` (token, expert) rows over X experts (remembered: a step asks for the
+    same few again and again)."""
+    got = _tile_rows_memo.get((n_rows, X))
+    if got is None:
+        fn = getattr(csrc.load("moe"), "lgml_moe_tile_rows")
+        fn.argtypes, fn.restype = [c_int, c_int], c_int
+        got = _tile_rows_memo[(n_rows, X)] = fn(n_rows, X)
+    return got
 
 
 def moe_experts_grouped(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor) -> torch.Tensor:
@@ -1040,7 +1054,7 @@ def moe_experts_tcgen05(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w
                         status: torch.Tensor, gated: bool = True, also: Optional[torch.Tensor] = None,
                         also_w: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``moe_experts_rows`` for many tokens, bfloat16, on tcgen05: the (token, chosen expert) rows are sorted by
-    expert on the device, the tokens' rows gathered into tiles of 128 rows of one expert, and the two products
+    expert on the device, the tokens' rows gathered into tiles of one expert's rows (128, or 16 to 64 where an expert gets few), and the two products
     run as grouped products of the tcgen05 kernel (a tile reads the matrices of its expert; the gate|up product
     applies the SiLU gate in its epilogue); a token's rows are then added, weighted, in the order of its experts.
     float32 [tokens, E].  No host value is read.  ``gated`` False: experts without a gate (``w_gu`` [X, F, E], the
@@ -1052,18 +1066,19 @@ def moe_experts_tcgen05(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w
     if not moe_grouped_supports(h, w_gu, gated):
         raise KernelError("moe_experts_tcgen05: widths and row strides must be multiples of 8 and the input 16-byte aligned")
     n_rows = n * top
-    max_tiles = _moe_tiles(n_rows, X)
+    tile_rows = moe_tile_rows(n_rows, X)
+    max_tiles = _moe_tiles(n_rows, X, tile_rows)
     dev = h.device
     rows = torch.empty(n_rows, dtype=torch.int32, device=dev)
     pos = torch.empty(n_rows, dtype=torch.int32, device=dev)
     tiles = torch.empty(3 * max_tiles + 1, dtype=torch.int32, device=dev)
-    a_perm = torch.empty((max_tiles * MOE_TILE_ROWS, E), dtype=torch.bfloat16, device=dev)
+    a_perm = torch.empty((max_tiles * tile_rows, E), dtype=torch.bfloat16, device=dev)
     out = torch.empty((n, E), dtype=torch.float32, device=dev)
     stream = _stream()
-    fn = _fn("moe", "lgml_moe_group_rows", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-    _check("moe", fn(_ptr(ids), _ptr(rows), _ptr(tiles), max_tiles, n, X, top, stream), "moe_group_rows")
-    fn = _fn("moe", "lgml_moe_gather_rows", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p])
-    _check("moe", fn(_ptr(h), ldh, _ptr(rows), _ptr(tiles), max_tiles, _ptr(a_perm), _ptr(pos), E, top, stream), "moe_gather_rows")
+    fn = _fn("moe", "lgml_moe_group_rows", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check("moe", fn(_ptr(ids), _ptr(rows), _ptr(tiles), max_tiles, tile_rows, n, X, top, stream), "moe_group_rows")
+    fn = _fn("moe", "lgml_moe_gather_rows", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p])
+    _check("moe", fn(_ptr(h), ldh, _ptr(rows), _ptr(tiles), max_tiles, tile_rows, _ptr(a_perm), _ptr(pos), E, top, stream), "moe_gather_rows")
     y = moe_tile_products(a_perm, tiles, w_gu, w_down, status, gated=gated)
     fn = _fn("moe", "lgml_moe_weighted_sum_form", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p,
                                                    c_void_p], label="moe_weighted_sum")
@@ -1073,38 +1088,39 @@ def moe_experts_tcgen05(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w
 
 def moe_tile_products(a_perm: torch.Tensor, tiles: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, status: torch.Tensor, gated: bool = True,
                       clamp=None) -> torch.Tensor:
-    """The experts' two products over tiles of 128 rows of one expert, bfloat16 on tcgen05: ``a_perm`` [max_tiles 128, E],
-    ``tiles`` int32 [3 max_tiles + 1] (per tile: expert, -, rows; the last word: how many tiles there are); float32 [max_tiles 128, E].
+    """The experts' two products over tiles of rows of one expert, bfloat16 on tcgen05: ``a_perm`` [max_tiles tile_rows, E],
+    ``tiles`` int32 [3 max_tiles + 1] (per tile: expert, -, rows; the last word: how many tiles there are); float32 [max_tiles tile_rows, E].
     The first product's epilogue is silu(gate) * up, with ``clamp`` = (alpha, limit) the clamped activation, without a gate relu
     squared.  Rows of a tile that hold no token come out as whatever they are."""
     _need(a_perm, "experts' rows", torch.bfloat16, 2)
     _need(tiles, "tiles", torch.int32, 1)
     X, F2, E = w_gu.shape
     F = F2 // 2 if gated else F2
-    max_tiles = a_perm.shape[0] // MOE_TILE_ROWS
-    if a_perm.shape != (max_tiles * MOE_TILE_ROWS, E) or not a_perm.is_contiguous() or tiles.numel() != 3 * max_tiles + 1 or not tiles.is_contiguous():
+    max_tiles = tiles.numel() // 3
+    tile_rows = a_perm.shape[0] // max_tiles
+    if a_perm.shape != (max_tiles * tile_rows, E) or not a_perm.is_contiguous() or tiles.numel() != 3 * max_tiles + 1 or not tiles.is_contiguous():
         raise KernelError(f"moe_tile_products: rows {tuple(a_perm.shape)} / tiles {tuple(tiles.shape)} do not fit matrices {tuple(w_gu.shape)}")
     if tuple(w_down.shape) != (X, E, F) or (clamp is not None and not gated):
         raise KernelError(f"moe_tile_products: matrices {tuple(w_gu.shape)} and {tuple(w_down.shape)} do not go together")
     alpha, limit = clamp if clamp is not None else (0.0, 0.0)
-    act = torch.empty((max_tiles * MOE_TILE_ROWS, F), dtype=torch.bfloat16, device=a_perm.device)
-    y = torch.empty((max_tiles * MOE_TILE_ROWS, E), dtype=torch.float32, device=a_perm.device)
+    act = torch.empty((max_tiles * tile_rows, F), dtype=torch.bfloat16, device=a_perm.device)
+    y = torch.empty((max_tiles * tile_rows, E), dtype=torch.float32, device=a_perm.device)
     stream = _stream()
-    fn = _fn("gemm_tcgen05", "lgml_gemm_tcgen05_grouped_act", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
+    fn = _fn("gemm_tcgen05", "lgml_gemm_tcgen05_grouped_tiles", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
                                                                c_float, c_float, c_void_p, c_void_p], label="gemm_tcgen05_grouped")
-    _check("gemm_tcgen05", fn(_ptr(a_perm), _ptr(w_gu), _ptr(act), 0, max_tiles, F2, E, X, F, _ptr(tiles), (3 if clamp is not None else 1) if gated else 2,
+    _check("gemm_tcgen05", fn(_ptr(a_perm), _ptr(w_gu), _ptr(act), 0, max_tiles, tile_rows, F2, E, X, F, _ptr(tiles), (3 if clamp is not None else 1) if gated else 2,
                               float(alpha), float(limit), _ptr(status), stream), "gemm_tcgen05_grouped")
-    _check("gemm_tcgen05", fn(_ptr(act), _ptr(w_down), _ptr(y), 1, max_tiles, E, F, X, E, _ptr(tiles), 0, 0.0, 0.0, _ptr(status), stream),
+    _check("gemm_tcgen05", fn(_ptr(act), _ptr(w_down), _ptr(y), 1, max_tiles, tile_rows, E, F, X, E, _ptr(tiles), 0, 0.0, 0.0, _ptr(status), stream),
            "gemm_tcgen05_grouped")
     return y
 
 
 class TableRoute:
     """Where the rows of one table's experts go in a step: ``ids`` int32 [tokens, top], ``places`` int32 [tokens, top] (the row
-    among the tiles), ``tiles`` int32 [3 max_tiles + 1]."""
+    among the tiles), ``tiles`` int32 [3 max_tiles + 1], each of ``tile_rows`` rows."""
 
-    def __init__(self, ids: torch.Tensor, places: torch.Tensor, tiles: torch.Tensor):
-        self.ids, self.places, self.tiles = ids, places, tiles
+    def __init__(self, ids: torch.Tensor, places: torch.Tensor, tiles: torch.Tensor, tile_rows: int):
+        self.ids, self.places, self.tiles, self.tile_rows = ids, places, tiles, tile_rows
 
     @property
     def max_tiles(self) -> int:
@@ -1123,13 +1139,14 @@ def table_route(token_ids: torch.Tensor, vocab: int, tables: torch.Tensor, desc:
         raise KernelError("table_route: one row (experts, top, first entry) per table")
     if tables.numel() != sum(vocab * top for _, top in shapes):
         raise KernelError(f"table_route: {tables.numel()} entries are not those of the tables")
-    sizes = [(n * top, _moe_tiles(n * top, X)) for X, top in shapes]
+    rows_of = [moe_tile_rows(n * top, X) for X, top in shapes]
+    sizes = [(n * top, _moe_tiles(n * top, X, m)) for (X, top), m in zip(shapes, rows_of)]
     out = torch.empty(sum(2 * r + 3 * t + 1 for r, t in sizes), dtype=torch.int32, device=token_ids.device)
     fn = _fn("moe", "lgml_table_route", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p])
     _check("moe", fn(_ptr(token_ids), n, int(vocab), _ptr(tables), _ptr(desc), len(shapes), max(X for X, _ in shapes), _ptr(out), _stream()), "table_route")
     routes, at = [], 0
-    for (r, t), (_, top) in zip(sizes, shapes):
-        routes.append(TableRoute(out[at:at + r].view(n, top), out[at + r:at + 2 * r].view(n, top), out[at + 2 * r:at + 2 * r + 3 * t + 1]))
+    for (r, t), (_, top), m in zip(sizes, shapes, rows_of):
+        routes.append(TableRoute(out[at:at + r].view(n, top), out[at + r:at + 2 * r].view(n, top), out[at + 2 * r:at + 2 * r + 3 * t + 1], m))
         at += 2 * r + 3 * t + 1
     return routes
 
@@ -1260,8 +1277,9 @@ def rglru_chunk_tokens() -> int:
 
 
 def _rglru_shapes(proj, ra, ra_b, ri, ri_b, sp8, who: str):
-    _need(proj, "projections", torch.float32, 2)
-    B, P, P2 = ra.shape
+    if proj is not None:
+        _need(proj, "projections", torch.float32, 2)
+    B, P, _ = ra.shape
     C = B * P
     for t, what in ((ra, "decay gate"), (ri, "input gate")):
         _need(t, f"{what}'s matrices", ra.dtype, 3)
@@ -1306,10 +1324,16 @@ def rglru_step(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, s
     return out
 
 
+def rglru_pieces_supported(ra: torch.Tensor, n_tokens: int) -> bool:
+    """Whether the gates of a step of that many tokens run on tensor cores, from inputs in three bfloat16 pieces."""
+    return n_tokens >= 32 and ra.dtype == torch.bfloat16 and ra.shape[1] % 8 == 0
+
+
 def rglru_conv(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, state: torch.Tensor, seq_of_token: torch.Tensor, seq_start: torch.Tensor,
-               slots: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+               slots: torch.Tensor, positions: torch.Tensor, pieces: bool = False) -> torch.Tensor:
     """The causal convolution of ``proj``'s first C columns, float32 [tokens, C]; the inputs of earlier steps come from the ring in
-    the request's state, which takes the step's last ones."""
+    the request's state, which takes the step's last ones.  ``pieces``: the result as bfloat16 [3, tokens, C], three numbers
+    whose sum is the float32 one (8 + 8 + 8 bits)."""
     _need(proj, "projections", torch.float32, 2)
     C = conv_b.numel()
     taps = _conv_shapes(conv_w, conv_b, C, "rglru_conv")
@@ -1317,28 +1341,29 @@ def rglru_conv(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, s
     if proj.shape[1] < C or positions.numel() != n or seq_of_token.numel() != n:
         raise KernelError(f"rglru_conv: projections {tuple(proj.shape)} hold no {C} channels")
     ld = _state_rows(state, rglru_state_floats(C, taps), "rglru_conv")
-    u = torch.empty((n, C), dtype=torch.float32, device=proj.device)
+    u = torch.empty((3, n, C), dtype=torch.bfloat16, device=proj.device) if pieces else torch.empty((n, C), dtype=torch.float32, device=proj.device)
     fn = _fn("rglru", "lgml_rglru_conv", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                          c_int, c_void_p])
+                                          c_int, c_int, c_void_p])
     _check("rglru", fn(_ptr(proj), ldp, _ptr(conv_w), _ptr(conv_b), _ptr(state), ld, _ptr(seq_of_token), _ptr(seq_start), _ptr(slots), _ptr(positions), _ptr(u),
-                       n, C, taps, _stream()), "rglru_conv")
+                       1 if pieces else 0, n, C, taps, _stream()), "rglru_conv")
     return u
 
 
-RGLRU_FORMS = {"auto": 0, "rows": 1, "mma": 2}
-
-
-def rglru_gates(u: torch.Tensor, ra: torch.Tensor, ra_b: torch.Tensor, ri: torch.Tensor, ri_b: torch.Tensor, sp8: torch.Tensor, form: str = "auto") -> torch.Tensor:
-    """From the convolved inputs ``u`` float32 [tokens, C]: float32 [2, tokens, C], the decay a = exp(-sigmoid(Ra u + ra_b) sp8) and the
-    pushed term sqrt(1 - a^2) sigmoid(Ri u + ri_b) u, Ra and Ri block-diagonal [parts, P, P].  The products are true 32-bit
-    sums over the float32 u in every form."""
-    C, P = _rglru_shapes(u, ra, ra_b, ri, ri_b, sp8, "rglru_gates")
-    n = u.shape[0]
-    if u.shape[1] != C or not u.is_contiguous():
+def rglru_gates(u: torch.Tensor, ra: torch.Tensor, ra_b: torch.Tensor, ri: torch.Tensor, ri_b: torch.Tensor, sp8: torch.Tensor) -> torch.Tensor:
+    """From the convolved inputs ``u`` (float32 [tokens, C], or bfloat16 [3, tokens, C] as ``rglru_conv(pieces=True)`` gives them): float32
+    [2, tokens, C], the decay a = exp(-sigmoid(Ra u + ra_b) sp8) and the pushed term sqrt(1 - a^2) sigmoid(Ri u + ri_b) u, Ra and Ri
+    block-diagonal [parts, P, P].  The products are true 32-bit sums over the float32 u in both forms."""
+    pieces = u.dtype == torch.bfloat16
+    B, P, _ = ra.shape
+    C = B * P
+    _need(u, "convolved inputs", torch.bfloat16 if pieces else torch.float32, 3 if pieces else 2)
+    _rglru_shapes(None, ra, ra_b, ri, ri_b, sp8, "rglru_gates")
+    n = u.shape[-2]
+    if tuple(u.shape) != ((3, n, C) if pieces else (n, C)) or not u.is_contiguous():
         raise KernelError(f"rglru_gates: inputs {tuple(u.shape)} do not fit {C} channels")
     ab = torch.empty((2, n, C), dtype=torch.float32, device=u.device)
-    fn = _fn("rglru", "lgml_rglru_gates", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
-    _check("rglru", fn(_ptr(u), _ptr(ra), _ptr(ra_b), _ptr(ri), _ptr(ri_b), _ptr(sp8), _ptr(ab), dtype_code(ra.dtype), n, C, P, RGLRU_FORMS[form], _stream()),
+    fn = _fn("rglru", "lgml_rglru_gates", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check("rglru", fn(_ptr(u), 1 if pieces else 0, _ptr(ra), _ptr(ra_b), _ptr(ri), _ptr(ri_b), _ptr(sp8), _ptr(ab), dtype_code(ra.dtype), n, C, P, _stream()),
            "rglru_gates")
     return ab
 

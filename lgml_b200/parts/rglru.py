@@ -65,7 +65,8 @@ class RealGatedLRU(Part):
         if batch.max_q_len == 1:
             out = ops.rglru_step(proj, self.conv_w, self.conv_b, cache.state, batch.slots, batch.positions, self.ra, self.ra_b, self.ri, self.ri_b, self.sp8)
             return rt.linear(out, self.wo, partials_ok=True)
-        u = ops.rglru_conv(proj, self.conv_w, self.conv_b, cache.state, batch.seq_of_token, batch.seq_start, batch.slots, batch.positions)
+        u = ops.rglru_conv(proj, self.conv_w, self.conv_b, cache.state, batch.seq_of_token, batch.seq_start, batch.slots, batch.positions,
+                           pieces=ops.rglru_pieces_supported(self.ra, h.shape[0]))
         ab = ops.rglru_gates(u, self.ra, self.ra_b, self.ri, self.ri_b, self.sp8)
         out = torch.empty((h.shape[0], self.inner), dtype=rt.dtype, device=h.device)
         chunks = chunk_start = None

@@ -111,7 +111,7 @@ class TableExperts(Part):
         route = self.routing.of(batch, self.number)
         if not rt.experts_in_tiles(route.ids.numel(), self.w_gu):
             return ExpertTiles(route)
-        return ExpertTiles(route, torch.empty((route.max_tiles * ops.MOE_TILE_ROWS, self.width), dtype=rt.dtype, device=route.ids.device))
+        return ExpertTiles(route, torch.empty((route.max_tiles * route.tile_rows, self.width), dtype=rt.dtype, device=route.ids.device))
 
     def forward(self, rt, h, routed: ExpertTiles):
         """float32 [tokens, width], or ``ops.ExpertRows`` that the next norm adds up."""
