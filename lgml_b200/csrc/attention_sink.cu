@@ -1199,8 +1199,9 @@ LGML_API int lgml_sink_decode(const void *q, int ldq, const int *positions, cons
     LGML_REQUIRE(gate_stride_ok(gate, ldg, H, Dv), "sink_decode: the gate's row stride %d is below its row", ldg);
     if (n_tokens == 0) return 0;
     const int group = H / Hkv;
-    float *part_o = scratch;
-    float2 *part_ml = reinterpret_cast<float2 *>(scratch + (size_t)n_tokens * H * n_splits * Dv);
+    // the pairs first: behind the values they would start on an odd float where heads, ranges and value size are all odd
+    float2 *part_ml = reinterpret_cast<float2 *>(scratch);
+    float *part_o = scratch != nullptr ? scratch + 2 * (size_t)n_tokens * H * n_splits : nullptr;
     if (D % 32 == 0 && Dv % 32 == 0 && D <= 128 && Dv <= 128 && ldq % 2 == 0 && ldv % 8 == 0 && (((uintptr_t)k_pages | (uintptr_t)v_pages) & 15) == 0 &&
         ((uintptr_t)q & 3) == 0) {
         // head sizes the tensor-core form is built for
