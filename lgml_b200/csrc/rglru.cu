@@ -11,8 +11,9 @@
 //
 //   rglru_step    one token a request: convolution, both gates, recurrence and output in one kernel, a block per (8 tokens, 32 channels)
 //   rglru_conv    the convolution alone for longer portions; also brings the ring up to date
-//   rglru_gates   a_t and the pushed term sqrt(1 - a^2) i u of longer portions: on tensor cores with u in three bfloat16
-//                 pieces (24 bits: what is multiplied is the float32 number), else as products of 8 rows
+//   rglru_gates   a_t and the pushed term sqrt(1 - a^2) i u of longer portions as products of 8 rows
+//   rglru_finish  the same from logits that a grouped product on tensor cores has left: a group a part of the channels, u in three
+//                 bfloat16 pieces side by side (24 bits: what is multiplied is the float32 number)
 //   rglru_scan    S_t = a_t S_(t-1) + push_t and the output, a thread a channel of a request
 //   rglru_chunks  the same for long portions in three passes: every chunk's (product of a, scan from zero), the chain over
 //                 a request's chunks, every chunk again from its true start
@@ -32,7 +33,8 @@ constexpr int CH = 32;           // channels a block of the row forms takes: eig
 constexpr int CHUNK = 32;        // tokens of a chunk of a long portion
 constexpr int MAX_TAPS = 16;
 
-__device__ __forceinline__ float sigmoid_(float v) { return 1.0f / (1.0f + expf(-v)); }
+// 1 / (1 + e^-v), right to two units in the last place; e^-v is kept below 2^126, where the fast division still divides
+__device__ __forceinline__ float sigmoid_(float v) { return __fdividef(1.0f, 1.0f + expf(fminf(-v, 80.0f))); }
 __device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
 
 // a and the pushed term from the gates' logits; sp8 = 8 softplus(lam)
@@ -122,7 +124,7 @@ __global__ void __launch_bounds__(256) rglru_step_kernel(const float *__restrict
                 for (int i = 0; i < TAPS; ++i) {
                     const int back = TAPS - 1 - i;
                     const bool there = j < nt && k < P && pos[j] >= back;
-                    in[j][i] = !there ? 0.f : (back == 0 ? act_load(proj + (size_t)(t0 + j) * ldp + c) : act_load(ring[j] + (size_t)((pos[j] - back) % TAPS) * C + c));
+                    in[j][i] = !there ? 0.f : (back == 0 ? act_load(proj + (size_t)(t0 + j) * ldp + c) : act_load(ring[j] + (size_t)((pos[j] - back) % (TAPS > 0 ? TAPS : 1)) * C + c));
                 }
 #pragma unroll
             for (int i = 0; i < TAPS; ++i) w[i] = k < P ? __ldg(conv_w + (size_t)i * C + c) : 0.f;
@@ -169,32 +171,48 @@ __global__ void __launch_bounds__(256) rglru_step_kernel(const float *__restrict
     if (taps > 1) row[C + (size_t)(pos_t % taps) * C + c] = x_in;
 }
 
-// A convolved input on its way out: a float32 number, or three bfloat16 numbers whose sum it is (8 + 8 + 8 bits), in three planes
-// of `plane` numbers (what the gates' tensor-core form multiplies).
+// A convolved input on its way out: a float32 number at [t, c], or three bfloat16 numbers whose sum it is (8 + 8 + 8 bits): channel
+// k of part b of token t in row b * rows + t of a matrix [B rows, 3 P], at columns k, P + k and 2 P + k.  A product of such rows with [R | R | R] is
+// R times the float32 number.
 struct AsFloat {
     float *u;
-    __device__ __forceinline__ void put(size_t i, float v) const { u[i] = v; }
-    __device__ __forceinline__ void put4(size_t i, const float4 &v) const { *reinterpret_cast<float4 *>(u + i) = v; }
+    int C;
+    __device__ __forceinline__ void put(int t, int c, float v) const { u[(size_t)t * C + c] = v; }
+    __device__ __forceinline__ void put4(int t, int c, const float4 &v) const { *reinterpret_cast<float4 *>(u + (size_t)t * C + c) = v; }
 };
 struct AsPieces {
     __nv_bfloat16 *u;
-    size_t plane;
-    __device__ __forceinline__ void put(size_t i, float v) const {
+    int rows, P;
+    __device__ __forceinline__ __nv_bfloat16 *at(int t, int c) const {
+        const int b = c / P;
+        return u + ((size_t)b * rows + t) * 3 * P + (c - b * P);
+    }
+    __device__ __forceinline__ void put(int t, int c, float v) const {
+        __nv_bfloat16 *p = at(t, c);
 #pragma unroll
         for (int k = 0; k < 3; ++k) {
             const __nv_bfloat16 h = __float2bfloat16_rn(v);
-            u[k * plane + i] = h;
+            p[k * P] = h;
             v -= __bfloat162float(h);
         }
     }
-    __device__ __forceinline__ void put4(size_t i, const float4 &v) const {
+    __device__ __forceinline__ void put4(int t, int c, const float4 &v) const {       // parts are multiples of 8 channels
+        __nv_bfloat16 *p = at(t, c);
         float x[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
         for (int k = 0; k < 3; ++k) {
             __nv_bfloat162 lo = __floats2bfloat162_rn(x[0], x[1]), hi = __floats2bfloat162_rn(x[2], x[3]);
-            *reinterpret_cast<uint2 *>(u + k * plane + i) = make_uint2(*reinterpret_cast<unsigned *>(&lo), *reinterpret_cast<unsigned *>(&hi));
+            *reinterpret_cast<uint2 *>(p + k * P) = make_uint2(*reinterpret_cast<unsigned *>(&lo), *reinterpret_cast<unsigned *>(&hi));
             x[0] -= __low2float(lo), x[1] -= __high2float(lo), x[2] -= __low2float(hi), x[3] -= __high2float(hi);
         }
+    }
+    // two neighbouring channels (c even) in three 4-byte loads
+    __device__ __forceinline__ float2 get2(int t, int c) const {
+        const unsigned *p = reinterpret_cast<const unsigned *>(at(t, c));
+        const unsigned hi = act_load(p), mid = act_load(p + P / 2), lo = act_load(p + P);
+        auto first = [](unsigned w) { return __uint_as_float(w << 16); };
+        auto second = [](unsigned w) { return __uint_as_float(w & 0xffff0000u); };
+        return make_float2(first(hi) + (first(mid) + first(lo)), second(hi) + (second(mid) + second(lo)));
     }
 };
 
@@ -217,11 +235,11 @@ __global__ void __launch_bounds__(256) rglru_conv_kernel(const float *__restrict
         if (t == t0) {
             float *ring = state + (size_t)slots[s] * state_ld + C;
             const int t1 = seq_start[s + 1], last = min(t1, t0 + max(taps - 1, 1)), pos0 = positions[t0];
-            for (int i = t0; i < last; ++i) u.put((size_t)i * C + c, conv_at(proj, ldp, conv_w, bias, ring, C, taps, i, t0, pos0 + i - t0, c));
+            for (int i = t0; i < last; ++i) u.put(i, c, conv_at(proj, ldp, conv_w, bias, ring, C, taps, i, t0, pos0 + i - t0, c));
             if (taps > 1)
                 for (int i = max(t0, t1 - (taps - 1)); i < t1; ++i) ring[(size_t)((pos0 + i - t0) % taps) * C + c] = act_load(proj + (size_t)i * ldp + c);
         } else if (t - t0 >= taps - 1) {
-            u.put(it, conv_at(proj, ldp, conv_w, bias, nullptr, C, taps, t, t0, positions[t], c));
+            u.put(t, c, conv_at(proj, ldp, conv_w, bias, nullptr, C, taps, t, t0, positions[t], c));
         }
     }
 }
@@ -263,13 +281,13 @@ __global__ void __launch_bounds__(256) rglru_conv_runs_kernel(const float *__res
                     v.x = fmaf(w[j].x, in[i + j].x, v.x), v.y = fmaf(w[j].y, in[i + j].y, v.y);
                     v.z = fmaf(w[j].z, in[i + j].z, v.z), v.w = fmaf(w[j].w, in[i + j].w, v.w);
                 }
-                u.put4((size_t)t * C + c, v);
+                u.put4(t, c, v);
             } else if (t == t0) {
                 float *ring = state + (size_t)slots[s] * state_ld + C;
                 const int t1 = seq_start[s + 1], last = min(t1, t0 + max(TAPS - 1, 1)), pos0 = positions[t0];
                 for (int e = 0; e < 4; ++e) {
                     for (int k = t0; k < last; ++k)
-                        u.put((size_t)k * C + c + e, conv_at(proj, ldp, conv_w, __ldg(conv_b + c + e), ring, C, TAPS, k, t0, pos0 + k - t0, c + e));
+                        u.put(k, c + e, conv_at(proj, ldp, conv_w, __ldg(conv_b + c + e), ring, C, TAPS, k, t0, pos0 + k - t0, c + e));
                     if (TAPS > 1)
                         for (int k = max(t0, t1 - (TAPS - 1)); k < t1; ++k)
                             ring[(size_t)((pos0 + k - t0) % TAPS) * C + c + e] = act_load(proj + (size_t)k * ldp + c + e);
@@ -306,117 +324,68 @@ __global__ void __launch_bounds__(256) rglru_gates_rows_kernel(const float *__re
     ab[(size_t)(n + t0 + j) * C + c] = push;
 }
 
-// Many tokens in bfloat16 (mma.sync m16n8k16, float32 accumulation): a block of eight warps takes 128 tokens x 64 channels of one part, both
-// gates at once (128 columns), a warp 32 tokens x 32 channels.  u comes as three bfloat16 planes whose sum is the float32 number, each
-// multiplied by the same matrix piece: bfloat16 products are exact in float32, so only the sums round.  Two stages of cp.async.
-constexpr int GT = 128, GK = 32, GLD = GK + 8, GSTAGE = (3 * GT + 128) * GLD;
-__device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void load_matrix(uint32_t (&r)[4], const __nv_bfloat16 *p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)));
-}
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void copy16(const __nv_bfloat16 *dst, const __nv_bfloat16 *src, bool ok) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(ok ? 16 : 0) : "memory");
-}
-__global__ void __launch_bounds__(256, 2) rglru_gates_mma_kernel(const __nv_bfloat16 *__restrict__ u, const __nv_bfloat16 *__restrict__ ra,
-                                                                 const float *__restrict__ ra_b, const __nv_bfloat16 *__restrict__ ri,
-                                                                 const float *__restrict__ ri_b, const float *__restrict__ sp8, float *__restrict__ ab, int n,
-                                                                 int C, int P) {
-    pdl_trigger();
-    extern __shared__ __align__(16) __nv_bfloat16 gm[];
-    const int t0 = blockIdx.x * GT, b = blockIdx.z, k_out = blockIdx.y * 64;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, wm = warp & 3, wn = warp >> 2;
-    const int mat = lane >> 3, mrow = lane & 7;
-    const size_t plane = (size_t)n * C;
-    auto matrices = [&](int k0, int buf) {
-        __nv_bfloat16 *Bs = gm + (size_t)buf * GSTAGE + 3 * GT * GLD;
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const int e = threadIdx.x + 256 * i, r = e / (GK / 8), col = (e % (GK / 8)) * 8, o = k_out + (r & 63);
-            const bool ok = o < P && k0 + col < P;
-            copy16(Bs + r * GLD + col, (r < 64 ? ra : ri) + ((size_t)b * P + (ok ? o : 0)) * P + (ok ? k0 + col : 0), ok);
-        }
-    };
-    auto inputs = [&](int k0, int buf) {
-        __nv_bfloat16 *As = gm + (size_t)buf * GSTAGE;
-#pragma unroll
-        for (int i = 0; i < 6; ++i) {
-            const int e = threadIdx.x + 256 * i, r = e / (GK / 8), col = (e % (GK / 8)) * 8, piece = r / GT, t = t0 + r % GT;
-            const bool ok = t < n && k0 + col < P;
-            copy16(As + r * GLD + col, u + piece * plane + (ok ? (size_t)t * C + b * P + k0 + col : 0), ok);
-        }
-    };
-    matrices(0, 0);                 // the matrices depend on no earlier kernel
-    pdl_wait();
-    inputs(0, 0);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    float acc[2][8][4];
-#pragma unroll
-    for (int m = 0; m < 2; ++m)
-#pragma unroll
-        for (int i = 0; i < 8; ++i) acc[m][i][0] = acc[m][i][1] = acc[m][i][2] = acc[m][i][3] = 0.f;
-    const int n_k = (P + GK - 1) / GK;
-    for (int kt = 0; kt < n_k; ++kt) {
-        if (kt + 1 < n_k) {
-            matrices((kt + 1) * GK, (kt + 1) & 1);
-            inputs((kt + 1) * GK, (kt + 1) & 1);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
-        __syncthreads();
-        const __nv_bfloat16 *As = gm + (size_t)(kt & 1) * GSTAGE, *Bs = As + 3 * GT * GLD;
-#pragma unroll
-        for (int ks = 0; ks < GK / 16; ++ks) {
-            uint32_t q[4][4];
-#pragma unroll
-            for (int np = 0; np < 4; ++np)          // 0, 1: Ra's rows of this warp's channels; 2, 3: Ri's
-                load_matrix(q[np], Bs + ((np >> 1) * 64 + wn * 32 + (np & 1) * 16 + (mat >> 1) * 8 + mrow) * GLD + ks * 16 + (mat & 1) * 8);
-#pragma unroll
-            for (int piece = 2; piece >= 0; --piece)         // the small pieces first
-#pragma unroll
-                for (int m = 0; m < 2; ++m) {
-                    uint32_t a[4];
-                    load_matrix(a, As + (piece * GT + wm * 32 + m * 16 + (mat & 1) * 8 + mrow) * GLD + ks * 16 + (mat >> 1) * 8);
-#pragma unroll
-                    for (int np = 0; np < 4; ++np) {
-                        mma_bf16(acc[m][2 * np], a, q[np][0], q[np][1]);
-                        mma_bf16(acc[m][2 * np + 1], a, q[np][2], q[np][3]);
-                    }
-                }
-        }
-        __syncthreads();            // everyone is done with this buffer before it is filled again
+// Many tokens in bfloat16: the gates' logits come from a product on tensor cores over the inputs in pieces, z float32 [B rows, 2 P]: row b *
+// rows + t, the decay gate's at column k, the input gate's at P + k.  A thread takes two neighbouring channels of a token, or, with chunks, of a
+// chunk's tokens, and then also forms the chunk's product of a and its scan from zero (pass 1 of the recurrence below).
+struct GatePair {
+    float2 zr, zi, u;
+    __device__ __forceinline__ void load(const float *__restrict__ z, const AsPieces &in, int t, int c, int b, int k) {
+        const float *row = z + ((size_t)b * in.rows + t) * 2 * in.P + k;
+        zr = act_load(reinterpret_cast<const float2 *>(row)), zi = act_load(reinterpret_cast<const float2 *>(row + in.P));
+        u = in.get2(t, c);
     }
-    // accumulators 0..3: Ra's columns, 4..7: Ri's, the same channels in the same thread
+    __device__ __forceinline__ void finish(const float2 &br, const float2 &bi, const float2 &sp, float2 &a, float2 &push) const {
+        gate_pair(zr.x + br.x, zi.x + bi.x, sp.x, u.x, a.x, push.x);
+        gate_pair(zr.y + br.y, zi.y + bi.y, sp.y, u.y, a.y, push.y);
+    }
+};
+__global__ void __launch_bounds__(256) rglru_finish_kernel(const float *__restrict__ z, const AsPieces u, const float *__restrict__ ra_b,
+                                                           const float *__restrict__ ri_b, const float *__restrict__ sp8, float *__restrict__ ab, int n, int C) {
+    pdl_trigger();
+    pdl_wait();
+    const size_t total = (size_t)n * (C / 2);
+    for (size_t it = (size_t)blockIdx.x * blockDim.x + threadIdx.x; it < total; it += (size_t)gridDim.x * blockDim.x) {
+        const int t = (int)(it / (C / 2)), c = (int)(it - (size_t)t * (C / 2)) * 2, b = c / u.P;
+        GatePair g;
+        g.load(z, u, t, c, b, c - b * u.P);
+        float2 a, push;
+        g.finish(__ldg(reinterpret_cast<const float2 *>(ra_b + c)), __ldg(reinterpret_cast<const float2 *>(ri_b + c)), __ldg(reinterpret_cast<const float2 *>(sp8 + c)),
+                 a, push);
+        *reinterpret_cast<float2 *>(ab + (size_t)t * C + c) = a;
+        *reinterpret_cast<float2 *>(ab + ((size_t)n + t) * C + c) = push;
+    }
+}
+__global__ void __launch_bounds__(64) rglru_finish_chunks_kernel(const float *__restrict__ z, const AsPieces u, const float *__restrict__ ra_b,
+                                                                 const float *__restrict__ ri_b, const float *__restrict__ sp8, float *__restrict__ ab,
+                                                                 const int *__restrict__ chunks, float *__restrict__ A, float *__restrict__ B, int n, int C) {
+    pdl_trigger();
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 2, k = blockIdx.y;
+    if (c >= C) return;
+    const int b = c / u.P;
+    const float2 br = __ldg(reinterpret_cast<const float2 *>(ra_b + c)), bi = __ldg(reinterpret_cast<const float2 *>(ri_b + c));
+    const float2 sp = __ldg(reinterpret_cast<const float2 *>(sp8 + c));
+    pdl_wait();
+    const int t0 = chunks[2 * k], t1 = chunks[2 * k + 1];
+    float2 prod = make_float2(1.f, 1.f), S = make_float2(0.f, 0.f);
+    constexpr int W = 8;            // tokens whose loads are in flight together
+    for (int t = t0; t < t1; t += W) {
+        GatePair g[W];
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt) {
-        const int k = k_out + wn * 32 + nt * 8 + (lane & 3) * 2;
-        if (k >= P) continue;
-        const int c = b * P + k;          // P and so k and c are even
-        const float2 br = __ldg(reinterpret_cast<const float2 *>(ra_b + c)), bi = __ldg(reinterpret_cast<const float2 *>(ri_b + c));
-        const float2 sp = __ldg(reinterpret_cast<const float2 *>(sp8 + c));
+        for (int i = 0; i < W; ++i)
+            if (t + i < t1) g[i].load(z, u, t + i, c, b, c - b * u.P);
 #pragma unroll
-        for (int m = 0; m < 2; ++m)
-#pragma unroll
-            for (int rr = 0; rr < 2; ++rr) {
-                const int t = t0 + wm * 32 + m * 16 + (lane >> 2) + rr * 8;
-                if (t >= n) continue;
-                float2 uv = make_float2(0.f, 0.f);
-#pragma unroll
-                for (int piece = 2; piece >= 0; --piece) {
-                    const unsigned raw = act_load(reinterpret_cast<const unsigned *>(u + piece * plane + (size_t)t * C + c));
-                    uv.x += __uint_as_float(raw << 16), uv.y += __uint_as_float(raw & 0xffff0000u);
-                }
+        for (int i = 0; i < W; ++i)
+            if (t + i < t1) {
                 float2 a, p;
-                gate_pair(acc[m][nt][rr * 2] + br.x, acc[m][nt + 4][rr * 2] + bi.x, sp.x, uv.x, a.x, p.x);
-                gate_pair(acc[m][nt][rr * 2 + 1] + br.y, acc[m][nt + 4][rr * 2 + 1] + bi.y, sp.y, uv.y, a.y, p.y);
-                *reinterpret_cast<float2 *>(ab + (size_t)t * C + c) = a;
-                *reinterpret_cast<float2 *>(ab + (size_t)(n + t) * C + c) = p;
+                g[i].finish(br, bi, sp, a, p);
+                *reinterpret_cast<float2 *>(ab + (size_t)(t + i) * C + c) = a;
+                *reinterpret_cast<float2 *>(ab + ((size_t)n + t + i) * C + c) = p;
+                S.x = fmaf(a.x, S.x, p.x), S.y = fmaf(a.y, S.y, p.y);
+                prod.x *= a.x, prod.y *= a.y;
             }
     }
+    *reinterpret_cast<float2 *>(A + (size_t)k * C + c) = prod;
+    *reinterpret_cast<float2 *>(B + (size_t)k * C + c) = S;
 }
 
 // ---- the recurrence ---------------------------------------------------------------------------------------
@@ -569,37 +538,25 @@ static int conv_run(const float *proj, int ldp, const float *conv_w, const float
     return lgml_launch_status("rglru_conv");
 }
 
-// u: float32 [n, C], or (pieces = 1) bfloat16 [3, n, C], three numbers whose sum is the float32 one
+// u: float32 [n, C], or (part > 0) bfloat16 [C / part * rows, 3 part], three numbers whose sum is the float32 one (AsPieces)
 LGML_API int lgml_rglru_conv(const float *proj, int ldp, const float *conv_w, const float *conv_b, float *state, long long state_ld, const int *seq_of_token,
-                             const int *seq_start, const int *slots, const int *positions, void *u, int pieces, int n_tokens, int C, int taps, cudaStream_t stream) {
+                             const int *seq_start, const int *slots, const int *positions, void *u, int part, int rows, int n_tokens, int C, int taps, cudaStream_t stream) {
     LGML_REQUIRE(n_tokens >= 0 && C > 0 && taps >= 1 && taps <= MAX_TAPS && ldp >= C && state_ld >= C + (taps > 1 ? (long long)taps * C : 0), "rglru_conv: bad sizes");
     if (n_tokens == 0) return 0;
     const bool vec = C % 4 == 0 && ldp % 4 == 0 && (((uintptr_t)proj | (uintptr_t)conv_w | (uintptr_t)conv_b | (uintptr_t)u) & 15) == 0;
-    if (pieces)
-        return conv_run(proj, ldp, conv_w, conv_b, state, state_ld, seq_of_token, seq_start, slots, positions, AsPieces{(__nv_bfloat16 *)u, (size_t)n_tokens * C},
-                        vec, n_tokens, C, taps, stream);
-    return conv_run(proj, ldp, conv_w, conv_b, state, state_ld, seq_of_token, seq_start, slots, positions, AsFloat{(float *)u}, vec, n_tokens, C, taps, stream);
+    if (part) {
+        LGML_REQUIRE(part > 0 && part % 8 == 0 && C % part == 0 && rows >= n_tokens, "rglru_conv: pieces of parts of %d channels, %d rows a part", part, rows);
+        return conv_run(proj, ldp, conv_w, conv_b, state, state_ld, seq_of_token, seq_start, slots, positions, AsPieces{(__nv_bfloat16 *)u, rows, part}, vec, n_tokens,
+                        C, taps, stream);
+    }
+    return conv_run(proj, ldp, conv_w, conv_b, state, state_ld, seq_of_token, seq_start, slots, positions, AsFloat{(float *)u, C}, vec, n_tokens, C, taps, stream);
 }
 
-// ab float32 [2, n, C].  u float32 [n, C] (products of 8 rows), or (pieces = 1) bfloat16 [3, n, C] (tensor cores: bfloat16 matrices, parts and
-// channels that are multiples of 8).
-LGML_API int lgml_rglru_gates(const void *u_any, int pieces, const void *ra, const float *ra_b, const void *ri, const float *ri_b, const float *sp8, float *ab,
+// The gates as products of 8 rows: u float32 [n, C] -> ab float32 [2, n, C].
+LGML_API int lgml_rglru_gates(const float *u, const void *ra, const float *ra_b, const void *ri, const float *ri_b, const float *sp8, float *ab,
                               int dtype, int n_tokens, int C, int P, cudaStream_t stream) {
     RGLRU_SIZES("rglru_gates");
     if (n_tokens == 0) return 0;
-    if (pieces) {
-        LGML_REQUIRE(dtype == LGML_BF16 && P % 8 == 0 &&
-                         (((uintptr_t)u_any | (uintptr_t)ra | (uintptr_t)ri | (uintptr_t)ra_b | (uintptr_t)ri_b | (uintptr_t)sp8 | (uintptr_t)ab) & 15) == 0,
-                     "rglru_gates: the tensor-core form takes bfloat16 matrices and parts that are multiples of 8, on 16-byte borders");
-        const size_t smem = sizeof(__nv_bfloat16) * 2 * (size_t)GSTAGE;
-        cudaError_t e = cudaFuncSetAttribute(rglru_gates_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) LGML_FAIL("rglru_gates: cannot have %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
-        dim3 grid((n_tokens + GT - 1) / GT, (P + 63) / 64, C / P);
-        lgml_launch(rglru_gates_mma_kernel, grid, 256, smem, stream, (const __nv_bfloat16 *)u_any, (const __nv_bfloat16 *)ra, ra_b, (const __nv_bfloat16 *)ri, ri_b,
-                    sp8, ab, n_tokens, C, P);
-        return lgml_launch_status("rglru_gates");
-    }
-    const float *u = (const float *)u_any;
     const size_t smem = sizeof(float) * NT * (size_t)((P + 3) & ~3);
     LGML_REQUIRE(smem <= 48 * 1024, "rglru_gates: parts of %d channels are too wide", P);
     dim3 grid((n_tokens + NT - 1) / NT, C / P, (P + CH - 1) / CH);
@@ -610,6 +567,25 @@ LGML_API int lgml_rglru_gates(const void *u_any, int pieces, const void *ra, con
         lgml_launch(rglru_gates_rows_kernel<__nv_bfloat16>, grid, 256, smem, stream, u, (const __nv_bfloat16 *)ra, ra_b, (const __nv_bfloat16 *)ri, ri_b, sp8, ab,
                     n_tokens, C, P, few_rows_lanes<__nv_bfloat16>(P), few_rows_vec<__nv_bfloat16>(ra, P) && few_rows_vec<__nv_bfloat16>(ri, P) ? 1 : 0);
     return lgml_launch_status("rglru_gates");
+}
+
+// The gates from their logits: z float32 [C / P * rows, 2 P] over the inputs in pieces u bfloat16 [C / P * rows, 3 P].  With chunks (int32 [n_chunks, 2]) also
+// every chunk's product of a and scan from zero, scratch float32 [2, n_chunks, C].
+LGML_API int lgml_rglru_finish(const float *z, const void *u, int rows, const float *ra_b, const float *ri_b, const float *sp8, float *ab, const int *chunks,
+                               int n_chunks, float *scratch, int n_tokens, int C, int P, cudaStream_t stream) {
+    LGML_REQUIRE(n_tokens >= 0 && C > 0 && P > 0 && C % P == 0 && P % 8 == 0 && rows >= n_tokens && n_chunks >= 0 && n_chunks <= 65535, "rglru_finish: bad sizes");
+    LGML_REQUIRE((((uintptr_t)z | (uintptr_t)u | (uintptr_t)ra_b | (uintptr_t)ri_b | (uintptr_t)sp8 | (uintptr_t)ab | (uintptr_t)scratch) & 15) == 0,
+                 "rglru_finish: operands must be 16-byte aligned");
+    if (n_tokens == 0) return 0;
+    const AsPieces in{(__nv_bfloat16 *)u, rows, P};
+    if (chunks != nullptr) {
+        lgml_launch(rglru_finish_chunks_kernel, dim3((C / 2 + 63) / 64, n_chunks), 64, 0, stream, z, in, ra_b, ri_b, sp8, ab, chunks, scratch,
+                    scratch + (size_t)n_chunks * C, n_tokens, C);
+    } else {
+        const size_t items = ((size_t)n_tokens * (C / 2) + 255) / 256;
+        lgml_launch(rglru_finish_kernel, (int)(items < 148 * 16 ? items : 148 * 16), 256, 0, stream, z, in, ra_b, ri_b, sp8, ab, n_tokens, C);
+    }
+    return lgml_launch_status("rglru_finish");
 }
 
 LGML_API int lgml_rglru_scan(const float *ab, const float *proj, int ldp, float *state, long long state_ld, const int *seq_start, const int *slots, void *out,
@@ -626,14 +602,16 @@ LGML_API int lgml_rglru_scan(const float *ab, const float *proj, int ldp, float 
     return lgml_launch_status("rglru_scan");
 }
 
-// chunks int32 [n_chunks, 2]: token rows [first, past the last), a request's chunks in a row; chunk_start int32 [n_seqs + 1]; scratch float32 [2, n_chunks, C]
+// chunks int32 [n_chunks, 2]: token rows [first, past the last), a request's chunks in a row; chunk_start int32 [n_seqs + 1]; scratch float32 [2, n_chunks, C],
+// with ends_known = 1 already holding pass 1's results (lgml_rglru_finish)
 LGML_API int lgml_rglru_chunks(const float *ab, const float *proj, int ldp, float *state, long long state_ld, const int *chunks, const int *chunk_start,
-                               int n_chunks, const int *slots, float *scratch, void *out, int dtype, int n_tokens, int n_seqs, int C, cudaStream_t stream) {
+                               int n_chunks, const int *slots, float *scratch, int ends_known, void *out, int dtype, int n_tokens, int n_seqs, int C,
+                               cudaStream_t stream) {
     LGML_REQUIRE(n_tokens >= 0 && n_chunks >= 0 && n_chunks <= 65535 && n_seqs >= 0 && n_seqs <= 65535 && C > 0 && ldp >= 2 * C && state_ld >= C, "rglru_chunks: bad sizes");
     if (n_chunks == 0) return 0;
     float *A = scratch, *B = scratch + (size_t)n_chunks * C;
     dim3 grid((C + 127) / 128, n_chunks), chain((C + 127) / 128, n_seqs);
-    lgml_launch(rglru_chunk_ends_kernel, grid, 128, 0, stream, ab, chunks, A, B, n_tokens, C);
+    if (!ends_known) lgml_launch(rglru_chunk_ends_kernel, grid, 128, 0, stream, ab, chunks, A, B, n_tokens, C);
     lgml_launch(rglru_chain_kernel, chain, 128, 0, stream, (const float *)A, B, chunk_start, state, state_ld, slots, C);
     if (dtype == LGML_F32)
         lgml_launch(rglru_chunk_scan_kernel<float>, grid, 128, 0, stream, ab, proj, ldp, chunks, (const float *)B, (float *)out, n_tokens, C);

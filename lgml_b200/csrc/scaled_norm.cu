@@ -78,11 +78,11 @@ __device__ __forceinline__ void store4(__nv_bfloat16 *p, int i, int E, int vec, 
 }
 
 // A block a row; thread i holds the quads i, i + threads, ... of it (NQ of them).  The number of threads is the width's, so that a
-// row's sums are formed in one order whatever else is in the batch.
+// row's sums are formed in one order whatever else is in the batch (but for few bfloat16 rows, which get a thread a quad).
 // PARTS: A comes in several parts (or halves): up to eight of them are in flight at a time.  Without them, for many rows, a
 // thread needs few enough registers for two blocks or more an SM.
 template <typename TO, int NQ, bool PARTS>
-__global__ void __launch_bounds__(NQ > 4 ? 1024 : 512, NQ > 2 || PARTS ? 1 : 2) scaled_norm_kernel(const Args a) {
+__global__ void __launch_bounds__(NQ > 4 || (NQ == 1 && PARTS) ? 1024 : 512, NQ > 2 || PARTS ? 1 : 2) scaled_norm_kernel(const Args a) {
     pdl_trigger();
     pdl_wait();
     __shared__ float red[32];
@@ -120,7 +120,7 @@ __global__ void __launch_bounds__(NQ > 4 ? 1024 : 512, NQ > 2 || PARTS ? 1 : 2) 
         if (ar) {
             if (PARTS) {
                 // the other parts (a row's halves one after the other), added in their order
-                constexpr int W = NQ > 4 ? 2 : 8;
+                constexpr int W = NQ > 4 ? 2 : (NQ == 1 ? 6 : 8);
                 const int total = a.a_second ? 2 * a.n_parts : a.n_parts;
                 for (int p = 1; p < total; p += W) {
                     float o[W][4];
@@ -211,6 +211,7 @@ int launch(const Args &a, int n_rows, cudaStream_t stream) {
         else lgml_launch(scaled_norm_kernel<TO, NQ, false>, n_rows, threads(NQ), 0, stream, a);                  \
     } while (0)
     if (quads <= 256) LGML_SN(1);
+    else if (sizeof(TO) == 2 && parts && n_rows <= 64 && quads <= 1024) LGML_SN(1);      // few rows: a thread a quad (a decode step is latency)
     else if (quads <= 1024) LGML_SN(2);
     else if (quads <= 2048) LGML_SN(4);
     else if (quads <= 8192) LGML_SN(8);

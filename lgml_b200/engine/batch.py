@@ -178,14 +178,18 @@ class StepBatch:
         alone at the end.  Made once per tile size."""
         cached = self._tiles.get(tile_tokens)
         if cached is None:
-            rows = []
-            start = 0
+            pieces, start = [], 0
             for s, n in enumerate(self.seq_lens):
-                for t0 in range(0, n, tile_tokens):
-                    rows.append((s, start + t0, min(tile_tokens, n - t0), self.pos0[s] + min(t0 + tile_tokens, n)))
+                t0 = np.arange(0, n, tile_tokens, dtype=np.int32)
+                part = np.empty((t0.size, 4), dtype=np.int32)
+                part[:, 0] = s
+                part[:, 1] = start + t0
+                part[:, 2] = np.minimum(tile_tokens, n - t0)
+                part[:, 3] = self.pos0[s] + np.minimum(t0 + tile_tokens, n)         # how far it has to look
+                pieces.append(part)
                 start += n
-            rows.sort(key=lambda r: -r[3])
-            arr = np.asarray(rows, dtype=np.int32).reshape(-1, 4)
+            arr = np.concatenate(pieces) if pieces else np.zeros((0, 4), dtype=np.int32)
+            arr = arr[np.argsort(-arr[:, 3], kind="stable")]
             arr[:, 3] = 0
             cached = self._to_device(arr.reshape(-1)).view(-1, 4)
             self._tiles[tile_tokens] = cached
@@ -214,14 +218,14 @@ class StepBatch:
         piece size."""
         cached = self._tiles.get(("pieces", piece_tokens))
         if cached is None:
-            pieces, first = [], [0]
-            start = 0
-            for n in self.seq_lens:
-                for t0 in range(0, n, piece_tokens):
-                    pieces.append((start + t0, start + min(t0 + piece_tokens, n)))
-                first.append(len(pieces))
-                start += n
-            both = self._to_device(np.concatenate([np.asarray(pieces, dtype=np.int32).reshape(-1), np.asarray(first, dtype=np.int32)]))
+            lens = np.asarray(self.seq_lens, dtype=np.int64)
+            counts = -(-lens // piece_tokens)
+            first = np.concatenate([[0], np.cumsum(counts)])
+            ends = np.cumsum(lens)
+            of = np.repeat(np.arange(len(lens)), counts)                              # the request of every piece
+            lo = (ends - lens)[of] + (np.arange(first[-1]) - first[of]) * piece_tokens
+            pieces = np.stack([lo, np.minimum(lo + piece_tokens, ends[of])], axis=1)
+            both = self._to_device(np.concatenate([pieces.reshape(-1), first]).astype(np.int32))
             cached = (both[:2 * len(pieces)].view(-1, 2), both[2 * len(pieces):])
             self._tiles[("pieces", piece_tokens)] = cached
         return cached

@@ -9,6 +9,8 @@
     python -m lgml_b200.kernel_bench token_side --rows 8 --width 4096 --dim 64
     python -m lgml_b200.kernel_bench chunk_scan --rows 2048 --heads 16 --kv-heads 8 --dim 128 --vdim 128 [--memory]
     python -m lgml_b200.kernel_bench stream_norm --rows 2048 --width 4096 --streams 2
+    python -m lgml_b200.kernel_bench scaled_norm --rows 2048 --width 4096 [--top 2] [--parts 9]
+    python -m lgml_b200.kernel_bench rglru --rows 2048 --width 4096 --part 256 [--requests 8]
 
 Each case is run over a ring of input buffers larger than the L2 cache, so that weights and
 cache pages come from HBM as they do in a decode step; warm-up launches first, then the timed
@@ -264,6 +266,66 @@ def case_stream_norm(a) -> None:
     print(f"stream_norm rows={n} width={E} streams={R}: {us:.2f} us, {byts / us / 1e3:.0f} GB/s")
 
 
+def case_scaled_norm(a) -> None:
+    """The seam between two parallel layers: a product (or its partial sums) and each token's experts, scaled channel by channel, into the
+    stream; the norm; its rows again into the experts' tiles."""
+    n, E, top = a.rows, a.width, a.top
+    nb = min(ring(n * E * 4 * (a.parts + top + 1)), 8)
+    xs = [torch.randn(n, E, device=DEV) for _ in range(nb)]
+    ds = [torch.randn(a.parts, n, E, device=DEV) for _ in range(nb)]
+    ys = [torch.randn(n * top, E, device=DEV) for _ in range(nb)]
+    places = torch.randperm(n * top, device=DEV).to(torch.int32).view(n, top)
+    w, s1, s2 = (torch.ones(E, device=DEV) for _ in range(3))
+    out = torch.empty(n, E, dtype=torch.bfloat16, device=DEV)
+    tiles = torch.empty(n * top, E, dtype=torch.bfloat16, device=DEV)
+
+    def run(i):
+        value = ops.Partials(ds[i]) if a.parts > 1 else ds[i][0]
+        ops.scaled_norm(xs[i], (ops.Term(value, s1), ops.Term(ops.ExpertRows(ys[i], places, 1.0 / top), s2)), 1e-6, w, out, tiles=tiles, places=places)
+
+    us = timed(run, nb, a.warmup, a.iters)
+    byts = n * E * (8 + 4 * a.parts + 4 * top + 2 + 2 * top)
+    print(f"scaled_norm rows={n} width={E} parts={a.parts} experts={top}: {us:.2f} us, {byts / us / 1e3:.0f} GB/s")
+
+
+def case_rglru(a) -> None:
+    """The gated linear recurrence between its projections: one token of every request (one kernel), or one request's portion
+    (convolution, the gates' product, the gates and the chunks' ends, the chain, the scan)."""
+    C, P, taps = a.width, a.part, 4
+    B = C // P
+    n = a.requests if a.requests > 1 else a.rows
+    nb = min(ring(n * C * 8), 8)
+    bufs = [torch.randn(n, 2 * C, device=DEV) for _ in range(nb)]
+    conv_w, conv_b = torch.randn(taps, C, device=DEV), torch.zeros(C, device=DEV)
+    ra, ri = ((torch.randn(B, P, P, device=DEV) / P ** 0.5).to(torch.bfloat16) for _ in range(2))
+    rb, sp8 = torch.zeros(C, device=DEV), torch.full((C,), 0.2, device=DEV)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=DEV)
+    slots = i32(list(range(a.requests)))
+    state = torch.zeros(a.requests, ops.rglru_state_floats(C, taps), device=DEV)
+    if a.requests > 1:
+        pos = i32([9] * n)
+        us = timed(lambda i: ops.rglru_step(bufs[i], conv_w, conv_b, state, slots, pos, ra, rb, ri, rb, sp8), nb, a.warmup, a.iters)
+        byts = 4 * B * P * P + n * C * (8 + 8 + 4 * taps + 2)
+        print(f"rglru step requests={n} channels={C} parts of {P}: {us:.2f} us, {byts / us / 1e3:.0f} GB/s")
+        return
+    rows, tile = ops.rglru_pieces_rows(n)
+    w = ops.rglru_pieces_matrices(ra, ri)
+    tiles = i32([v for b in range(B) for _ in range(rows // tile) for v in (b, 0, 0)] + [B * (rows // tile)])
+    status, step = torch.zeros(1, dtype=torch.int32, device=DEV), ops.rglru_chunk_tokens()
+    chunks = i32([(t, min(t + step, n)) for t in range(0, n, step)])
+    first, seq, start, pos = i32([0, chunks.shape[0]]), i32([0] * n), i32([0, n]), i32(list(range(n)))
+    out = torch.empty(n, C, dtype=torch.bfloat16, device=DEV)
+    conv = lambda i: ops.rglru_conv(bufs[i], conv_w, conv_b, state, seq, start, slots, pos, part=P)
+    u = conv(0)
+    gates = lambda i: ops.rglru_gates_pieces(u, n, w, tiles, rb, rb, sp8, status, chunks=chunks)
+    ab, ends = gates(0)
+    scan = lambda i: ops.rglru_scan(ab, bufs[i], state, start, slots, out, chunks, first, ends=ends.clone())
+    t_conv, t_gates, t_scan = (timed(f, nb, a.warmup, a.iters) for f in (conv, gates, scan))
+    print(f"rglru rows={n} channels={C} parts of {P}: convolution {t_conv:.2f} us ({n * C * 10 / t_conv / 1e3:.0f} GB/s), gates {t_gates:.2f} us "
+          f"({4.0 * n * C * P / t_gates / 1e6:.0f} TFLOP/s of float32 products, three times that on the tensor cores), scan {t_scan:.2f} us "
+          f"({n * C * 14 / t_scan / 1e3:.0f} GB/s)")
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="python -m lgml_b200.kernel_bench")
     ap.add_argument("--warmup", type=int, default=5)
@@ -311,6 +373,12 @@ def main(argv=None) -> int:
     c = sub.add_parser("stream_norm")
     for name, size in (("rows", 2048), ("width", 4096), ("streams", 2)):
         c.add_argument("--" + name, type=int, default=size)
+    c = sub.add_parser("scaled_norm")
+    for name, size in (("rows", 2048), ("width", 4096), ("top", 2), ("parts", 1)):
+        c.add_argument("--" + name, type=int, default=size)
+    c = sub.add_parser("rglru")
+    for name, size in (("rows", 2048), ("width", 4096), ("part", 256), ("requests", 1)):
+        c.add_argument("--" + name, type=int, default=size)
     a = ap.parse_args(argv)
     global USE_GRAPH
     USE_GRAPH = not a.no_graph
@@ -319,7 +387,7 @@ def main(argv=None) -> int:
         return 1
     {"gemm": case_gemm, "decode_attention": case_decode_attention, "prefill_attention": case_prefill_attention, "rmsnorm": case_rmsnorm,
      "token_shift": case_token_shift, "mingru": case_mingru, "token_side": case_token_side, "chunk_scan": case_chunk_scan,
-     "stream_norm": case_stream_norm}[a.case](a)
+     "stream_norm": case_stream_norm, "scaled_norm": case_scaled_norm, "rglru": case_rglru}[a.case](a)
     return 0
 
 

@@ -1324,55 +1324,95 @@ def rglru_step(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, s
     return out
 
 
-def rglru_pieces_supported(ra: torch.Tensor, n_tokens: int) -> bool:
-    """Whether the gates of a step of that many tokens run on tensor cores, from inputs in three bfloat16 pieces."""
-    return n_tokens >= 32 and ra.dtype == torch.bfloat16 and ra.shape[1] % 8 == 0
+def rglru_pieces_rows(n_tokens: int) -> int:
+    """(rows a part gets, rows of a tile) for a step's inputs in pieces: whole tiles of the grouped product."""
+    tile = 32 if n_tokens <= 32 else (64 if n_tokens <= 64 else MOE_TILE_ROWS)
+    return -(-n_tokens // tile) * tile, tile
 
 
 def rglru_conv(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, state: torch.Tensor, seq_of_token: torch.Tensor, seq_start: torch.Tensor,
-               slots: torch.Tensor, positions: torch.Tensor, pieces: bool = False) -> torch.Tensor:
+               slots: torch.Tensor, positions: torch.Tensor, part: int = 0) -> torch.Tensor:
     """The causal convolution of ``proj``'s first C columns, float32 [tokens, C]; the inputs of earlier steps come from the ring in
-    the request's state, which takes the step's last ones.  ``pieces``: the result as bfloat16 [3, tokens, C], three numbers
-    whose sum is the float32 one (8 + 8 + 8 bits)."""
+    the request's state, which takes the step's last ones.  ``part`` > 0: the result in three bfloat16 pieces whose sum is the float32
+    number (8 + 8 + 8 bits), [C / part, rows, 3, part] with ``rglru_pieces_rows`` rows of which the first ``tokens`` are written."""
     _need(proj, "projections", torch.float32, 2)
     C = conv_b.numel()
     taps = _conv_shapes(conv_w, conv_b, C, "rglru_conv")
     n, ldp = proj.shape[0], _rows_contiguous(proj, "projections")
-    if proj.shape[1] < C or positions.numel() != n or seq_of_token.numel() != n:
-        raise KernelError(f"rglru_conv: projections {tuple(proj.shape)} hold no {C} channels")
+    if proj.shape[1] < C or positions.numel() != n or seq_of_token.numel() != n or (part and C % part):
+        raise KernelError(f"rglru_conv: projections {tuple(proj.shape)} hold no {C} channels in parts of {part}")
     ld = _state_rows(state, rglru_state_floats(C, taps), "rglru_conv")
-    u = torch.empty((3, n, C), dtype=torch.bfloat16, device=proj.device) if pieces else torch.empty((n, C), dtype=torch.float32, device=proj.device)
+    rows = rglru_pieces_rows(n)[0] if part else n
+    u = torch.empty((C // part, rows, 3, part), dtype=torch.bfloat16, device=proj.device) if part else torch.empty((n, C), dtype=torch.float32, device=proj.device)
     fn = _fn("rglru", "lgml_rglru_conv", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                          c_int, c_int, c_void_p])
+                                          c_int, c_int, c_int, c_void_p])
     _check("rglru", fn(_ptr(proj), ldp, _ptr(conv_w), _ptr(conv_b), _ptr(state), ld, _ptr(seq_of_token), _ptr(seq_start), _ptr(slots), _ptr(positions), _ptr(u),
-                       1 if pieces else 0, n, C, taps, _stream()), "rglru_conv")
+                       int(part), rows, n, C, taps, _stream()), "rglru_conv")
     return u
 
 
 def rglru_gates(u: torch.Tensor, ra: torch.Tensor, ra_b: torch.Tensor, ri: torch.Tensor, ri_b: torch.Tensor, sp8: torch.Tensor) -> torch.Tensor:
-    """From the convolved inputs ``u`` (float32 [tokens, C], or bfloat16 [3, tokens, C] as ``rglru_conv(pieces=True)`` gives them): float32
-    [2, tokens, C], the decay a = exp(-sigmoid(Ra u + ra_b) sp8) and the pushed term sqrt(1 - a^2) sigmoid(Ri u + ri_b) u, Ra and Ri
-    block-diagonal [parts, P, P].  The products are true 32-bit sums over the float32 u in both forms."""
-    pieces = u.dtype == torch.bfloat16
-    B, P, _ = ra.shape
-    C = B * P
-    _need(u, "convolved inputs", torch.bfloat16 if pieces else torch.float32, 3 if pieces else 2)
-    _rglru_shapes(None, ra, ra_b, ri, ri_b, sp8, "rglru_gates")
-    n = u.shape[-2]
-    if tuple(u.shape) != ((3, n, C) if pieces else (n, C)) or not u.is_contiguous():
+    """From the convolved inputs ``u`` float32 [tokens, C]: float32 [2, tokens, C], the decay a = exp(-sigmoid(Ra u + ra_b) sp8) and the
+    pushed term sqrt(1 - a^2) sigmoid(Ri u + ri_b) u, Ra and Ri block-diagonal [parts, P, P]; float32 sums over the float32 u."""
+    C, P = _rglru_shapes(u, ra, ra_b, ri, ri_b, sp8, "rglru_gates")
+    n = u.shape[0]
+    if u.shape[1] != C or not u.is_contiguous():
         raise KernelError(f"rglru_gates: inputs {tuple(u.shape)} do not fit {C} channels")
     ab = torch.empty((2, n, C), dtype=torch.float32, device=u.device)
-    fn = _fn("rglru", "lgml_rglru_gates", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-    _check("rglru", fn(_ptr(u), 1 if pieces else 0, _ptr(ra), _ptr(ra_b), _ptr(ri), _ptr(ri_b), _ptr(sp8), _ptr(ab), dtype_code(ra.dtype), n, C, P, _stream()),
-           "rglru_gates")
+    fn = _fn("rglru", "lgml_rglru_gates", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check("rglru", fn(_ptr(u), _ptr(ra), _ptr(ra_b), _ptr(ri), _ptr(ri_b), _ptr(sp8), _ptr(ab), dtype_code(ra.dtype), n, C, P, _stream()), "rglru_gates")
     return ab
 
 
+def rglru_pieces_matrices(ra: torch.Tensor, ri: torch.Tensor) -> torch.Tensor:
+    """The gates' matrices as the product over inputs in pieces wants them: [parts, 2 P, 3 P], per part [Ra | Ra | Ra] above [Ri | Ri | Ri]."""
+    return torch.cat([ra, ri], dim=1).repeat(1, 1, 3).contiguous()
+
+
+def rglru_gates_pieces(u: torch.Tensor, n_tokens: int, w: torch.Tensor, tiles: torch.Tensor, ra_b: torch.Tensor, ri_b: torch.Tensor, sp8: torch.Tensor,
+                       status: torch.Tensor, chunks: Optional[torch.Tensor] = None):
+    """``rglru_gates`` for many tokens on tcgen05: ``u`` bfloat16 [parts, rows, 3, P] (``rglru_conv(part=P)``), ``w`` as ``rglru_pieces_matrices`` gives
+    it; one grouped product (``tiles`` int32: the part of every tile of rows, then how many tiles, as ``moe_tile_products`` takes them),
+    whose products are exact and whose sums are float32, then the gates.  With ``chunks`` the second result is every chunk's product of
+    decays and scan from zero (float32 [2, chunks, C]), which ``rglru_scan`` then need not form."""
+    _need(u, "inputs in pieces", torch.bfloat16, 4)
+    _need(w, "gates' matrices", torch.bfloat16, 3)
+    _need(tiles, "tiles", torch.int32, 1)
+    B, rows, _, P = u.shape
+    C, tile = B * P, rglru_pieces_rows(n_tokens)[1]
+    n_tiles = B * (rows // tile)
+    if rows != rglru_pieces_rows(n_tokens)[0] or tuple(w.shape) != (B, 2 * P, 3 * P) or not u.is_contiguous() or not w.is_contiguous() or P % 8 \
+            or tiles.numel() != 3 * n_tiles + 1 or not tiles.is_contiguous():
+        raise KernelError(f"rglru_gates_pieces: inputs {tuple(u.shape)} / matrices {tuple(w.shape)} / tiles {tuple(tiles.shape)} do not fit {n_tokens} tokens")
+    for t, what in ((ra_b, "decay gate's bias"), (ri_b, "input gate's bias"), (sp8, "decay rates")):
+        _need(t, what, torch.float32)
+        if t.numel() != C or not t.is_contiguous():
+            raise KernelError(f"rglru_gates_pieces: the {what} hold one number per channel")
+    z = torch.empty((B * rows, 2 * P), dtype=torch.float32, device=u.device)
+    stream = _stream()
+    fn = _fn("gemm_tcgen05", "lgml_gemm_tcgen05_grouped_tiles", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
+                                                                 c_float, c_float, c_void_p, c_void_p], label="gemm_tcgen05_grouped")
+    _check("gemm_tcgen05", fn(_ptr(u), _ptr(w), _ptr(z), 1, n_tiles, tile, 2 * P, 3 * P, B, 2 * P, _ptr(tiles), 0, 0.0, 0.0, _ptr(status), stream),
+           "gemm_tcgen05_grouped")
+    ab = torch.empty((2, n_tokens, C), dtype=torch.float32, device=u.device)
+    ends, n_chunks = None, 0
+    if chunks is not None:
+        _need(chunks, "chunks", torch.int32, 2)
+        n_chunks = chunks.shape[0]
+        ends = torch.empty((2, n_chunks, C), dtype=torch.float32, device=u.device)
+    fn = _fn("rglru", "lgml_rglru_finish", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
+                                            c_void_p])
+    _check("rglru", fn(_ptr(z), _ptr(u), rows, _ptr(ra_b), _ptr(ri_b), _ptr(sp8), _ptr(ab), _ptr(chunks), n_chunks, _ptr(ends), n_tokens, C, P, stream),
+           "rglru_finish")
+    return ab, ends
+
+
 def rglru_scan(ab: torch.Tensor, proj: torch.Tensor, state: torch.Tensor, seq_start: torch.Tensor, slots: torch.Tensor, out: torch.Tensor,
-               chunks: Optional[torch.Tensor] = None, chunk_start: Optional[torch.Tensor] = None) -> torch.Tensor:
+               chunks: Optional[torch.Tensor] = None, chunk_start: Optional[torch.Tensor] = None, ends: Optional[torch.Tensor] = None) -> torch.Tensor:
     """S <- a S + push over every request's tokens of this step, from ``state[slot]`` (which takes the last S); out[t] = S_t *
     gelu_tanh(y_t), y the columns C .. 2 C - 1 of ``proj``.  ``ab`` as ``rglru_gates`` gives it.  With ``chunks`` and ``chunk_start``
-    (``StepBatch.scan_pieces``) the pieces of a request's portion run side by side."""
+    (``StepBatch.scan_pieces``) the pieces of a request's portion run side by side; ``ends``: what ``rglru_gates_pieces`` knows of them already
+    (used up)."""
     _need(ab, "decays and pushed terms", torch.float32, 3)
     _need(proj, "projections", torch.float32, 2)
     _need(out, "recurrence output", ndim=2)
@@ -1392,10 +1432,13 @@ def rglru_scan(ab: torch.Tensor, proj: torch.Tensor, state: torch.Tensor, seq_st
     n_chunks = chunks.shape[0]
     if chunks.shape[1] != 2 or not chunks.is_contiguous() or chunk_start.numel() != n_seqs + 1:
         raise KernelError("rglru_scan: chunks are [n, 2] and chunk starts one more than the requests")
-    scratch = torch.empty((2, n_chunks, C), dtype=torch.float32, device=ab.device)
-    fn = _fn("rglru", "lgml_rglru_chunks", [c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                            c_int, c_int, c_void_p])
-    _check("rglru", fn(_ptr(ab), _ptr(proj), ldp, _ptr(state), ld, _ptr(chunks), _ptr(chunk_start), n_chunks, _ptr(slots), _ptr(scratch), _ptr(out),
+    if ends is not None and (tuple(ends.shape) != (2, n_chunks, C) or not ends.is_contiguous()):
+        raise KernelError(f"rglru_scan: chunk ends {tuple(ends.shape)} are not [2, {n_chunks}, {C}]")
+    scratch = torch.empty((2, n_chunks, C), dtype=torch.float32, device=ab.device) if ends is None else ends
+    fn = _fn("rglru", "lgml_rglru_chunks", [c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int,
+                                            c_int, c_int, c_int, c_void_p])
+    _check("rglru", fn(_ptr(ab), _ptr(proj), ldp, _ptr(state), ld, _ptr(chunks), _ptr(chunk_start), n_chunks, _ptr(slots), _ptr(scratch),
+                       0 if ends is None else 1, _ptr(out),
                        dtype_code(out.dtype), n, n_seqs, C, _stream()), "rglru_chunks")
     return out
 

@@ -22,6 +22,8 @@ from .base import Part, register_part
 
 # portions of a request longer than this run the recurrence in pieces side by side
 RGLRU_PIECES_FROM = 64
+# tokens of a step from which the gates' products run on tensor cores (bfloat16)
+RGLRU_PRODUCTS_FROM = 32
 
 
 class RealGatedLRU(Part):
@@ -32,7 +34,8 @@ class RealGatedLRU(Part):
             raise ValueError(f"{inner} channels do not fall into {blocks} equal parts")
         self.width, self.inner, self.blocks, self.taps = width, inner, blocks, taps
         self.w_in = self.b_in = self.wo = self.conv_w = self.conv_b = self.sp8 = None
-        self.ra = self.ri = self.ra_b = self.ri_b = None
+        self.ra = self.ri = self.ra_b = self.ri_b = self.w_gates = None
+        self._tiles = {}
 
     def cache_spec(self):
         return FixedState((ops.rglru_state_floats(self.inner, self.taps),), torch.float32)
@@ -53,6 +56,7 @@ class RealGatedLRU(Part):
         self.conv_w, self.conv_b = t(".conv").t().contiguous(), t(".conv.b").contiguous()
         self.ra, self.ri = t(".ra").contiguous(), t(".ri").contiguous()
         self.ra_b, self.ri_b = t(".ra.b").reshape(-1).contiguous(), t(".ri.b").reshape(-1).contiguous()
+        self.w_gates = ops.rglru_pieces_matrices(self.ra, self.ri) if rt.dtype == torch.bfloat16 and (self.inner // self.blocks) % 8 == 0 else None
         # 8 softplus(lam), from double precision
         self.sp8 = (8.0 * torch.nn.functional.softplus(t(".lam").double())).float().contiguous()
         self.wo = t(".o")
@@ -60,19 +64,34 @@ class RealGatedLRU(Part):
     def first_weights(self):
         return [self.w_in]
 
+    def _part_tiles(self, n: int, device) -> torch.Tensor:
+        """The grouped product's tile list for n tokens: the part of every tile, then how many tiles (made once per number of tiles)."""
+        rows, tile = ops.rglru_pieces_rows(n)
+        per = rows // tile
+        got = self._tiles.get(per)
+        if got is None:
+            flat = [v for b in range(self.blocks) for _ in range(per) for v in (b, 0, 0)] + [self.blocks * per]
+            got = self._tiles[per] = torch.tensor(flat, dtype=torch.int32).to(device)
+        return got
+
     def forward(self, rt, h, batch, cache):
         proj = rt.linear(h, self.w_in, bias=self.b_in, out_dtype=torch.float32)         # [tokens, x | y]
         if batch.max_q_len == 1:
             out = ops.rglru_step(proj, self.conv_w, self.conv_b, cache.state, batch.slots, batch.positions, self.ra, self.ra_b, self.ri, self.ri_b, self.sp8)
             return rt.linear(out, self.wo, partials_ok=True)
-        u = ops.rglru_conv(proj, self.conv_w, self.conv_b, cache.state, batch.seq_of_token, batch.seq_start, batch.slots, batch.positions,
-                           pieces=ops.rglru_pieces_supported(self.ra, h.shape[0]))
-        ab = ops.rglru_gates(u, self.ra, self.ra_b, self.ri, self.ri_b, self.sp8)
-        out = torch.empty((h.shape[0], self.inner), dtype=rt.dtype, device=h.device)
-        chunks = chunk_start = None
+        n = h.shape[0]
+        chunks = chunk_start = ends = None
         if batch.max_q_len > RGLRU_PIECES_FROM:
             chunks, chunk_start = batch.scan_pieces(ops.rglru_chunk_tokens())
-        ops.rglru_scan(ab, proj, cache.state, batch.seq_start, batch.slots, out, chunks, chunk_start)
+        products = self.w_gates is not None and n >= RGLRU_PRODUCTS_FROM
+        u = ops.rglru_conv(proj, self.conv_w, self.conv_b, cache.state, batch.seq_of_token, batch.seq_start, batch.slots, batch.positions,
+                           part=self.inner // self.blocks if products else 0)
+        if products:
+            ab, ends = ops.rglru_gates_pieces(u, n, self.w_gates, self._part_tiles(n, h.device), self.ra_b, self.ri_b, self.sp8, rt.status, chunks=chunks)
+        else:
+            ab = ops.rglru_gates(u, self.ra, self.ra_b, self.ri, self.ri_b, self.sp8)
+        out = torch.empty((n, self.inner), dtype=rt.dtype, device=h.device)
+        ops.rglru_scan(ab, proj, cache.state, batch.seq_start, batch.slots, out, chunks, chunk_start, ends=ends)
         return rt.linear(out, self.wo, partials_ok=True)
 
 

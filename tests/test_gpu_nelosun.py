@@ -431,14 +431,28 @@ def test_gates_are_32_bit_sums_in_every_form(dtype, C, B, taps):
     a, push = np.exp(log_a), np.sqrt(-np.expm1(2.0 * log_a)) * i * ud
     rough = P.sigmoid(P.block_linear(bf(ud), W["ri"], W["ri.b"]))
     assert np.abs(np.sqrt(-np.expm1(2.0 * log_a)) * rough * ud - push).max() > 1e-3, "rounded inputs would not show"
-    forms = [u]
+    ab = ops.rglru_gates(u, *gates)
+    assert worst(ab[0], a) < 2e-6 and worst(ab[1], push) < 1e-5 * (1 + np.abs(push).max())
     if dtype == torch.bfloat16 and (C // B) % 8 == 0:
-        pieces = ops.rglru_conv(*args, pieces=True)
-        assert bool((pieces.double().sum(dim=0) - u.double()).abs().max() < 1e-6)
-        forms.append(pieces)
-    for f in forms:
-        ab = ops.rglru_gates(f, *gates)
-        assert worst(ab[0], a) < (2e-6 if f is u else 1e-5) and worst(ab[1], push) < 1e-5 * (1 + np.abs(push).max())
+        rt = runtime(dtype)
+        for m in (150, 60, 32, 5):          # tiles of 128, 64 and 32 rows, whole and partly filled
+            P_ = C // B
+            few = (proj[:m], *conv, torch.zeros_like(state), i32([0] * m), i32([0, m]), i32([1]), i32(range(m)))
+            pieces = ops.rglru_conv(*few, part=P_)
+            rows, tile = ops.rglru_pieces_rows(m)
+            assert tuple(pieces.shape) == (B, rows, 3, P_)
+            assert worst(pieces[:, :m].double().sum(dim=2).permute(1, 0, 2).reshape(m, C), ud[:m]) < 1e-6
+            tiles = i32([v for b in range(B) for _ in range(rows // tile) for v in (b, 0, 0)] + [B * (rows // tile)])
+            chunks = i32([0, min(7, m), min(7, m), m]).view(2, 2)
+            for ch in (None, chunks):
+                ab, ends = ops.rglru_gates_pieces(pieces, m, ops.rglru_pieces_matrices(gates[0], gates[2]), tiles, gates[1], gates[3], gates[4], rt.status, chunks=ch)
+                rt.check_status()
+                assert worst(ab[0], a[:m]) < 1e-5 and worst(ab[1], push[:m]) < 1e-5 * (1 + np.abs(push).max())
+            for k, (lo, hi) in enumerate(chunks.tolist()):
+                S = np.zeros(C)
+                for t in range(lo, hi):
+                    S = a[t] * S + push[t]
+                assert worst(ends[0, k], np.prod(a[lo:hi], axis=0)) < 3e-5 and worst(ends[1, k], S) < 1e-4 * (1 + np.abs(S).max())
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
@@ -457,6 +471,7 @@ def test_recurrence_whole_in_pieces_and_token_by_token(dtype, C, B, taps):
     flip[0][0] *= -1
     assert np.abs(plain_recurrence(flip[0], ys[0], W)[3][-1] - want[0][-1]).max() > 1e-3, "the first token would not show at the end"
     conv, gates = bound_weights(W, dtype)
+    rt = runtime(dtype)
     slots = [3, 0, 2]
     plans = {"whole": [[330, 200, 75]], "single": [[1, 1, 1]] * 330, "mixed": [[1, 7, 75], [2, 1, 0], [64, 0, 0], [65, 3, 0], [1, 1, 0], [1, 1, 0], [129, 180, 0], [67, 7, 0]]}
     for name, plan in plans.items():
@@ -477,10 +492,8 @@ def test_recurrence_whole_in_pieces_and_token_by_token(dtype, C, B, taps):
             if max(n for _, n in here) == 1:
                 out = ops.rglru_step(proj, *conv, state, sl, pos, *gates)
             else:
-                u = ops.rglru_conv(proj, *conv, state, seq, start, sl, pos, pieces=ops.rglru_pieces_supported(gates[0], total))
-                ab = ops.rglru_gates(u, *gates)
                 out = torch.empty((total, C), dtype=dtype, device=DEV)
-                pieces = (None, None)
+                pieces, ends = (None, None), None
                 if max(n for _, n in here) > 64:
                     rows, first, t = [], [0], 0
                     for _, n in here:
@@ -488,7 +501,17 @@ def test_recurrence_whole_in_pieces_and_token_by_token(dtype, C, B, taps):
                         first.append(len(rows))
                         t += n
                     pieces = (i32(np.array(rows).reshape(-1)).view(-1, 2), i32(first))
-                ops.rglru_scan(ab, proj, state, start, sl, out, *pieces)
+                P_ = C // B
+                if dtype == torch.bfloat16 and P_ % 8 == 0 and total >= 32:
+                    u = ops.rglru_conv(proj, *conv, state, seq, start, sl, pos, part=P_)
+                    r_, tile = ops.rglru_pieces_rows(total)
+                    tiles = i32([v for b in range(B) for _ in range(r_ // tile) for v in (b, 0, 0)] + [B * (r_ // tile)])
+                    ab, ends = ops.rglru_gates_pieces(u, total, ops.rglru_pieces_matrices(gates[0], gates[2]), tiles, gates[1], gates[3], gates[4], rt.status,
+                                                      chunks=pieces[0])
+                    rt.check_status()
+                else:
+                    ab = ops.rglru_gates(ops.rglru_conv(proj, *conv, state, seq, start, sl, pos), *gates)
+                ops.rglru_scan(ab, proj, state, start, sl, out, *pieces, ends=ends)
             t = 0
             for r, n in here:
                 got[r][at[r]:at[r] + n] = out[t:t + n].float().cpu().numpy()
