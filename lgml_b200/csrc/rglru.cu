@@ -367,7 +367,7 @@ __global__ void __launch_bounds__(64) rglru_finish_chunks_kernel(const float *__
     pdl_wait();
     const int t0 = chunks[2 * k], t1 = chunks[2 * k + 1];
     float2 prod = make_float2(1.f, 1.f), S = make_float2(0.f, 0.f);
-    constexpr int W = 8;            // tokens whose loads are in flight together
+    constexpr int W = 4;            // tokens whose loads are in flight together (8 cost registers: 12 blocks an SM instead of 16, a second wave)
     for (int t = t0; t < t1; t += W) {
         GatePair g[W];
 #pragma unroll
