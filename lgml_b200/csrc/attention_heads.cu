@@ -6,9 +6,13 @@
 //                    latent c; its last Dr columns are a rotated key part shared by all heads;
 //                    both go into one cell of the cache [c | k_rot].  The queries' rotated part is
 //                    rotated and placed behind the R columns that head_linear fills
-//   head_linear      a product per head (FMA units; tensor cores from 32 tokens on): out[t, h, :] = W[h] x[t, h, :], for the up-projections of
+//   head_linear      a product per head (tensor cores from 32 tokens on, few bfloat16 rows with the matrix read sixteen bytes a lane, else
+//                    FMA tiles): out[t, h, :] = W[h] x[t, h, :], for the up-projections of
 //                    latent attention taken to the query side (q W_uk) and to the output side
 //                    (W_uv o), so that attention itself runs on the cached latent
+//   latent_down, latent_query   the same preparation where the queries come from a latent of their own: behind the one
+//                    down-projection both norms, the cell and the token's cosines and sines; behind the query product a head's
+//                    up-projection and turn in one kernel
 //
 // Norms, angles and the combination are float32 in both compute types.
 #include <math.h>
@@ -315,19 +319,24 @@ __global__ void __launch_bounds__(128) latent_down_kernel(const float *__restric
     pdl_trigger();
     pdl_wait();
     extern __shared__ float ld_sm[];        // the token's row, then its cosines and sines
-    __shared__ float red[32];
+    __shared__ float2 red[4];
     const int t = blockIdx.x, half = n_rot / 2;
     const int ps = halves ? 1 : 2, po = halves ? half : 1;
-    float *row = ld_sm, *cs = row + Rq + R + Dr, *sn = cs + half;
-    const int pos = positions[t];
+    float *row = ld_sm, *wn = row + Rq + R + Dr, *cs = wn + Rq + R, *sn = cs + half;          // wn: both norms' weights
+    const int pos = positions[t], blk = pos / page_size;
     const float *drow = down + (size_t)t * ldd;
     float sq = 0.f, sk = 0.f;
+#pragma unroll 4
     for (int k = threadIdx.x; k < Rq + R + Dr; k += blockDim.x) {
         const float v = act_load(drow + k);
+        if (k < Rq + R) wn[k] = k < Rq ? __ldg(wq + k) : __ldg(w + k - Rq);
         row[k] = v;
         if (k < Rq) sq = fmaf(v, v, sq);
         else if (k < Rq + R) sk = fmaf(v, v, sk);
     }
+    // the cell's page is looked up while the row is on its way
+    int page = -1;
+    if (pos >= 0 && blk < max_blocks) page = block_table[(size_t)seq_of_token[t] * max_blocks + blk];
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         float sv, cv;
         rope_sincos(pos, freq[i], freq_lo ? freq_lo[i] : 0.f, &sv, &cv);
@@ -335,20 +344,20 @@ __global__ void __launch_bounds__(128) latent_down_kernel(const float *__restric
         sn[i] = sv, cs[i] = cv;
         cos_sin[(size_t)t * n_rot + i] = cv, cos_sin[(size_t)t * n_rot + half + i] = sv;
     }
-    sq = block_sum(sq, red);
-    sk = block_sum(sk, red);
+    // both sums behind one barrier, in a fixed order
+    sq = warp_sum(sq), sk = warp_sum(sk);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(sq, sk);
+    __syncthreads();
+    sq = (red[0].x + red[1].x) + (red[2].x + red[3].x), sk = (red[0].y + red[1].y) + (red[2].y + red[3].y);
     const float iq = 1.0f / sqrtf(sq / (float)Rq + eps), ik = 1.0f / sqrtf(sk / (float)R + eps);
-    for (int k = threadIdx.x; k < Rq; k += blockDim.x) cq[(size_t)t * Rq + k] = from_f32<T>(row[k] * iq * wq[k]);
-    const int seq = seq_of_token[t], blk = pos / page_size;
-    int page = -1;
-    if (pos >= 0 && blk < max_blocks) page = block_table[(size_t)seq * max_blocks + blk];
+    for (int k = threadIdx.x; k < Rq; k += blockDim.x) cq[(size_t)t * Rq + k] = from_f32<T>(row[k] * iq * wn[k]);
     if (page < 0 || page >= n_pages) {      // the host reserves pages first; never write outside the pool
         if (threadIdx.x == 0) atomicExch(status, 2);
         return;
     }
     T *cell = k_pages + ((size_t)page * page_size + (size_t)(pos % page_size)) * (R + Dr);
     const float *c = row + Rq, *r = c + R;
-    for (int k = threadIdx.x; k < R; k += blockDim.x) cell[k] = from_f32<T>(c[k] * ik * w[k]);
+    for (int k = threadIdx.x; k < R; k += blockDim.x) cell[k] = from_f32<T>(c[k] * ik * wn[Rq + k]);
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         const float u = r[ps * i], v = r[ps * i + po];
         cell[R + ps * i] = from_f32<T>(u * cs[i] - v * sn[i]);
@@ -543,7 +552,7 @@ LGML_API int lgml_latent_down(const float *down, int ldd, const float *wq, const
     LGML_REQUIRE(n_rot >= 0 && n_rot <= Dr && n_rot % 2 == 0, "latent_down: %d rotated entries of %d", n_rot, Dr);
     LGML_REQUIRE(ldd >= Rq + R + Dr, "latent_down: row stride below the row");
     if (n_tokens == 0) return 0;
-    const size_t smem = sizeof(float) * ((size_t)Rq + R + Dr + n_rot);
+    const size_t smem = sizeof(float) * (2 * ((size_t)Rq + R) + Dr + n_rot);
     LGML_REQUIRE(smem <= 48 * 1024, "latent_down: rows of %d + %d + %d are too long", Rq, R, Dr);
     if (dtype == LGML_F32)
         lgml_launch(latent_down_kernel<float>, n_tokens, 128, smem, stream, down, ldd, wq, w, eps, freq, freq_lo, n_rot, positions, seq_of_token, block_table,
