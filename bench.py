@@ -16,8 +16,7 @@ measured copy bandwidth, and ``roofline_points`` the same fraction for every bat
 
 ``--shape llama32_3b`` runs that shape's own workload (32 prompts of 128 to 4,096 tokens in
 portions of 512 beside decodes, 512 new tokens each) through ``Engine.generate``;
-``--shape llama2_13b`` decodes at batch 16 after 3,584-token prompts; ``--design lefulorn`` (or ``gotulorn``, ``konovik``, ``dizepel``, ``tedisun``,
-``nelosun``)
+``--shape llama2_13b`` decodes at batch 16 after 3,584-token prompts; ``--design lefulorn`` (or ``gotulorn``, ``konovik``, ``dizepel``, ``tedisun``, ``nelosun``)
 times that design beside the Llama decoder at equal layer sizes; ``--cpu-baseline`` times the
 plain CPU implementation at the tiny configurations.
 """
