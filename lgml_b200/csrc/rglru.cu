@@ -355,7 +355,7 @@ __global__ void __launch_bounds__(256) rglru_finish_kernel(const float *__restri
         *reinterpret_cast<float2 *>(ab + ((size_t)n + t) * C + c) = push;
     }
 }
-__global__ void __launch_bounds__(64) rglru_finish_chunks_kernel(const float *__restrict__ z, const AsPieces u, const float *__restrict__ ra_b,
+__global__ void __launch_bounds__(64, 14) rglru_finish_chunks_kernel(const float *__restrict__ z, const AsPieces u, const float *__restrict__ ra_b,
                                                                  const float *__restrict__ ri_b, const float *__restrict__ sp8, float *__restrict__ ab,
                                                                  const int *__restrict__ chunks, float *__restrict__ A, float *__restrict__ B, int n, int C) {
     pdl_trigger();
@@ -367,7 +367,7 @@ __global__ void __launch_bounds__(64) rglru_finish_chunks_kernel(const float *__
     pdl_wait();
     const int t0 = chunks[2 * k], t1 = chunks[2 * k + 1];
     float2 prod = make_float2(1.f, 1.f), S = make_float2(0.f, 0.f);
-    constexpr int W = 4;            // tokens whose loads are in flight together (8 cost registers: 12 blocks an SM instead of 16, a second wave)
+    constexpr int W = 8;            // tokens whose loads are in flight together
     for (int t = t0; t < t1; t += W) {
         GatePair g[W];
 #pragma unroll
